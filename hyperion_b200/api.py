@@ -134,7 +134,7 @@ class Engine:
             num_pages=self.cache.num_pages, page_size=self.page_size, max_seq_len=limit,
             max_batch=min(max_batch or self.cache.max_requests, self.cache.max_requests), max_batch_tokens=max_batch_tokens,
             prefill_chunk_busy=prefill_chunk_busy, eos_token_ids=tuple(self.defaults.eos_token_ids), max_in_flight=2 if lookahead else 1,
-            group_windows=tuple(self.cache.group_windows)))
+            group_windows=tuple(self.cache.group_windows), group_keeps=tuple(self.cache.group_keeps)))
         # Requests are known to the scheduler by keys 0..n-1 (their order here) and to the cache by keys of its own.
         per_prompt = [p.validated() for p in per_prompt]  # once: an absent seed is drawn here, for the scheduler's copy and the sampler's alike
         sched_keys = [scheduler.enqueue(Request(index, prompt, params)) for index, (prompt, params) in enumerate(zip(prompts, per_prompt))]

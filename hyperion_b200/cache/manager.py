@@ -13,8 +13,9 @@ those operations and adds two things the reference's single kind of layer never 
   their own.  One page id addresses the same page in every member of its group.  What a user keeps
   per token is its own business: keys and values of some heads, one latent vector, anything of a
   fixed shape (:class:`hyperion_b200.parts.base.PagedTokens`).
-* *windows*: a group whose users only ever read the last ``window`` positions gives a page back as
-  soon as every position in it has fallen out of the window, while the request lives.
+* *windows*: a group whose users only ever read the last ``window`` positions (and perhaps the first
+  ``keep_first`` of the sequence, whose pages stay) gives a page back as soon as every position in it
+  has fallen out of the window, while the request lives.
 
 It is host code with no device dependency except the tensors it allocates when given a device; all
 bookkeeping can be exercised without one.
@@ -127,7 +128,8 @@ class CacheManager:
         self._lib = host.library()
         self._handle = ctypes.c_void_p()
         windows = host.ints([g.spec.window for g in self.paged])
-        host.check(self._lib.hb_cache_new(page_size, num_pages, max_requests, len(self.paged), host.address(windows), ctypes.byref(self._handle)))
+        keeps = host.ints([g.spec.keep_first for g in self.paged])
+        host.check(self._lib.hb_cache_new(page_size, num_pages, max_requests, len(self.paged), host.address(windows), host.address(keeps), ctypes.byref(self._handle)))
         self.keys = host.KeyMap()
         if device is not None:
             for g in self.paged:
@@ -158,6 +160,11 @@ class CacheManager:
     def group_windows(self) -> list[int]:
         """Per paged group its window (0 = it keeps every key): what the scheduler reserves pages by."""
         return [g.spec.window for g in self.paged]
+
+    @property
+    def group_keeps(self) -> list[int]:
+        """Per paged group the first positions it keeps beside its window."""
+        return [g.spec.keep_first for g in self.paged]
 
     def _key(self, request: Hashable) -> int:
         key = self.keys.known(request)

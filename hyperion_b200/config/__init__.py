@@ -5,5 +5,6 @@ from .mirovik import MirovikConfig
 from .nunivik import NunivikConfig
 from .qwen2 import Qwen2Config
 from .tobadra import TobadraConfig
+from .zurevik import ZurevikConfig
 
-__all__ = ["ConfigError", "ConfigReader", "read_json", "GenerationDefaults", "read_generation_defaults", "Qwen2Config", "NunivikConfig", "MirovikConfig", "KudazenConfig", "TobadraConfig"]
+__all__ = ["ConfigError", "ConfigReader", "read_json", "GenerationDefaults", "read_generation_defaults", "Qwen2Config", "NunivikConfig", "MirovikConfig", "KudazenConfig", "TobadraConfig", "ZurevikConfig"]

@@ -13,6 +13,9 @@
 // attention_split_rows_*_bf16 + attention_combine_rows_bf16 for decode rows
 // (helios/crates/helios-hal/kernels/elementwise.cu:576-729,749,875-937); mask: key position <= query
 // position (:660-663), optionally > position - window.
+// Beyond the reference: the first positions of a sequence may be seen from everywhere (keep_first), a softmax may have a sink per head, a
+// head's result a gate, and a head may have two softmax maps over the same values (`maps` 2): its queries and keys are then two halves of
+// D / 2 entries each, every map is a virtual head whose query is zero in the other half, and results leave as float.
 #include "common.cuh"
 
 #ifndef HB_HEAD_DIM
@@ -76,7 +79,7 @@ struct RowState {
 // thread's rows (hi < lo: nothing visible); `base`: position of the tile's key 0.
 template <int NT>
 __device__ __forceinline__ void process_keys(RowState& st, const bf16* qs, const bf16* ks, const bf16* vs, int key0, int base,
-                                             const int (&hi)[2], const int (&lo)[2], float scale_log2, float cap_pre, float cap_post) {
+                                             const int (&hi)[2], const int (&lo)[2], int keep, float scale_log2, float cap_pre, float cap_post) {
     const int lane = threadIdx.x & 31;
     float s[NT][4];
 #pragma unroll
@@ -102,7 +105,7 @@ __device__ __forceinline__ void process_keys(RowState& st, const bf16* qs, const
         for (int e = 0; e < 4; ++e) {
             const int r = e >> 1;
             const int pos = base + key0 + n * 8 + (lane & 3) * 2 + (e & 1);
-            const float v = (pos <= hi[r] && pos >= lo[r]) ? (cap_pre > 0.f ? capped_score_log2(s[n][e], cap_pre, cap_post) : s[n][e] * scale_log2) : -INFINITY;
+            const float v = (pos <= hi[r] && (pos >= lo[r] || pos < keep)) ? (cap_pre > 0.f ? capped_score_log2(s[n][e], cap_pre, cap_post) : s[n][e] * scale_log2) : -INFINITY;
             s[n][e] = v;
             mx[r] = fmaxf(mx[r], v);
         }
@@ -156,7 +159,7 @@ __device__ __forceinline__ void process_keys(RowState& st, const bf16* qs, const
 // Stage keys [base, base + 64) of one key/value head into the shared K and V tiles. Keys outside
 // [need_lo, need_hi] or without a page are zero-filled; a missing page inside the range sets the status.
 __device__ __forceinline__ void load_kv_tile(bf16* ks, bf16* vs, const bf16* cache, const int* table, int table_width, int base,
-                                             int need_lo, int need_hi, int kvh, int kv_heads, int page_size, int pages, int* status) {
+                                             int need_lo, int need_hi, int keep, int kvh, int kv_heads, int page_size, int pages, int* status) {
     // page_size is a power of two (the launcher refuses anything else).  All table entries are fetched first and the
     // copies issued afterwards, so the table reads of a tile overlap instead of each standing in front of its copy.
     const int shift = 31 - __clz(page_size);
@@ -167,7 +170,7 @@ __device__ __forceinline__ void load_kv_tile(bf16* ks, bf16* vs, const bf16* cac
     for (int i = 0; i < LOADS; ++i) {
         const int pos = base + (i * THREADS + (int)threadIdx.x) / CHUNKS;
         const int block = pos >> shift;
-        page[i] = (pos >= need_lo && pos <= need_hi) ? (block < table_width ? max(__ldg(table + block), -2) : -2) : -3;
+        page[i] = ((pos >= need_lo || pos < keep) && pos <= need_hi) ? (block < table_width ? max(__ldg(table + block), -2) : -2) : -3;
     }
 #pragma unroll
     for (int i = 0; i < LOADS; ++i) {
@@ -196,7 +199,21 @@ struct AttnArgs {
     float scale_log2;                  // scale * log2(e)
     int* status;
     float cap_pre, cap_post;  // scale / cap and cap * log2(e) of a smooth cap on the scores; cap_pre 0: none
+    int keep_first;                    // positions 0 .. keep_first - 1 are seen whatever the window
+    const float* sinks;                // [heads] or null: one more term exp(sink) in a softmax's denominator
+    const float* gate; int gate_stride;  // [tokens, gate_stride] float or null: head h's result takes sigmoid(gate[token, h])
+    int maps;                          // 1, or 2: heads are (head, map) pairs, map fastest, with queries of D / 2 entries each
+    int out_f32;                       // tile shape: the output is float
+    int pieces;                        // token shape: the unmerged pieces are the result, also with one split
 };
+
+// The 16-byte piece c of virtual head `head`'s query: with two maps per head, the half of the other map is zero.
+__device__ __forceinline__ const bf16* query_piece(const AttnArgs& a, int token, int head, int c, bool& valid) {
+    if (a.maps == 1) return valid ? a.q + (size_t)token * a.q_stride + (size_t)head * D + c * 8 : a.q;
+    const int inside = c * 8 - (head & 1) * (D / 2);
+    valid = valid && inside >= 0 && inside < D / 2;
+    return valid ? a.q + (size_t)token * a.q_stride + (size_t)head * (D / 2) + inside : a.q;
+}
 
 // ---------------------------------------------------------------------------------- tile shape
 // tiles[3*i] = first token (flat index), tiles[3*i+1] = token count, tiles[3*i+2] = batch row.
@@ -217,8 +234,8 @@ __global__ void __launch_bounds__(THREADS) attention_tiles_kernel(AttnArgs a, co
     for (int e = tid; e < BM * CHUNKS; e += THREADS) {
         const int v = e / CHUNKS, c = e - v * CHUNKS;
         const int tok = v / gc, hh = v - tok * gc;
-        const bool valid = tok < ntok && hh < heads_here;
-        const bf16* src = valid ? a.q + (size_t)(tok0 + tok) * a.q_stride + (size_t)(first_head + hh) * D + c * 8 : a.q;
+        bool valid = tok < ntok && hh < heads_here;
+        const bf16* src = query_piece(a, tok0 + tok, first_head + hh, c, valid);
         cp_async16(qs + v * LDS + c * 8, src, valid);
     }
     int hi[2], lo[2];
@@ -236,17 +253,18 @@ __global__ void __launch_bounds__(THREADS) attention_tiles_kernel(AttnArgs a, co
     const bool warp_has_rows = warp_first_tok < ntok;
 
     const int need_lo = first_seen(pos_first, a.window);
-    const int start = (need_lo / BN) * BN;
-    const int n_tiles = (pos_last - start) / BN + 1;
+    const int start = (need_lo / BN) * BN, n_kept = kept_tiles(a.keep_first, start, BN);
+    const int n_tiles = (pos_last - start) / BN + 1 + n_kept;
     RowState st;
     st.init();
-    load_kv_tile(kv, kv + BN * LDS, a.cache, table, a.table_width, start, need_lo, pos_last, kvh, a.kv_heads, a.page_size, a.pages, a.status);
+    load_kv_tile(kv, kv + BN * LDS, a.cache, table, a.table_width, key_tile_base(0, n_kept, start, BN), need_lo, pos_last, a.keep_first, kvh, a.kv_heads, a.page_size,
+                 a.pages, a.status);
     cp_async_commit();
     for (int it = 0; it < n_tiles; ++it) {
         bf16* ks = kv + (it & 1) * 2 * BN * LDS;
         if (it + 1 < n_tiles) {
             bf16* nk = kv + ((it + 1) & 1) * 2 * BN * LDS;
-            load_kv_tile(nk, nk + BN * LDS, a.cache, table, a.table_width, start + (it + 1) * BN, need_lo, pos_last, kvh, a.kv_heads,
+            load_kv_tile(nk, nk + BN * LDS, a.cache, table, a.table_width, key_tile_base(it + 1, n_kept, start, BN), need_lo, pos_last, a.keep_first, kvh, a.kv_heads,
                          a.page_size, a.pages, a.status);
             cp_async_commit();
             cp_async_wait<1>();
@@ -254,9 +272,9 @@ __global__ void __launch_bounds__(THREADS) attention_tiles_kernel(AttnArgs a, co
             cp_async_wait<0>();
         }
         __syncthreads();
-        const int base = start + it * BN;
-        if (warp_has_rows && base <= warp_hi && base + BN - 1 >= warp_lo)
-            process_keys<BN / 8>(st, qs + warp * 16 * LDS, ks, ks + BN * LDS, 0, base, hi, lo, a.scale_log2, a.cap_pre, a.cap_post);
+        const int base = key_tile_base(it, n_kept, start, BN);
+        if (warp_has_rows && base <= warp_hi && (base + BN - 1 >= warp_lo || base < a.keep_first))
+            process_keys<BN / 8>(st, qs + warp * 16 * LDS, ks, ks + BN * LDS, 0, base, hi, lo, a.keep_first, a.scale_log2, a.cap_pre, a.cap_post);
         __syncthreads();
     }
 #pragma unroll
@@ -264,7 +282,15 @@ __global__ void __launch_bounds__(THREADS) attention_tiles_kernel(AttnArgs a, co
         const int v = warp * 16 + (lane >> 2) + r * 8;
         const int tok = v / gc, hh = v - tok * gc;
         if (tok >= ntok || hh >= heads_here) continue;
-        const float inv = st.l[r] > 0.f ? 1.f / st.l[r] : 0.f;
+        const float l = st.l[r] + sink_share(a.sinks, first_head + hh, st.m[r]);
+        float inv = l > 0.f ? 1.f / l : 0.f;
+        if (a.gate) inv *= sigmoid_of(a.gate[(size_t)(tok0 + tok) * a.gate_stride + first_head + hh]);
+        if (a.out_f32) {
+            float* wide = reinterpret_cast<float*>(a.out) + (size_t)(tok0 + tok) * a.out_stride + (size_t)(first_head + hh) * D + (lane & 3) * 2;
+#pragma unroll
+            for (int n = 0; n < D / 8; ++n) *reinterpret_cast<float2*>(wide + n * 8) = make_float2(st.o[n][2 * r] * inv, st.o[n][2 * r + 1] * inv);
+            continue;
+        }
         bf16* dst = a.out + (size_t)(tok0 + tok) * a.out_stride + (size_t)(first_head + hh) * D + (lane & 3) * 2;
 #pragma unroll
         for (int n = 0; n < D / 8; ++n)
@@ -289,15 +315,16 @@ __global__ void __launch_bounds__(THREADS) attention_tokens_kernel(AttnArgs a, c
     const int pos = a.positions[t];
     const int* table = a.block_table + (size_t)a.token_row[t] * a.table_width;
     const int need_lo = first_seen(pos, a.window);
-    const int start = (need_lo / BN) * BN;
-    const int n_tiles = (pos - start) / BN + 1;
+    const int start = (need_lo / BN) * BN, n_kept = kept_tiles(a.keep_first, start, BN);
+    const int n_tiles = (pos - start) / BN + 1 + n_kept;
     const int per_split = (n_tiles + splits - 1) / splits;
     const int first = split * per_split, last = min(n_tiles, first + per_split);
 
     for (int e = tid; e < 16 * CHUNKS; e += THREADS) {
         const int v = e / CHUNKS, c = e - v * CHUNKS;
-        const bool valid = v < heads_here;
-        cp_async16(qs + v * LDS + c * 8, valid ? a.q + (size_t)t * a.q_stride + (size_t)(first_head + v) * D + c * 8 : a.q, valid);
+        bool valid = v < heads_here;
+        const bf16* src = query_piece(a, t, first_head + v, c, valid);
+        cp_async16(qs + v * LDS + c * 8, src, valid);
     }
     int hi[2], lo[2];
 #pragma unroll
@@ -314,7 +341,7 @@ __global__ void __launch_bounds__(THREADS) attention_tokens_kernel(AttnArgs a, c
     for (int s = 0; s < TOKEN_STAGES - 1; ++s) {
         if (first + s < last) {
             bf16* nk = kv + s * 2 * BN * LDS;
-            load_kv_tile(nk, nk + BN * LDS, a.cache, table, a.table_width, start + (first + s) * BN, need_lo, pos, kvh, a.kv_heads, a.page_size,
+            load_kv_tile(nk, nk + BN * LDS, a.cache, table, a.table_width, key_tile_base(first + s, n_kept, start, BN), need_lo, pos, a.keep_first, kvh, a.kv_heads, a.page_size,
                          a.pages, a.status);
         }
         cp_async_commit();
@@ -323,15 +350,15 @@ __global__ void __launch_bounds__(THREADS) attention_tokens_kernel(AttnArgs a, c
         const int ahead = it + TOKEN_STAGES - 1;
         if (ahead < last) {
             bf16* nk = kv + ((ahead - first) % TOKEN_STAGES) * 2 * BN * LDS;
-            load_kv_tile(nk, nk + BN * LDS, a.cache, table, a.table_width, start + ahead * BN, need_lo, pos, kvh, a.kv_heads, a.page_size,
+            load_kv_tile(nk, nk + BN * LDS, a.cache, table, a.table_width, key_tile_base(ahead, n_kept, start, BN), need_lo, pos, a.keep_first, kvh, a.kv_heads, a.page_size,
                          a.pages, a.status);
         }
         cp_async_commit();
         cp_async_wait<TOKEN_STAGES - 1>();
         __syncthreads();
         bf16* ks = kv + ((it - first) % TOKEN_STAGES) * 2 * BN * LDS;
-        const int base = start + it * BN;
-        if (base + warp * 16 <= pos) process_keys<2>(st, qs, ks, ks + BN * LDS, warp * 16, base, hi, lo, a.scale_log2, a.cap_pre, a.cap_post);
+        const int base = key_tile_base(it, n_kept, start, BN);
+        if (base + warp * 16 <= pos) process_keys<2>(st, qs, ks, ks + BN * LDS, warp * 16, base, hi, lo, a.keep_first, a.scale_log2, a.cap_pre, a.cap_post);
         __syncthreads();
     }
     cp_async_wait<0>();
@@ -364,7 +391,9 @@ __global__ void __launch_bounds__(THREADS) attention_tokens_kernel(AttnArgs a, c
             o += f * wo[((size_t)w * 16 + row) * D + c];
         }
         const int head = first_head + row;
-        if (splits == 1) {
+        if (splits == 1 && !a.pieces) {
+            l += sink_share(a.sinks, head, m);
+            if (a.gate) o *= sigmoid_of(a.gate[(size_t)t * a.gate_stride + head]);
             a.out[(size_t)t * a.out_stride + (size_t)head * D + c] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
         } else {
             const size_t slot = ((size_t)item * a.heads + head) * splits + split;
@@ -375,7 +404,8 @@ __global__ void __launch_bounds__(THREADS) attention_tokens_kernel(AttnArgs a, c
 }
 
 __global__ void attention_merge_kernel(const int* __restrict__ items, const float* __restrict__ ws_o, const float* __restrict__ ws_ml,
-                                       bf16* __restrict__ out, int out_stride, int heads, int splits) {
+                                       bf16* __restrict__ out, int out_stride, int heads, int splits, const float* __restrict__ sinks,
+                                       const float* __restrict__ gate, int gate_stride) {
     const int item = blockIdx.x, head = blockIdx.y, t = items[item];
     const size_t slot0 = ((size_t)item * heads + head) * splits;
     float m = -INFINITY;
@@ -388,6 +418,8 @@ __global__ void attention_merge_kernel(const int* __restrict__ items, const floa
             l += f * ws_ml[(slot0 + s) * 2 + 1];
             o += f * ws_o[(slot0 + s) * D + c];
         }
+        l += sink_share(sinks, head, m);
+        if (gate) o *= sigmoid_of(gate[(size_t)t * gate_stride + head]);
         out[(size_t)t * out_stride + (size_t)head * D + c] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
     }
 }
@@ -399,14 +431,15 @@ constexpr size_t TOKENS_SMEM = 16 * LDS * sizeof(bf16) + (TOKENS_KV_SMEM > TOKEN
 
 int fill_args(AttnArgs& a, const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
               int table_width, const int* token_row, const int* positions, int heads, int kv_heads, int head_dim, int page_size,
-              int pages, float scale, float softcap, int window, int* status) {
+              int pages, float scale, float softcap, int window, int keep_first, const float* sinks, const float* gate, int gate_stride, int maps, int* status) {
     if (head_dim != D) return HB_UNSUPPORTED_SIZE;
+    if (keep_first < 0 || maps < 1 || maps > 2 || (maps == 2 && (sinks || gate || (heads / (kv_heads > 0 ? kv_heads : 1)) % 2))) return HB_BAD_ARGUMENT;
     if (kv_heads <= 0 || heads % kv_heads || page_size <= 0 || q_stride % 8 || out_stride % 2) return HB_BAD_ARGUMENT;
     if (page_size & (page_size - 1)) return HB_UNSUPPORTED_SIZE;  // pages hold a power of two of tokens
     if (((uintptr_t)q | (uintptr_t)cache) & 15) return HB_BAD_ARGUMENT;
     a = AttnArgs{(const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)cache, block_table, table_width, token_row, positions,
                  heads, kv_heads, page_size, pages, window, scale * 1.4426950408889634f, status,
-                 softcap > 0.f ? scale / softcap : 0.f, softcap * 1.4426950408889634f};
+                 softcap > 0.f ? scale / softcap : 0.f, softcap * 1.4426950408889634f, window ? keep_first : 0, sinks, gate, gate_stride, maps, maps == 2, maps == 2};
     return 0;
 }
 }  // namespace
@@ -419,14 +452,16 @@ HB_EXPORT int hb_attention_tile_tokens(int heads, int kv_heads) {
     return BM / (group < BM ? group : BM);
 }
 
-HB_EXPORT int hb_attention_tiles_capped(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
+// keep_first, sinks, gate: see AttnArgs.  maps 2: `heads` counts (head, map) pairs, the query row is [heads, D / 2], the tile shape stores float
+// [tokens, heads, D] and the token shape leaves its pieces in the workspace (also with one split) and starts no merge.
+HB_EXPORT int hb_attention_tiles_extended(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
                                  int table_width, const int* token_row, const int* positions, const int* tiles, int n_tiles, int heads,
-                                 int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap, int window, int* status,
-                                 cudaStream_t stream) {
+                                 int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap, int window, int keep_first,
+                                 const float* sinks, const float* gate, int gate_stride, int maps, int* status, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     AttnArgs a;
     if (int code = fill_args(a, q, q_stride, out, out_stride, cache, block_table, table_width, token_row, positions, heads, kv_heads,
-                             head_dim, page_size, pages, scale, softcap, window, status)) return code;
+                             head_dim, page_size, pages, scale, softcap, window, keep_first, sinks, gate, gate_stride, maps, status)) return code;
     const int group = heads / kv_heads, gc = group < BM ? group : BM, head_chunks = (group + gc - 1) / gc;
     if ((long long)kv_heads * head_chunks > 65535) return HB_UNSUPPORTED_SIZE;
     static bool configured = false;
@@ -437,6 +472,14 @@ HB_EXPORT int hb_attention_tiles_capped(const void* q, int q_stride, void* out, 
     }
     attention_tiles_kernel<<<dim3(n_tiles, kv_heads * head_chunks), THREADS, TILES_SMEM, stream>>>(a, tiles, gc, head_chunks);
     return launch_status();
+}
+
+HB_EXPORT int hb_attention_tiles_capped(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
+                                 int table_width, const int* token_row, const int* positions, const int* tiles, int n_tiles, int heads,
+                                 int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap, int window, int* status,
+                                 cudaStream_t stream) {
+    return hb_attention_tiles_extended(q, q_stride, out, out_stride, cache, block_table, table_width, token_row, positions, tiles, n_tiles, heads, kv_heads, head_dim,
+                                       page_size, pages, scale, softcap, window, 0, nullptr, nullptr, 0, 1, status, stream);
 }
 
 HB_EXPORT int hb_attention_tiles(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
@@ -451,16 +494,16 @@ HB_EXPORT long long hb_attention_tokens_workspace(int n_items, int heads, int sp
     return splits <= 1 ? 0 : (long long)n_items * heads * splits * (D + 2);
 }
 
-HB_EXPORT int hb_attention_tokens_capped(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
+HB_EXPORT int hb_attention_tokens_extended(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
                                   int table_width, const int* token_row, const int* positions, const int* items, int n_items, int splits,
                                   float* workspace, int heads, int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap,
-                                  int window, int* status, cudaStream_t stream) {
+                                  int window, int keep_first, const float* sinks, const float* gate, int gate_stride, int maps, int* status, cudaStream_t stream) {
     if (n_items <= 0) return 0;
     AttnArgs a;
     if (int code = fill_args(a, q, q_stride, out, out_stride, cache, block_table, table_width, token_row, positions, heads, kv_heads,
-                             head_dim, page_size, pages, scale, softcap, window, status)) return code;
+                             head_dim, page_size, pages, scale, softcap, window, keep_first, sinks, gate, gate_stride, maps, status)) return code;
     const int group = heads / kv_heads, head_chunks = (group + 15) / 16;
-    if (splits < 1 || splits > 65535 || (long long)kv_heads * head_chunks > 65535 || (splits > 1 && !workspace)) return HB_BAD_ARGUMENT;
+    if (splits < 1 || splits > 65535 || (long long)kv_heads * head_chunks > 65535 || ((splits > 1 || a.pieces) && !workspace)) return HB_BAD_ARGUMENT;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(attention_tokens_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TOKENS_SMEM);
@@ -471,9 +514,18 @@ HB_EXPORT int hb_attention_tokens_capped(const void* q, int q_stride, void* out,
     float* ws_ml = workspace ? workspace + (size_t)n_items * heads * splits * D : nullptr;
     attention_tokens_kernel<<<dim3(n_items, kv_heads * head_chunks, splits), THREADS, TOKENS_SMEM, stream>>>(a, items, head_chunks, splits, ws_o, ws_ml);
     int code = launch_status();
-    if (code || splits == 1) return code;
-    attention_merge_kernel<<<dim3(n_items, heads), D < 64 ? 32 : (D < 128 ? 64 : 128), 0, stream>>>(items, ws_o, ws_ml, (bf16*)out, out_stride, heads, splits);
+    if (code || splits == 1 || a.pieces) return code;
+    attention_merge_kernel<<<dim3(n_items, heads), D < 64 ? 32 : (D < 128 ? 64 : 128), 0, stream>>>(items, ws_o, ws_ml, (bf16*)out, out_stride, heads, splits, sinks, gate,
+                                                                                                   gate_stride);
     return launch_status();
+}
+
+HB_EXPORT int hb_attention_tokens_capped(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
+                                  int table_width, const int* token_row, const int* positions, const int* items, int n_items, int splits,
+                                  float* workspace, int heads, int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap,
+                                  int window, int* status, cudaStream_t stream) {
+    return hb_attention_tokens_extended(q, q_stride, out, out_stride, cache, block_table, table_width, token_row, positions, items, n_items, splits, workspace, heads,
+                                        kv_heads, head_dim, page_size, pages, scale, softcap, window, 0, nullptr, nullptr, 0, 1, status, stream);
 }
 
 HB_EXPORT int hb_attention_tokens(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,

@@ -12,7 +12,9 @@
 // distance may be added to the score, and the result may pass a sigmoid gate.  Further options, each absent unless its
 // argument is given: a factor per head on the scaled score; a slope per head, slope * (query position - key position)
 // being taken off the score; sight limited to the query's own chunk of positions (chunks of `chunk` positions counted
-// from position 0); a sink per head, one more term exp(sink) in the softmax's denominator that has no key and no value.
+// from position 0); a sink per head, one more term exp(sink) in the softmax's denominator that has no key and no value; the first
+// `keep_first` positions of the sequence seen from everywhere beside the window; one gate per head instead of one per entry; several
+// softmax maps per head, each with queries and keys of its own, over the same values (the maps' results lie side by side in the row).
 // Heads of up to 640 entries take the kernel's second size (more shared memory and registers).
 #include "common.cuh"
 
@@ -24,11 +26,14 @@ struct ScoreExtras {
     const float* slopes;      // [heads] or null
     const float* sinks;       // [heads] or null
     int chunk;                // 0: no chunks
+    int keep_first;           // positions 0 .. keep_first - 1 are seen whatever the window
+    int gate_per_head;        // the gate has one column per head
+    int maps;                 // softmax maps per head: query row (head * maps + map), key at map * head_dim of the key/value head's keys
 };
 
-template <typename T, int DMAX>
+template <typename T, typename TO, int DMAX>
 __global__ void __launch_bounds__(THREADS) attention_generic_kernel(
-    const T* __restrict__ q, int q_stride, T* __restrict__ out, int out_stride, const T* __restrict__ k_cache,
+    const T* __restrict__ q, int q_stride, TO* __restrict__ out, int out_stride, const T* __restrict__ k_cache,
     const T* __restrict__ v_cache, size_t page_stride, size_t head_stride, int token_stride,
     const int* __restrict__ block_table, int table_width, const int* __restrict__ token_row,
     const int* __restrict__ positions, int heads, int kv_heads, int head_dim, int v_dim, int page_size, int pages, float scale,
@@ -39,7 +44,8 @@ __global__ void __launch_bounds__(THREADS) attention_generic_kernel(
     __shared__ float m_run[GMAX], l_run[GMAX], alpha[GMAX];
     __shared__ int tile_page[TILE];
 
-    const int t = blockIdx.x, kvh = blockIdx.y;
+    const int maps = extras.maps;
+    const int t = blockIdx.x, kvh = blockIdx.y / maps, map = blockIdx.y - kvh * maps;
     const int group = heads / kv_heads;
     const int g0 = blockIdx.z * GMAX;
     const int g = min(GMAX, group - g0);
@@ -50,7 +56,7 @@ __global__ void __launch_bounds__(THREADS) attention_generic_kernel(
 
     for (int e = tid; e < g * head_dim; e += THREADS) {
         const int hh = e / head_dim, d = e - hh * head_dim;
-        qs[hh][d] = to_float(q[(size_t)t * q_stride + (size_t)(kvh * group + g0 + hh) * head_dim + d]);
+        qs[hh][d] = to_float(q[(size_t)t * q_stride + (size_t)((kvh * group + g0 + hh) * maps + map) * head_dim + d]);
     }
     if (tid < GMAX) {  // a sink enters as a key whose score is the sink itself and whose value is nothing
         const bool sunk = extras.sinks && tid < g;
@@ -65,15 +71,17 @@ __global__ void __launch_bounds__(THREADS) attention_generic_kernel(
 
     int lo = window > 0 ? max(0, pos - window + 1) : 0;
     if (extras.chunk > 0) lo = max(lo, (pos / extras.chunk) * extras.chunk);
+    const int keep = min(extras.keep_first, lo);  // what lies below the window and is seen all the same
     bool bad_page = false;
     __syncthreads();
 
-    for (int base = (lo / TILE) * TILE; base <= pos; base += TILE) {
+    for (int base = keep > 0 ? 0 : (lo / TILE) * TILE; base <= pos; base += TILE) {
+        if (base >= keep && base + TILE <= lo) base = (lo / TILE) * TILE;  // nothing of what lies between is seen
         // pages of the tile's keys
         if (tid < TILE) {
             const int j = base + tid;
             int page = -1;
-            if (j >= lo && j <= pos) {
+            if ((j >= lo || j < keep) && j <= pos) {
                 const int block = j / page_size;
                 page = block < table_width ? table[block] : -1;
                 if (page < 0 || page >= pages) { bad_page = true; page = -1; }
@@ -89,7 +97,7 @@ __global__ void __launch_bounds__(THREADS) attention_generic_kernel(
 #pragma unroll
             for (int hh = 0; hh < GMAX; ++hh) part[hh] = 0.f;
             if (page >= 0) {
-                const T* kp = k_cache + (size_t)page * page_stride + (size_t)kvh * head_stride + (size_t)(j % page_size) * token_stride;
+                const T* kp = k_cache + (size_t)page * page_stride + (size_t)kvh * head_stride + (size_t)(j % page_size) * token_stride + map * head_dim;
                 for (int d = lane; d < head_dim; d += 32) {
                     const float kv = to_float(kp[d]);
 #pragma unroll
@@ -163,10 +171,11 @@ __global__ void __launch_bounds__(THREADS) attention_generic_kernel(
             for (int hh = 0; hh < GMAX; ++hh)
                 if (hh < g) {
                     const float l = l_run[hh];
-                    const size_t column = (size_t)(kvh * group + g0 + hh) * v_dim + d;
+                    const int head = kvh * group + g0 + hh;
+                    const size_t column = (size_t)(head * maps + map) * v_dim + d;
                     float result = l > 0.f ? acc[hh][c] / l : 0.f;
-                    if (gate) result *= out_scale / (1.f + expf(-gate[(size_t)t * gate_stride + gate_off + column]));
-                    out[(size_t)t * out_stride + column] = from_float<T>(result);
+                    if (gate) result *= out_scale / (1.f + expf(-gate[(size_t)t * gate_stride + gate_off + (extras.gate_per_head ? (size_t)head : column)]));
+                    out[(size_t)t * out_stride + column] = from_float<TO>(result);
                 }
         }
     }
@@ -178,6 +187,43 @@ __global__ void __launch_bounds__(THREADS) attention_generic_kernel(
 // key position j takes dist_bias[head, min(p - j, bias_span - 1)] after scale and cap.  gate [tokens, gate_stride] float (optional): the
 // result of (token, head, d) is multiplied by out_scale * sigmoid(gate[token, gate_off + head * v_dim + d]) before its one rounding.
 // head_scale, slopes, sinks: [heads] float each or null; chunk: 0 or the size of the chunks of positions a query stays inside.
+// keep_first: that many first positions are seen beside the window.  gate_per_head: the gate has one column per head.  maps: softmax maps
+// per head (queries [heads, maps, head_dim], a key/value head's keys [maps, head_dim], results [heads, maps, v_dim]; bias, factors, slopes,
+// sinks and the gate go by the head).  out_f32: the result is stored as float whatever the element type.
+HB_EXPORT int hb_attention_mapped(const void* q, int q_stride, void* out, int out_stride, int is_bf16, const void* k_cache,
+                                    const void* v_cache, long long page_stride, long long head_stride, int token_stride,
+                                    const int* block_table, int table_width, const int* token_row, const int* positions,
+                                    int tokens, int heads, int kv_heads, int head_dim, int v_dim, int page_size, int pages, float scale,
+                                    float softcap, int window, const float* dist_bias, int bias_span, const float* gate, int gate_stride,
+                                    int gate_off, float out_scale, const float* head_scale, const float* slopes, const float* sinks, int chunk,
+                                    int keep_first, int gate_per_head, int maps, int out_f32, int* status, cudaStream_t stream) {
+    if ((dist_bias && bias_span <= 0) || chunk < 0 || keep_first < 0 || maps < 1) return HB_BAD_ARGUMENT;
+    if (tokens <= 0) return 0;
+    const int largest = head_dim > v_dim ? head_dim : v_dim;
+    if (head_dim <= 0 || v_dim <= 0 || largest > 640 || kv_heads <= 0 || heads % kv_heads || page_size <= 0) return HB_UNSUPPORTED_SIZE;
+    const int group = heads / kv_heads;
+    dim3 grid(tokens, kv_heads * maps, (group + GMAX - 1) / GMAX);
+    if (grid.y > 65535 || grid.z > 65535) return HB_UNSUPPORTED_SIZE;
+    const ScoreExtras extras{head_scale, slopes, sinks, chunk, keep_first, gate_per_head, maps};
+#define HB_ATTEND(T, TO, DMAX)                                                                                                                   \
+    attention_generic_kernel<T, TO, DMAX><<<grid, THREADS, 0, stream>>>((const T*)q, q_stride, (TO*)out, out_stride, (const T*)k_cache, (const T*)v_cache, \
+                                                                    (size_t)page_stride, (size_t)head_stride, token_stride, block_table, table_width, \
+                                                                    token_row, positions, heads, kv_heads, head_dim, v_dim, page_size, pages, scale,  \
+                                                                    softcap, window, dist_bias, bias_span, gate, gate_stride, gate_off, out_scale,    \
+                                                                    extras, status)
+    if (largest <= 256) {
+        if (is_bf16 && out_f32) HB_ATTEND(__nv_bfloat16, float, 256);
+        else if (is_bf16) HB_ATTEND(__nv_bfloat16, __nv_bfloat16, 256);
+        else HB_ATTEND(float, float, 256);
+    } else {
+        if (is_bf16 && out_f32) HB_ATTEND(__nv_bfloat16, float, 640);
+        else if (is_bf16) HB_ATTEND(__nv_bfloat16, __nv_bfloat16, 640);
+        else HB_ATTEND(float, float, 640);
+    }
+#undef HB_ATTEND
+    return launch_status();
+}
+
 HB_EXPORT int hb_attention_extended(const void* q, int q_stride, void* out, int out_stride, int is_bf16, const void* k_cache,
                                     const void* v_cache, long long page_stride, long long head_stride, int token_stride,
                                     const int* block_table, int table_width, const int* token_row, const int* positions,
@@ -185,29 +231,10 @@ HB_EXPORT int hb_attention_extended(const void* q, int q_stride, void* out, int 
                                     float softcap, int window, const float* dist_bias, int bias_span, const float* gate, int gate_stride,
                                     int gate_off, float out_scale, const float* head_scale, const float* slopes, const float* sinks, int chunk,
                                     int* status, cudaStream_t stream) {
-    if ((dist_bias && bias_span <= 0) || chunk < 0) return HB_BAD_ARGUMENT;
-    if (tokens <= 0) return 0;
-    const int largest = head_dim > v_dim ? head_dim : v_dim;
-    if (head_dim <= 0 || v_dim <= 0 || largest > 640 || kv_heads <= 0 || heads % kv_heads || page_size <= 0) return HB_UNSUPPORTED_SIZE;
-    const int group = heads / kv_heads;
-    dim3 grid(tokens, kv_heads, (group + GMAX - 1) / GMAX);
-    if (grid.y > 65535 || grid.z > 65535) return HB_UNSUPPORTED_SIZE;
-    const ScoreExtras extras{head_scale, slopes, sinks, chunk};
-#define HB_ATTEND(T, DMAX)                                                                                                                       \
-    attention_generic_kernel<T, DMAX><<<grid, THREADS, 0, stream>>>((const T*)q, q_stride, (T*)out, out_stride, (const T*)k_cache, (const T*)v_cache, \
-                                                                    (size_t)page_stride, (size_t)head_stride, token_stride, block_table, table_width, \
-                                                                    token_row, positions, heads, kv_heads, head_dim, v_dim, page_size, pages, scale,  \
-                                                                    softcap, window, dist_bias, bias_span, gate, gate_stride, gate_off, out_scale,    \
-                                                                    extras, status)
-    if (largest <= 256) {
-        if (is_bf16) HB_ATTEND(__nv_bfloat16, 256);
-        else HB_ATTEND(float, 256);
-    } else {
-        if (is_bf16) HB_ATTEND(__nv_bfloat16, 640);
-        else HB_ATTEND(float, 640);
-    }
-#undef HB_ATTEND
-    return launch_status();
+    return hb_attention_mapped(q, q_stride, out, out_stride, is_bf16, k_cache, v_cache, page_stride, head_stride, token_stride, block_table,
+                               table_width, token_row, positions, tokens, heads, kv_heads, head_dim, v_dim, page_size, pages, scale, softcap,
+                               window, dist_bias, bias_span, gate, gate_stride, gate_off, out_scale, head_scale, slopes, sinks, chunk, 0, 0, 1, 0,
+                               status, stream);
 }
 
 HB_EXPORT int hb_attention_biased(const void* q, int q_stride, void* out, int out_stride, int is_bf16, const void* k_cache,

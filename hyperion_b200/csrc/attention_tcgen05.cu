@@ -21,6 +21,11 @@
 // A product of 64 keys cannot feed the tensor core: it is bound by reading Q out of shared memory (measured: 54 clocks
 // for M 128, N 64, K 16 against 64 for N 128, which does twice the arithmetic), and the hand-overs between the roles
 // cost the same per tile whatever its width; hence tiles of 128 keys.
+// Two softmax maps per head over the same values (`MAPS`, D = 128: queries and keys of a head are two halves of 64 entries, values have 128):
+// the halves H and L then are the two maps of the same 128 (token, head) rows.  They share the key and value tiles, S_H meets the first 64
+// columns of a key tile and S_L the last, and at an item's end the two softmax threads of a row, whose tensor-memory lanes are the same, take
+// half of the row's columns each:  o = a1 - lambda a2, o / sqrt(mean(o^2) + eps) * post * sigmoid(gate), exchanging what they need of one
+// another (1 / sum, the sum of squares) through shared memory.
 // Every mbarrier wait is bounded; a wait that runs out sets HB_STATUS_WAIT_EXPIRED, all roles leave their loops, the block
 // takes no further item, tensor memory is freed and the block returns.
 //
@@ -219,6 +224,10 @@ struct AttnArgs {
                         // bias_span < 0: [heads], and a key n positions back adds n * bias[head]
     int bias_span;
     float bias_to_raw;  // 1 / scale_log2: a bias is added to the raw score as bias * bias_to_raw, so that the one scaling that follows stands
+    int keep_first;                      // positions 0 .. keep_first - 1 are seen whatever the window
+    const float* sinks;                  // [heads] or null: one more term exp(sink) in a softmax's denominator
+    const float* gate; int gate_stride;  // [tokens, gate_stride] float or null: one column per head, with MAPS one per head and value entry
+    float lambda, eps, post;             // MAPS: the second map's weight, and what follows (see above)
 };
 
 // tiles[3*i] = first token (flat index), tiles[3*i+1] = token count, tiles[3*i+2] = batch row; virtual row v of a tile is
@@ -231,7 +240,9 @@ struct AttnArgs {
 // tile all of them; with one block per item the longest item alone would set the kernel's time, now the items spread
 // evenly over the blocks. `work` = {items handed out beyond every block's first, blocks that have finished}: the block
 // that finishes last sets both back to zero for the next launch in the stream.
-template <int BIASED>  // a bias by distance on the scores (1: a table, 2: a number per head times the distance): kernels of their own, so that the others keep their registers
+// BIASED: a bias by distance on the scores (1: a table, 2: a number per head times the distance); MAPS: two softmax maps per head; EXTRAS: the first
+// positions seen beside the window, sinks, a gate per head.  Kernels of their own, so that the others keep their registers.
+template <int BIASED, bool MAPS, bool EXTRAS>
 __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const __grid_constant__ CUtensorMap q_map,
                                                                   const AttnArgs a,
                                                                   const int* __restrict__ tiles, int n_work_tiles, int ys, int gc, int head_chunks,
@@ -255,12 +266,14 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
     unsigned long long* q_empty = q_full + 1;         // [1]: the item's last S has been computed
     unsigned long long* round_done = q_empty + 1;     // [1]: the eight softmax warps have finished the item
     unsigned long long* q_seen = round_done + 1;      // [1]: the eight softmax warps have seen the item's queries land
+    unsigned long long* maps_done = q_seen + 1;       // [2]: MAPS: both maps' results and sums are there; both halves' sums of squares are
     const int total_items = n_work_tiles * ys;
-    unsigned* tmem_slot = reinterpret_cast<unsigned*>(q_seen + 1);
+    unsigned* tmem_slot = reinterpret_cast<unsigned*>(maps_done + 2);
     volatile int* failed = reinterpret_cast<volatile int*>(tmem_slot + 1);
     // [4][5]: the items in flight, each with what every thread wants to know of it (item, first token, token count, batch
     // row, first position), fetched by the producer while the item before is still being worked on
     volatile int* item_slot = failed + 1;
+    volatile float* exchange = reinterpret_cast<volatile float*>(item_slot + 20);  // MAPS: [2][2][128]
     auto note_item = [&](int slot, int item) {  // one thread
         volatile int* info = item_slot + 5 * slot;
         info[0] = item;
@@ -287,6 +300,8 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
         mbar_init(q_empty, 1);
         mbar_init(round_done, 8);
         mbar_init(q_seen, 8);
+        mbar_init(&maps_done[0], 8);
+        mbar_init(&maps_done[1], 8);
         *failed = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -315,14 +330,15 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
         asm volatile("prefetch.tensormap [%0];" ::"l"(&kv_map) : "memory");
         asm volatile("prefetch.tensormap [%0];" ::"l"(&q_map) : "memory");
     }
-    const int tokens_per_tile = ROWS / gc;
+    const int tokens_per_tile = (MAPS ? BM : ROWS) / gc;
+    const int keep = EXTRAS ? a.keep_first : 0;
 
     // The roles run through the items each at its own pace, held together by the barriers of the data alone: the producer
     // fetches the next item's keys while the last tiles of this one are worked on, its queries as soon as this item's last
     // S has been issued, and the first S of the next item follows the last product of this one without a pause.
     // g0: key tiles of the items before this one; the rings of K and V run on across items (stage g % STAGES, phase by g).
     // h0[x]: key tiles half x has seen; its three barriers change phase once per tile of an item the half takes part in.
-    struct Item { int tok0, ntok, kvh, first_head, heads_here, pos_first, pos_last, need_lo, start, n_tiles, halves; const int* table; };
+    struct Item { int tok0, ntok, kvh, first_head, heads_here, pos_first, pos_last, need_lo, start, n_kept, n_tiles, halves; const int* table; };
     auto read_item = [&](int round, Item& it) -> bool {  // false: no item left
         volatile int* info = item_slot + 5 * (round & 3);
         const int item = info[0];
@@ -339,8 +355,9 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
         it.pos_last = it.pos_first + it.ntok - 1;
         it.need_lo = first_seen(it.pos_first, a.window);
         it.start = (it.need_lo / BN) * BN;
-        it.n_tiles = (it.pos_last - it.start) / BN + 1;
-        it.halves = it.ntok * gc > BM ? 2 : 1;
+        it.n_kept = EXTRAS ? kept_tiles(keep, it.start, BN) : 0;
+        it.n_tiles = (it.pos_last - it.start) / BN + 1 + it.n_kept;
+        it.halves = MAPS || it.ntok * gc > BM ? 2 : 1;
         return true;
     };
 
@@ -373,16 +390,17 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
                 if (!mbar_wait(q_empty, (round & 1) ^ 1, failed) || !mbar_wait(q_seen, (round & 1) ^ 1, failed)) { *failed = 1; alive = false; }
                 if (alive) {
                     mbar_expect_tx(q_full, (unsigned)(PANELS * 128 * gc * tokens_per_tile));
-                    for (int h = 0; h < PANELS; ++h) tma_load_3d(qs + h * Q_PANEL, &q_map, q_full, h * 64, it.first_head, it.tok0);
+                    // (MAPS: the first map's 128 rows and below them the second's, in one panel)
+                    for (int h = 0; h < PANELS; ++h) tma_load_3d(qs + h * (MAPS ? BM * 64 : Q_PANEL), &q_map, q_full, h * 64, it.first_head, it.tok0);
                 }
             }
             alive = __shfl_sync(0xffffffffu, alive ? 1 : 0, 0) != 0;
             for (int t = 0; t < it.n_tiles && alive; ++t) {
                 const int g = g0 + t, s = g % STAGES, turn = g / STAGES;
-                const int tile_base = it.start + t * BN;
+                const int tile_base = key_tile_base(t, it.n_kept, it.start, BN);
                 int my_page = -1;
                 const int k0 = tile_base + lane * a.page_size;
-                if (lane < pages_per_tile && k0 <= it.pos_last && k0 + a.page_size - 1 >= it.need_lo) {
+                if (lane < pages_per_tile && k0 <= it.pos_last && (k0 + a.page_size - 1 >= it.need_lo || (EXTRAS && k0 < keep))) {
                     const int block = k0 >> shift;
                     const int id = block < a.table_width ? __ldg(it.table + block) : -1;
                     if (id >= 0 && id < a.pages) my_page = id;
@@ -423,8 +441,8 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
             const unsigned q_empty_at = smem_u32(q_empty);
             auto issue_s = [&](int x, int g) {  // S_x = Q_x K(g)^T
                 const unsigned k_low = k_low0 + (unsigned)(g % STAGES) * (TILE_BYTES >> 4), q_low = q_low0 + (unsigned)x * (BM * 128 >> 4);
-                umma_s_panel(tmem + x * BN, q_low, k_low, idesc_s, 0u);
-                if (PANELS == 2) umma_s_panel(tmem + x * BN, q_low + (Q_PANEL * 2 >> 4), k_low + (KV_PANEL * 2 >> 4), idesc_s, 1u);
+                umma_s_panel(tmem + x * BN, q_low, MAPS ? k_low + (unsigned)x * (KV_PANEL * 2 >> 4) : k_low, idesc_s, 0u);
+                if (PANELS == 2 && !MAPS) umma_s_panel(tmem + x * BN, q_low + (Q_PANEL * 2 >> 4), k_low + (KV_PANEL * 2 >> 4), idesc_s, 1u);
                 umma_commit_at(s_full0 + 8u * (unsigned)x);
             };
             auto issue_pv = [&](int x, int g, unsigned accumulate) {  // O_x (+)= P_x V(g); P_x lies over the first 64 columns of S_x
@@ -494,7 +512,8 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
             if (!read_item(round, it)) break;
             if (x < it.halves) {
                 const int n_tiles = it.n_tiles;
-                const int tok = v / gc, hh = v - tok * gc;
+                const int row = MAPS ? r : v;
+                const int tok = row / gc, hh = row - tok * gc;
                 const bool row_valid = tok < it.ntok && hh < it.heads_here;
                 // A row beyond the tile's end (or beyond the heads of the chunk) is computed like the tile's last token and never
                 // stored: it takes the same way through the code as its neighbours, so no warp has to walk two ways.
@@ -512,7 +531,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
 #pragma unroll
                         for (int i = 0; i < BN; ++i) s[i] = capped_score_log2(s[i], a.cap_pre, a.cap_post);
                     }
-                    const int tile_base = it.start + j * BN;
+                    const int tile_base = key_tile_base(j, it.n_kept, it.start, BN);
                     // A bias by distance: from bias_span - 1 positions back it is one value per head.  A tile that lies that far
                     // behind every row of the warp takes it as a shift of the whole tile (nothing per score); only the tiles
                     // near the diagonal look their scores' biases up.
@@ -535,7 +554,13 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
                     }
                     // one way for the whole warp: the masked walk only where some row of the warp needs it
                     const int last_visible = hi - tile_base, first_visible = lo - tile_base;  // among the tile's keys 0 .. BN - 1
-                    if (!__all_sync(0xffffffffu, last_visible >= BN - 1 && first_visible <= 0)) {
+                    if (EXTRAS) {
+                        const int kept = keep - tile_base;  // the tile's keys below this one are seen whatever the window
+                        if (!__all_sync(0xffffffffu, last_visible >= BN - 1 && (first_visible <= 0 || kept >= BN))) {
+#pragma unroll
+                            for (int i = 0; i < BN; ++i) s[i] = (i <= last_visible && (i >= first_visible || i < kept)) ? s[i] : -INFINITY;
+                        }
+                    } else if (!__all_sync(0xffffffffu, last_visible >= BN - 1 && first_visible <= 0)) {
 #pragma unroll
                         for (int i = 0; i < BN; ++i) s[i] = (i <= last_visible && i >= first_visible) ? s[i] : -INFINITY;
                     }
@@ -593,8 +618,69 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
                 if (ok) ok = mbar_wait(&o_done[x], (hx + n_tiles - 1) & 1, failed);
                 if (!ok) *failed = 1;
                 tc_fence_after();
-                if (ok) {
-                    const float inv = l > 0.f ? 1.f / l : 0.f;
+                if constexpr (MAPS) {
+                    auto meet = [&](int which) {  // the eight softmax warps; each phase is waited for by everyone, once per item
+                        tc_fence_before();
+                        __syncwarp();
+                        if (lane == 0) mbar_arrive(&maps_done[which]);
+                        if (ok && !mbar_wait(&maps_done[which], round & 1, failed)) { *failed = 1; ok = false; }
+                        tc_fence_after();
+                    };
+                    exchange[x * BM + r] = l > 0.f ? 1.f / l : 0.f;
+                    meet(0);
+                    const float inv1 = exchange[r], inv2 = exchange[BM + r] * a.lambda;
+                    auto difference = [&](int c, float (&o)[16]) {  // 16 columns of a1 - lambda a2, by the whole warp
+                        float second[16];
+                        tmem_ld16(lane_addr + O_COL + x * 64 + c, o);
+                        tmem_ld16(lane_addr + O_COL + BM + x * 64 + c, second);
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) o[i] = o[i] * inv1 - second[i] * inv2;
+                    };
+                    float part[4] = {0.f, 0.f, 0.f, 0.f};
+                    if (ok) {
+#pragma unroll 1
+                        for (int c = 0; c < 64; c += 16) {
+                            float o[16];
+                            difference(c, o);
+#pragma unroll
+                            for (int i = 0; i < 16; ++i) part[i & 3] = fmaf(o[i], o[i], part[i & 3]);
+                        }
+                    }
+                    exchange[2 * BM + x * BM + r] = (part[0] + part[1]) + (part[2] + part[3]);
+                    meet(1);
+                    if (ok) {
+                        const float scale_o = a.post / sqrtf((exchange[2 * BM + r] + exchange[3 * BM + r]) / (float)D + a.eps);
+                        const size_t column = (size_t)(it.first_head + hh) * D + x * 64;
+                        const float* g = a.gate + (size_t)(it.tok0 + tok) * a.gate_stride + column;
+                        uint4* dst = reinterpret_cast<uint4*>(a.out + (size_t)(it.tok0 + tok) * a.out_stride + column);
+#pragma unroll 1
+                        for (int c = 0; c < 64; c += 16) {
+                            float o[16];
+                            difference(c, o);
+                            if (!row_valid) continue;
+#pragma unroll
+                            for (int half = 0; half < 2; ++half) {
+                                uint4 w;
+                                unsigned* packed = reinterpret_cast<unsigned*>(&w);
+#pragma unroll
+                                for (int i = 0; i < 8; i += 4) {
+                                    float z[4];
+                                    load4(g + c + half * 8 + i, z);
+#pragma unroll
+                                    for (int e = 0; e < 4; ++e) z[e] = o[half * 8 + i + e] * __fdividef(scale_o, 1.f + fast_exp2(-1.4426950408889634f * z[e]));
+                                    packed[i / 2] = pack_bf16x2(z[0], z[1]);
+                                    packed[i / 2 + 1] = pack_bf16x2(z[2], z[3]);
+                                }
+                                dst[c / 8 + half] = w;
+                            }
+                        }
+                    }
+                    tc_fence_before();
+                } else if (ok) {
+                    const int head = it.first_head + (row_valid ? hh : 0);
+                    if (EXTRAS) l += sink_share(a.sinks, head, m);
+                    float inv = l > 0.f ? 1.f / l : 0.f;
+                    if (EXTRAS && a.gate && row_valid) inv *= sigmoid_of(a.gate[(size_t)(it.tok0 + tok) * a.gate_stride + head]);
 #pragma unroll
                     for (int c = 0; c < D; c += 16) {
                         float o[16];
@@ -658,7 +744,7 @@ EncodeTiled encode_tiled() {
 }
 
 // More than half of an SM's shared memory, so that one block is all an SM takes: the block holds all of its tensor memory.
-constexpr size_t SMEM_USED = 1024 + (size_t)2 * STAGES * TILE_BYTES + (size_t)PANELS * Q_PANEL * sizeof(bf16) + (4 * STAGES + 10) * 8 + 96;
+constexpr size_t SMEM_USED = 1024 + (size_t)2 * STAGES * TILE_BYTES + (size_t)PANELS * Q_PANEL * sizeof(bf16) + (4 * STAGES + 12) * 8 + 96 + 4 * BM * sizeof(float);
 constexpr size_t SMEM_BYTES = SMEM_USED > 120 * 1024 ? SMEM_USED : 120 * 1024;
 }  // namespace
 
@@ -667,13 +753,19 @@ constexpr size_t SMEM_BYTES = SMEM_USED > 120 * 1024 ? SMEM_USED : 120 * 1024;
 HB_EXPORT int hb_attention_tc_tile_rows() { return ROWS; }
 
 // bias [heads, bias_span] float (optional), already times log2(e), or with bias_span < 0 one number per head that multiplies the
-// distance: see AttnArgs.  Not together with a cap.
-HB_EXPORT int hb_attention_tc_tiles_biased(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
+// distance: see AttnArgs.  Not together with a cap.  keep_first, sinks, gate: see AttnArgs.  maps 2 (D = 128): two softmax maps per head, `heads` counts
+// heads, the query row is [heads, 2, 64], the gate [heads, 128] per token (rows of 16-byte pieces); neither bias, cap nor sinks with it.
+HB_EXPORT int hb_attention_tc_tiles_extended(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
                                     int table_width, const int* token_row, const int* positions, const int* tiles, int n_tiles, int n_tokens,
                                     int heads, int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap, int window,
-                                    const float* bias, int bias_span, int* status, int* work, cudaStream_t stream) {
+                                    const float* bias, int bias_span, int keep_first, const float* sinks, const float* gate, int gate_stride, int maps,
+                                    float lambda, float eps, float post, int* status, int* work, cudaStream_t stream) {
     (void)token_row;
     if (!work) return HB_BAD_ARGUMENT;
+    if (keep_first < 0 || maps < 1 || maps > 2) return HB_BAD_ARGUMENT;
+    if (maps == 2 && (D != 128 || bias || sinks || softcap > 0.f || !gate || gate_stride % 4 || ((uintptr_t)gate & 15))) return HB_BAD_ARGUMENT;
+    if (!window) keep_first = 0;
+    if ((keep_first || sinks || gate) && bias) return HB_BAD_ARGUMENT;
     if (bias && (bias_span == 0 || softcap > 0.f)) return HB_BAD_ARGUMENT;
     if (n_tiles <= 0) return 0;
     if (n_tokens <= 0) return HB_BAD_ARGUMENT;
@@ -693,11 +785,12 @@ HB_EXPORT int hb_attention_tc_tiles_biased(const void* q, int q_stride, void* ou
                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
         return HB_BAD_ARGUMENT;
     // the queries as (column, head, token): a tile's box is 64 columns of gc heads of its tokens
-    const int group = heads / kv_heads, gc = group < ROWS ? group : ROWS, head_chunks = (group + gc - 1) / gc;
+    const int rows = maps == 2 ? BM : ROWS;  // (token, head) rows of a tile
+    const int group = heads / kv_heads, gc = group < rows ? group : rows, head_chunks = (group + gc - 1) / gc;
     CUtensorMap q_map;
     const cuuint64_t q_dims[3] = {(cuuint64_t)D, (cuuint64_t)heads, (cuuint64_t)n_tokens};
     const cuuint64_t q_strides[2] = {(cuuint64_t)D * 2, (cuuint64_t)q_stride * 2};
-    const cuuint32_t q_box[3] = {64, (cuuint32_t)gc, (cuuint32_t)(ROWS / gc)};
+    const cuuint32_t q_box[3] = {64, (cuuint32_t)gc, (cuuint32_t)(rows / gc)};
     const cuuint32_t q_elem[3] = {1, 1, 1};
     if (encode(&q_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(q), q_dims, q_strides, q_box, q_elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
@@ -705,13 +798,17 @@ HB_EXPORT int hb_attention_tc_tiles_biased(const void* q, int q_stride, void* ou
     AttnArgs a{(const bf16*)q, q_stride, (bf16*)out, out_stride, block_table, table_width, positions,
                heads, kv_heads, page_size, pages, window, softcap > 0.f ? 1.f : scale * 1.4426950408889634f, status,
                (((uintptr_t)out & 31) == 0 && out_stride % 16 == 0) ? 1 : 0, softcap > 0.f ? scale / softcap : 0.f, softcap * 1.4426950408889634f,
-               bias, bias_span, 1.f / (scale * 1.4426950408889634f)};
+               bias, bias_span, 1.f / (scale * 1.4426950408889634f), keep_first, sinks, gate, gate_stride, lambda, eps, post};
     if ((long long)kv_heads * head_chunks > 65535) return HB_UNSUPPORTED_SIZE;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_tc_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_tc_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
+        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<0, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_tc_kernel<1, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_tc_kernel<2, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_tc_kernel<0, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
+#if HB_HEAD_DIM == 128
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_tc_kernel<0, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
+#endif
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
@@ -722,14 +819,26 @@ HB_EXPORT int hb_attention_tc_tiles_biased(const void* q, int q_stride, void* ou
     const long long items = (long long)n_tiles * kv_heads * head_chunks;
     if (items > 0x7fffffffLL) return HB_UNSUPPORTED_SIZE;
     const int blocks = (int)(items < (long long)sms ? items : (long long)sms);
-    if (bias && bias_span < 0)
-        return launch_after_previous(attention_tc_kernel<2>, dim3(blocks), THREADS, SMEM_BYTES, stream, map, q_map, a, tiles, n_tiles,
-                                     kv_heads * head_chunks, gc, head_chunks, work);
-    if (bias)
-        return launch_after_previous(attention_tc_kernel<1>, dim3(blocks), THREADS, SMEM_BYTES, stream, map, q_map, a, tiles, n_tiles,
-                                     kv_heads * head_chunks, gc, head_chunks, work);
-    return launch_after_previous(attention_tc_kernel<0>, dim3(blocks), THREADS, SMEM_BYTES, stream, map, q_map, a, tiles, n_tiles, kv_heads * head_chunks, gc,
-                                 head_chunks, work);
+#define HB_TC_LAUNCH(BIASED, MAPS, EXTRAS)                                                                                                              \
+    return launch_after_previous(attention_tc_kernel<BIASED, MAPS, EXTRAS>, dim3(blocks), THREADS, SMEM_BYTES, stream, map, q_map, a, tiles, n_tiles,   \
+                                 kv_heads * head_chunks, gc, head_chunks, work)
+#if HB_HEAD_DIM == 128
+    if (maps == 2) HB_TC_LAUNCH(0, true, true);
+#endif
+    if (bias && bias_span < 0) HB_TC_LAUNCH(2, false, false);
+    if (bias) HB_TC_LAUNCH(1, false, false);
+    if (keep_first || sinks || gate) HB_TC_LAUNCH(0, false, true);
+    HB_TC_LAUNCH(0, false, false);
+#undef HB_TC_LAUNCH
+}
+
+HB_EXPORT int hb_attention_tc_tiles_biased(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
+                                    int table_width, const int* token_row, const int* positions, const int* tiles, int n_tiles, int n_tokens,
+                                    int heads, int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap, int window,
+                                    const float* bias, int bias_span, int* status, int* work, cudaStream_t stream) {
+    return hb_attention_tc_tiles_extended(q, q_stride, out, out_stride, cache, block_table, table_width, token_row, positions, tiles, n_tiles, n_tokens, heads,
+                                          kv_heads, head_dim, page_size, pages, scale, softcap, window, bias, bias_span, 0, nullptr, nullptr, 0, 1, 0.f, 0.f, 0.f,
+                                          status, work, stream);
 }
 
 HB_EXPORT int hb_attention_tc_tiles_capped(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,

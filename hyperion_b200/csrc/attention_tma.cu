@@ -11,6 +11,9 @@
 // Pages a tile does not need (beyond the query's position, or released by a window) are not fetched; the
 // ring is zeroed once so that what they leave in shared memory is finite.
 //
+// Also here: the first positions of a sequence seen from everywhere (keep_first), a sink per head in the softmax, a gate per head on the
+// result, and two softmax maps per head over the same values (see attention_bf16.cu).
+//
 // Every mbarrier wait is bounded; a wait that runs out sets HB_STATUS_WAIT_EXPIRED and the block leaves.
 // Counterparts in the reference: attention_mma_paged_*_bf16 and attention_split_rows_*_bf16 +
 // attention_combine_rows_bf16 (helios/crates/helios-hal/kernels/elementwise.cu:576-729,749,875-937).
@@ -101,7 +104,7 @@ struct RowState {
 // One warp: 16 query rows (padded tile `qs`) against NT * 8 keys starting at key `key0` of the swizzled K / V tiles.
 template <int NT>
 __device__ __forceinline__ void process_keys(RowState& st, const bf16* qs, const bf16* ks, const bf16* vs, int key0, int base,
-                                             const int (&hi)[2], const int (&lo)[2], float scale_log2, float cap_pre, float cap_post,
+                                             const int (&hi)[2], const int (&lo)[2], int keep, float scale_log2, float cap_pre, float cap_post,
                                              const float* const (&bias)[2], int bias_span) {
     const int lane = threadIdx.x & 31, m = lane >> 3;
     float s[NT][4];
@@ -127,7 +130,7 @@ __device__ __forceinline__ void process_keys(RowState& st, const bf16* qs, const
             const int r = e >> 1;
             const int pos = base + key0 + n * 8 + (lane & 3) * 2 + (e & 1);
             float v = -INFINITY;
-            if (pos <= hi[r] && pos >= lo[r]) {
+            if (pos <= hi[r] && (pos >= lo[r] || pos < keep)) {
                 v = cap_pre > 0.f ? capped_score_log2(s[n][e], cap_pre, cap_post) : s[n][e] * scale_log2;
                 if (bias[r]) v += bias[r][min(hi[r] - pos, bias_span - 1)];
             }
@@ -191,6 +194,12 @@ struct AttnArgs {
     float cap_pre, cap_post;  // scale / cap and cap * log2(e) of a smooth cap on the scores; cap_pre 0: none
     const float* bias;  // [heads, bias_span] floats times log2(e), or null: a key n positions back adds bias[head, min(n, bias_span - 1)] to its score
     int bias_span;
+    int keep_first;                      // positions 0 .. keep_first - 1 are seen whatever the window
+    const float* sinks;                  // [heads] or null: one more term exp(sink) in a softmax's denominator
+    const float* gate; int gate_stride;  // [tokens, gate_stride] float or null: head h's result takes sigmoid(gate[token, h])
+    int maps;                            // 1, or 2: heads are (head, map) pairs, map fastest, with queries of D / 2 entries each
+    int out_f32;                         // tile shape: the output is float
+    int pieces;                          // token shape: the unmerged pieces are the result, also with one split
 };
 
 __host__ __device__ constexpr int stages_for(bool tokens) { return D <= 64 ? 4 : (tokens && D <= 128 ? 3 : 2); }
@@ -224,8 +233,8 @@ __global__ void __launch_bounds__(THREADS) attention_tma_kernel(const __grid_con
     const int* table = a.block_table + (size_t)brow * a.table_width;
     const int pos_first = a.positions[tok0], pos_last = pos_first + ntok - 1;
     const int need_lo = first_seen(pos_first, a.window);
-    const int start = (need_lo / BN) * BN;
-    const int n_tiles = (pos_last - start) / BN + 1;
+    const int start = (need_lo / BN) * BN, n_kept = kept_tiles(a.keep_first, start, BN);
+    const int n_tiles = (pos_last - start) / BN + 1 + n_kept;
     int first = 0, last = n_tiles;
     if (TOKENS) {
         const int per_split = (n_tiles + splits - 1) / splits;
@@ -240,10 +249,10 @@ __global__ void __launch_bounds__(THREADS) attention_tma_kernel(const __grid_con
     }
     // Pages that are not fetched (before a window's start, beyond the last position) leave whatever the stage held
     // before under masked keys; that is earlier key/value data, which is finite, unless the stage was never written.
-    // So a stage is zeroed when its first tile is one of the two that can be fetched in part.
+    // So a stage is zeroed when its first tile is one of those that can be fetched in part.
     for (int s = 0; s < STAGES && first + s < last; ++s) {
         const int tile = first + s;
-        if (tile != n_tiles - 1 && !(tile == 0 && need_lo > start)) continue;
+        if (tile != n_tiles - 1 && tile >= n_kept && !(tile == n_kept && need_lo > start)) continue;
         uint4* stage = reinterpret_cast<uint4*>(ring + (size_t)s * STAGE_BYTES);
         for (int e = tid; e < STAGE_BYTES / 16; e += THREADS) stage[e] = make_uint4(0, 0, 0, 0);
     }
@@ -262,8 +271,15 @@ __global__ void __launch_bounds__(THREADS) attention_tma_kernel(const __grid_con
             const int v = e / (D / 8), c = e - v * (D / 8);
             const int tok = v / gc, hh = v - tok * gc;
             uint4 value = make_uint4(0, 0, 0, 0);
-            if (tok < ntok && hh < heads_here)
-                value = *reinterpret_cast<const uint4*>(a.q + (size_t)(tok0 + tok) * a.q_stride + (size_t)(first_head + hh) * D + c * 8);
+            if (tok < ntok && hh < heads_here) {
+                if (a.maps == 1) {
+                    value = *reinterpret_cast<const uint4*>(a.q + (size_t)(tok0 + tok) * a.q_stride + (size_t)(first_head + hh) * D + c * 8);
+                } else {  // two maps per head: the half of the other map is zero
+                    const int inside = c * 8 - ((first_head + hh) & 1) * (D / 2);
+                    if (inside >= 0 && inside < D / 2)
+                        value = *reinterpret_cast<const uint4*>(a.q + (size_t)(tok0 + tok) * a.q_stride + (size_t)(first_head + hh) * (D / 2) + inside);
+                }
+            }
             *reinterpret_cast<uint4*>(qs + v * LDQ + c * 8) = value;
         }
     }
@@ -296,7 +312,8 @@ __global__ void __launch_bounds__(THREADS) attention_tma_kernel(const __grid_con
         int looked_from = first, looked_id = -1;
         auto look_up = [&](int from) {
             looked_from = from;
-            const int block = (start + from * BN + lane * a.page_size) >> shift;
+            const int tile = from + lane / pages_per_tile;
+            const int block = (key_tile_base(tile, n_kept, start, BN) + (lane % pages_per_tile) * a.page_size) >> shift;
             looked_id = block < a.table_width ? __ldg(table + block) : -1;
         };
         if (looks_ahead) look_up(first);
@@ -311,7 +328,7 @@ __global__ void __launch_bounds__(THREADS) attention_tma_kernel(const __grid_con
                 if (lane == 0) { *failed = 1; atomicOr(a.status, HB_STATUS_WAIT_EXPIRED | (TOKENS ? HB_STATUS_IN_ATTENTION_TMA_TOKENS : HB_STATUS_IN_ATTENTION_TMA_TILES)); }
                 break;
             }
-            const int base = start + it * BN;
+            const int base = key_tile_base(it, n_kept, start, BN);
             if (!waited && base + BN - 1 >= fresh_from) {
                 wait_for_previous_kernels();
                 waited = true;
@@ -319,7 +336,7 @@ __global__ void __launch_bounds__(THREADS) attention_tma_kernel(const __grid_con
             int my_page = -1;
             const int k0 = base + lane * a.page_size;
             const int looked = looks_ahead ? __shfl_sync(0xffffffffu, looked_id, ((it - looked_from) * pages_per_tile + lane) & 31) : -1;
-            if (lane < pages_per_tile && k0 <= pos_last && k0 + a.page_size - 1 >= need_lo) {
+            if (lane < pages_per_tile && k0 <= pos_last && (k0 + a.page_size - 1 >= need_lo || k0 < a.keep_first)) {
                 const int block = k0 >> shift;
                 const int id = looks_ahead ? looked : (block < a.table_width ? __ldg(table + block) : -1);
                 if (id >= 0 && id < a.pages) my_page = id;
@@ -369,12 +386,12 @@ __global__ void __launch_bounds__(THREADS) attention_tma_kernel(const __grid_con
         const int s = (it - first) % STAGES, round = (it - first) / STAGES;
         if (!mbar_wait(&full[s], round & 1, failed)) { *failed = 1; atomicOr(a.status, HB_STATUS_WAIT_EXPIRED | (TOKENS ? HB_STATUS_IN_ATTENTION_TMA_TOKENS : HB_STATUS_IN_ATTENTION_TMA_TILES)); ok = false; break; }
         const bf16* ks = reinterpret_cast<const bf16*>(ring + (size_t)s * STAGE_BYTES);
-        const int base = start + it * BN;
+        const int base = key_tile_base(it, n_kept, start, BN);
         if (TOKENS) {
-            if (base + warp * 16 <= pos_last) process_keys<2>(st, qs, ks, ks + TILE_ELEMS, warp * 16, base, hi, lo, a.scale_log2, a.cap_pre, a.cap_post, bias, a.bias_span);
+            if (base + warp * 16 <= pos_last) process_keys<2>(st, qs, ks, ks + TILE_ELEMS, warp * 16, base, hi, lo, a.keep_first, a.scale_log2, a.cap_pre, a.cap_post, bias, a.bias_span);
         } else if (!TOKENS) {
-            if (warp_has_rows && base <= warp_hi && base + BN - 1 >= warp_lo)
-                process_keys<BN / 8>(st, qs + warp * 16 * LDQ, ks, ks + TILE_ELEMS, 0, base, hi, lo, a.scale_log2, a.cap_pre, a.cap_post, bias, a.bias_span);
+            if (warp_has_rows && base <= warp_hi && (base + BN - 1 >= warp_lo || base < a.keep_first))
+                process_keys<BN / 8>(st, qs + warp * 16 * LDQ, ks, ks + TILE_ELEMS, 0, base, hi, lo, a.keep_first, a.scale_log2, a.cap_pre, a.cap_post, bias, a.bias_span);
         }
         __syncwarp();
         if (lane == 0) mbar_arrive(&empty[s]);
@@ -386,7 +403,15 @@ __global__ void __launch_bounds__(THREADS) attention_tma_kernel(const __grid_con
             const int v = warp * 16 + (lane >> 2) + r * 8;
             const int tok = v / gc, hh = v - tok * gc;
             if (tok >= ntok || hh >= heads_here) continue;
-            const float inv = st.l[r] > 0.f ? 1.f / st.l[r] : 0.f;
+            const float l = st.l[r] + sink_share(a.sinks, first_head + hh, st.m[r]);
+            float inv = l > 0.f ? 1.f / l : 0.f;
+            if (a.gate) inv *= sigmoid_of(a.gate[(size_t)(tok0 + tok) * a.gate_stride + first_head + hh]);
+            if (a.out_f32) {
+                float* wide = reinterpret_cast<float*>(a.out) + (size_t)(tok0 + tok) * a.out_stride + (size_t)(first_head + hh) * D + (lane & 3) * 2;
+#pragma unroll
+                for (int n = 0; n < D / 8; ++n) *reinterpret_cast<float2*>(wide + n * 8) = make_float2(st.o[n][2 * r] * inv, st.o[n][2 * r + 1] * inv);
+                continue;
+            }
             bf16* dst = a.out + (size_t)(tok0 + tok) * a.out_stride + (size_t)(first_head + hh) * D + (lane & 3) * 2;
 #pragma unroll
             for (int n = 0; n < D / 8; ++n)
@@ -425,7 +450,9 @@ __global__ void __launch_bounds__(THREADS) attention_tma_kernel(const __grid_con
             o += f * wo[((size_t)w * 16 + row) * D + c];
         }
         const int head = first_head + row;
-        if (splits == 1) {
+        if (splits == 1 && !a.pieces) {
+            l += sink_share(a.sinks, head, m);
+            if (a.gate) o *= sigmoid_of(a.gate[(size_t)tok0 * a.gate_stride + head]);
             a.out[(size_t)tok0 * a.out_stride + (size_t)head * D + c] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
         } else {
             const size_t slot = ((size_t)blockIdx.x * a.heads + head) * splits + split;
@@ -440,7 +467,8 @@ __global__ void __launch_bounds__(THREADS) attention_tma_kernel(const __grid_con
 // sums stays the order of the splits.
 constexpr int MERGE_AHEAD = 16;
 __global__ void attention_merge_kernel(const int* __restrict__ items, const float* __restrict__ ws_o, const float* __restrict__ ws_ml,
-                                       bf16* __restrict__ out, int out_stride, int heads, int splits) {
+                                       bf16* __restrict__ out, int out_stride, int heads, int splits, const float* __restrict__ sinks,
+                                       const float* __restrict__ gate, int gate_stride) {
     const int item = blockIdx.x, head = blockIdx.y, t = items[item];
     let_next_kernel_start();
     wait_for_previous_kernels();
@@ -475,6 +503,8 @@ __global__ void attention_merge_kernel(const int* __restrict__ items, const floa
             l += f * p.y;
             o += f * ws_o[(slot0 + s) * D + c];
         }
+        l += sink_share(sinks, head, m);
+        if (gate) o *= sigmoid_of(gate[(size_t)t * gate_stride + head]);
         out[(size_t)t * out_stride + (size_t)head * D + c] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
     }
 }
@@ -502,8 +532,11 @@ constexpr size_t smem_bytes() {
 // The cache layer as a matrix [pages * 2 * kv_heads * page_size, D] fetched in boxes of page_size rows x 64 columns.
 int prepare(CUtensorMap* map, AttnArgs& a, const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
             int table_width, const int* token_row, const int* positions, int heads, int kv_heads, int head_dim, int page_size, int pages,
-            float scale, float softcap, int window, const float* bias, int bias_span, int* status) {
+            float scale, float softcap, int window, const float* bias, int bias_span, int keep_first, const float* sinks, const float* gate, int gate_stride,
+            int maps, int* status) {
     if (head_dim != D) return HB_UNSUPPORTED_SIZE;
+    if (keep_first < 0 || maps < 1 || maps > 2) return HB_BAD_ARGUMENT;
+    if (maps == 2 && (sinks || gate || bias || kv_heads <= 0 || (heads / kv_heads) % 2)) return HB_BAD_ARGUMENT;
     if (bias && bias_span <= 0) return HB_BAD_ARGUMENT;
     if (kv_heads <= 0 || heads % kv_heads || q_stride % 8 || out_stride % 2) return HB_BAD_ARGUMENT;
     if (page_size < 8 || page_size > 64 || (page_size & (page_size - 1))) return HB_UNSUPPORTED_SIZE;
@@ -519,21 +552,25 @@ int prepare(CUtensorMap* map, AttnArgs& a, const void* q, int q_stride, void* ou
         return HB_BAD_ARGUMENT;
     a = AttnArgs{(const bf16*)q, q_stride, (bf16*)out, out_stride, block_table, table_width, token_row, positions,
                  heads, kv_heads, page_size, pages, window, scale * 1.4426950408889634f, status,
-                 softcap > 0.f ? scale / softcap : 0.f, softcap * 1.4426950408889634f, bias, bias_span};
+                 softcap > 0.f ? scale / softcap : 0.f, softcap * 1.4426950408889634f, bias, bias_span, window ? keep_first : 0, sinks, gate, gate_stride,
+                 maps, maps == 2, maps == 2};
     return 0;
 }
 }  // namespace
 
 // bias [heads, bias_span] float (optional), already times log2(e): a key n positions back adds bias[head, min(n, bias_span - 1)] to its score.
-HB_EXPORT int hb_attention_tma_tiles_biased(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
+// keep_first, sinks, gate: see AttnArgs.  maps 2: `heads` counts (head, map) pairs, the query row is [heads, D / 2], the tile shape stores float
+// [tokens, heads, D] and the token shape leaves its pieces in the workspace (also with one split) and starts no merge.
+HB_EXPORT int hb_attention_tma_tiles_extended(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
                                      int table_width, const int* token_row, const int* positions, const int* tiles, int n_tiles, int heads,
                                      int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap, int window,
-                                     const float* bias, int bias_span, int* status, cudaStream_t stream) {
+                                     const float* bias, int bias_span, int keep_first, const float* sinks, const float* gate, int gate_stride, int maps,
+                                     int* status, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     CUtensorMap map;
     AttnArgs a;
     if (int code = prepare(&map, a, q, q_stride, out, out_stride, cache, block_table, table_width, token_row, positions, heads, kv_heads,
-                           head_dim, page_size, pages, scale, softcap, window, bias, bias_span, status)) return code;
+                           head_dim, page_size, pages, scale, softcap, window, bias, bias_span, keep_first, sinks, gate, gate_stride, maps, status)) return code;
     const int group = heads / kv_heads, gc = group < 64 ? group : 64, head_chunks = (group + gc - 1) / gc;
     if ((long long)kv_heads * head_chunks > 65535) return HB_UNSUPPORTED_SIZE;
     static bool configured = false;
@@ -544,6 +581,14 @@ HB_EXPORT int hb_attention_tma_tiles_biased(const void* q, int q_stride, void* o
     }
     return launch_after_previous(attention_tma_kernel<false>, dim3(n_tiles, kv_heads * head_chunks), THREADS, smem_bytes<false>(), stream, map, a, tiles,
                                  gc, head_chunks, 1, nullptr, nullptr);
+}
+
+HB_EXPORT int hb_attention_tma_tiles_biased(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
+                                     int table_width, const int* token_row, const int* positions, const int* tiles, int n_tiles, int heads,
+                                     int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap, int window,
+                                     const float* bias, int bias_span, int* status, cudaStream_t stream) {
+    return hb_attention_tma_tiles_extended(q, q_stride, out, out_stride, cache, block_table, table_width, token_row, positions, tiles, n_tiles, heads, kv_heads,
+                                           head_dim, page_size, pages, scale, softcap, window, bias, bias_span, 0, nullptr, nullptr, 0, 1, status, stream);
 }
 
 HB_EXPORT int hb_attention_tma_tiles_capped(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
@@ -561,17 +606,18 @@ HB_EXPORT int hb_attention_tma_tiles(const void* q, int q_stride, void* out, int
     return hb_attention_tma_tiles_capped(q, q_stride, out, out_stride, cache, block_table, table_width, token_row, positions, tiles, n_tiles, heads, kv_heads, head_dim, page_size, pages, scale, 0.f, window, status, stream);
 }
 
-HB_EXPORT int hb_attention_tma_tokens_biased(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
+HB_EXPORT int hb_attention_tma_tokens_extended(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
                                       int table_width, const int* token_row, const int* positions, const int* items, int n_items, int splits,
                                       float* workspace, int heads, int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap,
-                                      int window, const float* bias, int bias_span, int* status, cudaStream_t stream) {
+                                      int window, const float* bias, int bias_span, int keep_first, const float* sinks, const float* gate, int gate_stride,
+                                      int maps, int* status, cudaStream_t stream) {
     if (n_items <= 0) return 0;
     CUtensorMap map;
     AttnArgs a;
     if (int code = prepare(&map, a, q, q_stride, out, out_stride, cache, block_table, table_width, token_row, positions, heads, kv_heads,
-                           head_dim, page_size, pages, scale, softcap, window, bias, bias_span, status)) return code;
+                           head_dim, page_size, pages, scale, softcap, window, bias, bias_span, keep_first, sinks, gate, gate_stride, maps, status)) return code;
     const int group = heads / kv_heads, head_chunks = (group + 15) / 16;
-    if (splits < 1 || splits > 65535 || (long long)kv_heads * head_chunks > 65535 || (splits > 1 && !workspace)) return HB_BAD_ARGUMENT;
+    if (splits < 1 || splits > 65535 || (long long)kv_heads * head_chunks > 65535 || ((splits > 1 || a.pieces) && !workspace)) return HB_BAD_ARGUMENT;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(attention_tma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_bytes<true>());
@@ -582,9 +628,18 @@ HB_EXPORT int hb_attention_tma_tokens_biased(const void* q, int q_stride, void* 
     float* ws_ml = workspace ? workspace + (size_t)n_items * heads * splits * D : nullptr;
     int code = launch_after_previous(attention_tma_kernel<true>, dim3(n_items, kv_heads * head_chunks, splits), THREADS, smem_bytes<true>(), stream, map, a,
                                      items, 16, head_chunks, splits, ws_o, ws_ml);
-    if (code || splits == 1) return code;
+    if (code || splits == 1 || a.pieces) return code;
     return launch_after_previous(attention_merge_kernel, dim3(n_items, heads), D < 128 ? 64 : 128, 0, stream, items, (const float*)ws_o,
-                                 (const float*)ws_ml, (bf16*)out, out_stride, heads, splits);
+                                 (const float*)ws_ml, (bf16*)out, out_stride, heads, splits, sinks, gate, gate_stride);
+}
+
+HB_EXPORT int hb_attention_tma_tokens_biased(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,
+                                      int table_width, const int* token_row, const int* positions, const int* items, int n_items, int splits,
+                                      float* workspace, int heads, int kv_heads, int head_dim, int page_size, int pages, float scale, float softcap,
+                                      int window, const float* bias, int bias_span, int* status, cudaStream_t stream) {
+    return hb_attention_tma_tokens_extended(q, q_stride, out, out_stride, cache, block_table, table_width, token_row, positions, items, n_items, splits, workspace,
+                                            heads, kv_heads, head_dim, page_size, pages, scale, softcap, window, bias, bias_span, 0, nullptr, nullptr, 0, 1,
+                                            status, stream);
 }
 
 HB_EXPORT int hb_attention_tma_tokens_capped(const void* q, int q_stride, void* out, int out_stride, const void* cache, const int* block_table,

@@ -87,6 +87,16 @@ __device__ __forceinline__ float capped_score_log2(float raw, float pre, float p
     return post * (1.f - __fdividef(2.f, 1.f + e));
 }
 
+// The activations a product's epilogue can apply to what it stores.
+enum : int { HB_ACT_NONE = 0, HB_ACT_RELU_SQUARED = 1 };
+__device__ __forceinline__ float activated(float v, int act) {
+    if (act == HB_ACT_RELU_SQUARED) {
+        v = fmaxf(v, 0.f);
+        return v * v;
+    }
+    return v;
+}
+
 static inline int launch_status() { return (int)cudaGetLastError(); }
 
 // ---------------------------------------------------------------- programmatic dependent launch
@@ -134,6 +144,19 @@ __host__ __device__ __forceinline__ int first_seen(int pos, int window) {
     if (window < 0) return pos >= 0 ? pos - pos % (-window) : 0;
     return 0;
 }
+
+// A query may also see the first `keep` positions of the sequence, however far its window has moved on: how many key tiles of `bn` positions
+// a walk that begins at `start` (a multiple of bn) takes from position 0 on before it goes there.  Positions below `keep` that lie in the tiles
+// from `start` on need no tile of their own.
+__host__ __device__ __forceinline__ int kept_tiles(int keep, int start, int bn) {
+    const int tiles = (keep + bn - 1) / bn, below = start / bn;
+    return tiles < below ? tiles : below;
+}
+__device__ __forceinline__ int key_tile_base(int tile, int n_kept, int start, int bn) { return tile < n_kept ? tile * bn : start + (tile - n_kept) * bn; }
+
+// What a softmax's denominator takes beside its keys: exp(sink) of the head, in units of the running maximum m (exp2 domain).
+__device__ __forceinline__ float sink_share(const float* sinks, int head, float m) { return sinks ? exp2f(sinks[head] * 1.4426950408889634f - m) : 0.f; }
+__device__ __forceinline__ float sigmoid_of(float z) { return 1.f / (1.f + expf(-z)); }
 
 // Four consecutive elements as floats, by one 16-byte (float) or 8-byte (bfloat16) access; p is aligned to that.
 __device__ __forceinline__ void load4(const float* p, float (&v)[4]) {

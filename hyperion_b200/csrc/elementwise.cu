@@ -1086,3 +1086,169 @@ HB_EXPORT int hb_scale_rows(float* x, float scale, long long count, cudaStream_t
     scale_rows_kernel<<<blocks, 256, 0, stream>>>(x, scale, (size_t)count);
     return launch_status();
 }
+
+// ---------------------------------------------------------------- the sum of two sublayers, then one norm or two of the same stream
+// h <- h + (a + b) in the float stream, then out1 = h / sqrt(mean(h^2) + eps) * w1 and, where a second weight is given, out2 likewise with w2: two
+// sublayers that read the same stream through norms of their own share its root mean square.  `a` is dense, or a product still in its split-K
+// pieces (float, added up in split order); `b` is dense, or rows sorted by expert of which a token takes `top` with a weight each (added
+// in the order of the choices).  With `rows` only those rows are worked on and h stays as it was.  Everything is float until the
+// rounding of a result.  A row stays in the block's registers between the sum and the norm.
+struct PairInputs {
+    const void* a;          // [tokens, hidden], or float [splits, tokens, hidden] when a_splits > 0
+    int a_splits;
+    size_t a_split_stride;
+    const void* b;          // [tokens, hidden], or [slots, hidden] when slot_of is given
+    const int* slot_of;     // [tokens, top]
+    const float* weights;   // [tokens, top]
+    int top;
+};
+
+template <typename TD, int VEC>
+__device__ __forceinline__ void read_entries(const TD* p, float (&v)[VEC]) {
+    if constexpr (VEC == 4) load4(p, v);
+    else v[0] = to_float(p[0]);
+}
+
+template <typename TD, typename TO, int VEC, int CHUNKS>
+__global__ void __launch_bounds__(512) add_pair_norms_kernel(float* __restrict__ h, const PairInputs in, const float* __restrict__ w1, const float* __restrict__ w2,
+                                                             TO* __restrict__ out1, TO* __restrict__ out2, const int* __restrict__ rows, int hidden, float eps,
+                                                             int write_h) {
+    __shared__ float scratch[32];
+    const int r = blockIdx.x, step = blockDim.x * VEC;
+    float weight1[CHUNKS][VEC];
+    let_next_kernel_start();
+#pragma unroll
+    for (int c = 0; c < CHUNKS; ++c) {  // no kernel writes weights: these loads overlap the kernel before
+        const int i = c * step + threadIdx.x * VEC;
+        if (i < hidden) read_entries<float, VEC>(w1 + i, weight1[c]);
+    }
+    wait_for_previous_kernels();
+    const int s = rows ? rows[r] : r;
+    float* hrow = h + (size_t)s * hidden;
+    float v[CHUNKS][VEC];
+    float sum = 0.f;
+#pragma unroll
+    for (int c = 0; c < CHUNKS; ++c) {
+        const int i = c * step + threadIdx.x * VEC;
+        if (i >= hidden) continue;
+        read_entries<float, VEC>(hrow + i, v[c]);
+        float add[VEC], x[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) add[e] = 0.f;
+        if (in.a_splits > 0) {
+            const float* p = (const float*)in.a + (size_t)s * hidden + i;
+#pragma unroll 4
+            for (int k = 0; k < in.a_splits; ++k) {
+                read_entries<float, VEC>(p + (size_t)k * in.a_split_stride, x);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) add[e] += x[e];
+            }
+        } else if (in.a) {
+            read_entries<TD, VEC>((const TD*)in.a + (size_t)s * hidden + i, add);
+        }
+        if (in.slot_of) {
+            float fed[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) fed[e] = 0.f;
+#pragma unroll 4
+            for (int k = 0; k < in.top; ++k) {
+                const int slot = in.slot_of[(size_t)s * in.top + k];
+                const float w = in.weights[(size_t)s * in.top + k];
+                if (slot < 0) continue;
+                read_entries<TD, VEC>((const TD*)in.b + (size_t)slot * hidden + i, x);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) fed[e] = fmaf(w, x[e], fed[e]);
+            }
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) add[e] += fed[e];
+        } else if (in.b) {
+            read_entries<TD, VEC>((const TD*)in.b + (size_t)s * hidden + i, x);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) add[e] += x[e];
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[c][e] += add[e];
+        if (write_h && (in.a || in.b)) {
+            if constexpr (VEC == 4) store4(hrow + i, v[c]);
+            else hrow[i] = v[c][0];
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) sum = fmaf(v[c][e], v[c][e], sum);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(sum, scratch) / (float)hidden + eps);
+#pragma unroll
+    for (int c = 0; c < CHUNKS; ++c) {
+        const int i = c * step + threadIdx.x * VEC;
+        if (i >= hidden) continue;
+        float o[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) o[e] = v[c][e] * inv * weight1[c][e];
+        if constexpr (VEC == 4) store4(out1 + (size_t)r * hidden + i, o);
+        else out1[(size_t)r * hidden + i] = from_float<TO>(o[0]);
+        if (w2) {
+            float w[VEC];
+            read_entries<float, VEC>(w2 + i, w);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) o[e] = v[c][e] * inv * w[e];
+            if constexpr (VEC == 4) store4(out2 + (size_t)r * hidden + i, o);
+            else out2[(size_t)r * hidden + i] = from_float<TO>(o[0]);
+        }
+    }
+}
+
+// Rows that are no multiple of four entries (or not aligned to them) may have up to 4,096, others up to 16,384; bfloat16 sublayer outputs go with
+// bfloat16 results.
+HB_EXPORT int hb_add_pair_norms(float* h, const void* a, int a_splits, long long a_split_stride, const void* b, const int* slot_of, const float* weights, int top,
+                                int delta_is_bf16, const float* w1, const float* w2, void* out1, void* out2, int out_is_bf16, const int* rows, int n_rows,
+                                int hidden, float eps, int write_h, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (!w1 || !out1 || (w2 && !out2) || (slot_of && (!b || !weights || top <= 0)) || (a_splits > 0 && !a)) return HB_BAD_ARGUMENT;
+    if (hidden <= 0 || hidden > 512 * 32 || (delta_is_bf16 && !out_is_bf16)) return HB_UNSUPPORTED_SIZE;
+    const uintptr_t all = (uintptr_t)h | (uintptr_t)a | (uintptr_t)b | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)out1 | (uintptr_t)out2;
+    const bool by_four = hidden % 4 == 0 && (all & 15) == 0 && (a_split_stride & 3) == 0;
+    const PairInputs in{a, a_splits, (size_t)a_split_stride, b, slot_of, weights, top};
+    const int pieces = by_four ? hidden / 4 : hidden;
+    // the block's size and a thread's share follow from the row alone, so a row's sum has one shape whatever else is in the launch
+    const int threads = pieces <= 128 ? 128 : (pieces <= 512 ? 256 : 512), chunks = (pieces + threads - 1) / threads;
+#define HB_PAIR_LAUNCH(TD, TO, VEC, CHUNKS)                                                                                                                   \
+    return launch_after_previous(add_pair_norms_kernel<TD, TO, VEC, CHUNKS>, dim3(n_rows), dim3(threads), 0, stream, h, in, w1, w2, (TO*)out1, (TO*)out2, rows, \
+                                 hidden, eps, write_h)
+#define HB_PAIR(TD, TO)                                    \
+    if (by_four) {                                         \
+        if (chunks <= 2) HB_PAIR_LAUNCH(TD, TO, 4, 2);     \
+        HB_PAIR_LAUNCH(TD, TO, 4, 8);                      \
+    }                                                      \
+    if (chunks <= 2) HB_PAIR_LAUNCH(TD, TO, 1, 2);         \
+    if (chunks > 8) return HB_UNSUPPORTED_SIZE;            \
+    HB_PAIR_LAUNCH(TD, TO, 1, 8)
+    if (delta_is_bf16 && out_is_bf16) { HB_PAIR(__nv_bfloat16, __nv_bfloat16); }
+    if (out_is_bf16) { HB_PAIR(float, __nv_bfloat16); }
+    HB_PAIR(float, float);
+#undef HB_PAIR
+#undef HB_PAIR_LAUNCH
+}
+
+// ---------------------------------------------------------------- a smooth cap in place
+// x <- cap * tanh(x / cap) over a dense float tensor.
+__global__ void soft_cap_kernel(float* __restrict__ x, float cap, size_t count) {
+    let_next_kernel_start();
+    wait_for_previous_kernels();
+    for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4; i < count; i += (size_t)gridDim.x * blockDim.x * 4) {
+        if (i + 4 <= count) {
+            float v[4];
+            load4(x + i, v);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[e] = cap * tanhf(v[e] / cap);
+            store4(x + i, v);
+        } else {
+            for (size_t j = i; j < count; ++j) x[j] = cap * tanhf(x[j] / cap);
+        }
+    }
+}
+
+HB_EXPORT int hb_soft_cap(float* x, float cap, long long count, cudaStream_t stream) {
+    if (count <= 0) return 0;
+    if (!(cap > 0.f) || ((uintptr_t)x & 15)) return HB_BAD_ARGUMENT;
+    const long long blocks = (count + 1023) / 1024;
+    return launch_after_previous(soft_cap_kernel, dim3((unsigned)(blocks < 8192 ? blocks : 8192)), dim3(256), 0, stream, x, cap, (size_t)count);
+}

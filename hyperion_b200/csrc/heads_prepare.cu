@@ -508,3 +508,134 @@ HB_EXPORT int hb_rotate_heads(void* x, int is_bf16, int tokens, int stride, int 
     else rotate_heads_kernel<<<grid, ROTATE_THREADS, 0, stream>>>((float*)x, stride, col0, heads, head_dim, rot_dims, rot_half, inv_freq, positions, sign);
     return launch_status();
 }
+
+// ---------------------------------------------------------------- heads that nothing rotates
+// Float projections [tokens, stride] with queries at q_off, keys at k_off and values at v_off: an optional bias per column is added, every query
+// and key head passes an optional RMS norm (one weight for all of them), queries go to a dense buffer, keys and values to their pages.
+// A key/value head may hold several keys per token (`maps` of them side by side, each a head of its own to the norm).  A group of lanes
+// serves a head, so a norm's sum has one shape whatever the launch; a lane takes VEC consecutive entries per access.
+namespace {
+constexpr int STORE_THREADS = 256;
+
+template <int VEC>
+__device__ __forceinline__ void fetch_entries(const float* p, const float* bias, float (&v)[VEC]) {
+    if constexpr (VEC == 4) {
+        load4(p, v);
+        if (bias) {
+            float b[4];
+            load4(bias, b);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[e] += b[e];
+        }
+    } else {
+        v[0] = bias ? p[0] + bias[0] : p[0];
+    }
+}
+
+// Heads `part`, `part + parts`, ... of a projection; `place(head)` is where a head goes (null: nowhere).  Every lane of a warp makes the same
+// number of rounds, because the norm's sum crosses lanes.
+template <int VEC, typename TO, typename Place>
+__device__ __forceinline__ void store_heads(const float* all, const float* bias, int heads, int dim, const float* weight, float eps, int lanes, int part, int parts,
+                                            Place place) {
+    const int per_block = STORE_THREADS / lanes, group = threadIdx.x / lanes, lane = threadIdx.x & (lanes - 1);
+    const int groups_per_warp = 32 / lanes, warp_first = (threadIdx.x >> 5) * groups_per_warp;
+    for (int round = 0; round * per_block * parts + part * per_block + warp_first < heads; ++round) {
+        const int head = round * per_block * parts + part * per_block + group;
+        const bool there = head < heads;
+        const float* p = all + (size_t)(there ? head : 0) * dim;
+        const float* b = bias ? bias + (size_t)(there ? head : 0) * dim : nullptr;
+        float inv = 1.f;
+        if (weight) {
+            float sum = 0.f;
+            for (int i = lane * VEC; i < dim; i += lanes * VEC) {
+                float v[VEC];
+                fetch_entries<VEC>(p + i, b ? b + i : nullptr, v);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) sum = fmaf(v[e], v[e], sum);
+            }
+            for (int offset = lanes / 2; offset > 0; offset >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
+            inv = 1.0f / sqrtf(sum / (float)dim + eps);
+        }
+        TO* dst = there ? place(head) : nullptr;
+        if (!dst) continue;
+        for (int i = lane * VEC; i < dim; i += lanes * VEC) {
+            float v[VEC];
+            fetch_entries<VEC>(p + i, b ? b + i : nullptr, v);
+            if (weight) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[e] *= inv * weight[i + e];
+            }
+            if constexpr (VEC == 4) store4(dst + i, v);
+            else dst[i] = from_float<TO>(v[0]);
+        }
+    }
+}
+
+template <int VEC, typename TO>
+__global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float* __restrict__ x, int stride, const float* __restrict__ bias, int q_off, int k_off,
+                                                                    int v_off, int q_heads, int k_heads, int v_heads, int maps, int head_dim, int v_dim,
+                                                                    const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, int lanes,
+                                                                    int v_lanes, const int* __restrict__ positions, TO* __restrict__ q_out, int q_out_stride,
+                                                                    TO* __restrict__ k_cache, TO* __restrict__ v_cache, size_t page_stride, size_t head_stride,
+                                                                    int token_stride, const int* __restrict__ block_table, int table_width,
+                                                                    const int* __restrict__ token_row, int page_size, int pages, int* status) {
+    let_next_kernel_start();
+    wait_for_previous_kernels();
+    const int t = blockIdx.x, part = blockIdx.y, parts = gridDim.y;
+    const float* row = x + (size_t)t * stride;
+    store_heads<VEC, TO>(row + q_off, bias ? bias + q_off : nullptr, q_heads, head_dim, q_norm, eps, lanes, part, parts,
+                         [&](int head) { return q_out + (size_t)t * q_out_stride + (size_t)head * head_dim; });
+    if (!k_cache) return;
+    const int pos = positions[t], block = pos / page_size;
+    int page = (pos >= 0 && block < table_width) ? block_table[(size_t)token_row[t] * table_width + block] : -1;
+    if (page < 0 || page >= pages) {
+        if (threadIdx.x == 0) atomicOr(status, HB_STATUS_BAD_PAGE);
+        page = -1;
+    }
+    const size_t at = page >= 0 ? (size_t)page * page_stride + (size_t)(pos - block * page_size) * token_stride : 0;
+    store_heads<VEC, TO>(row + k_off, bias ? bias + k_off : nullptr, k_heads, head_dim, k_norm, eps, lanes, part, parts, [&](int head) {
+        return page >= 0 ? k_cache + at + (size_t)(head / maps) * head_stride + (size_t)(head % maps) * head_dim : nullptr;
+    });
+    store_heads<VEC, TO>(row + v_off, bias ? bias + v_off : nullptr, v_heads, v_dim, nullptr, 0.f, v_lanes, part, parts,
+                         [&](int head) { return page >= 0 ? v_cache + at + (size_t)head * head_stride : nullptr; });
+}
+
+int lanes_for(int pieces) {
+    int lanes = 1;
+    while (lanes < pieces && lanes < 32) lanes *= 2;
+    return lanes;
+}
+}  // namespace
+
+// q_heads and k_heads count every map; k_cache null: queries only.  A key head h goes to the key/value head h / maps, its map h % maps.
+HB_EXPORT int hb_heads_store(const float* x, int tokens, int stride, const float* bias, int q_off, int k_off, int v_off, int q_heads, int k_heads, int v_heads,
+                             int maps, int head_dim, int v_dim, const float* q_norm, const float* k_norm, float eps, const int* positions, void* q_out,
+                             int q_out_stride, int out_is_bf16, void* k_cache, void* v_cache, long long page_stride, long long head_stride, int token_stride,
+                             const int* block_table, int table_width, const int* token_row, int page_size, int pages, int* status, cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (head_dim <= 0 || v_dim <= 0 || q_heads <= 0 || !q_out || maps < 1) return HB_UNSUPPORTED_SIZE;
+    if (k_cache && (k_heads <= 0 || v_heads <= 0 || k_heads != v_heads * maps || !v_cache || page_size <= 0)) return HB_BAD_ARGUMENT;
+    const uintptr_t store_mask = out_is_bf16 ? 7 : 15;
+    bool by_four = ((stride | q_off | head_dim | q_out_stride) & 3) == 0 && (((uintptr_t)x | (uintptr_t)bias) & 15) == 0 && ((uintptr_t)q_out & store_mask) == 0;
+    if (k_cache)
+        by_four = by_four && ((k_off | v_off | v_dim | token_stride) & 3) == 0 && ((page_stride | head_stride) & 3) == 0 &&
+                  (((uintptr_t)k_cache | (uintptr_t)v_cache) & store_mask) == 0;
+    const int vec = by_four ? 4 : 1, lanes = lanes_for((head_dim + vec - 1) / vec), v_lanes = lanes_for((v_dim + vec - 1) / vec);
+    const int most = q_heads > k_heads ? q_heads : k_heads, rounds = (most * lanes + STORE_THREADS - 1) / STORE_THREADS;
+    int parts = tokens >= 512 ? 1 : 512 / tokens;  // few tokens: a token's heads over several blocks
+    parts = parts > rounds ? rounds : parts;
+    parts = parts < 1 ? 1 : (parts > 1024 ? 1024 : parts);
+    const dim3 grid(tokens, parts);
+#define HB_STORE(VEC, TO)                                                                                                                                     \
+    return launch_after_previous(heads_store_kernel<VEC, TO>, grid, dim3(STORE_THREADS), 0, stream, x, stride, bias, q_off, k_off, v_off, q_heads, k_heads,    \
+                                 v_heads, maps, head_dim, v_dim, q_norm, k_norm, eps, lanes, v_lanes, positions, (TO*)q_out, q_out_stride, (TO*)k_cache,       \
+                                 (TO*)v_cache, (size_t)page_stride, (size_t)head_stride, token_stride, block_table, table_width, token_row, page_size, pages,  \
+                                 status)
+    if (out_is_bf16) {
+        if (by_four) HB_STORE(4, __nv_bfloat16);
+        HB_STORE(1, __nv_bfloat16);
+    }
+    if (by_four) HB_STORE(4, float);
+    HB_STORE(1, float);
+#undef HB_STORE
+}

@@ -65,10 +65,11 @@ HB_API int hb_pool_check(const HbPool* pool) {
 }
 
 // ---------------------------------------------------------------- cache index
-HB_API int hb_cache_new(int page_size, int num_pages, int max_requests, int n_groups, const int* windows, HbCache** out) {
+HB_API int hb_cache_new(int page_size, int num_pages, int max_requests, int n_groups, const int* windows, const int* keeps, HbCache** out) {
     return guarded([&] {
         require(n_groups >= 0, "the number of groups must not be negative");
-        *out = new HbCache{hb::CacheIndex(page_size, num_pages, max_requests, std::vector<int>(windows, windows + n_groups))};
+        *out = new HbCache{hb::CacheIndex(page_size, num_pages, max_requests, std::vector<int>(windows, windows + n_groups),
+                                          keeps ? std::vector<int>(keeps, keeps + n_groups) : std::vector<int>())};
     });
 }
 HB_API void hb_cache_delete(HbCache* cache) { delete cache; }
@@ -148,8 +149,8 @@ HB_API int hb_cache_lengths(const HbCache* cache, int n, const int64_t* keys, in
 HB_API int hb_cache_check(const HbCache* cache) {
     return guarded([&] { cache->index.check(); });
 }
-HB_API int hb_cache_worst_case_pages(int page_size, int window, int tokens, int largest_portion, int* pages) {
-    return guarded([&] { *pages = hb::CacheIndex::worst_case_pages(page_size, window, tokens, largest_portion); });
+HB_API int hb_cache_worst_case_pages(int page_size, int window, int keep, int tokens, int largest_portion, int* pages) {
+    return guarded([&] { *pages = hb::CacheIndex::worst_case_pages(page_size, window, tokens, largest_portion, keep); });
 }
 
 // ---------------------------------------------------------------- step assembly
@@ -275,13 +276,14 @@ HB_API int hb_plan_attention(int n_rows, const int* counts, int tokens_per_tile,
 }
 
 // ---------------------------------------------------------------- scheduler
-HB_API int hb_sched_new(int num_pages, int page_size, int n_groups, const int* group_windows, int max_seq_len, int max_batch, int max_batch_tokens,
-                        int prefill_chunk_busy, int max_queue, int max_in_flight, int n_eos, const int* eos, HbScheduler** out) {
+HB_API int hb_sched_new(int num_pages, int page_size, int n_groups, const int* group_windows, const int* group_keeps, int max_seq_len, int max_batch,
+                        int max_batch_tokens, int prefill_chunk_busy, int max_queue, int max_in_flight, int n_eos, const int* eos, HbScheduler** out) {
     return guarded([&] {
         if (n_groups < 0) throw hb::Failure{hb::BAD_ARGUMENT, "n_groups must not be negative"};
         hb::SchedulerConfig config;
         config.num_pages = num_pages;
         config.group_windows.assign(group_windows, group_windows + n_groups);
+        if (group_keeps) config.group_keeps.assign(group_keeps, group_keeps + n_groups);
         config.page_size = page_size;
         config.max_seq_len = max_seq_len;
         config.max_batch = max_batch;

@@ -37,11 +37,14 @@ void PagePool::check() const {
     if (held != held_count_ || (int)free_.size() + held != num_pages()) throw Failure{CACHE_ERROR, "page accounting broken"};
 }
 
-CacheIndex::CacheIndex(int page_size, int num_pages, int max_requests, std::vector<int> windows)
-    : page_size_(page_size), max_requests_(max_requests), windows_(std::move(windows)) {
+CacheIndex::CacheIndex(int page_size, int num_pages, int max_requests, std::vector<int> windows, std::vector<int> keeps)
+    : page_size_(page_size), max_requests_(max_requests), windows_(std::move(windows)), keeps_(std::move(keeps)) {
     if (page_size <= 0 || (page_size & (page_size - 1)))
         throw Failure{BAD_ARGUMENT, "page_size must be a power of two, got " + std::to_string(page_size)};
     if (max_requests < 0) throw Failure{BAD_ARGUMENT, "max_requests must not be negative"};
+    keeps_.resize(windows_.size(), 0);
+    for (int keep : keeps_)
+        if (keep < 0) throw Failure{BAD_ARGUMENT, "the number of first positions a group keeps must not be negative"};
     for (size_t g = 0; g < windows_.size(); ++g) pools_.emplace_back(num_pages);
     for (int slot = 0; slot < max_requests; ++slot) free_slots_.push_back(slot);
 }
@@ -83,14 +86,14 @@ int CacheIndex::first_needed_block(int group, int length) const {
     return std::max(0, length - window + 1) / page_size_;
 }
 
-int CacheIndex::worst_case_pages(int page_size, int window, int tokens, int largest_portion) {
-    if (page_size < 1 || window < 0 || tokens < 0 || largest_portion < 1) throw Failure{BAD_ARGUMENT, "worst_case_pages: bad sizes"};
+int CacheIndex::worst_case_pages(int page_size, int window, int tokens, int largest_portion, int keep) {
+    if (page_size < 1 || window < 0 || tokens < 0 || largest_portion < 1 || keep < 0) throw Failure{BAD_ARGUMENT, "worst_case_pages: bad sizes"};
     const long long all = ((long long)tokens + page_size - 1) / page_size;
     if (window == 0) return (int)all;
     // before a step the table holds blocks from first_needed_block(length) on; the step adds blocks up to its last token:
     // ceil((a + window - 1 + n) / page) - floor(a / page) <= ceil((window + n - 1) / page) + 1 for every start a
     const long long spanned = ((long long)window + largest_portion - 1 + page_size - 1) / page_size + 1;
-    return (int)std::min(all, spanned);
+    return (int)std::min(all, spanned + ((long long)keep + page_size - 1) / page_size);
 }
 
 void CacheIndex::pages_needed(int64_t key, int new_tokens, int* out) const {
@@ -125,7 +128,7 @@ void CacheIndex::advance(int64_t key, int new_tokens, std::vector<std::pair<int,
     for (int g = 0; g < groups(); ++g) {
         std::vector<int>& table = r.tables[g];
         const int passed = std::min(first_needed_block(g, r.length), (int)table.size());
-        for (int block = 0; block < passed; ++block) {
+        for (int block = (keeps_[g] + page_size_ - 1) / page_size_; block < passed; ++block) {  // the blocks of the first positions stay
             if (table[block] == NO_PAGE) continue;
             pools_[g].give_back(table[block]);
             if (released) released->emplace_back(g, table[block]);

@@ -58,8 +58,9 @@ struct RequestRecord {
 
 class CacheIndex {
   public:
-    // windows[g] > 0: group g only ever reads the last windows[g] positions.
-    CacheIndex(int page_size, int num_pages, int max_requests, std::vector<int> windows);
+    // windows[g] > 0: group g only ever reads the last windows[g] positions and the first keeps[g] of the sequence (a missing
+    // entry of keeps is 0; a group that keeps every key has no use for one).
+    CacheIndex(int page_size, int num_pages, int max_requests, std::vector<int> windows, std::vector<int> keeps = {});
 
     int page_size() const { return page_size_; }
     int groups() const { return (int)pools_.size(); }
@@ -81,15 +82,15 @@ class CacheIndex {
 
     // The most pages of one group that a request of up to `tokens` tokens can hold at any moment, when no step brings it
     // more than `largest_portion` tokens: all its blocks for a group that keeps every key (window 0), else the blocks
-    // that the window behind the next position and one portion ahead of it can touch.
-    static int worst_case_pages(int page_size, int window, int tokens, int largest_portion);
+    // that the window behind the next position and one portion ahead of it can touch, plus those of the first `keep` positions.
+    static int worst_case_pages(int page_size, int window, int tokens, int largest_portion, int keep = 0);
 
   private:
     RequestRecord& mutable_record(int64_t key);
     int first_needed_block(int group, int length) const;
 
     int page_size_, max_requests_;
-    std::vector<int> windows_;
+    std::vector<int> windows_, keeps_;
     std::vector<PagePool> pools_;
     std::unordered_map<int64_t, RequestRecord> requests_;
     std::vector<int64_t> order_;  // live requests, oldest first

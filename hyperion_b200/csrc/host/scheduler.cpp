@@ -10,6 +10,7 @@ Scheduler::Scheduler(SchedulerConfig config) : config_(std::move(config)) {
     if (config_.page_size < 1 || config_.max_in_flight < 1) throw Failure{BAD_ARGUMENT, "page_size and max_in_flight must be at least 1"};
     for (int window : config_.group_windows)
         if (window < 0) throw Failure{BAD_ARGUMENT, "a group's window must not be negative"};
+    config_.group_keeps.resize(config_.group_windows.size(), 0);
 }
 
 void Scheduler::enqueue(int64_t key, std::vector<int> prompt, int max_tokens, bool ignore_eos) {
@@ -59,7 +60,7 @@ void Scheduler::admit() {
         int most = 0;
         bool fits = true;
         for (size_t g = 0; g < groups; ++g) {
-            need[g] = CacheIndex::worst_case_pages(c.page_size, c.group_windows[g], tokens, portion);
+            need[g] = CacheIndex::worst_case_pages(c.page_size, c.group_windows[g], tokens, portion, c.group_keeps[g]);
             most = std::max(most, need[g]);
             fits = fits && reserved[g] + need[g] <= c.num_pages;
         }

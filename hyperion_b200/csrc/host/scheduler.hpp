@@ -31,6 +31,7 @@ struct SchedulerConfig {
     int num_pages = 0;             // pages in the pool of every paged group
     int page_size = 1;
     std::vector<int> group_windows{0};  // one entry per paged group of the cache: 0 = keeps every key, else its window
+    std::vector<int> group_keeps;       // per group the first positions a windowed group keeps beside its window (empty: none)
     int max_seq_len = 0;
     int max_batch = 64;            // most requests live at a time
     int max_batch_tokens = 2048;   // token budget of one step

@@ -19,6 +19,10 @@
 //                      best c can be chosen; the `top` largest c; weight = s * scale
 //   plan:              a choice >= experts takes no slot (slot_of = -1); without weights every slot's weight is 1
 //   combine_weighted:  out[token] = sigmoid(gate[token]) * base[token] + sum over choices of w * (y[slot] or, without a slot, x[token])
+//
+// A third router adds a bias to the logits, chooses by them and weighs the chosen by a softmax over the chosen alone:
+//   route_softmax:     z = W_r x + b; the `top` largest z; weight = exp(z) / sum over the chosen of exp(z)
+// A product may apply the experts' activation to what it stores (`act`, see activated() in common.cuh).
 #include "common.cuh"
 
 namespace {
@@ -163,6 +167,97 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_scored_kernel(const T
     }
 }
 
+// Softmax over the chosen logits alone.  A block serves TOKENS tokens, so that a prompt-sized step reads the router's matrix once per TOKENS
+// tokens; a logit is summed in the same order whatever TOKENS is.  Warp j then searches and weighs token j.
+template <typename T, int TOKENS>
+__global__ void __launch_bounds__(ROUTE_THREADS) moe_route_softmax_kernel(const T* __restrict__ x, int x_stride, const float* __restrict__ router,
+                                                                          const float* __restrict__ bias, int tokens, int hidden, int experts, int top,
+                                                                          int* __restrict__ chosen, float* __restrict__ weights) {
+    static_assert(TOKENS <= ROUTE_THREADS / 32, "a warp per token");
+    extern __shared__ __align__(16) float shared[];  // TOKENS rows, then per token: a logit per expert, the chosen logits
+    const int padded = (hidden + 3) & ~3;
+    float* logits = shared + (size_t)TOKENS * padded;
+    float* picked = logits + TOKENS * experts;
+    const int first = blockIdx.x * TOKENS, count = min(TOKENS, tokens - first), lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    let_next_kernel_start();
+    wait_for_previous_kernels();
+    const bool rows_by_four = (hidden & 3) == 0 && (x_stride & 3) == 0 && (((uintptr_t)x) & (4 * sizeof(T) - 1)) == 0;
+    for (int j = 0; j < TOKENS; ++j) {
+        float* row = shared + (size_t)j * padded;
+        const T* from = x + (size_t)(first + min(j, count - 1)) * x_stride;
+        if (rows_by_four) {
+            for (int i = threadIdx.x * 4; i < hidden; i += ROUTE_THREADS * 4) {
+                float v[4];
+                load4(from + i, v);
+                store4(row + i, v);
+            }
+        } else {
+            for (int i = threadIdx.x; i < padded; i += ROUTE_THREADS) row[i] = i < hidden ? to_float(from[i]) : 0.f;
+        }
+    }
+    __syncthreads();
+    const bool by_four = (hidden & 3) == 0 && (((uintptr_t)router) & 15) == 0;
+    for (int e = warp; e < experts; e += ROUTE_THREADS / 32) {
+        const float* w = router + (size_t)e * hidden;
+        float part[TOKENS][4];
+#pragma unroll
+        for (int j = 0; j < TOKENS; ++j) part[j][0] = part[j][1] = part[j][2] = part[j][3] = 0.f;
+        if (by_four) {
+#pragma unroll 4
+            for (int i = lane * 4; i < hidden; i += 128) {
+                const float4 wv = *reinterpret_cast<const float4*>(w + i);
+#pragma unroll
+                for (int j = 0; j < TOKENS; ++j) {
+                    const float4 rv = *reinterpret_cast<const float4*>(shared + (size_t)j * padded + i);
+                    part[j][0] = fmaf(rv.x, wv.x, part[j][0]); part[j][1] = fmaf(rv.y, wv.y, part[j][1]);
+                    part[j][2] = fmaf(rv.z, wv.z, part[j][2]); part[j][3] = fmaf(rv.w, wv.w, part[j][3]);
+                }
+            }
+        } else {
+            for (int i = lane * 4; i < hidden; i += 128)
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+                    if (i + c < hidden)
+#pragma unroll
+                        for (int j = 0; j < TOKENS; ++j) part[j][c] = fmaf(shared[(size_t)j * padded + i + c], w[i + c], part[j][c]);
+        }
+        const float b = bias ? bias[e] : 0.f;
+#pragma unroll
+        for (int j = 0; j < TOKENS; ++j) {
+            const float sum = warp_sum((part[j][0] + part[j][1]) + (part[j][2] + part[j][3]));
+            if (lane == 0) logits[j * experts + e] = sum + b;
+        }
+    }
+    __syncthreads();
+    if (warp >= count) return;
+    float* z = logits + warp * experts;
+    float* mine = picked + warp * top;
+    const size_t t = first + warp;
+    for (int k = 0; k < top; ++k) {
+        float value = -INFINITY;
+        int index = 0x7fffffff;
+        for (int e = lane; e < experts; e += 32)
+            if (z[e] > value) { value = z[e]; index = e; }
+        warp_best(value, index);
+        if (index == 0x7fffffff) {  // only when every logit left is minus infinity or not a number: a place is filled without weight
+            index = 0;
+            value = -INFINITY;
+        }
+        __syncwarp();
+        if (lane == 0) {
+            chosen[t * top + k] = index;
+            mine[k] = value;
+            z[index] = -INFINITY;
+        }
+        __syncwarp();
+    }
+    const float most = mine[0];
+    float sum = 0.f;
+    for (int k = lane; k < top; k += 32) sum += expf(mine[k] - most);
+    sum = warp_sum(sum);
+    for (int k = lane; k < top; k += 32) weights[t * top + k] = expf(mine[k] - most) / sum;
+}
+
 constexpr int PLAN_THREADS = 1024;
 
 // One block.  counts and cursors live in shared memory (experts <= 1024).
@@ -219,7 +314,7 @@ constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
 
 template <typename T>
 __global__ void __launch_bounds__(256) moe_gemm_kernel(const T* __restrict__ a, const T* __restrict__ w, T* __restrict__ c, const int* __restrict__ tile_expert,
-                                                       int pad, int n, int k) {
+                                                       int pad, int n, int k, int act) {
     __shared__ float as[BK][BM + 4];
     __shared__ float ws[BK][BN + 4];
     const int tid = threadIdx.x;
@@ -263,7 +358,7 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(const T* __restrict__ a, 
 #pragma unroll
         for (int j = 0; j < TN; ++j) {
             const int col = col0 + tx * TN + j;
-            if (col < n) c[(size_t)r * n + col] = from_float<T>(acc[i][j]);
+            if (col < n) c[(size_t)r * n + col] = from_float<T>(activated(acc[i][j], act));
         }
     }
 }
@@ -430,6 +525,29 @@ HB_EXPORT int hb_moe_route(const void* x, int is_bf16, int x_stride, const float
     return launch_status();
 }
 
+HB_EXPORT int hb_moe_route_softmax(const void* x, int is_bf16, int x_stride, const float* router, const float* bias, int tokens, int hidden, int experts,
+                                   int top, int* chosen, float* weights, cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (experts <= 0 || experts > 1024 || top <= 0 || top > experts || hidden <= 0) return HB_UNSUPPORTED_SIZE;
+    auto bytes = [&](int at_once) { return (size_t)at_once * (((hidden + 3) & ~3) + experts + top) * sizeof(float); };
+    const int at_once = tokens >= 512 && bytes(4) <= 100 * 1024 ? 4 : 1;  // a step of few tokens fills more of the device with a token per block
+    const size_t shared = bytes(at_once);
+    if (shared > 200 * 1024) return HB_UNSUPPORTED_SIZE;
+#define HB_ROUTE(T, N)                                                                                                                                  \
+    {                                                                                                                                                   \
+        if (shared > 48 * 1024) cudaFuncSetAttribute(moe_route_softmax_kernel<T, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared);          \
+        return launch_after_previous(moe_route_softmax_kernel<T, N>, dim3((tokens + N - 1) / N), dim3(ROUTE_THREADS), shared, stream, (const T*)x, x_stride, \
+                                     router, bias, tokens, hidden, experts, top, chosen, weights);                                                      \
+    }
+    if (is_bf16) {
+        if (at_once == 4) HB_ROUTE(__nv_bfloat16, 4);
+        HB_ROUTE(__nv_bfloat16, 1);
+    }
+    if (at_once == 4) HB_ROUTE(float, 4);
+    HB_ROUTE(float, 1);
+#undef HB_ROUTE
+}
+
 // capacity: a multiple of pad, at least pairs + experts * (pad - 1) rounded up to it.  tile_expert and tile_rows (the real rows at the start
 // of a tile) have capacity / pad entries.
 HB_EXPORT int hb_moe_plan(const int* chosen, const float* weights, int pairs, int top, int experts, int pad, int capacity, int* slot_of,
@@ -456,14 +574,14 @@ HB_EXPORT int hb_moe_gather(const void* x, int is_bf16, int x_stride, const int*
 }
 
 // a [capacity, k] and c [capacity, n] dense, w [experts, n, k] dense; pad a multiple of 64.
-HB_EXPORT int hb_moe_gemm(const void* a, const void* w, void* c, int is_bf16, const int* tile_expert, int pad, int capacity, int n, int k,
+HB_EXPORT int hb_moe_gemm(const void* a, const void* w, void* c, int is_bf16, const int* tile_expert, int pad, int capacity, int n, int k, int act,
                           cudaStream_t stream) {
     if (capacity <= 0 || n <= 0) return 0;
     if (k <= 0 || pad % BM || capacity % pad) return HB_BAD_ARGUMENT;
     const dim3 grid((n + BN - 1) / BN, capacity / BM);
     if (grid.y > 65535) return HB_UNSUPPORTED_SIZE;
-    if (is_bf16) moe_gemm_kernel<<<grid, 256, 0, stream>>>((const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (__nv_bfloat16*)c, tile_expert, pad, n, k);
-    else moe_gemm_kernel<<<grid, 256, 0, stream>>>((const float*)a, (const float*)w, (float*)c, tile_expert, pad, n, k);
+    if (is_bf16) moe_gemm_kernel<<<grid, 256, 0, stream>>>((const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (__nv_bfloat16*)c, tile_expert, pad, n, k, act);
+    else moe_gemm_kernel<<<grid, 256, 0, stream>>>((const float*)a, (const float*)w, (float*)c, tile_expert, pad, n, k, act);
     return launch_status();
 }
 

@@ -31,6 +31,7 @@ struct GroupedParams {
     bf16* c;                 // [rows, n]
     const int* tile_expert;  // [tiles_m]
     int rows, n, k, ldc;     // n: columns per expert
+    int act;                 // what is applied to an accumulator before its one rounding (activated() in common.cuh)
     int* status;
 };
 
@@ -40,6 +41,10 @@ __device__ __forceinline__ void store_grouped_row(const GroupedParams& p, unsign
     for (int c = 0; c < BN; c += 16) {
         float v[16];
         tmem_ld16(lane_addr + c, v);
+        if (p.act != HB_ACT_NONE) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = activated(v[j], p.act);
+        }
         const int col = col0 + c;
         if (r < p.rows && col < p.n) {
             bf16* dst = p.c + (size_t)r * p.ldc + col;
@@ -182,7 +187,7 @@ constexpr int ROWS_AT_ONCE = 8, COLUMNS_PER_BLOCK = 32, ROWS_THREADS = 256;
 
 __global__ void __launch_bounds__(ROWS_THREADS) gemm_grouped_rows_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, bf16* __restrict__ c,
                                                                          const int* __restrict__ tile_expert, const int* __restrict__ tile_rows, int pad,
-                                                                         int n, int k) {
+                                                                         int n, int k, int act) {
     extern __shared__ __align__(16) unsigned char rows_raw[];
     bf16* rows = reinterpret_cast<bf16*>(rows_raw);  // [ROWS_AT_ONCE, k]
     let_next_kernel_start();
@@ -236,7 +241,7 @@ __global__ void __launch_bounds__(ROWS_THREADS) gemm_grouped_rows_kernel(const b
 #pragma unroll
                 for (int r = 1; r < ROWS_AT_ONCE; ++r)
                     if (lane == r) mine = sum[r];
-                c[(size_t)(tile * pad + first + lane) * n + col] = __float2bfloat16_rn(mine);
+                c[(size_t)(tile * pad + first + lane) * n + col] = __float2bfloat16_rn(activated(mine, act));
             }
         }
     }
@@ -244,8 +249,8 @@ __global__ void __launch_bounds__(ROWS_THREADS) gemm_grouped_rows_kernel(const b
 }  // namespace
 
 // a [rows, k] and c [rows, n] dense bfloat16 (rows a multiple of 128), w [experts, n, k] dense bfloat16, k a multiple of 8.
-HB_EXPORT int hb_moe_gemm_tiles(const void* a, const void* w, void* c, const int* tile_expert, int rows, int experts, int n, int k, int* status,
-                                cudaStream_t stream) {
+HB_EXPORT int hb_moe_gemm_tiles(const void* a, const void* w, void* c, const int* tile_expert, int rows, int experts, int n, int k, int act,
+                                int* status, cudaStream_t stream) {
     if (rows <= 0 || n <= 0) return 0;
     if (k <= 0 || rows % BM || experts <= 0 || (k % 8) || !tile_expert) return HB_BAD_ARGUMENT;
     if ((long long)experts * n > 0x7fffffffLL) return HB_UNSUPPORTED_SIZE;
@@ -256,14 +261,14 @@ HB_EXPORT int hb_moe_gemm_tiles(const void* a, const void* w, void* c, const int
     const int tiles_m = rows / BM, tiles_n = (n + bn - 1) / bn;
     if ((long long)tiles_m * tiles_n > 0x7fffffffLL) return HB_UNSUPPORTED_SIZE;
     const int blocks = min(tiles_m * tiles_n, sm_count());
-    const GroupedParams p{(bf16*)c, tile_expert, rows, n, k, n, status};
+    const GroupedParams p{(bf16*)c, tile_expert, rows, n, k, n, act, status};
     return bn == 256 ? launch_grouped<256>(map_x, map_w, p, tiles_m, tiles_n, blocks, stream)
                      : launch_grouped<128>(map_x, map_w, p, tiles_m, tiles_n, blocks, stream);
 }
 
 // The same product for steps of a few rows; tile_rows[i]: the real rows at the start of tile i.
 HB_EXPORT int hb_moe_gemm_rows(const void* a, const void* w, void* c, const int* tile_expert, const int* tile_rows, int pad, int rows, int n, int k,
-                               cudaStream_t stream) {
+                               int act, cudaStream_t stream) {
     if (rows <= 0 || n <= 0) return 0;
     if (k <= 0 || pad <= 0 || rows % pad || (k % 8) || !tile_expert || !tile_rows) return HB_BAD_ARGUMENT;
     if ((((uintptr_t)a | (uintptr_t)w) & 15)) return HB_BAD_ARGUMENT;
@@ -277,5 +282,5 @@ HB_EXPORT int hb_moe_gemm_rows(const void* a, const void* w, void* c, const int*
     }
     const dim3 grid((n + COLUMNS_PER_BLOCK - 1) / COLUMNS_PER_BLOCK, rows / pad);
     return launch_after_previous(gemm_grouped_rows_kernel, grid, dim3(ROWS_THREADS), shared, stream, (const bf16*)a, (const bf16*)w, (bf16*)c, tile_expert,
-                                 tile_rows, pad, n, k);
+                                 tile_rows, pad, n, k, act);
 }

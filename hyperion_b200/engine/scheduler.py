@@ -67,6 +67,7 @@ class SchedulerConfig:
     # one entry per paged group of the cache, 0 = the group keeps every key, else its window; pages are reserved per
     # group (a windowed group costs what its window and one portion span, a model without paged groups nothing)
     group_windows: tuple[int, ...] = (0,)
+    group_keeps: tuple[int, ...] = ()  # per group the first positions a windowed group keeps beside its window (empty: none)
 
 
 @dataclass
@@ -113,7 +114,11 @@ class Scheduler:
         self._handle = ctypes.c_void_p()
         eos = host.ints(list(config.eos_token_ids))
         windows = host.ints(list(config.group_windows))
-        host.check(self._lib.hb_sched_new(config.num_pages, config.page_size, len(windows), host.address(windows), config.max_seq_len, config.max_batch,
+        if config.group_keeps and len(config.group_keeps) != len(config.group_windows):
+            raise ValueError("group_keeps has one entry per paged group, like group_windows")
+        keeps = host.ints(list(config.group_keeps)) if config.group_keeps else None
+        host.check(self._lib.hb_sched_new(config.num_pages, config.page_size, len(windows), host.address(windows),
+                                          host.address(keeps) if keeps is not None else None, config.max_seq_len, config.max_batch,
                                           config.max_batch_tokens,
                                           config.prefill_chunk_busy, config.max_queue, config.max_in_flight, len(eos), host.address(eos),
                                           ctypes.byref(self._handle)))

@@ -39,6 +39,21 @@ def _entry(head_dim: int, page_size: int, shape: str):
     return getattr(library("attention_bf16", HB_HEAD_DIM=head_dim), f"hb_attention_{shape}_capped")
 
 
+def _plain_vector(t, heads: int, what: str):
+    if t is not None and (t.dtype != torch.float32 or t.numel() != heads or not t.is_contiguous()):
+        raise KernelError(f"attention: {what} are a dense float32 vector with one entry per head")
+
+
+def _gate_arguments(gate, tokens: int, columns: int):
+    """(pointer, row stride) of a float gate [tokens, >= columns]; a view of some columns of a wider matrix is fine."""
+    if gate is None:
+        return ptr(None), i32(0)
+    require_cuda(gate)
+    if gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1 or gate.shape[0] != tokens or gate.shape[1] < columns:
+        raise KernelError(f"attention: the gate is a float32 matrix [tokens, {columns}] with unit inner stride")
+    return ptr(gate), i32(gate.stride(0))
+
+
 def takes_distance_bias(head_dim: int, page_size: int) -> bool:
     """A bias per head and distance on the scores is an argument of the TMA-fed kernels and of the tcgen05 kernel."""
     return uses_tma(head_dim, page_size)
@@ -109,13 +124,36 @@ def _common(q, out, cache, block_table, token_row, positions):
 
 
 def attention_tiles(q, heads, cache, block_table, token_row, positions, tiles, n_tiles, scale, window, out, tile_size: int = TILE_ROWS,
-                    softcap: float = 0.0, bias=None, bias_per_position=None):
+                    softcap: float = 0.0, bias=None, bias_per_position=None, keep_first: int = 0, sinks=None, gate=None):
     """``tile_size``: the virtual rows per tile the tiles were planned for (64, or 256 for the tcgen05 kernel).
     ``softcap`` > 0: scores become cap * tanh(score / cap) before the softmax.  ``bias`` [heads, span] float, times log2(e):
     the score of a key n positions back takes ``bias[head, min(n, span - 1)]``.  ``bias_per_position`` [heads] float, times log2(e):
-    where the bias is n times a number per head, the tcgen05 kernel computes it instead of looking it up (the others take ``bias``)."""
+    where the bias is n times a number per head, the tcgen05 kernel computes it instead of looking it up (the others take ``bias``).  ``keep_first``: that many
+    first positions of the sequence are seen beside the window; ``sinks`` [heads] float: one more term exp(sink) in each softmax's denominator;
+    ``gate`` [tokens, heads] float: a head's result takes sigmoid(gate).  These three do not go together with a bias."""
     _common(q, out, cache, block_table, token_row, positions)
     pages, _, kv_heads, page_size, head_dim = cache.shape
+    if keep_first or sinks is not None or gate is not None:
+        if bias is not None or bias_per_position is not None:
+            raise KernelError("attention: a distance bias does not go together with kept first tokens, sinks or a gate")
+        require_cuda(sinks)
+        _plain_vector(sinks, heads, "sinks")
+        gate_ptr, gate_stride = _gate_arguments(gate, q.shape[0], heads)
+        extras = (i32(keep_first), ptr(sinks), gate_ptr, gate_stride, i32(1))
+        common = (ptr(q), i32(q.stride(0)), ptr(out), i32(out.stride(0)), ptr(cache), ptr(block_table), i32(block_table.shape[1]), ptr(token_row), ptr(positions),
+                  ptr(tiles), i32(n_tiles))
+        sizes = (i32(heads), i32(kv_heads), i32(head_dim), i32(page_size), i32(pages), f32(scale), f32(softcap or 0.0), i32(window or 0))
+        if uses_tcgen05(head_dim, page_size) and tile_size == TC_TILE_ROWS:
+            check(library("attention_tcgen05", HB_HEAD_DIM=head_dim).hb_attention_tc_tiles_extended(
+                *common, i32(q.shape[0]), *sizes, ptr(None), i32(0), *extras, f32(0.0), f32(0.0), f32(0.0), ptr(status_word(q.device)),
+                ptr(work_counters(q.device)), stream_ptr()), "attention_tiles")
+        elif uses_tma(head_dim, page_size):
+            check(library("attention_tma", HB_HEAD_DIM=head_dim).hb_attention_tma_tiles_extended(
+                *common, *sizes, ptr(None), i32(0), *extras, ptr(status_word(q.device)), stream_ptr()), "attention_tiles")
+        else:
+            check(library("attention_bf16", HB_HEAD_DIM=head_dim).hb_attention_tiles_extended(*common, *sizes, *extras, ptr(status_word(q.device)), stream_ptr()),
+                  "attention_tiles")
+        return
     if bias_per_position is not None and uses_tcgen05(head_dim, page_size) and tile_size == TC_TILE_ROWS:
         require_cuda(bias_per_position)
         if bias_per_position.dtype != torch.float32 or bias_per_position.numel() != heads or not bias_per_position.is_contiguous():
@@ -155,7 +193,8 @@ def attention_tiles(q, heads, cache, block_table, token_row, positions, tiles, n
 
 
 def attention_tokens(q, heads, cache, block_table, token_row, positions, items, n_items, splits, scale, window, out, workspace=None,
-                     softcap: float = 0.0, bias=None):
+                     softcap: float = 0.0, bias=None, keep_first: int = 0, sinks=None, gate=None):
+    """The token shape; ``keep_first``, ``sinks`` and ``gate`` as for :func:`attention_tiles`."""
     _common(q, out, cache, block_table, token_row, positions)
     pages, _, kv_heads, page_size, head_dim = cache.shape
     if splits > 1:
@@ -164,7 +203,15 @@ def attention_tokens(q, heads, cache, block_table, token_row, positions, items, 
             workspace = torch.empty(need, dtype=torch.float32, device=q.device)
         elif workspace.numel() < need or workspace.dtype != torch.float32:
             raise KernelError(f"attention_tokens: workspace of {need} floats needed")
-    if bias is not None:
+    if keep_first or sinks is not None or gate is not None:
+        if bias is not None:
+            raise KernelError("attention: a distance bias does not go together with kept first tokens, sinks or a gate")
+        require_cuda(sinks)
+        _plain_vector(sinks, heads, "sinks")
+        gate_ptr, gate_stride = _gate_arguments(gate, q.shape[0], heads)
+        _tokens_extended(q, out, cache, block_table, token_row, positions, items, n_items, splits, workspace, heads, scale, softcap, window,
+                         (i32(keep_first), ptr(sinks), gate_ptr, gate_stride, i32(1)))
+    elif bias is not None:
         require_cuda(bias)
         bias_ptr, span = _bias_arguments(bias, heads, head_dim, page_size)
         check(library("attention_tma", HB_HEAD_DIM=head_dim).hb_attention_tma_tokens_biased(
@@ -180,6 +227,86 @@ def attention_tokens(q, heads, cache, block_table, token_row, positions, items, 
         from . import native
 
         native.LAUNCHES[0] += 1  # the merge kernel
+
+
+def _tokens_extended(q, out, cache, block_table, token_row, positions, items, n_items, splits, workspace, heads, scale, softcap, window, extras):
+    pages, _, kv_heads, page_size, head_dim = cache.shape
+    tma = uses_tma(head_dim, page_size)
+    entry = (library("attention_tma", HB_HEAD_DIM=head_dim).hb_attention_tma_tokens_extended if tma
+             else library("attention_bf16", HB_HEAD_DIM=head_dim).hb_attention_tokens_extended)
+    check(entry(ptr(q), i32(q.stride(0)), ptr(out), i32(out.stride(0) if out is not None else 0), ptr(cache), ptr(block_table), i32(block_table.shape[1]), ptr(token_row), ptr(positions),
+                ptr(items), i32(n_items), i32(splits), ptr(workspace), i32(heads), i32(kv_heads), i32(head_dim), i32(page_size), i32(pages), f32(scale),
+                f32(softcap or 0.0), i32(window or 0), *((ptr(None), i32(0)) if tma else ()), *extras, ptr(status_word(q.device)), stream_ptr()), "attention_tokens")
+
+
+# ------------------------------------------------------------------ two softmax maps per head over the same values
+def differential_supported(head_dim: int, value_dim: int) -> bool:
+    """Shapes the tensor-core kernels take: a head's two keys fill a row as wide as its value (a multiple of 16 up to 256)."""
+    return 2 * head_dim == value_dim and supported(value_dim)
+
+
+def fuses_differential(value_dim: int, page_size: int) -> bool:
+    """Whether prompt portions take the tcgen05 kernel that forms the maps' difference itself."""
+    return value_dim == 128 and uses_tcgen05(value_dim, page_size)
+
+
+def _differential_common(q, cache, heads):
+    pages, two, kv_heads, page_size, width = cache.shape
+    if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or q.stride(-1) != 1 or not cache.is_contiguous() or q.shape[1] < heads * width:
+        raise KernelError("differential attention: dense bfloat16 queries [tokens, heads * 2 * d] and a cache [pages, 2, kv_heads, page, 2 * d]")
+    return pages, kv_heads, page_size, width
+
+
+def differential_tiles(q, heads, cache, block_table, token_row, positions, tiles, n_tiles, scale, window, keep_first, gate, weight, eps, post, out) -> None:
+    """Prompt tiles with two maps per head: ``q`` [tokens, heads * 2 * d] (a head's two queries side by side) against ``cache`` [pages, 2, kv_heads,
+    page, 2 * d] (a head's two keys side by side; its value).  ``out`` [tokens, heads * 2 * d] bfloat16 receives the finished heads:
+    o = a1 - weight * a2, o / sqrt(mean(o^2) + eps) * post * sigmoid(``gate``), ``gate`` [tokens, heads * 2 * d] float.  ``tiles`` as planned
+    for 2 * heads heads.  Where the kernel does not form the difference itself, ``combine`` does (through a float buffer of all tokens)."""
+    require_cuda(q, cache, block_table, token_row, positions, tiles, gate, out)
+    pages, kv_heads, page_size, width = _differential_common(q, cache, heads)
+    tokens = q.shape[0]
+    common = (i32(block_table.shape[1]), ptr(token_row), ptr(positions), ptr(tiles), i32(n_tiles))
+    if fuses_differential(width, page_size) and gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0:
+        gate_ptr, gate_stride = _gate_arguments(gate, tokens, heads * width)
+        check(library("attention_tcgen05", HB_HEAD_DIM=width).hb_attention_tc_tiles_extended(
+            ptr(q), i32(q.stride(0)), ptr(out), i32(out.stride(0)), ptr(cache), ptr(block_table), *common, i32(tokens), i32(heads), i32(kv_heads), i32(width),
+            i32(page_size), i32(pages), f32(scale), f32(0.0), i32(window or 0), ptr(None), i32(0), i32(keep_first), ptr(None), gate_ptr, gate_stride, i32(2),
+            f32(weight), f32(eps), f32(post), ptr(status_word(q.device)), ptr(work_counters(q.device)), stream_ptr()), "differential_tiles")
+        return
+    wide = torch.empty((tokens, 2 * heads * width), dtype=torch.float32, device=q.device)
+    sizes = (i32(2 * heads), i32(kv_heads), i32(width), i32(page_size), i32(pages), f32(scale), f32(0.0), i32(window or 0))
+    extras = (i32(keep_first), ptr(None), ptr(None), i32(0), i32(2))
+    head = (ptr(q), i32(q.stride(0)), ptr(wide), i32(wide.stride(0)), ptr(cache), ptr(block_table))
+    if uses_tma(width, page_size):
+        check(library("attention_tma", HB_HEAD_DIM=width).hb_attention_tma_tiles_extended(*head, *common, *sizes, ptr(None), i32(0), *extras, ptr(status_word(q.device)),
+                                                                                         stream_ptr()), "differential_tiles")
+    else:
+        check(library("attention_bf16", HB_HEAD_DIM=width).hb_attention_tiles_extended(*head, *common, *sizes, *extras, ptr(status_word(q.device)), stream_ptr()),
+              "differential_tiles")
+    differential_combine(wide, None, None, tokens, heads, 1, width, weight, eps, post, gate, out)
+
+
+def differential_tokens(q, heads, cache, block_table, token_row, positions, items, n_items, splits, scale, window, keep_first, gate, weight, eps, post, out) -> None:
+    """The token shape of :func:`differential_tiles`: the pieces of both maps, then one kernel that merges them and finishes the heads."""
+    require_cuda(q, cache, block_table, token_row, positions, items, gate, out)
+    _, _, _, width = _differential_common(q, cache, heads)
+    pieces = n_items * 2 * heads * splits
+    workspace = torch.empty(pieces * (width + 2), dtype=torch.float32, device=q.device)
+    _tokens_extended(q, None, cache, block_table, token_row, positions, items, n_items, splits, workspace, 2 * heads, scale, 0.0, window,
+                     (i32(keep_first), ptr(None), ptr(None), i32(0), i32(2)))
+    differential_combine(workspace, workspace[pieces * width:], items, n_items, heads, splits, width, weight, eps, post, gate, out)
+
+
+def differential_combine(pieces, ml, items, n_items: int, heads: int, splits: int, value_dim: int, weight: float, eps: float, post: float, gate, out) -> None:
+    """``pieces`` [items, heads, 2, splits, value_dim] float (``ml``: each piece's maximum in the exp2 domain and sum) or whole results [tokens, heads,
+    2, value_dim] (``ml`` None) -> ``out`` [tokens, heads * value_dim]: o = a1 - weight * a2, o / sqrt(mean(o^2) + eps) * post * sigmoid(gate)."""
+    require_cuda(pieces, ml, items, gate, out)
+    gate_ptr, gate_stride = _gate_arguments(gate, out.shape[0], heads * value_dim)
+    if pieces.dtype != torch.float32 or out.stride(1) != 1:
+        raise KernelError("differential_combine: float32 pieces and an output with unit inner stride")
+    check(library("attention_combine").hb_differential_combine(ptr(pieces), ptr(ml), ptr(items), i32(n_items), i32(heads), i32(splits), i32(value_dim), f32(weight),
+                                                               f32(eps), f32(post), gate_ptr, gate_stride, i32(0), ptr(out), i32(out.stride(0)),
+                                                               i32(1 if out.dtype == torch.bfloat16 else 0), stream_ptr()), "differential_combine")
 
 
 # ------------------------------------------------------------------ attention over latent records (csrc/attention_latent.cu)

@@ -237,7 +237,8 @@ def attention_general(q: torch.Tensor, heads: int, kv_heads: int, head_dim: int,
                       token_row: torch.Tensor, positions: torch.Tensor, page_size: int, scale: float, softcap: float = 0.0, window: int = 0, *,
                       distance_bias: torch.Tensor | None = None, gate: torch.Tensor | None = None, gate_off: int = 0, out_scale: float = 1.0,
                       out: torch.Tensor | None = None, head_scale: torch.Tensor | None = None, slopes: torch.Tensor | None = None,
-                      sinks: torch.Tensor | None = None, chunk: int = 0, value_prefix: bool = False) -> torch.Tensor:
+                      sinks: torch.Tensor | None = None, chunk: int = 0, value_prefix: bool = False, keep_first: int = 0, gate_per_head: bool = False,
+                      maps: int = 1, wide_out: bool = False) -> torch.Tensor:
     """Causal attention of every token over its request's pages with keys of ``head_dim`` and values of ``v_dim``, a smooth
     cap on the scores (0 = none) and a window (0 = all keys); the cache in either arrangement of :func:`paged_strides`.
     ``distance_bias`` [heads, span] float: the score of a key ``n`` positions back takes ``distance_bias[head, min(n, span - 1)]``
@@ -246,7 +247,10 @@ def attention_general(q: torch.Tensor, heads: int, kv_heads: int, head_dim: int,
     ``slopes`` [heads] float: ``slopes[head] * (query position - key position)`` is taken off the score; ``sinks`` [heads] float: one more
     term ``exp(sinks[head])`` in the softmax's denominator, with no key and no value; ``chunk`` > 0: a query sees only the keys of its own
     chunk of ``chunk`` positions (counted from position 0).  ``value_prefix``: the cache is [pages, kv_heads, page, head_dim] and a
-    token's value is the first ``v_dim`` entries of its key (attention over a latent)."""
+    token's value is the first ``v_dim`` entries of its key (attention over a latent).  ``keep_first``: that many first positions of the
+    sequence are seen beside the window.  ``gate_per_head``: the gate has one column per head.  ``maps``: softmax maps per head over the same
+    values: queries [heads, maps, head_dim], keys [kv_heads, maps, head_dim] in the cache, results [heads, maps, v_dim].  ``wide_out``: the
+    result is float whatever the element type."""
     require_cuda(q, cache, block_table, token_row, positions, distance_bias, gate, out, head_scale, slopes, sinks)
     for t in (head_scale, slopes, sinks):
         if t is not None and (t.dtype != torch.float32 or t.numel() != heads or not t.is_contiguous()):
@@ -263,19 +267,21 @@ def attention_general(q: torch.Tensor, heads: int, kv_heads: int, head_dim: int,
             raise KernelError("attention: a cache of [pages, kv_heads, page, head_dim] whose values are the keys' first v_dim entries")
         v_off, page_stride, head_stride, token_stride = 0, kv_heads * cache.shape[2] * head_dim, cache.shape[2] * head_dim, head_dim
     else:
-        v_off, page_stride, head_stride, token_stride = paged_strides(cache, head_dim, v_dim)
+        v_off, page_stride, head_stride, token_stride = paged_strides(cache, maps * head_dim, v_dim)
     tokens = q.shape[0]
+    out_dtype = torch.float32 if wide_out else q.dtype
     if out is None:
-        out = torch.empty((tokens, heads * v_dim), dtype=q.dtype, device=q.device)
-    elif out.dtype != q.dtype or out.shape[0] != tokens or out.shape[1] < heads * v_dim or out.stride(1) != 1:
+        out = torch.empty((tokens, heads * maps * v_dim), dtype=out_dtype, device=q.device)
+    elif out.dtype != out_dtype or out.shape[0] != tokens or out.shape[1] < heads * maps * v_dim or out.stride(1) != 1:
         raise KernelError("attention: the output is a [tokens, >= heads * v_dim] view of the queries' element type")
     v_cache = ctypes.c_void_p(cache.data_ptr() + v_off * cache.element_size())
-    check(library("attention_generic").hb_attention_extended(
+    check(library("attention_generic").hb_attention_mapped(
         ptr(q), i32(q.stride(0)), ptr(out), i32(out.stride(0)), i32(is_bf16(q)), ptr(cache), v_cache, ctypes.c_longlong(page_stride),
         ctypes.c_longlong(head_stride), i32(token_stride), ptr(block_table), i32(block_table.shape[1]), ptr(token_row), ptr(positions), i32(tokens),
         i32(heads), i32(kv_heads), i32(head_dim), i32(v_dim), i32(page_size), i32(cache.shape[0]), f32(scale), f32(softcap or 0.0), i32(window or 0),
         ptr(distance_bias), i32(distance_bias.shape[1] if distance_bias is not None else 0), ptr(gate), i32(gate.stride(0) if gate is not None else 0),
-        i32(gate_off), f32(out_scale), ptr(head_scale), ptr(slopes), ptr(sinks), i32(chunk or 0), ptr(status_word(q.device)), stream_ptr()),
+        i32(gate_off), f32(out_scale), ptr(head_scale), ptr(slopes), ptr(sinks), i32(chunk or 0), i32(keep_first), i32(1 if gate_per_head else 0),
+        i32(maps), i32(1 if out.dtype == torch.float32 else 0), ptr(status_word(q.device)), stream_ptr()),
         "attention_general")
     return out
 
@@ -510,3 +516,95 @@ def rotate_heads_(x: torch.Tensor, col0: int, heads: int, head_dim: int, positio
         raise KernelError("rotate_heads: the heads lie outside the rows")
     check(library("heads_prepare").hb_rotate_heads(ptr(x), i32(is_bf16(x)), i32(x.shape[0]), i32(x.stride(0)), i32(col0), i32(heads), i32(head_dim), i32(rot_dims),
                                                    i32(1 if rot_half else 0), ptr(inv_freq), ptr(positions), f32(sign), stream_ptr()), "rotate_heads")
+
+
+def heads_store(x: torch.Tensor, q_off: int, k_off: int, v_off: int, q_heads: int, kv_heads: int, head_dim: int, v_dim: int, positions: torch.Tensor, *,
+                q_out: torch.Tensor, maps: int = 1, bias: torch.Tensor | None = None, q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None,
+                eps: float = 0.0, cache: torch.Tensor | None = None, block_table: torch.Tensor | None = None, token_row: torch.Tensor | None = None,
+                page_size: int = 0) -> None:
+    """Float projections ``x`` [tokens, *] of heads that nothing rotates: ``bias`` [columns] float is added, query and key heads pass an optional RMS
+    norm (one weight [head_dim] for all of them), queries [q_heads, maps, head_dim] go to ``q_out``, keys [kv_heads, maps, head_dim] and values
+    [kv_heads, v_dim] to ``cache`` (either arrangement of :func:`paged_strides`, with maps * head_dim as the keys' size).  Without a cache:
+    queries only."""
+    require_cuda(x, positions, q_out, bias, q_norm, k_norm, cache, block_table, token_row)
+    if x.dtype != torch.float32 or x.stride(-1) != 1 or q_out.stride(-1) != 1 or q_out.shape[1] < q_heads * maps * head_dim:
+        raise KernelError("heads_store: float32 projections and queries with unit inner stride")
+    if bias is not None and (bias.dtype != torch.float32 or not bias.is_contiguous() or bias.numel() > x.shape[1]):
+        raise KernelError("heads_store: the bias is a dense float32 vector over the projections' columns")
+    for t in (q_norm, k_norm):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or t.numel() != head_dim):
+            raise KernelError("heads_store: norm weights are dense float32 vectors of a head's size")
+    v_cache_off = page_stride = head_stride = token_stride = pages = 0
+    if cache is not None:
+        if cache.dtype != q_out.dtype:
+            raise KernelError("heads_store: queries and cache must share their element type")
+        v_cache_off, page_stride, head_stride, token_stride = paged_strides(cache, maps * head_dim, v_dim)
+        pages = cache.shape[0]
+    v_cache = ctypes.c_void_p(cache.data_ptr() + v_cache_off * cache.element_size()) if cache is not None else ctypes.c_void_p(0)
+    check(library("heads_prepare").hb_heads_store(
+        ptr(x), i32(x.shape[0]), i32(x.stride(0)), ptr(bias), i32(q_off), i32(k_off), i32(v_off), i32(q_heads * maps), i32(kv_heads * maps), i32(kv_heads), i32(maps),
+        i32(head_dim), i32(v_dim), ptr(q_norm), ptr(k_norm), f32(eps), ptr(positions), ptr(q_out), i32(q_out.stride(0)), i32(is_bf16(q_out)), ptr(cache), v_cache,
+        ctypes.c_longlong(page_stride), ctypes.c_longlong(head_stride), i32(token_stride), ptr(block_table),
+        i32(block_table.shape[1] if block_table is not None else 0), ptr(token_row), i32(page_size), i32(pages), ptr(status_word(x.device)), stream_ptr()),
+        "heads_store")
+
+
+def pair_norms_take(hidden: int) -> bool:
+    """Whether ``add_pair_norms`` takes rows of this width (a row stays in its block's registers)."""
+    return hidden <= (16384 if hidden % 4 == 0 else 4096)
+
+
+def add_pair_norms(h: torch.Tensor, first, second, w1: torch.Tensor, w2: torch.Tensor | None, eps: float, out_dtype: torch.dtype,
+                   rows: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """``h + (first + second)`` (either may be absent; the two are added to one another first), then the sum divided by its root mean square, times
+    ``w1`` and, unless None, times ``w2``: (rows for one reader, rows for the other or None).  Without ``rows`` the sum is written back into the
+    float stream ``h``; with ``rows`` (int32 indices) only those rows are read and ``h`` is left alone.  ``first`` may be a product still in its
+    split-K pieces (``ops.gemm.SplitSum`` without a bias), ``second`` rows sorted by expert with a weight per choice (``ops.moe.WeightedRows``)."""
+    from .gemm import SplitSum
+    from .moe import WeightedRows
+
+    if h.dtype != torch.float32 or not h.is_contiguous() or h.dim() != 2:
+        raise KernelError("add_pair_norms: a dense float32 stream")
+    tokens, hidden = h.shape
+    splits = stride = 0
+    if isinstance(second, SplitSum):
+        second = second.tensor()
+    if isinstance(first, SplitSum):
+        if first.bias is None and first.partials.is_contiguous() and first.shape == (tokens, hidden):
+            splits, stride = first.partials.shape[0], tokens * hidden
+        else:
+            first = first.tensor()
+    dense = [d for d in (first if not splits else None, second if not isinstance(second, WeightedRows) else None) if d is not None]
+    a = first.partials if splits else first
+    b, slot_of, weights, top = second, None, None, 0
+    if isinstance(second, WeightedRows):
+        b, slot_of, weights, top = second.y, second.where.slot_of, second.weights, second.where.top
+        if b.shape[1] != hidden or not b.is_contiguous() or weights.shape != (tokens, top) or weights.dtype != torch.float32 or not weights.is_contiguous():
+            raise KernelError("add_pair_norms: dense expert rows of the stream's width and float32 weights [tokens, top]")
+    types = {d.dtype for d in dense} | ({b.dtype} if slot_of is not None else set())
+    if len(types) > 1 or (types == {torch.bfloat16} and out_dtype == torch.float32):  # sublayers of unlike precision
+        wide = [None if d is None else (d.tensor() if hasattr(d, "tensor") else d).float() for d in (first, second)]
+        return add_pair_norms(h, *wide, w1, w2, eps, out_dtype, rows)
+    for d in dense:
+        if d.shape != h.shape or not d.is_contiguous():
+            raise KernelError("add_pair_norms: sublayer outputs are dense and of the stream's shape")
+    for w in (w1, w2):
+        if w is not None and (w.dtype != torch.float32 or w.numel() != hidden or not w.is_contiguous()):
+            raise KernelError("add_pair_norms: norm weights are dense float32 vectors of the stream's width")
+    require_cuda(h, a, b, slot_of, weights, w1, w2, rows)
+    n_rows = rows.numel() if rows is not None else tokens
+    out1 = torch.empty((n_rows, hidden), dtype=out_dtype, device=h.device)
+    out2 = torch.empty_like(out1) if w2 is not None else None
+    check(library("elementwise").hb_add_pair_norms(
+        ptr(h), ptr(a), i32(splits), ctypes.c_longlong(stride), ptr(b), ptr(slot_of), ptr(weights), i32(top), i32(1 if torch.bfloat16 in (types or {out_dtype}) else 0), ptr(w1), ptr(w2),
+        ptr(out1), ptr(out2), i32(is_bf16(out1)), ptr(rows), i32(n_rows), i32(hidden), f32(eps), i32(0 if rows is not None else 1), stream_ptr()), "add_pair_norms")
+    return out1, out2
+
+
+def soft_cap_(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x <- cap * tanh(x / cap) in place over a dense float32 tensor."""
+    require_cuda(x)
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise KernelError("soft_cap_: a dense float32 tensor")
+    check(library("elementwise").hb_soft_cap(ptr(x), f32(cap), ctypes.c_longlong(x.numel()), stream_ptr()), "soft_cap")
+    return x

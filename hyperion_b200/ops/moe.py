@@ -64,6 +64,22 @@ def route_scored(x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor
     return chosen, weights
 
 
+def route_softmax(x: torch.Tensor, router: torch.Tensor, bias: torch.Tensor | None, top: int) -> tuple[torch.Tensor, torch.Tensor]:
+    """Router logits ``x router^T + bias`` in float, the ``top`` largest per token (lowest index first among equals), weights = softmax over the
+    chosen logits alone: ([tokens, top] int32, [tokens, top] float)."""
+    require_cuda(x, router, bias)
+    if router.dtype != torch.float32 or not router.is_contiguous() or x.stride(-1) != 1 or x.shape[1] != router.shape[1]:
+        raise KernelError("moe.route_softmax: a dense float32 router matrix [experts, hidden] and rows with unit inner stride")
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != router.shape[0] or not bias.is_contiguous()):
+        raise KernelError("moe.route_softmax: the bias is a dense float32 vector with one entry per expert")
+    tokens, hidden = x.shape
+    chosen = torch.empty((tokens, top), dtype=torch.int32, device=x.device)
+    weights = torch.empty((tokens, top), dtype=torch.float32, device=x.device)
+    check(library("moe").hb_moe_route_softmax(ptr(x), i32(is_bf16(x)), i32(x.stride(0)), ptr(router), ptr(bias), i32(tokens), i32(hidden), i32(router.shape[0]), i32(top),
+                                              ptr(chosen), ptr(weights), stream_ptr()), "moe_route_softmax")
+    return chosen, weights
+
+
 def capacity_for(pairs: int, experts: int, pad: int = PAD) -> int:
     """Rows the sorted buffers need whatever the routing: all pairs, each expert's run padded to whole tiles."""
     return -(-(pairs + experts * (pad - 1)) // pad) * pad
@@ -103,8 +119,15 @@ def takes_tensor_cores(a: torch.Tensor, w: torch.Tensor) -> bool:
     return a.dtype == torch.bfloat16 and a.shape[1] % 8 == 0 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
 
 
-def grouped_linear(a: torch.Tensor, w: torch.Tensor, where: Plan) -> torch.Tensor:
-    """``a`` [capacity, k] times the matrix of each tile's expert: ``w`` [experts, n, k] -> [capacity, n], float accumulation."""
+ACTIVATIONS = {None: 0, "relu_squared": 1}  # what a grouped product can apply to its result before the one rounding
+
+
+def grouped_linear(a: torch.Tensor, w: torch.Tensor, where: Plan, activation: str | None = None) -> torch.Tensor:
+    """``a`` [capacity, k] times the matrix of each tile's expert: ``w`` [experts, n, k] -> [capacity, n], float accumulation; ``activation``
+    (a key of ``ACTIVATIONS``) is applied to the float result."""
+    if activation not in ACTIVATIONS:
+        raise KernelError(f"moe.grouped_linear: no activation {activation!r} (known: {sorted(k for k in ACTIVATIONS if k)})")
+    act = i32(ACTIVATIONS[activation])
     require_cuda(a, w)
     if a.dtype != w.dtype or not a.is_contiguous() or not w.is_contiguous() or w.dim() != 3 or w.shape[2] != a.shape[1] or a.shape[0] != where.capacity:
         raise KernelError("moe.grouped_linear: dense operands of one element type, rows [capacity, k] and matrices [experts, n, k]")
@@ -113,13 +136,13 @@ def grouped_linear(a: torch.Tensor, w: torch.Tensor, where: Plan) -> torch.Tenso
         lib = library("moe_gemm_tcgen05")
         if where.pairs <= FEW_PAIRS:
             check(lib.hb_moe_gemm_rows(ptr(a), ptr(w), ptr(out), ptr(where.tile_expert), ptr(where.tile_rows), i32(PAD), i32(where.capacity), i32(w.shape[1]),
-                                       i32(w.shape[2]), stream_ptr()), "moe_gemm_rows")
+                                       i32(w.shape[2]), act, stream_ptr()), "moe_gemm_rows")
         else:
             check(lib.hb_moe_gemm_tiles(ptr(a), ptr(w), ptr(out), ptr(where.tile_expert), i32(where.capacity), i32(w.shape[0]), i32(w.shape[1]),
-                                        i32(w.shape[2]), ptr(status_word(a.device)), stream_ptr()), "moe_gemm_tiles")
+                                        i32(w.shape[2]), act, ptr(status_word(a.device)), stream_ptr()), "moe_gemm_tiles")
         return out
     check(library("moe").hb_moe_gemm(ptr(a), ptr(w), ptr(out), i32(is_bf16(a)), ptr(where.tile_expert), i32(PAD), i32(where.capacity), i32(w.shape[1]),
-                                     i32(w.shape[2]), stream_ptr()), "moe_gemm")
+                                     i32(w.shape[2]), act, stream_ptr()), "moe_gemm")
     return out
 
 
@@ -151,3 +174,17 @@ def combine_weighted(y: torch.Tensor, where: Plan, weights: torch.Tensor, x: tor
     check(library("moe").hb_moe_combine_weighted(ptr(y), ptr(where.slot_of), ptr(weights), i32(where.top), ptr(x), i32(x.stride(0)), ptr(base), ptr(base_gate),
                                                  ptr(out), i32(is_bf16(y)), i32(tokens), i32(hidden), stream_ptr()), "moe_combine_weighted")
     return out
+
+
+@dataclass
+class WeightedRows:
+    """A feed-forward's result before a token's rows have been added up: ``y`` [capacity, hidden] sorted by expert, ``weights`` [tokens, top] float.
+    A reader that can weigh and add them itself (``ops.add_pair_norms``) saves a pass over the tokens; any other calls :meth:`tensor`."""
+
+    y: torch.Tensor
+    where: Plan
+    weights: torch.Tensor
+    x: torch.Tensor  # the rows the feed-forward read
+
+    def tensor(self) -> torch.Tensor:
+        return combine_weighted(self.y, self.where, self.weights, self.x, None, None)

@@ -112,8 +112,10 @@ class GroupedQueryAttention(Mixer):
         """Per-step metadata: the rows cut into tiles and single tokens (shared by all layers with the same tiling)."""
         if not self.fast:
             return {}
-        heads, kv_heads, head_dim = self.heads, self.kv_heads, self.head_dim
+        return GroupedQueryAttention.plans_for(self.heads, self.kv_heads, self.head_dim)
 
+    @staticmethod
+    def plans_for(heads: int, kv_heads: int, head_dim: int) -> dict:
         def plan(rows, packer, host):
             size = fast_attention.tile_rows(head_dim, host.get("page_size"))
             tokens_per_tile = fast_attention.tile_tokens(heads, kv_heads, size)
@@ -138,9 +140,9 @@ class GroupedQueryAttention(Mixer):
             return int((rows.positions[short] + rows.counts[short]).max())
         return max(row.position + row.count for row in rows if row.count <= fast_attention.TOKEN_SHAPE_MAX)
 
-    def _attend_fast(self, qkv, step, cache, out=None, bias=None, bias_per_position=None):
+    def _attend_fast(self, qkv, step, cache, out=None, bias=None, bias_per_position=None, sinks=None, gate=None):
         """``out``: a [tokens, >= heads * head_dim] view to write to; ``bias``: a table by distance, ``bias_per_position``: the same bias
-        as one number per head where it is linear in the distance (``ops.attention.attention_tiles``)."""
+        as one number per head where it is linear in the distance; ``sinks`` and ``gate`` as ``ops.attention.attention_tiles`` takes them."""
         if out is None:
             out = torch.empty((step.n_tokens, self.heads * self.head_dim), dtype=self.dtype, device=qkv.device)
         size = fast_attention.tile_rows(self.head_dim, step.host.get("page_size"))
@@ -149,7 +151,7 @@ class GroupedQueryAttention(Mixer):
         if n_tiles:
             fast_attention.attention_tiles(qkv, self.heads, cache.kv, cache.block_table, step.token_row, step.positions,
                                            step.extra[key], n_tiles, self.scale, self.window, out, tile_size=size, softcap=self.softcap, bias=bias,
-                                           bias_per_position=bias_per_position)
+                                           bias_per_position=bias_per_position, sinks=sinks, gate=gate)
         if n_items:
             # a step replayed from a CUDA graph fixes its launch shape for every context its tables can hold
             longest = step.host.get("context_cap") or self._longest_short_row(step.rows)
@@ -157,7 +159,8 @@ class GroupedQueryAttention(Mixer):
                 longest = min(longest, abs(self.window) + fast_attention.KEY_TILE)
             splits = fast_attention.choose_splits(n_items, self.heads, self.kv_heads, longest)
             fast_attention.attention_tokens(qkv, self.heads, cache.kv, cache.block_table, step.token_row, step.positions,
-                                            step.extra["attn_items"], n_items, splits, self.scale, self.window, out, softcap=self.softcap, bias=bias)
+                                            step.extra["attn_items"], n_items, splits, self.scale, self.window, out, softcap=self.softcap, bias=bias,
+                                            sinks=sinks, gate=gate)
         return out
 
 

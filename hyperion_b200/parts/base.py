@@ -40,7 +40,8 @@ class PagedTokens:
     """A payload of fixed shape per token, kept in pages.  The cache manager gives the mixer a tensor
     [pages, *outer, page_size, *inner]: a token at position p of a request lies at
     ``[block_table[row, p // page_size], ..., p % page_size, ...]``.  ``window`` > 0: only the last
-    ``window`` positions are ever read again, so older pages are given back while the request lives.
+    ``window`` positions are ever read again, so older pages are given back while the request lives;
+    ``keep_first`` > 0 (with a window): the first ``keep_first`` positions of the sequence are read for ever, so their pages stay.
     ``dtype`` None: the model's activation type.  Users with equal requests share one pool of pages
     and one block table per request."""
 
@@ -48,6 +49,7 @@ class PagedTokens:
     inner: tuple[int, ...] = ()
     window: int = 0
     dtype: Optional[torch.dtype] = None
+    keep_first: int = 0
 
     @property
     def values_per_token(self) -> int:
@@ -60,9 +62,9 @@ class PagedTokens:
         return (num_pages, *self.outer, page_size, *self.inner)
 
 
-def PagedKV(kv_heads: int, head_dim: int, window: int = 0) -> PagedTokens:
+def PagedKV(kv_heads: int, head_dim: int, window: int = 0, keep_first: int = 0) -> PagedTokens:
     """Keys and values per token: pages of [2, kv_heads, page_size, head_dim]."""
-    return PagedTokens((2, int(kv_heads)), (int(head_dim),), int(window))
+    return PagedTokens((2, int(kv_heads)), (int(head_dim),), int(window), keep_first=int(keep_first))
 
 
 @dataclass(frozen=True)

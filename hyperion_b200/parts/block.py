@@ -93,3 +93,21 @@ class SideBySideBlock(Arrangement):
 
 
 register_arrangement("side_by_side", SideBySideBlock)
+
+
+class SideBySideTwoNormsBlock(Arrangement):
+    """Mixer and feed-forward read the same stream through norms of their own and their results are added to it together:
+    h <- h + (mixer(norm_a(h)) + feed_forward(norm_c(h))).  Norm names: ``input`` and, when the layer has a feed-forward, ``feed_forward_in``.  Both
+    norms divide by the same root mean square, so one launch adds what is pending and makes both (``ops.add_pair_norms``); what the two sublayers
+    return travels on as a :class:`SumOfTwo`."""
+
+    def forward(self, h, delta, step, cache, own_cache):
+        from .norm import SumOfTwo
+
+        if self.feed_forward is None:
+            return h, SumOfTwo(self.mixer.forward(self.norms["input"].forward(h, delta), step, cache, own_cache), None)
+        x, y = self.norms["input"].forward_pair(h, delta, self.norms["feed_forward_in"])
+        return h, SumOfTwo(self.mixer.forward(x, step, cache, own_cache), self.feed_forward.forward(y, step))
+
+
+register_arrangement("side_by_side_two_norms", SideBySideTwoNormsBlock)

@@ -7,7 +7,8 @@ Parameters: ``vocab_size``, ``hidden_size``, ``weight_name`` (the tensor's name 
 unless stated); the embedding also ``scale`` (the looked-up row is multiplied by it in float, 1 unless
 stated) and ``norm_weight_name`` with ``eps`` (unless absent: the looked-up row passes an RMS norm with that weight
 before it becomes the stream); the head also ``tied`` (then it owns no tensor and is handed the embedding's table)
-and ``scale`` (the logits are multiplied by it, 1 unless stated).
+and ``scale`` (the logits are multiplied by it, 1 unless stated) and ``softcap`` (the logits become
+cap * tanh(logits / cap) after that, unless 0).
 
 ``offset_table`` is a learned table [count, hidden] of vectors that the schedule adds to the stream before an entry
 runs (a model that passes some layers several times marks each pass this way).  Parameters: ``count``, ``hidden_size``,
@@ -67,6 +68,7 @@ class LinearHead(Head):
         self.tied = bool(spec.params.get("tied", False))
         self.weight_name = str(spec.params.get("weight_name", "weight"))
         self.scale = float(spec.params.get("scale", 1.0))
+        self.softcap = float(spec.params.get("softcap") or 0.0)
         self.weight = None
 
     def weights(self):
@@ -85,11 +87,13 @@ class LinearHead(Head):
         self.weight = table
 
     def kernel_modules(self):
-        return [("sgemm_f32", {}) if self.dtype == torch.float32 else ("gemm_tcgen05", {})] + ([("elementwise", {})] if self.scale != 1.0 else [])
+        return [("sgemm_f32", {}) if self.dtype == torch.float32 else ("gemm_tcgen05", {})] + ([("elementwise", {})] if self.scale != 1.0 or self.softcap else [])
 
     def forward(self, x):
         logits = ops.linear(x, self.weight, None, torch.float32)
-        return ops.scale_(logits, self.scale) if self.scale != 1.0 else logits
+        if self.scale != 1.0:
+            ops.scale_(logits, self.scale)
+        return ops.soft_cap_(logits, self.softcap) if self.softcap else logits
 
 
 register_embedding("token_embedding", TokenEmbedding)

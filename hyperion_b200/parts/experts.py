@@ -20,6 +20,13 @@ the same form runs for every token and is added times sigmoid(w_sg . x), one num
 Parameters: ``hidden_size``, ``experts`` (those with matrices), ``identity``, ``top``, ``expert_size``, ``activation``, ``scale``, ``group_count``
 (0: no groups), ``group_keep``, ``shared_size`` (None for none).  Tensors: router [experts + identity, hidden], correction
 [experts + identity], e<i>.{up,down}, shared.{up,down,sg}.
+
+``chosen_softmax_experts`` chooses by the logits themselves, z = W_r x + b in float, and weighs the ``top`` chosen by a softmax over the chosen
+logits alone; the weight multiplies what an expert returns.  Experts are down(act(up(h))) without a gate and without biases, the activation
+applied by the grouped product that makes its argument.  There is no shared expert.  The result leaves as rows with weights
+(``ops.moe.WeightedRows``), which the norm that adds it to the stream weighs and adds up itself.
+Parameters: ``hidden_size``, ``experts``, ``top``, ``expert_size``, ``activation`` (``relu_squared``).  Tensors: router [experts, hidden], router.b [experts],
+e<i>.{up,down}.
 """
 from __future__ import annotations
 
@@ -149,3 +156,43 @@ class ScoredExperts(FeedForward):
 
 
 register_feed_forward("scored_experts", ScoredExperts)
+
+
+class ChosenSoftmaxExperts(FeedForward):
+    def __init__(self, spec: PartSpec, build: BuildContext):
+        super().__init__(spec, build)
+        p = spec.params
+        self.hidden, self.experts, self.top, self.inter = int(p["hidden_size"]), int(p["experts"]), int(p["top"]), int(p["expert_size"])
+        self.activation = str(p.get("activation", "relu_squared"))
+        if not 0 < self.top <= self.experts or self.experts > 1024:
+            raise ValueError(f"{self.top} of {self.experts} experts: the router takes up to 1,024 experts and at least one of them per token")
+        if self.activation not in moe.ACTIVATIONS:
+            raise ValueError(f"no activation {self.activation!r} (known: {sorted(k for k in moe.ACTIVATIONS if k)})")
+
+    def weights(self) -> dict[str, WeightSpec]:
+        wanted = {"router": WeightSpec((self.experts, self.hidden)), "router.b": WeightSpec((self.experts,))}
+        for e in range(self.experts):
+            wanted[f"e{e}.up"] = WeightSpec((self.inter, self.hidden))
+            wanted[f"e{e}.down"] = WeightSpec((self.hidden, self.inter))
+        return wanted
+
+    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        self.router = tensors["router"].to(torch.float32).contiguous()
+        self.router_bias = tensors["router.b"].to(torch.float32).contiguous()
+        self.w_up = torch.stack([tensors[f"e{e}.up"] for e in range(self.experts)]).contiguous()  # [experts, inter, hidden]
+        self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(self.experts)]).contiguous()  # [experts, hidden, inter]
+
+    def kernel_modules(self):
+        modules = [("moe", {}), ("elementwise", {})]
+        if self.dtype == torch.bfloat16 and (self.hidden % 8 == 0 or self.inter % 8 == 0):
+            modules.append(("moe_gemm_tcgen05", {}))
+        return modules
+
+    def forward(self, x, step):
+        chosen, weights = moe.route_softmax(x, self.router, self.router_bias, self.top)
+        where = moe.plan(chosen, None, self.experts)  # the weights multiply what an expert returns, so the rows are gathered as they are
+        act = moe.grouped_linear(moe.gather(x, where), self.w_up, where, self.activation)
+        return moe.WeightedRows(moe.grouped_linear(act, self.w_down, where), where, weights, x)
+
+
+register_feed_forward("chosen_softmax_experts", ChosenSoftmaxExperts)

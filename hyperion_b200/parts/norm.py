@@ -19,6 +19,7 @@ from typing import Mapping, Optional
 import torch
 
 from .. import ops
+from ..ops.moe import WeightedRows
 from .base import BuildContext, Norm, WeightSpec, register_norm
 from .spec import PartSpec
 
@@ -70,10 +71,11 @@ class NormedDelta:
 @dataclass
 class SumOfTwo:
     """What two sublayers that read the same rows returned, still to be added to the stream: first to one another, then to the
-    stream.  The next norm that reads the stream does it in its own launch (``ops.add_group_rmsnorm``).  Either may be absent."""
+    stream.  The next norm that reads the stream does it in its own launch (``ops.add_pair_norms``, which also takes ``first`` in its split-K
+    pieces and ``second`` as an expert feed-forward's rows with their weights, or ``ops.add_group_rmsnorm``).  Either may be absent."""
 
-    first: Optional[torch.Tensor]
-    second: Optional[torch.Tensor]
+    first: object
+    second: object
 
     def parts(self) -> tuple[Optional[torch.Tensor], Optional[torch.Tensor]]:
         return tuple(d.tensor() if hasattr(d, "tensor") else d for d in (self.first, self.second))
@@ -120,7 +122,18 @@ class RMSNorm(Norm):
     def kernel_modules(self):
         return [("elementwise", {})]
 
+    def forward_pair(self, h, delta, other: "RMSNorm"):
+        """This norm and ``other`` of the same stream, in one launch: (rows for this norm's reader, rows for the other's)."""
+        if other.eps != self.eps or self.groups > 1 or other.groups > 1 or other.dtype != self.dtype or not ops.pair_norms_take(h.shape[1]) or isinstance(delta, (NormedDelta, GatedResult)):
+            return self.forward(h, delta), other.forward(h, None)
+        first, second = (delta.first, delta.second) if isinstance(delta, SumOfTwo) else (delta, None)
+        return ops.add_pair_norms(h, first, second, self.weight, other.weight, self.eps, self.dtype)
+
     def forward(self, h, delta, rows=None):
+        if isinstance(delta, SumOfTwo) and self.groups == 1 and ops.pair_norms_take(h.shape[1]):
+            return ops.add_pair_norms(h, delta.first, delta.second, self.weight, None, self.eps, self.dtype, rows)[0]
+        if isinstance(delta, WeightedRows):
+            delta = delta.tensor()
         if isinstance(delta, GatedResult):  # a gated result that no norm stands on: multiplied here, added below
             delta = delta.tensor()
         if self.groups > 1 or isinstance(delta, SumOfTwo):

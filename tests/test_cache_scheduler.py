@@ -577,21 +577,23 @@ def test_worst_case_pages_bounds_what_a_windowed_request_ever_holds():
 
     from hyperion_b200 import host
 
-    def bound(page, window, tokens, portion):
+    def bound(page, window, tokens, portion, keep=0):
         value = ctypes.c_int()
-        host.check(host.library().hb_cache_worst_case_pages(page, window, tokens, portion, ctypes.byref(value)))
+        host.check(host.library().hb_cache_worst_case_pages(page, window, keep, tokens, portion, ctypes.byref(value)))
         return value.value
 
     assert bound(4, 0, 33, 7) == 9 and bound(4, 6, 5, 100) == 2 and bound(16, 0, 0, 1) == 0
+    assert bound(4, 8, 1000, 4) == 4 and bound(4, 8, 1000, 4, keep=5) == 6 and bound(4, 8, 12, 4, keep=5) == 3
     rng = random.Random(5)
     for _ in range(60):
         page = rng.choice([1, 2, 4, 8, 16])
         window = rng.randint(1, 40)
         portion = rng.randint(1, 30)
         total = rng.randint(1, 200)
-        m = CacheManager([(0, PagedKV(1, 8, window=window))], page, 400, 1)
+        keep = rng.choice([0, 0, 1, 5, 16, 33])
+        m = CacheManager([(0, PagedKV(1, 8, window=window, keep_first=keep))], page, 400, 1)
         m.add_request("r")
-        limit, fed, most = bound(page, window, total, portion), 0, 0
+        limit, fed, most = bound(page, window, total, portion, keep), 0, 0
         while fed < total:
             n = min(rng.randint(1, portion), total - fed)
             m.extend("r", n)
@@ -599,7 +601,37 @@ def test_worst_case_pages_bounds_what_a_windowed_request_ever_holds():
             m.advance("r", n)
             fed += n
         assert most <= limit, (page, window, portion, total, most, limit)
+        m.check()
         m.free("r")
+
+
+def test_the_first_pages_stay_while_a_window_passes_the_others():
+    """A window of 6 beside 5 kept first positions over pages of 4: the two pages that hold the kept positions stay in the table for the
+    request's life, the ones between them and the window go back, and admission counts them."""
+    from hyperion_b200.host import CacheError
+
+    m = CacheManager([(0, PagedKV(1, 8, window=6, keep_first=5)), (1, PagedKV(1, 8, window=6)), (2, PagedKV(1, 8, window=6, keep_first=5))], 4, 40, 1)
+    assert [g.users for g in m.paged] == [[0, 2], [1]] and m.group_windows == [6, 6] and m.group_keeps == [5, 0]
+    m.add_request("r")
+    m.extend("r", 10)
+    assert m.advance("r", 10) == [(1, m.table(0, "r")[0])]  # the next query sees 5 .. 10: block 0 goes where nothing is kept
+    m.extend("r", 30)
+    released = m.advance("r", 30)
+    kept, plain = m.table(0, "r"), m.table(1, "r")
+    assert [b for b, page in enumerate(kept) if page >= 0] == [0, 1, 8, 9] and [b for b, page in enumerate(plain) if page >= 0] == [8, 9]
+    assert sorted(group for group, _ in released) == [0] * 6 + [1] * 7
+    m.check()
+    m.free("r")
+    assert m.free_pages(0) == m.free_pages(1) == 40
+    with pytest.raises(CacheError):
+        m.length("r")
+    # admission: without the kept positions a request of this window costs 4 pages, with them 6
+    for keeps, running in (((), 2), ((5,), 1)):
+        s = Scheduler(SchedulerConfig(num_pages=8, page_size=4, max_seq_len=1000, max_batch_tokens=4, group_windows=(8,), group_keeps=keeps))
+        for name in "ab":
+            s.enqueue(Request(name, list(range(30)), params(500)))
+        s.next_plan()
+        assert 2 - len(s.waiting) == running
 
 
 def test_admission_counts_pages_per_group_of_the_cache():
