@@ -656,6 +656,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_tc_kernel(const __grid_c
 #pragma unroll 1
                         for (int c = 0; c < 64; c += 16) {
                             float o[16];
+                            __syncwarp();
                             difference(c, o);
                             if (!row_valid) continue;
 #pragma unroll

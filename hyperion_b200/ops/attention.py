@@ -250,6 +250,11 @@ def fuses_differential(value_dim: int, page_size: int) -> bool:
     return value_dim == 128 and uses_tcgen05(value_dim, page_size)
 
 
+def differential_tile_rows(value_dim: int, page_size) -> int:
+    """Virtual rows (tokens x heads of a group x maps) per tile of the kernel that will run."""
+    return TC_TILE_ROWS if page_size is not None and fuses_differential(value_dim, page_size) else TILE_ROWS
+
+
 def _differential_common(q, cache, heads):
     pages, two, kv_heads, page_size, width = cache.shape
     if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or q.stride(-1) != 1 or not cache.is_contiguous() or q.shape[1] < heads * width:
@@ -261,12 +266,12 @@ def differential_tiles(q, heads, cache, block_table, token_row, positions, tiles
     """Prompt tiles with two maps per head: ``q`` [tokens, heads * 2 * d] (a head's two queries side by side) against ``cache`` [pages, 2, kv_heads,
     page, 2 * d] (a head's two keys side by side; its value).  ``out`` [tokens, heads * 2 * d] bfloat16 receives the finished heads:
     o = a1 - weight * a2, o / sqrt(mean(o^2) + eps) * post * sigmoid(``gate``), ``gate`` [tokens, heads * 2 * d] float.  ``tiles`` as planned
-    for 2 * heads heads.  Where the kernel does not form the difference itself, ``combine`` does (through a float buffer of all tokens)."""
+    for 2 * heads heads of :func:`differential_tile_rows`.  Where the kernel does not form the difference itself, ``combine`` does (through a float buffer of all tokens)."""
     require_cuda(q, cache, block_table, token_row, positions, tiles, gate, out)
     pages, kv_heads, page_size, width = _differential_common(q, cache, heads)
     tokens = q.shape[0]
     common = (i32(block_table.shape[1]), ptr(token_row), ptr(positions), ptr(tiles), i32(n_tiles))
-    if fuses_differential(width, page_size) and gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0:
+    if fuses_differential(width, page_size):
         gate_ptr, gate_stride = _gate_arguments(gate, tokens, heads * width)
         check(library("attention_tcgen05", HB_HEAD_DIM=width).hb_attention_tc_tiles_extended(
             ptr(q), i32(q.stride(0)), ptr(out), i32(out.stride(0)), ptr(cache), ptr(block_table), *common, i32(tokens), i32(heads), i32(kv_heads), i32(width),

@@ -115,9 +115,12 @@ class GroupedQueryAttention(Mixer):
         return GroupedQueryAttention.plans_for(self.heads, self.kv_heads, self.head_dim)
 
     @staticmethod
-    def plans_for(heads: int, kv_heads: int, head_dim: int) -> dict:
+    def plans_for(heads: int, kv_heads: int, head_dim: int, rows_of=None) -> dict:
+        """``rows_of(page_size)``: the virtual rows per tile, where another kernel than the usual one for this head size will run."""
+        rows_of = rows_of or (lambda page_size: fast_attention.tile_rows(head_dim, page_size))
+
         def plan(rows, packer, host):
-            size = fast_attention.tile_rows(head_dim, host.get("page_size"))
+            size = rows_of(host.get("page_size"))
             tokens_per_tile = fast_attention.tile_tokens(heads, kv_heads, size)
             key = f"attn_tiles_{tokens_per_tile}"
             if key in host:
@@ -130,7 +133,7 @@ class GroupedQueryAttention(Mixer):
             if len(items) and "attn_items" not in [name for name, *_ in packer._items]:
                 packer.add("attn_items", items)
 
-        return {("attention_plan", heads // kv_heads, head_dim): plan}
+        return {("attention_plan", heads // kv_heads, head_dim, rows_of(None), rows_of(16)): plan}
 
     @staticmethod
     def _longest_short_row(rows) -> int:

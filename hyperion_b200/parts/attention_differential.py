@@ -93,11 +93,14 @@ class DifferentialAttention(Mixer):
         """As for a grouped-query attention of 2 * heads heads of e entries."""
         if not self.fast:
             return {}
-        return GroupedQueryAttention.plans_for(2 * self.heads, self.kv_heads, self.value_dim)
+        return GroupedQueryAttention.plans_for(2 * self.heads, self.kv_heads, self.value_dim, self._tile_rows)
+
+    def _tile_rows(self, page_size) -> int:
+        return fast_attention.differential_tile_rows(self.value_dim, page_size)
 
     def _attend_fast(self, q, gate, step, cache, out):
         heads, kv_heads = 2 * self.heads, self.kv_heads
-        size = fast_attention.tile_rows(self.value_dim, step.host.get("page_size"))
+        size = self._tile_rows(step.host.get("page_size"))
         key = f"attn_tiles_{fast_attention.tile_tokens(heads, kv_heads, size)}"
         n_tiles, n_items = step.host.get(key, 0), step.host.get("attn_items", 0)
         after = (self.scale, self.window, self.keep_first, gate, self.map_weight, self.eps, 1.0 - self.diff, out)
