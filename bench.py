@@ -1008,6 +1008,190 @@ def tobadra_workload(args) -> int:
     return 0
 
 
+ZUREVIK_SIZES = {
+    # width; heads and kv heads of both attentions; differential attention (size of a map's query, value size, window, kept first tokens); windowed
+    # attention with sinks (head size, window); experts (count, per token, inner width).  Eight layers S D D S' D S D S' (S = windowed attention with sinks,
+    # S' = the same over the keys and values of the S before it, D = differential attention), every layer with experts, 32,000 tokens
+    "2k": {"width": 2048, "heads": (16, 4), "differential": (64, 128, 1024, 4), "sinks": (128, 1024), "experts": (16, 2, 2048)},
+    "4k": {"width": 4096, "heads": (32, 8), "differential": (64, 128, 2048, 4), "sinks": (128, 2048), "experts": (16, 2, 3584)},
+}
+
+
+def zurevik_document(size: dict, vocab: int = 32000) -> dict:
+    heads, kv_heads = size["heads"]
+    dim, vdim, window, keep = size["differential"]
+    s_dim, s_window = size["sinks"]
+    count, top, inner = size["experts"]
+    mlp = {"kind": "moe", "expert": {"ff": inner}, "router": {"experts": count, "top": top}}
+    d = {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "diff": 0.5,
+                                                    "mask": {"size": window, "keep_first": keep}}}
+
+    def s(kv_from=None):
+        mixer = {"heads": heads, "kv_heads": kv_heads, "dim": s_dim, "vdim": s_dim, "scale": s_dim ** -0.5, "mask": {"size": s_window}}
+        return {"type": "attention_2", "mlp": mlp, "mixer": {**mixer, "kv_from": kv_from} if kv_from is not None else mixer}
+
+    return {"architecture": "Zurevik", "vocab": vocab, "width": size["width"], "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+            "layers": [s(), d, d, s(0), d, s(), d, s(5)]}
+
+
+def zurevik_like_document(size: dict, vocab: int = 32000) -> dict:
+    """The closest model of the package at equal size: Tobadra with windowed attention and experts in all eight layers, no input convolution, no groups, no
+    shared expert (its sublayers keep their gates)."""
+    heads, kv_heads = size["heads"]
+    dim, window = size["sinks"]
+    count, top, inner = size["experts"]
+    layer = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window}},
+             "mlp": {"kind": "moe", "expert": {"ff": inner}, "router": {"experts": count, "top": top, "scale": 1.0, "identity": 0}}}
+    return {"architecture": "Tobadra", "vocab": vocab, "width": size["width"], "norm": {"eps": 1e-6}, "logit_scale": 1.0, "layers": [layer] * 8}
+
+
+def zurevik_kernels(size: dict, measured: dict) -> dict:
+    """The design's own kernels alone at this size, a prompt of 2,048 tokens in one row and 8 rows of one decoded token behind 2,048: time, the bytes
+    each must move against the measured copy bandwidth, for attention and the experts' products the bfloat16 operations against the measured product
+    rate; beside each the like kernel of the closest models (Tobadra's windowed attention, router, product and sum; Kudazen's norm)."""
+    import types
+
+    import torch
+
+    from hyperion_b200 import ops
+    from hyperion_b200.ops import attention as fast, moe
+
+    dev = torch.device("cuda")
+    hbm, peak = measured["hbm_gbs"] * 1e9, measured["bf16_tflops"] * 1e12
+    out: dict = {}
+    width, page = size["width"], 16
+
+    def report(name, ms, bytes_moved, bf16_flops=None):
+        entry = {"us": round(ms * 1e3, 2), "bytes": int(bytes_moved), "of_measured_bandwidth": round(bytes_moved / (ms / 1e3) / hbm, 3)}
+        if bf16_flops is not None:
+            entry["of_measured_bf16_rate"] = round(bf16_flops / (ms / 1e3) / peak, 3)
+        out[name] = entry
+
+    heads, kv_heads = size["heads"]
+    dim, vdim, window, keep = size["differential"]
+    s_dim, s_window = size["sinks"]
+    count, top, inner = size["experts"]
+    for shape, counts, before in (("prefill_2048", [PROMPT], 0), ("decode_8", [1] * 8, PROMPT)):
+        tokens, rows = sum(counts), len(counts)
+        token_row = torch.tensor([r for r, c in enumerate(counts) for _ in range(c)], dtype=torch.int32, device=dev)
+        positions = torch.cat([torch.arange(c, dtype=torch.int32) + before for c in counts]).to(dev)
+        context = before + max(counts)
+        per_row = -(-context // page)
+        table = torch.arange(rows * per_row, dtype=torch.int32, device=dev).view(rows, per_row)
+        # the sum of two sublayers with two norms behind it: dense results, and the experts' rows
+        h = torch.randn(tokens, width, device=dev)
+        x = torch.randn(tokens, width, device=dev).to(torch.bfloat16)
+        a, b = (torch.randn(tokens, width, device=dev).to(torch.bfloat16) for _ in range(2))
+        weight = torch.ones(width, device=dev)
+        router, bias = torch.randn(count, width, device=dev) * 0.05, torch.randn(count, device=dev) * 0.05
+        chosen, weights = moe.route_softmax(x, router, bias, top)
+        where = moe.plan(chosen, None, count)
+        z = torch.randn(where.capacity, width, device=dev).to(torch.bfloat16)
+        rows_of = moe.WeightedRows(z, where, weights, x)
+        report(f"add_pair_norms/{shape}", timed(lambda: ops.add_pair_norms(h, a, b, weight, weight, 1e-6, torch.bfloat16)), tokens * width * (4 + 4 + 2 + 2 + 2 + 2))
+        report(f"add_pair_norms_of_expert_rows/{shape}", timed(lambda: ops.add_pair_norms(h, a, rows_of, weight, weight, 1e-6, torch.bfloat16)),
+               tokens * width * (4 + 4 + 2 + 2 * top + 2 + 2))
+        report(f"kudazen.add_group_rmsnorm/{shape}", timed(lambda: ops.add_group_rmsnorm(h, a, b, weight, 1, 1e-6, torch.bfloat16)), tokens * width * (4 + 4 + 2 + 2 + 2))
+        report(f"tobadra.combine_weighted/{shape}", timed(lambda: moe.combine_weighted(z, where, weights, x, None, None)), tokens * (top + 1) * width * 2)
+        # heads to their buffers and pages
+        proj = torch.randn(tokens, 2 * heads * dim + 2 * kv_heads * dim + kv_heads * vdim + heads * vdim, device=dev)
+        q = torch.empty(tokens, 2 * heads * dim, dtype=torch.bfloat16, device=dev)
+        cache = (torch.randn(rows * per_row, 2, kv_heads, page, vdim, device=dev) * 0.5).to(torch.bfloat16)
+        ones = torch.ones(dim, device=dev)
+        k_off, v_off = 2 * heads * dim, 2 * (heads + kv_heads) * dim
+        g_off = v_off + kv_heads * vdim
+        report(f"differential.heads_store/{shape}", timed(lambda: ops.heads_store(proj, 0, k_off, v_off, heads, kv_heads, dim, vdim, positions, q_out=q, maps=2, q_norm=ones, k_norm=ones,
+                                                                               eps=1e-6, cache=cache, block_table=table, token_row=token_row, page_size=page)), tokens * g_off * 6)
+        s_cols = (heads + 2 * kv_heads) * s_dim
+        s_proj, s_bias = torch.randn(tokens, s_cols + 8 * -(-heads // 8), device=dev), torch.randn(s_cols, device=dev)
+        s_q = torch.empty(tokens, heads * s_dim, dtype=torch.bfloat16, device=dev)
+        s_cache = (torch.randn(rows * per_row, 2, kv_heads, page, s_dim, device=dev) * 0.5).to(torch.bfloat16)
+        report(f"sinks.heads_store/{shape}", timed(lambda: ops.heads_store(s_proj, 0, heads * s_dim, (heads + kv_heads) * s_dim, heads, kv_heads, s_dim, s_dim, positions, q_out=s_q, bias=s_bias,
+                                                                        cache=s_cache, block_table=table, token_row=token_row, page_size=page)), tokens * s_cols * 6)
+        report(f"tobadra.heads_prepare/{shape}", timed(lambda: ops.heads_prepare_wide(s_proj, 0, heads * s_dim, (heads + kv_heads) * s_dim, heads, kv_heads, s_dim, s_dim, positions, q_out=s_q,
+                                                                                   cache=s_cache, block_table=table, token_row=token_row, page_size=page)), tokens * s_cols * 6)
+        # attention: two maps per head; sinks and a gate per head; the windowed attention of the closest model
+        fake_rows = [types.SimpleNamespace(count=c, position=before) for c in counts]
+        seen = lambda w: sum(min(p + 1, w) for p in positions.tolist())
+        gate = proj[:, g_off:]
+        attn = torch.empty(tokens, heads * vdim, dtype=torch.bfloat16, device=dev)
+        d_tiles, d_items = fast.plan(fake_rows, fast.tile_tokens(2 * heads, kv_heads, fast.differential_tile_rows(vdim, page)))
+        after = (dim ** -0.5, window, keep, gate, 0.5, 1e-6, 0.5, attn)
+        if len(d_tiles):
+            d_dev = torch.tensor(d_tiles, dtype=torch.int32, device=dev)
+            run = lambda: fast.differential_tiles(q, heads, cache, table, token_row, positions, d_dev, len(d_tiles) // 3, *after)
+        else:
+            d_dev = torch.tensor(d_items, dtype=torch.int32, device=dev)
+            d_splits = fast.choose_splits(len(d_items), 2 * heads, kv_heads, min(context, window + keep + 2 * fast.KEY_TILE))
+            run = lambda: fast.differential_tokens(q, heads, cache, table, token_row, positions, d_dev, len(d_items), d_splits, *after)
+        keys = rows * min(context, window + keep)
+        report(f"differential.attention/{shape}", timed(run), keys * kv_heads * (2 * dim + vdim) * 2 + tokens * heads * (2 * dim * 2 + vdim * (2 + 4)),
+               bf16_flops=4.0 * (seen(window) + keep * tokens) * heads * (dim + vdim))
+        tile = fast.tile_rows(s_dim, page)
+        tiles, items = fast.plan(fake_rows, fast.tile_tokens(heads, kv_heads, tile))
+        sink = torch.zeros(heads, device=dev)
+        s_gate = s_proj[:, s_cols:][:, :heads]
+        s_attn = torch.empty(tokens, heads * s_dim, dtype=torch.bfloat16, device=dev)
+        work = torch.tensor(tiles if len(tiles) else items, dtype=torch.int32, device=dev)
+        splits = fast.choose_splits(max(1, len(items)), heads, kv_heads, min(context, s_window + fast.KEY_TILE))
+        for label, extras in (("sinks.attention", {"sinks": sink, "gate": s_gate}), ("tobadra.windowed_attention", {})):
+            if len(tiles):
+                run = lambda: fast.attention_tiles(s_q, heads, s_cache, table, token_row, positions, work, len(tiles) // 3, s_dim ** -0.5, s_window, s_attn, tile_size=tile, **extras)
+            else:
+                run = lambda: fast.attention_tokens(s_q, heads, s_cache, table, token_row, positions, work, len(items), splits, s_dim ** -0.5, s_window, s_attn, **extras)
+            report(f"{label}/{shape}", timed(run), rows * min(context, s_window) * 2 * kv_heads * s_dim * 2 + tokens * heads * s_dim * 4, bf16_flops=4.0 * seen(s_window) * heads * s_dim)
+        # experts: router, plan, gather, the products with and without the activation in the first one's epilogue
+        report(f"experts.route_softmax/{shape}", timed(lambda: moe.route_softmax(x, router, bias, top)), tokens * width * 2 + count * width * 4)
+        report(f"tobadra.route_scored/{shape}", timed(lambda: moe.route_scored(x, router, bias, top, 0, 0, 1.0)), tokens * width * 2 + count * width * 4)
+        report(f"experts.plan/{shape}", timed(lambda: moe.plan(chosen, None, count)), tokens * top * 16)
+        report(f"experts.gather/{shape}", timed(lambda: moe.gather(x, where)), tokens * top * width * 4)
+        gathered = moe.gather(x, where)
+        w_up = (torch.randn(count, inner, width, device=dev) * 0.02).to(torch.bfloat16)
+        w_down = (torch.randn(count, width, inner, device=dev) * 0.02).to(torch.bfloat16)
+        used = int(torch.unique(chosen).numel())
+        moved = used * inner * width * 2 + tokens * top * (width + inner) * 2
+        flops = 2.0 * tokens * top * inner * width
+        report(f"experts.up_product_with_activation/{shape}", timed(lambda: moe.grouped_linear(gathered, w_up, where, "relu_squared")), moved, bf16_flops=flops)
+        act = moe.grouped_linear(gathered, w_up, where, "relu_squared")
+        report(f"experts.down_product/{shape}", timed(lambda: moe.grouped_linear(act, w_down, where)), moved, bf16_flops=flops)
+        report(f"tobadra.up_product_then_gelu/{shape}", timed(lambda: ops.gelu_erf(moe.grouped_linear(gathered, w_up, where))), moved, bf16_flops=flops)
+    logits = torch.randn(8, 32000, device=dev)
+    report("soft_cap/decode_8", timed(lambda: ops.soft_cap_(logits, 30.0)), logits.numel() * 8)
+    report("tobadra.scale_logits/decode_8", timed(lambda: ops.scale_(logits, 1.0)), logits.numel() * 8)
+    return out
+
+
+def zurevik_workload(args) -> int:
+    """Prefill (one prompt of 2,048 tokens in one step) and decode (batch 8 from a context of 2,048) of the Zurevik design at two sizes that
+    resemble real layers, beside the closest model of the package, Tobadra with windowed attention and experts in every layer, at equal width, heads, windows,
+    experts and number of layers; random weights."""
+    import torch
+
+    from hyperion_b200.api import Engine
+    from hyperion_b200.config import TobadraConfig, ZurevikConfig
+
+    measured, kind = peaks()
+    for name, size in ZUREVIK_SIZES.items():
+        if args.size and name != args.size:
+            continue
+        arms = {"zurevik": ("Zurevik", ZurevikConfig.from_dict(zurevik_document(size))), "tobadra": ("Tobadra", TobadraConfig.from_dict(zurevik_like_document(size)))}
+        line = {"workload": "zurevik", "size": name, "dtype": "bf16", "data": "synthetic: random weights and token ids",
+                "layers": "S D D S' D S D S', all with experts, beside eight layers of windowed attention with experts", "peaks": kind}
+        for arm, (architecture, config) in arms.items():
+            engine = Engine.from_random(architecture, config, seed=0, dtype="bfloat16", page_size=16, max_tokens=8 * (PROMPT + 256), max_requests=8)
+            prefill = time_prefill(engine)
+            decode = time_decode(engine, 8, 16, max(3, args.warmup), decode_tokens=max(3, args.warmup) + 160)
+            line[arm] = {"prefill_ms": round(prefill["ms"], 3), "prefill_tokens_per_s": round(PROMPT / prefill["ms"] * 1e3),
+                         "decode_ms_per_step": round(decode["ms_per_step"], 4), "decode_tokens_per_s": round(decode["tok_s"], 1),
+                         "decode_launches_per_step": round(decode["launches"] / decode["steps"], 1)}
+            del engine
+            torch.cuda.empty_cache()
+        if not args.skip_points:
+            line["kernels"] = zurevik_kernels(size, measured)
+        print(json.dumps(line), flush=True)
+    return 0
+
+
 def main() -> int:
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
@@ -1020,13 +1204,13 @@ def main() -> int:
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
     parser.add_argument("--skip-points", action="store_true", help="leave out the batch 1 / 64 points, prefill and e2e")
     parser.add_argument("--only", default=None, choices=["prefill"], help="time one part alone (for profiling)")
-    parser.add_argument("--workload", default=None, choices=["mixed-1.5b", "batch-32b", "reference-tables", "nunivik", "mirovik", "kudazen", "tobadra"],
+    parser.add_argument("--workload", default=None, choices=["mixed-1.5b", "batch-32b", "reference-tables", "nunivik", "mirovik", "kudazen", "tobadra", "zurevik"],
                         help="one of the other workloads instead: 128 requests with prompts of 16..4096 tokens and 256 decoded tokens "
                              "each through generate() at the 1.5B shape; batch 16 with prompts of 4,096 and 512 decoded tokens at the 32B shape; "
                              "or the reference's own published tables (decode by batch at context 512, prefill by length) at the 0.5B and 7B shapes; "
                              "or the Nunivik design at two layer sizes beside the Qwen2 model of equal size, with its own kernels timed alone; "
                              "or the Mirovik design at two layer sizes beside the Nunivik model of equal size, likewise")
-    parser.add_argument("--size", default=None, choices=["2k", "4k"], help="with --workload nunivik, mirovik, kudazen or tobadra: one of its sizes only")
+    parser.add_argument("--size", default=None, choices=["2k", "4k"], help="with --workload nunivik, mirovik, kudazen, tobadra or zurevik: one of its sizes only")
     args = parser.parse_args()
     if args.impl == "reference":
         return reference_arm()
@@ -1040,6 +1224,8 @@ def main() -> int:
         return kudazen_workload(args)
     if args.workload == "tobadra":
         return tobadra_workload(args)
+    if args.workload == "zurevik":
+        return zurevik_workload(args)
     if args.workload:
         return other_workload(args.workload)
     if args.gpus != 1 or int(os.environ.get("WORLD_SIZE", "1")) != 1:
