@@ -532,72 +532,96 @@ __device__ __forceinline__ void fetch_entries(const float* p, const float* bias,
     }
 }
 
-// Heads `part`, `part + parts`, ... of a projection; `place(head)` is where a head goes (null: nowhere).  Every lane of a warp makes the same
-// number of rounds, because the norm's sum crosses lanes.
-template <int VEC, typename TO, typename Place>
-__device__ __forceinline__ void store_heads(const float* all, const float* bias, int heads, int dim, const float* weight, float eps, int lanes, int part, int parts,
-                                            Place place) {
-    const int per_block = STORE_THREADS / lanes, group = threadIdx.x / lanes, lane = threadIdx.x & (lanes - 1);
-    const int groups_per_warp = 32 / lanes, warp_first = (threadIdx.x >> 5) * groups_per_warp;
-    for (int round = 0; round * per_block * parts + part * per_block + warp_first < heads; ++round) {
-        const int head = round * per_block * parts + part * per_block + group;
-        const bool there = head < heads;
-        const float* p = all + (size_t)(there ? head : 0) * dim;
-        const float* b = bias ? bias + (size_t)(there ? head : 0) * dim : nullptr;
-        float inv = 1.f;
+// A head of `dim` entries by a group of `lanes` lanes.  Every lane of a warp comes through here together, because the norm's sum crosses lanes (a
+// lane without a head brings `dst` null and any readable p).
+template <int VEC, typename TO>
+__device__ __forceinline__ void store_head(const float* p, const float* bias, int dim, const float* weight, float eps, int lanes, bool norm_anywhere, TO* dst) {
+    const int lane = threadIdx.x & (lanes - 1);
+    float kept[VEC];  // a head that its lanes hold in one round is read once
+    float inv = 1.f;
+    const bool one_round = dim <= lanes * VEC;
+    if (one_round && lane * VEC < dim) fetch_entries<VEC>(p + lane * VEC, bias ? bias + lane * VEC : nullptr, kept);
+    if (norm_anywhere) {
+        float sum = 0.f;
         if (weight) {
-            float sum = 0.f;
             for (int i = lane * VEC; i < dim; i += lanes * VEC) {
                 float v[VEC];
-                fetch_entries<VEC>(p + i, b ? b + i : nullptr, v);
+                if (one_round) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) v[e] = kept[e];
+                } else {
+                    fetch_entries<VEC>(p + i, bias ? bias + i : nullptr, v);
+                }
 #pragma unroll
                 for (int e = 0; e < VEC; ++e) sum = fmaf(v[e], v[e], sum);
             }
-            for (int offset = lanes / 2; offset > 0; offset >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
-            inv = 1.0f / sqrtf(sum / (float)dim + eps);
         }
-        TO* dst = there ? place(head) : nullptr;
-        if (!dst) continue;
-        for (int i = lane * VEC; i < dim; i += lanes * VEC) {
-            float v[VEC];
-            fetch_entries<VEC>(p + i, b ? b + i : nullptr, v);
-            if (weight) {
+        for (int offset = lanes / 2; offset > 0; offset >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
+        if (weight) inv = 1.0f / sqrtf(sum / (float)dim + eps);
+    }
+    if (!dst) return;
+    for (int i = lane * VEC; i < dim; i += lanes * VEC) {
+        float v[VEC];
+        if (one_round) {
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) v[e] *= inv * weight[i + e];
-            }
-            if constexpr (VEC == 4) store4(dst + i, v);
-            else dst[i] = from_float<TO>(v[0]);
+            for (int e = 0; e < VEC; ++e) v[e] = kept[e];
+        } else {
+            fetch_entries<VEC>(p + i, bias ? bias + i : nullptr, v);
         }
+        if (weight) {
+            float w[VEC];
+            if constexpr (VEC == 4) load4(weight + i, w);
+            else w[0] = weight[i];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[e] *= inv * w[e];
+        }
+        if constexpr (VEC == 4) store4(dst + i, v);
+        else dst[i] = from_float<TO>(v[0]);
     }
 }
 
+// A group of `lanes` lanes per head: the token's query heads first, then its keys, then its values (a value is stored in runs of head_dim entries, so
+// that every group does the same amount of work).
 template <int VEC, typename TO>
 __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float* __restrict__ x, int stride, const float* __restrict__ bias, int q_off, int k_off,
                                                                     int v_off, int q_heads, int k_heads, int v_heads, int maps, int head_dim, int v_dim,
                                                                     const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, int lanes,
-                                                                    int v_lanes, const int* __restrict__ positions, TO* __restrict__ q_out, int q_out_stride,
+                                                                    const int* __restrict__ positions, TO* __restrict__ q_out, int q_out_stride,
                                                                     TO* __restrict__ k_cache, TO* __restrict__ v_cache, size_t page_stride, size_t head_stride,
                                                                     int token_stride, const int* __restrict__ block_table, int table_width,
                                                                     const int* __restrict__ token_row, int page_size, int pages, int* status) {
     let_next_kernel_start();
     wait_for_previous_kernels();
-    const int t = blockIdx.x, part = blockIdx.y, parts = gridDim.y;
+    const int t = blockIdx.x, runs = (v_dim + head_dim - 1) / head_dim;
+    const int item = blockIdx.y * (STORE_THREADS / lanes) + threadIdx.x / lanes;
+    const int stored = k_cache ? k_heads + v_heads * runs : 0;
     const float* row = x + (size_t)t * stride;
-    store_heads<VEC, TO>(row + q_off, bias ? bias + q_off : nullptr, q_heads, head_dim, q_norm, eps, lanes, part, parts,
-                         [&](int head) { return q_out + (size_t)t * q_out_stride + (size_t)head * head_dim; });
-    if (!k_cache) return;
-    const int pos = positions[t], block = pos / page_size;
-    int page = (pos >= 0 && block < table_width) ? block_table[(size_t)token_row[t] * table_width + block] : -1;
-    if (page < 0 || page >= pages) {
-        if (threadIdx.x == 0) atomicOr(status, HB_STATUS_BAD_PAGE);
-        page = -1;
+    int col = q_off, dim = head_dim;
+    const float* weight = nullptr;
+    TO* dst = nullptr;
+    if (item < q_heads) {
+        col = q_off + item * head_dim;
+        weight = q_norm;
+        dst = q_out + (size_t)t * q_out_stride + (size_t)item * head_dim;
+    } else if (item < q_heads + stored) {
+        const int pos = positions[t], block = pos / page_size;
+        const int page = (pos >= 0 && block < table_width) ? block_table[(size_t)token_row[t] * table_width + block] : -1;
+        const bool there = page >= 0 && page < pages;
+        if (!there) atomicOr(status, HB_STATUS_BAD_PAGE);
+        const size_t at = there ? (size_t)page * page_stride + (size_t)(pos - block * page_size) * token_stride : 0;
+        const int which = item - q_heads;
+        if (which < k_heads) {
+            col = k_off + which * head_dim;
+            weight = k_norm;
+            if (there) dst = k_cache + at + (size_t)(which / maps) * head_stride + (size_t)(which % maps) * head_dim;
+        } else {
+            const int head = (which - k_heads) / runs, first = ((which - k_heads) % runs) * head_dim;
+            col = v_off + head * v_dim + first;
+            dim = min(head_dim, v_dim - first);
+            if (there) dst = v_cache + at + (size_t)head * head_stride + first;
+        }
     }
-    const size_t at = page >= 0 ? (size_t)page * page_stride + (size_t)(pos - block * page_size) * token_stride : 0;
-    store_heads<VEC, TO>(row + k_off, bias ? bias + k_off : nullptr, k_heads, head_dim, k_norm, eps, lanes, part, parts, [&](int head) {
-        return page >= 0 ? k_cache + at + (size_t)(head / maps) * head_stride + (size_t)(head % maps) * head_dim : nullptr;
-    });
-    store_heads<VEC, TO>(row + v_off, bias ? bias + v_off : nullptr, v_heads, v_dim, nullptr, 0.f, v_lanes, part, parts,
-                         [&](int head) { return page >= 0 ? v_cache + at + (size_t)head * head_stride : nullptr; });
+    store_head<VEC, TO>(row + col, bias ? bias + col : nullptr, dim, weight, eps, lanes, q_norm || k_norm, dst);
 }
 
 int lanes_for(int pieces) {
@@ -616,19 +640,17 @@ HB_EXPORT int hb_heads_store(const float* x, int tokens, int stride, const float
     if (head_dim <= 0 || v_dim <= 0 || q_heads <= 0 || !q_out || maps < 1) return HB_UNSUPPORTED_SIZE;
     if (k_cache && (k_heads <= 0 || v_heads <= 0 || k_heads != v_heads * maps || !v_cache || page_size <= 0)) return HB_BAD_ARGUMENT;
     const uintptr_t store_mask = out_is_bf16 ? 7 : 15;
-    bool by_four = ((stride | q_off | head_dim | q_out_stride) & 3) == 0 && (((uintptr_t)x | (uintptr_t)bias) & 15) == 0 && ((uintptr_t)q_out & store_mask) == 0;
+    bool by_four = ((stride | q_off | head_dim | q_out_stride) & 3) == 0 && (((uintptr_t)x | (uintptr_t)bias | (uintptr_t)q_norm | (uintptr_t)k_norm) & 15) == 0 && ((uintptr_t)q_out & store_mask) == 0;
     if (k_cache)
         by_four = by_four && ((k_off | v_off | v_dim | token_stride) & 3) == 0 && ((page_stride | head_stride) & 3) == 0 &&
                   (((uintptr_t)k_cache | (uintptr_t)v_cache) & store_mask) == 0;
-    const int vec = by_four ? 4 : 1, lanes = lanes_for((head_dim + vec - 1) / vec), v_lanes = lanes_for((v_dim + vec - 1) / vec);
-    const int most = q_heads > k_heads ? q_heads : k_heads, rounds = (most * lanes + STORE_THREADS - 1) / STORE_THREADS;
-    int parts = tokens >= 512 ? 1 : 512 / tokens;  // few tokens: a token's heads over several blocks
-    parts = parts > rounds ? rounds : parts;
-    parts = parts < 1 ? 1 : (parts > 1024 ? 1024 : parts);
-    const dim3 grid(tokens, parts);
+    const int vec = by_four ? 4 : 1, lanes = lanes_for((head_dim + vec - 1) / vec), runs = (v_dim + head_dim - 1) / head_dim;
+    const long long items = (long long)q_heads + (k_cache ? k_heads + (long long)v_heads * runs : 0), blocks = (items * lanes + STORE_THREADS - 1) / STORE_THREADS;
+    if (blocks > 65535) return HB_UNSUPPORTED_SIZE;
+    const dim3 grid(tokens, (unsigned)blocks);
 #define HB_STORE(VEC, TO)                                                                                                                                     \
     return launch_after_previous(heads_store_kernel<VEC, TO>, grid, dim3(STORE_THREADS), 0, stream, x, stride, bias, q_off, k_off, v_off, q_heads, k_heads,    \
-                                 v_heads, maps, head_dim, v_dim, q_norm, k_norm, eps, lanes, v_lanes, positions, (TO*)q_out, q_out_stride, (TO*)k_cache,       \
+                                 v_heads, maps, head_dim, v_dim, q_norm, k_norm, eps, lanes, positions, (TO*)q_out, q_out_stride, (TO*)k_cache,       \
                                  (TO*)v_cache, (size_t)page_stride, (size_t)head_stride, token_stride, block_table, table_width, token_row, page_size, pages,  \
                                  status)
     if (out_is_bf16) {

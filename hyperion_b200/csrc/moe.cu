@@ -197,20 +197,27 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_softmax_kernel(const 
     }
     __syncthreads();
     const bool by_four = (hidden & 3) == 0 && (((uintptr_t)router) & 15) == 0;
-    for (int e = warp; e < experts; e += ROUTE_THREADS / 32) {
-        const float* w = router + (size_t)e * hidden;
-        float part[TOKENS][4];
+    // a warp takes two experts at a time, so that what it reads of the rows serves both
+    for (int e = 2 * warp; e < experts; e += ROUTE_THREADS / 16) {
+        const int there = min(2, experts - e);
+        const float* w[2] = {router + (size_t)e * hidden, router + (size_t)(e + there - 1) * hidden};
+        float part[2][TOKENS][4];
 #pragma unroll
-        for (int j = 0; j < TOKENS; ++j) part[j][0] = part[j][1] = part[j][2] = part[j][3] = 0.f;
+        for (int s = 0; s < 2; ++s)
+#pragma unroll
+            for (int j = 0; j < TOKENS; ++j) part[s][j][0] = part[s][j][1] = part[s][j][2] = part[s][j][3] = 0.f;
         if (by_four) {
 #pragma unroll 4
             for (int i = lane * 4; i < hidden; i += 128) {
-                const float4 wv = *reinterpret_cast<const float4*>(w + i);
+                const float4 wv[2] = {*reinterpret_cast<const float4*>(w[0] + i), *reinterpret_cast<const float4*>(w[1] + i)};
 #pragma unroll
                 for (int j = 0; j < TOKENS; ++j) {
                     const float4 rv = *reinterpret_cast<const float4*>(shared + (size_t)j * padded + i);
-                    part[j][0] = fmaf(rv.x, wv.x, part[j][0]); part[j][1] = fmaf(rv.y, wv.y, part[j][1]);
-                    part[j][2] = fmaf(rv.z, wv.z, part[j][2]); part[j][3] = fmaf(rv.w, wv.w, part[j][3]);
+#pragma unroll
+                    for (int s = 0; s < 2; ++s) {
+                        part[s][j][0] = fmaf(rv.x, wv[s].x, part[s][j][0]); part[s][j][1] = fmaf(rv.y, wv[s].y, part[s][j][1]);
+                        part[s][j][2] = fmaf(rv.z, wv[s].z, part[s][j][2]); part[s][j][3] = fmaf(rv.w, wv[s].w, part[s][j][3]);
+                    }
                 }
             }
         } else {
@@ -219,13 +226,18 @@ __global__ void __launch_bounds__(ROUTE_THREADS) moe_route_softmax_kernel(const 
                 for (int c = 0; c < 4; ++c)
                     if (i + c < hidden)
 #pragma unroll
-                        for (int j = 0; j < TOKENS; ++j) part[j][c] = fmaf(shared[(size_t)j * padded + i + c], w[i + c], part[j][c]);
-        }
-        const float b = bias ? bias[e] : 0.f;
+                        for (int s = 0; s < 2; ++s)
 #pragma unroll
-        for (int j = 0; j < TOKENS; ++j) {
-            const float sum = warp_sum((part[j][0] + part[j][1]) + (part[j][2] + part[j][3]));
-            if (lane == 0) logits[j * experts + e] = sum + b;
+                            for (int j = 0; j < TOKENS; ++j) part[s][j][c] = fmaf(shared[(size_t)j * padded + i + c], w[s][i + c], part[s][j][c]);
+        }
+#pragma unroll
+        for (int s = 0; s < 2; ++s) {
+            const float b = bias && s < there ? bias[e + s] : 0.f;
+#pragma unroll
+            for (int j = 0; j < TOKENS; ++j) {
+                const float sum = warp_sum((part[s][j][0] + part[s][j][1]) + (part[s][j][2] + part[s][j][3]));
+                if (lane == 0 && s < there) logits[j * experts + e + s] = sum + b;
+            }
         }
     }
     __syncthreads();

@@ -12,8 +12,8 @@
 //   the plan kernel just before) and skip the same tiles, so their counters stay in step.  Every wait is bounded; when one runs
 //   out the status word says so, all roles leave their loops, tensor memory is freed and the block returns.
 // * The rows kernel (steps of a few tokens) streams each used expert's matrix once: a block takes the real rows of one
-//   tile (tile_rows[i] of them, eight at a time) into shared memory and its warps walk output columns, every lane reading
-//   16 bytes of the matrix row per step.  Such a step is bound by the bytes of the matrices it touches, not by arithmetic.
+//   tile (tile_rows[i] of them, eight at a time) into shared memory and its warps walk output columns two at a time, every lane reading
+//   16 bytes of both matrix rows per step.  Such a step is bound by the bytes of the matrices it touches, not by arithmetic.
 #include "gemm_tcgen05.cuh"
 
 namespace {
@@ -183,11 +183,76 @@ int launch_grouped(const CUtensorMap& map_x, const CUtensorMap& map_w, const Gro
 }
 
 // ---------------------------------------------------------------- a few rows per expert: the matrices stream once
-constexpr int ROWS_AT_ONCE = 8, COLUMNS_PER_BLOCK = 32, ROWS_THREADS = 256;
+constexpr int ROWS_AT_ONCE = 8, COLUMNS_PER_BLOCK = 32, COLUMNS_AT_ONCE = 2, ROWS_THREADS = 256;
 
-__global__ void __launch_bounds__(ROWS_THREADS) gemm_grouped_rows_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, bf16* __restrict__ c,
-                                                                         const int* __restrict__ tile_expert, const int* __restrict__ tile_rows, int pad,
-                                                                         int n, int k, int act) {
+// Columns `col` and `col + 1` of ROWS rows in shared memory: a lane takes every 32nd 16-byte piece of the matrix rows, several of them asked for
+// before the first is used (the step is bound by how many bytes are on their way), the lanes meet in a butterfly.  Every sum has the same
+// shape whatever ROWS is.
+template <int ROWS>
+__device__ __forceinline__ void stream_columns(const bf16* __restrict__ first_row, int columns, const bf16* rows, int chunks, float (&sum)[COLUMNS_AT_ONCE][ROWS]) {
+    const int lane = threadIdx.x & 31;
+    const size_t k = (size_t)chunks * 8;
+#pragma unroll
+    for (int c = 0; c < COLUMNS_AT_ONCE; ++c)
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) sum[c][r] = 0.f;
+    const bf16* second = first_row + (columns > 1 ? k : 0);  // an odd last column is read twice and stored once
+#pragma unroll 4
+    for (int piece = lane; piece < chunks; piece += 32) {
+        const uint4 raw[COLUMNS_AT_ONCE] = {__ldg(reinterpret_cast<const uint4*>(first_row + piece * 8)), __ldg(reinterpret_cast<const uint4*>(second + piece * 8))};
+        float w[COLUMNS_AT_ONCE][8];
+#pragma unroll
+        for (int c = 0; c < COLUMNS_AT_ONCE; ++c) {
+            const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw[c]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(p[i]); w[c][2 * i] = f.x; w[c][2 * i + 1] = f.y; }
+        }
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            const uint4 xr = *reinterpret_cast<const uint4*>(rows + (size_t)r * k + piece * 8);
+            const __nv_bfloat162* xp = reinterpret_cast<const __nv_bfloat162*>(&xr);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float2 f = __bfloat1622float2(xp[i]);
+#pragma unroll
+                for (int c = 0; c < COLUMNS_AT_ONCE; ++c) {
+                    sum[c][r] = fmaf(f.x, w[c][2 * i], sum[c][r]);
+                    sum[c][r] = fmaf(f.y, w[c][2 * i + 1], sum[c][r]);
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int c = 0; c < COLUMNS_AT_ONCE; ++c)
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) sum[c][r] = warp_sum(sum[c][r]);
+}
+
+template <int ROWS>
+__device__ __forceinline__ void stream_tile(const bf16* __restrict__ we, const bf16* rows, bf16* __restrict__ c, int count, int n, int k, int act) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int j = warp * COLUMNS_AT_ONCE; j < COLUMNS_PER_BLOCK; j += ROWS_THREADS / 32 * COLUMNS_AT_ONCE) {
+        const int col = blockIdx.x * COLUMNS_PER_BLOCK + j;
+        if (col >= n) break;
+        float sum[COLUMNS_AT_ONCE][ROWS];
+        stream_columns<ROWS>(we + (size_t)col * k, n - col, rows, k / 8, sum);
+        const int r = lane % ROWS, which = lane / ROWS;  // lane: row r of column col + which
+        if (which < COLUMNS_AT_ONCE && r < count && col + which < n) {
+            float mine = sum[0][0];
+#pragma unroll
+            for (int cc = 0; cc < COLUMNS_AT_ONCE; ++cc)
+#pragma unroll
+                for (int rr = 0; rr < ROWS; ++rr)
+                    if (which == cc && r == rr) mine = sum[cc][rr];
+            c[(size_t)r * n + col + which] = __float2bfloat16_rn(activated(mine, act));
+        }
+    }
+}
+
+// row_token: null, or the row of `a` that stands in a slot (the rows then need not be gathered first).
+__global__ void __launch_bounds__(ROWS_THREADS) gemm_grouped_rows_kernel(const bf16* __restrict__ a, int a_stride, const int* __restrict__ row_token,
+                                                                         const bf16* __restrict__ w, bf16* __restrict__ c, const int* __restrict__ tile_expert,
+                                                                         const int* __restrict__ tile_rows, int pad, int n, int k, int act) {
     extern __shared__ __align__(16) unsigned char rows_raw[];
     bf16* rows = reinterpret_cast<bf16*>(rows_raw);  // [ROWS_AT_ONCE, k]
     let_next_kernel_start();
@@ -196,54 +261,26 @@ __global__ void __launch_bounds__(ROWS_THREADS) gemm_grouped_rows_kernel(const b
     const int expert = tile_expert[tile];
     if (expert < 0) return;
     const int real = tile_rows[tile];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bf16* we = w + (size_t)expert * n * k;
     const int chunks = k / 8;  // 16-byte pieces of a row
     for (int first = 0; first < real; first += ROWS_AT_ONCE) {
-        const int count = min(ROWS_AT_ONCE, real - first);
+        const int count = min(ROWS_AT_ONCE, real - first), filled = count <= 2 ? count : (count <= 4 ? 4 : ROWS_AT_ONCE);
         __syncthreads();
-        for (int e = threadIdx.x; e < ROWS_AT_ONCE * chunks; e += ROWS_THREADS) {
+        for (int e = threadIdx.x; e < filled * chunks; e += ROWS_THREADS) {
             const int r = e / chunks, piece = e - r * chunks;
             uint4 value = make_uint4(0, 0, 0, 0);
-            if (r < count) value = *reinterpret_cast<const uint4*>(a + (size_t)(tile * pad + first + r) * k + piece * 8);
+            if (r < count) {
+                const int slot = tile * pad + first + r;
+                value = *reinterpret_cast<const uint4*>(a + (size_t)(row_token ? row_token[slot] : slot) * a_stride + piece * 8);
+            }
             *reinterpret_cast<uint4*>(rows + (size_t)r * k + piece * 8) = value;
         }
         __syncthreads();
-        for (int j = warp; j < COLUMNS_PER_BLOCK; j += ROWS_THREADS / 32) {
-            const int col = blockIdx.x * COLUMNS_PER_BLOCK + j;
-            if (col >= n) break;
-            const bf16* wrow = we + (size_t)col * k;
-            float sum[ROWS_AT_ONCE];
-#pragma unroll
-            for (int r = 0; r < ROWS_AT_ONCE; ++r) sum[r] = 0.f;
-            for (int piece = lane; piece < chunks; piece += 32) {
-                const uint4 raw = *reinterpret_cast<const uint4*>(wrow + piece * 8);
-                const __nv_bfloat162* wp = reinterpret_cast<const __nv_bfloat162*>(&raw);
-                float wf[8];
-#pragma unroll
-                for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(wp[i]); wf[2 * i] = f.x; wf[2 * i + 1] = f.y; }
-#pragma unroll
-                for (int r = 0; r < ROWS_AT_ONCE; ++r) {
-                    const uint4 xr = *reinterpret_cast<const uint4*>(rows + (size_t)r * k + piece * 8);
-                    const __nv_bfloat162* xp = reinterpret_cast<const __nv_bfloat162*>(&xr);
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) {
-                        const float2 f = __bfloat1622float2(xp[i]);
-                        sum[r] = fmaf(f.x, wf[2 * i], sum[r]);
-                        sum[r] = fmaf(f.y, wf[2 * i + 1], sum[r]);
-                    }
-                }
-            }
-#pragma unroll
-            for (int r = 0; r < ROWS_AT_ONCE; ++r) sum[r] = warp_sum(sum[r]);
-            if (lane < count) {
-                float mine = sum[0];
-#pragma unroll
-                for (int r = 1; r < ROWS_AT_ONCE; ++r)
-                    if (lane == r) mine = sum[r];
-                c[(size_t)(tile * pad + first + lane) * n + col] = __float2bfloat16_rn(activated(mine, act));
-            }
-        }
+        bf16* out = c + (size_t)(tile * pad + first) * n;
+        if (count == 1) stream_tile<1>(we, rows, out, count, n, k, act);
+        else if (count == 2) stream_tile<2>(we, rows, out, count, n, k, act);
+        else if (count <= 4) stream_tile<4>(we, rows, out, count, n, k, act);
+        else stream_tile<ROWS_AT_ONCE>(we, rows, out, count, n, k, act);
     }
 }
 }  // namespace
@@ -266,11 +303,12 @@ HB_EXPORT int hb_moe_gemm_tiles(const void* a, const void* w, void* c, const int
                      : launch_grouped<128>(map_x, map_w, p, tiles_m, tiles_n, blocks, stream);
 }
 
-// The same product for steps of a few rows; tile_rows[i]: the real rows at the start of tile i.
-HB_EXPORT int hb_moe_gemm_rows(const void* a, const void* w, void* c, const int* tile_expert, const int* tile_rows, int pad, int rows, int n, int k,
+// The same product for steps of a few rows; tile_rows[i]: the real rows at the start of tile i.  row_token (or null): the row of `a` that stands in
+// a slot, rows a_stride elements apart.
+HB_EXPORT int hb_moe_gemm_rows(const void* a, int a_stride, const int* row_token, const void* w, void* c, const int* tile_expert, const int* tile_rows, int pad, int rows, int n, int k,
                                int act, cudaStream_t stream) {
     if (rows <= 0 || n <= 0) return 0;
-    if (k <= 0 || pad <= 0 || rows % pad || (k % 8) || !tile_expert || !tile_rows) return HB_BAD_ARGUMENT;
+    if (k <= 0 || pad <= 0 || rows % pad || (k % 8) || (a_stride % 8) || !tile_expert || !tile_rows) return HB_BAD_ARGUMENT;
     if ((((uintptr_t)a | (uintptr_t)w) & 15)) return HB_BAD_ARGUMENT;
     const size_t shared = (size_t)ROWS_AT_ONCE * k * sizeof(bf16);
     if (shared > 200 * 1024 || rows / pad > 65535) return HB_UNSUPPORTED_SIZE;
@@ -281,6 +319,6 @@ HB_EXPORT int hb_moe_gemm_rows(const void* a, const void* w, void* c, const int*
         configured = shared;
     }
     const dim3 grid((n + COLUMNS_PER_BLOCK - 1) / COLUMNS_PER_BLOCK, rows / pad);
-    return launch_after_previous(gemm_grouped_rows_kernel, grid, dim3(ROWS_THREADS), shared, stream, (const bf16*)a, (const bf16*)w, (bf16*)c, tile_expert,
+    return launch_after_previous(gemm_grouped_rows_kernel, grid, dim3(ROWS_THREADS), shared, stream, (const bf16*)a, a_stride, row_token, (const bf16*)w, (bf16*)c, tile_expert,
                                  tile_rows, pad, n, k, act);
 }

@@ -12,6 +12,7 @@ from .basic import status_word
 from .native import KernelError, check, f32, i32, is_bf16, library, ptr, require_cuda, stream_ptr
 
 PAD = 128  # an expert's rows are padded to whole tiles of this many rows
+STREAM_ROWS = 8  # rows the streaming kernel takes at once
 FEW_PAIRS = 128  # steps of at most this many (token, choice) pairs stream the matrices of the experts they use instead of taking tensor-core tiles
 
 
@@ -27,6 +28,8 @@ class Plan:
     tile_expert: torch.Tensor  # [capacity / PAD] int32: the expert of a tile of rows, -1 beyond the last used tile
     tile_rows: torch.Tensor  # [capacity / PAD] int32: how many rows of a tile are taken (they come first)
     pairs: int = 0
+    pad: int = PAD  # an expert's rows are padded to tiles of this many
+    streams: bool = False  # every product of the step goes to the streaming kernel, which takes tiles of few rows and rows that are not gathered
 
 
 def route(x: torch.Tensor, router: torch.Tensor, top: int, weighted: bool = True) -> tuple[torch.Tensor, torch.Tensor]:
@@ -85,18 +88,21 @@ def capacity_for(pairs: int, experts: int, pad: int = PAD) -> int:
     return -(-(pairs + experts * (pad - 1)) // pad) * pad
 
 
-def plan(chosen: torch.Tensor, weights: torch.Tensor | None, experts: int) -> Plan:
+def plan(chosen: torch.Tensor, weights: torch.Tensor | None, experts: int, streams: bool = False) -> Plan:
     """``weights`` None: every row's weight is 1 (the weights then multiply what the experts return: :func:`combine_weighted`).  A choice
-    of ``experts`` or above (a router output without matrices) takes no row; its ``slot_of`` is -1."""
+    of ``experts`` or above (a router output without matrices) takes no row; its ``slot_of`` is -1.  ``streams``: the caller's products can all
+    take the streaming kernel (:func:`can_stream`), so a step of few pairs pads its experts to that kernel's few rows and needs no gather."""
     require_cuda(chosen, weights)
     tokens, top = chosen.shape
     pairs = tokens * top
-    capacity = capacity_for(pairs, experts)
+    streams = streams and pairs <= FEW_PAIRS
+    pad = STREAM_ROWS if streams else PAD
+    capacity = capacity_for(pairs, experts, pad)
     device = chosen.device
     out = Plan(capacity, top, torch.empty(pairs, dtype=torch.int32, device=device), torch.empty(capacity, dtype=torch.int32, device=device),
-               torch.empty(capacity, dtype=torch.float32, device=device), torch.empty(capacity // PAD, dtype=torch.int32, device=device),
-               torch.empty(capacity // PAD, dtype=torch.int32, device=device), pairs)
-    check(library("moe").hb_moe_plan(ptr(chosen), ptr(weights), i32(pairs), i32(top), i32(experts), i32(PAD), i32(capacity), ptr(out.slot_of),
+               torch.empty(capacity, dtype=torch.float32, device=device), torch.empty(capacity // pad, dtype=torch.int32, device=device),
+               torch.empty(capacity // pad, dtype=torch.int32, device=device), pairs, pad, streams)
+    check(library("moe").hb_moe_plan(ptr(chosen), ptr(weights), i32(pairs), i32(top), i32(experts), i32(pad), i32(capacity), ptr(out.slot_of),
                                      ptr(out.slot_token), ptr(out.slot_weight), ptr(out.tile_expert), ptr(out.tile_rows), stream_ptr()), "moe_plan")
     return out
 
@@ -113,6 +119,11 @@ def gather(x: torch.Tensor, where: Plan) -> torch.Tensor:
     return out
 
 
+def can_stream(dtype: torch.dtype, *inner: int) -> bool:
+    """Whether products over these inner sizes can take the streaming kernel."""
+    return dtype == torch.bfloat16 and all(k % 8 == 0 and STREAM_ROWS * k * 2 <= 200 * 1024 for k in inner)
+
+
 def takes_tensor_cores(a: torch.Tensor, w: torch.Tensor) -> bool:
     """bfloat16 operands whose rows are multiples of 16 bytes go to ``csrc/moe_gemm_tcgen05.cu``; everything else (float32, where
     every output is one chain of fused multiply-adds whatever the step's size, and odd sizes) to the plain kernel."""
@@ -124,24 +135,27 @@ ACTIVATIONS = {None: 0, "relu_squared": 1}  # what a grouped product can apply t
 
 def grouped_linear(a: torch.Tensor, w: torch.Tensor, where: Plan, activation: str | None = None) -> torch.Tensor:
     """``a`` [capacity, k] times the matrix of each tile's expert: ``w`` [experts, n, k] -> [capacity, n], float accumulation; ``activation``
-    (a key of ``ACTIVATIONS``) is applied to the float result."""
+    (a key of ``ACTIVATIONS``) is applied to the float result.  Where the plan says so (``streams``), ``a`` may be the tokens' own rows [tokens, k],
+    of which every slot takes its token's."""
     if activation not in ACTIVATIONS:
         raise KernelError(f"moe.grouped_linear: no activation {activation!r} (known: {sorted(k for k in ACTIVATIONS if k)})")
     act = i32(ACTIVATIONS[activation])
     require_cuda(a, w)
-    if a.dtype != w.dtype or not a.is_contiguous() or not w.is_contiguous() or w.dim() != 3 or w.shape[2] != a.shape[1] or a.shape[0] != where.capacity:
+    ungathered = where.streams and a.shape[0] != where.capacity
+    if a.dtype != w.dtype or not a.is_contiguous() or not w.is_contiguous() or w.dim() != 3 or w.shape[2] != a.shape[1] or (a.shape[0] != where.capacity and not ungathered):
         raise KernelError("moe.grouped_linear: dense operands of one element type, rows [capacity, k] and matrices [experts, n, k]")
     out = torch.empty((where.capacity, w.shape[1]), dtype=a.dtype, device=a.device)
     if takes_tensor_cores(a, w):
         lib = library("moe_gemm_tcgen05")
         if where.pairs <= FEW_PAIRS:
-            check(lib.hb_moe_gemm_rows(ptr(a), ptr(w), ptr(out), ptr(where.tile_expert), ptr(where.tile_rows), i32(PAD), i32(where.capacity), i32(w.shape[1]),
+            check(lib.hb_moe_gemm_rows(ptr(a), i32(a.shape[1]), ptr(where.slot_token if ungathered else None), ptr(w), ptr(out), ptr(where.tile_expert),
+                                       ptr(where.tile_rows), i32(where.pad), i32(where.capacity), i32(w.shape[1]),
                                        i32(w.shape[2]), act, stream_ptr()), "moe_gemm_rows")
         else:
             check(lib.hb_moe_gemm_tiles(ptr(a), ptr(w), ptr(out), ptr(where.tile_expert), i32(where.capacity), i32(w.shape[0]), i32(w.shape[1]),
                                         i32(w.shape[2]), act, ptr(status_word(a.device)), stream_ptr()), "moe_gemm_tiles")
         return out
-    check(library("moe").hb_moe_gemm(ptr(a), ptr(w), ptr(out), i32(is_bf16(a)), ptr(where.tile_expert), i32(PAD), i32(where.capacity), i32(w.shape[1]),
+    check(library("moe").hb_moe_gemm(ptr(a), ptr(w), ptr(out), i32(is_bf16(a)), ptr(where.tile_expert), i32(where.pad), i32(where.capacity), i32(w.shape[1]),
                                      i32(w.shape[2]), act, stream_ptr()), "moe_gemm")
     return out
 

@@ -190,8 +190,8 @@ class ChosenSoftmaxExperts(FeedForward):
 
     def forward(self, x, step):
         chosen, weights = moe.route_softmax(x, self.router, self.router_bias, self.top)
-        where = moe.plan(chosen, None, self.experts)  # the weights multiply what an expert returns, so the rows are gathered as they are
-        act = moe.grouped_linear(moe.gather(x, where), self.w_up, where, self.activation)
+        where = moe.plan(chosen, None, self.experts, moe.can_stream(x.dtype, self.hidden, self.inter))  # the weights multiply what an expert returns
+        act = moe.grouped_linear(x if where.streams else moe.gather(x, where), self.w_up, where, self.activation)
         return moe.WeightedRows(moe.grouped_linear(act, self.w_down, where), where, weights, x)
 
 
