@@ -532,57 +532,19 @@ __device__ __forceinline__ void fetch_entries(const float* p, const float* bias,
     }
 }
 
-// A head of `dim` entries by a group of `lanes` lanes.  Every lane of a warp comes through here together, because the norm's sum crosses lanes (a
-// lane without a head brings `dst` null and any readable p).
-template <int VEC, typename TO>
-__device__ __forceinline__ void store_head(const float* p, const float* bias, int dim, const float* weight, float eps, int lanes, bool norm_anywhere, TO* dst) {
-    const int lane = threadIdx.x & (lanes - 1);
-    float kept[VEC];  // a head that its lanes hold in one round is read once
-    float inv = 1.f;
-    const bool one_round = dim <= lanes * VEC;
-    if (one_round && lane * VEC < dim) fetch_entries<VEC>(p + lane * VEC, bias ? bias + lane * VEC : nullptr, kept);
-    if (norm_anywhere) {
-        float sum = 0.f;
-        if (weight) {
-            for (int i = lane * VEC; i < dim; i += lanes * VEC) {
-                float v[VEC];
-                if (one_round) {
-#pragma unroll
-                    for (int e = 0; e < VEC; ++e) v[e] = kept[e];
-                } else {
-                    fetch_entries<VEC>(p + i, bias ? bias + i : nullptr, v);
-                }
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) sum = fmaf(v[e], v[e], sum);
-            }
-        }
-        for (int offset = lanes / 2; offset > 0; offset >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
-        if (weight) inv = 1.0f / sqrtf(sum / (float)dim + eps);
-    }
-    if (!dst) return;
-    for (int i = lane * VEC; i < dim; i += lanes * VEC) {
-        float v[VEC];
-        if (one_round) {
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) v[e] = kept[e];
-        } else {
-            fetch_entries<VEC>(p + i, bias ? bias + i : nullptr, v);
-        }
-        if (weight) {
-            float w[VEC];
-            if constexpr (VEC == 4) load4(weight + i, w);
-            else w[0] = weight[i];
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) v[e] *= inv * w[e];
-        }
-        if constexpr (VEC == 4) store4(dst + i, v);
-        else dst[i] = from_float<TO>(v[0]);
-    }
-}
+// What a group of lanes does with one head: `dim` float entries at column `col` of the token's row go to `dst` (null: nowhere).
+template <typename TO>
+struct HeadJob {
+    int col, dim;
+    const float* weight;
+    TO* dst;
+};
 
-// A group of `lanes` lanes per head: the token's query heads first, then its keys, then its values (a value is stored in runs of head_dim entries, so
-// that every group does the same amount of work).
-template <int VEC, typename TO>
+// A group of `lanes` lanes per head, JOBS heads to a group: the token's query heads first, then its keys, then its values (a value is stored in runs of
+// head_dim entries, so that every group does the same amount of work).  Every lane of a warp comes through the norm's sum together, because the
+// sum crosses lanes; a lane without a head has `dst` null.  Heads that their lanes hold in one round (ONE_ROUND) are read once, all of a group's heads
+// before the first is used.
+template <int VEC, typename TO, int JOBS, bool ONE_ROUND>
 __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float* __restrict__ x, int stride, const float* __restrict__ bias, int q_off, int k_off,
                                                                     int v_off, int q_heads, int k_heads, int v_heads, int maps, int head_dim, int v_dim,
                                                                     const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, int lanes,
@@ -592,36 +554,97 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
                                                                     const int* __restrict__ token_row, int page_size, int pages, int* status) {
     let_next_kernel_start();
     wait_for_previous_kernels();
-    const int t = blockIdx.x, runs = (v_dim + head_dim - 1) / head_dim;
-    const int item = blockIdx.y * (STORE_THREADS / lanes) + threadIdx.x / lanes;
+    const int t = blockIdx.x, runs = (v_dim + head_dim - 1) / head_dim, groups = STORE_THREADS / lanes, lane = threadIdx.x & (lanes - 1);
+    const int first_item = blockIdx.y * groups * JOBS + threadIdx.x / lanes;
     const int stored = k_cache ? k_heads + v_heads * runs : 0;
     const float* row = x + (size_t)t * stride;
-    int col = q_off, dim = head_dim;
-    const float* weight = nullptr;
-    TO* dst = nullptr;
-    if (item < q_heads) {
-        col = q_off + item * head_dim;
-        weight = q_norm;
-        dst = q_out + (size_t)t * q_out_stride + (size_t)item * head_dim;
-    } else if (item < q_heads + stored) {
+    TO* key_at = nullptr;
+    TO* value_at = nullptr;
+    if (stored && first_item + (JOBS - 1) * groups >= q_heads) {  // some head of this group goes to the token's page
         const int pos = positions[t], block = pos / page_size;
         const int page = (pos >= 0 && block < table_width) ? block_table[(size_t)token_row[t] * table_width + block] : -1;
-        const bool there = page >= 0 && page < pages;
-        if (!there) atomicOr(status, HB_STATUS_BAD_PAGE);
-        const size_t at = there ? (size_t)page * page_stride + (size_t)(pos - block * page_size) * token_stride : 0;
-        const int which = item - q_heads;
-        if (which < k_heads) {
-            col = k_off + which * head_dim;
-            weight = k_norm;
-            if (there) dst = k_cache + at + (size_t)(which / maps) * head_stride + (size_t)(which % maps) * head_dim;
+        if (page >= 0 && page < pages) {
+            const size_t at = (size_t)page * page_stride + (size_t)(pos - block * page_size) * token_stride;
+            key_at = k_cache + at;
+            value_at = v_cache + at;
         } else {
-            const int head = (which - k_heads) / runs, first = ((which - k_heads) % runs) * head_dim;
-            col = v_off + head * v_dim + first;
-            dim = min(head_dim, v_dim - first);
-            if (there) dst = v_cache + at + (size_t)head * head_stride + first;
+            atomicOr(status, HB_STATUS_BAD_PAGE);
         }
     }
-    store_head<VEC, TO>(row + col, bias ? bias + col : nullptr, dim, weight, eps, lanes, q_norm || k_norm, dst);
+    auto job_of = [&](int item) {
+        HeadJob<TO> job{q_off, head_dim, nullptr, nullptr};
+        if (item < q_heads) {
+            job.col = q_off + item * head_dim;
+            job.weight = q_norm;
+            job.dst = q_out + (size_t)t * q_out_stride + (size_t)item * head_dim;
+        } else if (item < q_heads + stored) {
+            const int which = item - q_heads;
+            if (which < k_heads) {
+                job.col = k_off + which * head_dim;
+                job.weight = k_norm;
+                if (key_at) job.dst = key_at + (size_t)(which / maps) * head_stride + (size_t)(which % maps) * head_dim;
+            } else {
+                const int head = (which - k_heads) / runs, first = ((which - k_heads) % runs) * head_dim;
+                job.col = v_off + head * v_dim + first;
+                job.dim = min(head_dim, v_dim - first);
+                if (value_at) job.dst = value_at + (size_t)head * head_stride + first;
+            }
+        }
+        return job;
+    };
+    float kept[JOBS][VEC];
+    if (ONE_ROUND) {
+#pragma unroll
+        for (int u = 0; u < JOBS; ++u) {
+            const HeadJob<TO> job = job_of(first_item + u * groups);
+            const int i = lane * VEC;
+            if (i < job.dim) fetch_entries<VEC>(row + job.col + i, bias ? bias + job.col + i : nullptr, kept[u]);
+        }
+    }
+#pragma unroll
+    for (int u = 0; u < JOBS; ++u) {
+        const HeadJob<TO> job = job_of(first_item + u * groups);
+        const float* p = row + job.col;
+        const float* b = bias ? bias + job.col : nullptr;
+        float inv = 1.f;
+        if (q_norm || k_norm) {
+            float sum = 0.f;
+            if (job.weight) {
+                for (int i = lane * VEC; i < job.dim; i += lanes * VEC) {
+                    float v[VEC];
+                    if (!ONE_ROUND) fetch_entries<VEC>(p + i, b ? b + i : nullptr, v);
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        const float value = ONE_ROUND ? kept[u][e] : v[e];
+                        sum = fmaf(value, value, sum);
+                    }
+                    if (ONE_ROUND) break;
+                }
+            }
+            for (int offset = lanes / 2; offset > 0; offset >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
+            if (job.weight) inv = 1.0f / sqrtf(sum / (float)job.dim + eps);
+        }
+        if (!job.dst) continue;
+        for (int i = lane * VEC; i < job.dim; i += lanes * VEC) {
+            float v[VEC];
+            if (ONE_ROUND) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[e] = kept[u][e];
+            } else {
+                fetch_entries<VEC>(p + i, b ? b + i : nullptr, v);
+            }
+            if (job.weight) {
+                float w[VEC];
+                if constexpr (VEC == 4) load4(job.weight + i, w);
+                else w[0] = job.weight[i];
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[e] *= inv * w[e];
+            }
+            if constexpr (VEC == 4) store4(job.dst + i, v);
+            else job.dst[i] = from_float<TO>(v[0]);
+            if (ONE_ROUND) break;
+        }
+    }
 }
 
 int lanes_for(int pieces) {
@@ -645,19 +668,24 @@ HB_EXPORT int hb_heads_store(const float* x, int tokens, int stride, const float
         by_four = by_four && ((k_off | v_off | v_dim | token_stride) & 3) == 0 && ((page_stride | head_stride) & 3) == 0 &&
                   (((uintptr_t)k_cache | (uintptr_t)v_cache) & store_mask) == 0;
     const int vec = by_four ? 4 : 1, lanes = lanes_for((head_dim + vec - 1) / vec), runs = (v_dim + head_dim - 1) / head_dim;
-    const long long items = (long long)q_heads + (k_cache ? k_heads + (long long)v_heads * runs : 0), blocks = (items * lanes + STORE_THREADS - 1) / STORE_THREADS;
+    const long long items = (long long)q_heads + (k_cache ? k_heads + (long long)v_heads * runs : 0);
+    const bool one_round = head_dim <= lanes * vec;
+    const int jobs = one_round && by_four && tokens >= 256 ? 4 : 1;  // a step of few tokens spreads a token's heads over more blocks
+    const long long blocks = (items * lanes + (long long)STORE_THREADS * jobs - 1) / ((long long)STORE_THREADS * jobs);
     if (blocks > 65535) return HB_UNSUPPORTED_SIZE;
     const dim3 grid(tokens, (unsigned)blocks);
-#define HB_STORE(VEC, TO)                                                                                                                                     \
-    return launch_after_previous(heads_store_kernel<VEC, TO>, grid, dim3(STORE_THREADS), 0, stream, x, stride, bias, q_off, k_off, v_off, q_heads, k_heads,    \
-                                 v_heads, maps, head_dim, v_dim, q_norm, k_norm, eps, lanes, positions, (TO*)q_out, q_out_stride, (TO*)k_cache,       \
-                                 (TO*)v_cache, (size_t)page_stride, (size_t)head_stride, token_stride, block_table, table_width, token_row, page_size, pages,  \
+#define HB_STORE(VEC, TO, JOBS, ONE)                                                                                                                          \
+    return launch_after_previous(heads_store_kernel<VEC, TO, JOBS, ONE>, grid, dim3(STORE_THREADS), 0, stream, x, stride, bias, q_off, k_off, v_off, q_heads, \
+                                 k_heads, v_heads, maps, head_dim, v_dim, q_norm, k_norm, eps, lanes, positions, (TO*)q_out, q_out_stride, (TO*)k_cache,      \
+                                 (TO*)v_cache, (size_t)page_stride, (size_t)head_stride, token_stride, block_table, table_width, token_row, page_size, pages, \
                                  status)
-    if (out_is_bf16) {
-        if (by_four) HB_STORE(4, __nv_bfloat16);
-        HB_STORE(1, __nv_bfloat16);
-    }
-    if (by_four) HB_STORE(4, float);
-    HB_STORE(1, float);
+#define HB_STORE_TYPE(TO)                         \
+    if (jobs == 4) HB_STORE(4, TO, 4, true);      \
+    if (by_four && one_round) HB_STORE(4, TO, 1, true); \
+    if (by_four) HB_STORE(4, TO, 1, false);       \
+    HB_STORE(1, TO, 1, false)
+    if (out_is_bf16) { HB_STORE_TYPE(__nv_bfloat16); }
+    HB_STORE_TYPE(float);
+#undef HB_STORE_TYPE
 #undef HB_STORE
 }
