@@ -209,6 +209,8 @@ def all_modules() -> list[tuple[str, dict]]:
         text = path.read_text()
         if "HB_HEAD_DIM" in text:
             requests += [(module, {"HB_HEAD_DIM": d}) for d in (64, 128)]
+        elif "HB_STREAMS" in text:
+            requests += [(module, {"HB_STREAMS": n}) for n in (2, 4)]
         else:
             requests.append((module, {}))
     return requests

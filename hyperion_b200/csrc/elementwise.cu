@@ -1252,3 +1252,39 @@ HB_EXPORT int hb_soft_cap(float* x, float cap, long long count, cudaStream_t str
     const long long blocks = (count + 1023) / 1024;
     return launch_after_previous(soft_cap_kernel, dim3((unsigned)(blocks < 8192 ? blocks : 8192)), dim3(256), 0, stream, x, cap, (size_t)count);
 }
+
+// ---------------------------------------------------------------- the square of relu
+// out = max(z, 0)^2, in float, rounded once.
+template <typename T>
+__global__ void relu_squared_kernel(const T* __restrict__ x, T* __restrict__ out, size_t count) {
+    let_next_kernel_start();
+    wait_for_previous_kernels();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < count; i += (size_t)gridDim.x * blockDim.x)
+        out[i] = from_float<T>(activated(to_float(x[i]), HB_ACT_RELU_SQUARED));
+}
+
+// Eight entries per thread and access, for 16-byte aligned tensors of a multiple of eight entries.
+__global__ void relu_squared_bf16x8_kernel(const uint4* __restrict__ x, uint4* __restrict__ out, size_t eights) {
+    let_next_kernel_start();
+    wait_for_previous_kernels();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < eights; i += (size_t)gridDim.x * blockDim.x) {
+        uint4 raw = x[i];
+        __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const float2 f = __bfloat1622float2(pairs[k]);
+            pairs[k] = __floats2bfloat162_rn(activated(f.x, HB_ACT_RELU_SQUARED), activated(f.y, HB_ACT_RELU_SQUARED));
+        }
+        out[i] = raw;
+    }
+}
+
+HB_EXPORT int hb_relu_squared(const void* x, void* out, int is_bf16, long long count, cudaStream_t stream) {
+    if (count <= 0) return 0;
+    const bool eights = is_bf16 && count % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0;
+    const long long items = eights ? count / 8 : count, wanted = (items + 255) / 256;
+    const dim3 blocks((unsigned)(wanted < 16384 ? wanted : 16384));
+    if (eights) return launch_after_previous(relu_squared_bf16x8_kernel, blocks, dim3(256), 0, stream, (const uint4*)x, (uint4*)out, (size_t)items);
+    if (is_bf16) return launch_after_previous(relu_squared_kernel<__nv_bfloat16>, blocks, dim3(256), 0, stream, (const __nv_bfloat16*)x, (__nv_bfloat16*)out, (size_t)count);
+    return launch_after_previous(relu_squared_kernel<float>, blocks, dim3(256), 0, stream, (const float*)x, (float*)out, (size_t)count);
+}

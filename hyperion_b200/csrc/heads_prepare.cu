@@ -509,13 +509,25 @@ HB_EXPORT int hb_rotate_heads(void* x, int is_bf16, int tokens, int stride, int 
     return launch_status();
 }
 
-// ---------------------------------------------------------------- heads that nothing rotates
+// ---------------------------------------------------------------- heads to their buffers and pages, by groups of lanes
 // Float projections [tokens, stride] with queries at q_off, keys at k_off and values at v_off: an optional bias per column is added, every query
 // and key head passes an optional RMS norm (one weight for all of them), queries go to a dense buffer, keys and values to their pages.
+// With TURN (hb_heads_turn) queries and keys may also be divided by their root mean square without a weight, turn by their position (pairs of a
+// head's first rot_dims entries; cosine and sine times `amplitude`), and queries are multiplied by a temperature that grows with the position,
+// 1 + coef * ln(floor((p + 1) / every) + 1).
 // A key/value head may hold several keys per token (`maps` of them side by side, each a head of its own to the norm).  A group of lanes
 // serves a head, so a norm's sum has one shape whatever the launch; a lane takes VEC consecutive entries per access.
 namespace {
-constexpr int STORE_THREADS = 256;
+constexpr int STORE_THREADS = 256, TURN_PAIRS = 320;
+
+struct TurnArgs {
+    const float* inv_freq;  // [rot_dims / 2], or null: nothing turns
+    int rot_dims, rot_half; // pairs (i, i + rot_dims / 2), or (2i, 2i + 1)
+    float amplitude;
+    int unit_norm;          // queries and keys are divided by sqrt(mean(x^2) + eps)
+    float temp_coef;        // 0: no temperature
+    int temp_every;
+};
 
 template <int VEC>
 __device__ __forceinline__ void fetch_entries(const float* p, const float* bias, float (&v)[VEC]) {
@@ -538,21 +550,34 @@ struct HeadJob {
     int col, dim;
     const float* weight;
     TO* dst;
+    int kind;  // 0: a query, 1: a key, 2: a value
 };
 
 // A group of `lanes` lanes per head, JOBS heads to a group: the token's query heads first, then its keys, then its values (a value is stored in runs of
 // head_dim entries, so that every group does the same amount of work).  Every lane of a warp comes through the norm's sum together, because the
 // sum crosses lanes; a lane without a head has `dst` null.  Heads that their lanes hold in one round (ONE_ROUND) are read once, all of a group's heads
 // before the first is used.
-template <int VEC, typename TO, int JOBS, bool ONE_ROUND>
+template <int VEC, typename TO, int JOBS, bool ONE_ROUND, bool TURN>
 __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float* __restrict__ x, int stride, const float* __restrict__ bias, int q_off, int k_off,
                                                                     int v_off, int q_heads, int k_heads, int v_heads, int maps, int head_dim, int v_dim,
                                                                     const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, int lanes,
                                                                     const int* __restrict__ positions, TO* __restrict__ q_out, int q_out_stride,
                                                                     TO* __restrict__ k_cache, TO* __restrict__ v_cache, size_t page_stride, size_t head_stride,
                                                                     int token_stride, const int* __restrict__ block_table, int table_width,
-                                                                    const int* __restrict__ token_row, int page_size, int pages, int* status) {
+                                                                    const int* __restrict__ token_row, int page_size, int pages, int* status, const TurnArgs turn) {
+    __shared__ float2 turned[TURN ? TURN_PAIRS : 1];  // (cosine, sine) of every pair at this token's position
     let_next_kernel_start();
+    if constexpr (TURN) {  // positions come with the step's one copy from the host, not from a kernel
+        if (turn.inv_freq) {
+            const float at = (float)positions[blockIdx.x];
+            for (int i = threadIdx.x; i < turn.rot_dims / 2; i += STORE_THREADS) {
+                float sine, cosine;
+                sincosf(at * turn.inv_freq[i], &sine, &cosine);
+                turned[i] = make_float2(cosine * turn.amplitude, sine * turn.amplitude);
+            }
+            __syncthreads();
+        }
+    }
     wait_for_previous_kernels();
     const int t = blockIdx.x, runs = (v_dim + head_dim - 1) / head_dim, groups = STORE_THREADS / lanes, lane = threadIdx.x & (lanes - 1);
     const int first_item = blockIdx.y * groups * JOBS + threadIdx.x / lanes;
@@ -572,7 +597,7 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
         }
     }
     auto job_of = [&](int item) {
-        HeadJob<TO> job{q_off, head_dim, nullptr, nullptr};
+        HeadJob<TO> job{q_off, head_dim, nullptr, nullptr, 0};
         if (item < q_heads) {
             job.col = q_off + item * head_dim;
             job.weight = q_norm;
@@ -582,10 +607,12 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
             if (which < k_heads) {
                 job.col = k_off + which * head_dim;
                 job.weight = k_norm;
+                job.kind = 1;
                 if (key_at) job.dst = key_at + (size_t)(which / maps) * head_stride + (size_t)(which % maps) * head_dim;
             } else {
                 const int head = (which - k_heads) / runs, first = ((which - k_heads) % runs) * head_dim;
                 job.col = v_off + head * v_dim + first;
+                job.kind = 2;
                 job.dim = min(head_dim, v_dim - first);
                 if (value_at) job.dst = value_at + (size_t)head * head_stride + first;
             }
@@ -607,9 +634,10 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
         const float* p = row + job.col;
         const float* b = bias ? bias + job.col : nullptr;
         float inv = 1.f;
-        if (q_norm || k_norm) {
+        if (q_norm || k_norm || (TURN && turn.unit_norm)) {
+            const bool normed = job.weight || (TURN && turn.unit_norm && job.kind < 2);
             float sum = 0.f;
-            if (job.weight) {
+            if (normed) {
                 for (int i = lane * VEC; i < job.dim; i += lanes * VEC) {
                     float v[VEC];
                     if (!ONE_ROUND) fetch_entries<VEC>(p + i, b ? b + i : nullptr, v);
@@ -622,9 +650,13 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
                 }
             }
             for (int offset = lanes / 2; offset > 0; offset >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
-            if (job.weight) inv = 1.0f / sqrtf(sum / (float)job.dim + eps);
+            if (normed) inv = 1.0f / sqrtf(sum / (float)job.dim + eps);
         }
         if (!job.dst) continue;
+        float after = 1.f;
+        if constexpr (TURN) {
+            if (job.kind == 0 && turn.temp_coef != 0.f) after = 1.f + turn.temp_coef * logf((float)((positions[t] + 1) / turn.temp_every + 1));
+        }
         for (int i = lane * VEC; i < job.dim; i += lanes * VEC) {
             float v[VEC];
             if (ONE_ROUND) {
@@ -639,6 +671,39 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
                 else w[0] = job.weight[i];
 #pragma unroll
                 for (int e = 0; e < VEC; ++e) v[e] *= inv * w[e];
+            }
+            if constexpr (TURN) {
+                if (!job.weight) {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) v[e] *= inv;
+                }
+                if (turn.inv_freq && job.kind < 2 && i < turn.rot_dims) {
+                    const int half = turn.rot_dims / 2;
+                    float other[VEC];  // the partners of this lane's entries
+                    if (turn.rot_half && half % VEC == 0) {
+                        const int from = i < half ? i + half : i - half;
+                        fetch_entries<VEC>(p + from, b ? b + from : nullptr, other);
+#pragma unroll
+                        for (int e = 0; e < VEC; ++e) other[e] *= job.weight ? inv * job.weight[from + e] : inv;
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < VEC; ++e) {
+                            const int at = i + e, from = at >= turn.rot_dims ? at : (turn.rot_half ? (at < half ? at + half : at - half) : (at ^ 1));
+                            other[e] = (b ? p[from] + b[from] : p[from]) * (job.weight ? inv * job.weight[from] : inv);
+                        }
+                    }
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        const int at = i + e;
+                        if (at < turn.rot_dims) {
+                            const bool lower = turn.rot_half ? at < half : !(at & 1);
+                            const float2 cs = turned[turn.rot_half ? (lower ? at : at - half) : at / 2];
+                            v[e] = lower ? v[e] * cs.x - other[e] * cs.y : v[e] * cs.x + other[e] * cs.y;
+                        }
+                    }
+                }
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[e] *= after;
             }
             if constexpr (VEC == 4) store4(job.dst + i, v);
             else job.dst[i] = from_float<TO>(v[0]);
@@ -655,10 +720,10 @@ int lanes_for(int pieces) {
 }  // namespace
 
 // q_heads and k_heads count every map; k_cache null: queries only.  A key head h goes to the key/value head h / maps, its map h % maps.
-HB_EXPORT int hb_heads_store(const float* x, int tokens, int stride, const float* bias, int q_off, int k_off, int v_off, int q_heads, int k_heads, int v_heads,
-                             int maps, int head_dim, int v_dim, const float* q_norm, const float* k_norm, float eps, const int* positions, void* q_out,
-                             int q_out_stride, int out_is_bf16, void* k_cache, void* v_cache, long long page_stride, long long head_stride, int token_stride,
-                             const int* block_table, int table_width, const int* token_row, int page_size, int pages, int* status, cudaStream_t stream) {
+static int store_heads(const float* x, int tokens, int stride, const float* bias, int q_off, int k_off, int v_off, int q_heads, int k_heads, int v_heads, int maps,
+                       int head_dim, int v_dim, const float* q_norm, const float* k_norm, float eps, const int* positions, void* q_out, int q_out_stride, int out_is_bf16,
+                       void* k_cache, void* v_cache, long long page_stride, long long head_stride, int token_stride, const int* block_table, int table_width,
+                       const int* token_row, int page_size, int pages, int* status, bool turns, const TurnArgs& turn, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (head_dim <= 0 || v_dim <= 0 || q_heads <= 0 || !q_out || maps < 1) return HB_UNSUPPORTED_SIZE;
     if (k_cache && (k_heads <= 0 || v_heads <= 0 || k_heads != v_heads * maps || !v_cache || page_size <= 0)) return HB_BAD_ARGUMENT;
@@ -674,18 +739,43 @@ HB_EXPORT int hb_heads_store(const float* x, int tokens, int stride, const float
     const long long blocks = (items * lanes + (long long)STORE_THREADS * jobs - 1) / ((long long)STORE_THREADS * jobs);
     if (blocks > 65535) return HB_UNSUPPORTED_SIZE;
     const dim3 grid(tokens, (unsigned)blocks);
-#define HB_STORE(VEC, TO, JOBS, ONE)                                                                                                                          \
-    return launch_after_previous(heads_store_kernel<VEC, TO, JOBS, ONE>, grid, dim3(STORE_THREADS), 0, stream, x, stride, bias, q_off, k_off, v_off, q_heads, \
-                                 k_heads, v_heads, maps, head_dim, v_dim, q_norm, k_norm, eps, lanes, positions, (TO*)q_out, q_out_stride, (TO*)k_cache,      \
-                                 (TO*)v_cache, (size_t)page_stride, (size_t)head_stride, token_stride, block_table, table_width, token_row, page_size, pages, \
-                                 status)
-#define HB_STORE_TYPE(TO)                         \
-    if (jobs == 4) HB_STORE(4, TO, 4, true);      \
-    if (by_four && one_round) HB_STORE(4, TO, 1, true); \
-    if (by_four) HB_STORE(4, TO, 1, false);       \
-    HB_STORE(1, TO, 1, false)
-    if (out_is_bf16) { HB_STORE_TYPE(__nv_bfloat16); }
-    HB_STORE_TYPE(float);
+#define HB_STORE(VEC, TO, JOBS, ONE, TURN)                                                                                                                          \
+    return launch_after_previous(heads_store_kernel<VEC, TO, JOBS, ONE, TURN>, grid, dim3(STORE_THREADS), 0, stream, x, stride, bias, q_off, k_off, v_off, q_heads, \
+                                 k_heads, v_heads, maps, head_dim, v_dim, q_norm, k_norm, eps, lanes, positions, (TO*)q_out, q_out_stride, (TO*)k_cache,            \
+                                 (TO*)v_cache, (size_t)page_stride, (size_t)head_stride, token_stride, block_table, table_width, token_row, page_size, pages,       \
+                                 status, turn)
+#define HB_STORE_TYPE(TO, TURN)                               \
+    if (jobs == 4) HB_STORE(4, TO, 4, true, TURN);            \
+    if (by_four && one_round) HB_STORE(4, TO, 1, true, TURN); \
+    if (by_four) HB_STORE(4, TO, 1, false, TURN);             \
+    HB_STORE(1, TO, 1, false, TURN)
+    if (turns) {
+        if (out_is_bf16) { HB_STORE_TYPE(__nv_bfloat16, true); }
+        HB_STORE_TYPE(float, true);
+    }
+    if (out_is_bf16) { HB_STORE_TYPE(__nv_bfloat16, false); }
+    HB_STORE_TYPE(float, false);
 #undef HB_STORE_TYPE
 #undef HB_STORE
+}
+
+HB_EXPORT int hb_heads_store(const float* x, int tokens, int stride, const float* bias, int q_off, int k_off, int v_off, int q_heads, int k_heads, int v_heads,
+                             int maps, int head_dim, int v_dim, const float* q_norm, const float* k_norm, float eps, const int* positions, void* q_out,
+                             int q_out_stride, int out_is_bf16, void* k_cache, void* v_cache, long long page_stride, long long head_stride, int token_stride,
+                             const int* block_table, int table_width, const int* token_row, int page_size, int pages, int* status, cudaStream_t stream) {
+    return store_heads(x, tokens, stride, bias, q_off, k_off, v_off, q_heads, k_heads, v_heads, maps, head_dim, v_dim, q_norm, k_norm, eps, positions, q_out, q_out_stride,
+                       out_is_bf16, k_cache, v_cache, page_stride, head_stride, token_stride, block_table, table_width, token_row, page_size, pages, status, false,
+                       TurnArgs{nullptr, 0, 0, 1.f, 0, 0.f, 1}, stream);
+}
+
+// The same with what TurnArgs says: a norm without a weight, a rotation, a temperature on the queries.
+HB_EXPORT int hb_heads_turn(const float* x, int tokens, int stride, const float* bias, int q_off, int k_off, int v_off, int q_heads, int k_heads, int v_heads,
+                            int maps, int head_dim, int v_dim, const float* q_norm, const float* k_norm, float eps, const int* positions, void* q_out,
+                            int q_out_stride, int out_is_bf16, void* k_cache, void* v_cache, long long page_stride, long long head_stride, int token_stride,
+                            const int* block_table, int table_width, const int* token_row, int page_size, int pages, const float* inv_freq, int rot_dims, int rot_half,
+                            float amplitude, int unit_norm, float temp_coef, int temp_every, int* status, cudaStream_t stream) {
+    if (rot_dims < 0 || (rot_dims & 1) || (inv_freq && (rot_dims > head_dim || rot_dims / 2 > TURN_PAIRS)) || (temp_coef != 0.f && temp_every < 1)) return HB_UNSUPPORTED_SIZE;
+    return store_heads(x, tokens, stride, bias, q_off, k_off, v_off, q_heads, k_heads, v_heads, maps, head_dim, v_dim, q_norm, k_norm, eps, positions, q_out, q_out_stride,
+                       out_is_bf16, k_cache, v_cache, page_stride, head_stride, token_stride, block_table, table_width, token_row, page_size, pages, status, true,
+                       TurnArgs{inv_freq, inv_freq ? rot_dims : 0, rot_half, amplitude, unit_norm, temp_coef, temp_every < 1 ? 1 : temp_every}, stream);
 }

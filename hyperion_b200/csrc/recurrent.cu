@@ -14,6 +14,8 @@
 //                   (a decay per key entry computed from the token, and a bonus u that only the current token gets)
 //     channel delta: S <- diag(g) S;  u = b (v - S^T k);  S <- S + k u^T;  o = S^T q,  g_i = exp(-exp(A_log) softplus(x_i + bias_i))
 //                   (the delta rule with a decay per key entry computed from the token)
+//     given:        S <- a S + b k v^T;                              o = S^T q  with a and b given per token and head (a kernel ahead made them);
+//                   a column beyond the values takes the constant 1, so that it sums the keys: the normaliser of a matrix memory
 // Column j of S (one value dimension) never meets another column, so the work is cut by columns:
 // eight lanes share a column, each holding n / 8 of its entries in registers (groups of four
 // consecutive entries, stored as S^T so that they are one 16-byte access), and a block of 128
@@ -25,7 +27,7 @@
 
 namespace {
 constexpr int SCAN_THREADS = 128;
-enum : int { MODE_DELTA = 0, MODE_STATE_SPACE = 1, MODE_RETENTION = 2, MODE_WKV = 3, MODE_CHANNEL_DELTA = 4 };
+enum : int { MODE_DELTA = 0, MODE_STATE_SPACE = 1, MODE_RETENTION = 2, MODE_WKV = 3, MODE_CHANNEL_DELTA = 4, MODE_GIVEN = 5 };
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
@@ -86,6 +88,9 @@ struct ScanArgs {
     float* out;          // [tokens, heads * e], or null: only the states are wanted
     int heads, groups, n, n_padded, e;
     float q_scale;
+    int values;          // value columns of a head (0: e); a column from there on takes the constant 1
+    int out_e;           // columns of a head in `out` (0: e)
+    float* decays;       // [rows, heads] or null: the product of a row's decays per head (what joins segments scanned side by side)
 };
 
 template <int NG, int LPC, int CPT, int MODE>  // NG groups of four entries per lane, LPC lanes per column (n <= NG * 4 * LPC), CPT columns per thread
@@ -125,9 +130,9 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
             s[c][r][0] = v.x; s[c][r][1] = v.y; s[c][r][2] = v.z; s[c][r][3] = v.w;
         }
     }
-    const float a_rate = (MODE == MODE_RETENTION || WKV) ? 0.f : expf(a.a_log[head]);
+    const float a_rate = (MODE == MODE_RETENTION || MODE == MODE_GIVEN || WKV) ? 0.f : expf(a.a_log[head]);
     const float fixed_decay = MODE == MODE_RETENTION ? a.a_log[head] : 0.f;
-    const float bias = (MODE == MODE_RETENTION || VEC) ? 0.f : a.dt_bias[head];
+    const float bias = (MODE == MODE_RETENTION || MODE == MODE_GIVEN || VEC) ? 0.f : a.dt_bias[head];
     float w0[NPR], bonus[NPR];  // wkv: this lane's entries of the head's decay offset and bonus; channel delta: of the decay's bias
 #pragma unroll
     for (int r = 0; r < NPR; ++r) {
@@ -136,6 +141,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
         bonus[r] = (WKV && index < a.n) ? a.dt_bias[(size_t)head * a.n + index] : 0.f;
     }
     const float skip = MODE == MODE_STATE_SPACE ? a.skip[head] : 0.f;
+    float faded = 1.f;
 
     float pk[PER_WARP][NPR], pq[PER_WARP][NPR], pv[PER_WARP][VR], pdecay[PER_WARP], pstep[PER_WARP], pw[PER_WARP][VEC ? NPR : 1];
     auto prefetch = [&](int first) {
@@ -146,7 +152,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
             const size_t at = (size_t)(live ? t : t0);
             const float* k = a.k + at * a.k_stride + (size_t)group * a.n;
             const float* q = a.q + at * a.q_stride + (size_t)group * a.n;
-            const float* vals = a.v + at * a.v_stride + (size_t)head * a.e;
+            const float* vals = a.v + at * a.v_stride + (size_t)head * a.values;
 #pragma unroll
             for (int r = 0; r < NPR; ++r) {
                 const int index = lane + 32 * r;
@@ -156,7 +162,8 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
 #pragma unroll
             for (int r = 0; r < VR; ++r) {
                 const int column = lane + 32 * r;
-                pv[i][r] = (live && column < COLUMNS && col0 + column < a.e) ? vals[col0 + column] : 0.f;
+                pv[i][r] = (live && column < COLUMNS && col0 + column < a.values) ? vals[col0 + column] : 0.f;
+                if (MODE == MODE_GIVEN && live && col0 + column >= a.values) pv[i][r] = 1.f;
             }
             const float* p = a.proj + at * a.proj_stride;
             if (VEC) {
@@ -167,14 +174,14 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
                 }
             }
             pdecay[i] = (live && MODE != MODE_RETENTION && !VEC) ? p[a.decay_off + head] : 0.f;
-            pstep[i] = (live && DELTA) ? a.step[at * a.step_stride + a.step_off + head] : 0.f;
+            pstep[i] = (live && (DELTA || MODE == MODE_GIVEN)) ? a.step[at * a.step_stride + a.step_off + head] : 0.f;
         }
     };
     auto publish = [&](int buffer) {
 #pragma unroll
         for (int i = 0; i < PER_WARP; ++i) {
             const int j = warp + 4 * i;
-            float ik = 1.f, iq = 1.f;
+            float ik = 1.f, iq = MODE == MODE_GIVEN ? a.q_scale : 1.f;
             if (DELTA) {  // keys and queries become unit vectors; the query also takes the scale
                 float sum_k = 0.f, sum_q = 0.f;
 #pragma unroll
@@ -216,6 +223,9 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
                 } else if (MODE == MODE_RETENTION) {  // the head's decay is a constant of the model; keys enter as they are
                     decay = fixed_decay;
                     step = 1.f;
+                } else if (MODE == MODE_GIVEN) {
+                    decay = pdecay[i];
+                    step = pstep[i];
                 } else {
                     step = softplus_f(pdecay[i] + bias);
                     decay = expf(-a_rate * step);
@@ -305,6 +315,16 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
                         for (int i = 0; i < 4; ++i) s[c][r][i] *= decay;
                     u[c] = step * cv[c];
                 }
+                faded *= decay;
+                if (!a.out) {  // only the states are wanted: the query meets nothing
+#pragma unroll
+                    for (int c = 0; c < CPT; ++c)
+#pragma unroll
+                        for (int r = 0; r < NG; ++r)
+#pragma unroll
+                            for (int i = 0; i < 4; ++i) s[c][r][i] = fmaf(ck[r][i], u[c], s[c][r][i]);
+                    continue;
+                }
             }
 #pragma unroll
             for (int c = 0; c < CPT; ++c) {
@@ -323,13 +343,14 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
             for (int c = 0; c < CPT; ++c) {
                 const int col = col0 + cw + GROUPS * c;
                 const float out = MODE == MODE_STATE_SPACE ? fmaf(skip, cv[c], o[c]) : o[c];
-                if (l == 0 && col < a.e && a.out) a.out[((size_t)(first + j) * a.heads + head) * a.e + col] = out;
+                if (l == 0 && col < a.e && a.out) a.out[((size_t)(first + j) * a.heads + head) * a.out_e + col] = out;
             }
         }
         if (!more) break;
         publish(buffer ^ 1);
         __syncthreads();
     }
+    if (a.decays && blockIdx.x == 0 && threadIdx.x == 0) a.decays[(size_t)row * a.heads + head] = faded;
 #pragma unroll
     for (int c = 0; c < CPT; ++c) {
         const int col = col0 + cw + GROUPS * c;
@@ -343,7 +364,10 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
 }
 
 template <int MODE>
-int launch_scan(const ScanArgs& a, int rows, cudaStream_t stream) {
+int launch_scan(const ScanArgs& given, int rows, cudaStream_t stream) {
+    ScanArgs a = given;
+    if (a.values <= 0) a.values = a.e;
+    if (a.out_e <= 0) a.out_e = a.e;
     // Eight lanes per column; one column per thread for the delta rule, two for the state-space recurrence, whatever the batch (a
     // token's sums must not change with it).  Measured on a B200 at heads x e = 2,048 and 4,096 with n = 128, a prompt of 2,048
     // tokens: sixteen or thirty-two lanes per column (more warps, fewer entries each) took 1.3 to 2 times as long, because every
@@ -448,15 +472,17 @@ HB_EXPORT int hb_conv_state_update(const float* x, int x_stride, int col0, int c
 // mode 0: gated delta rule (keys and queries made unit vectors, q times q_scale; decay = exp(-exp(a_log) softplus(proj[decay_off] + dt_bias)),
 // step = sigmoid(proj[step_off])).  mode 1: state space (step = softplus(proj[decay_off] + dt_bias), decay = exp(-exp(a_log) step), skip = D).
 // The state of (slot, head) is S^T [e, n_padded] at state + slot * slot_stride + state_off; n_padded, state_off and slot_stride are multiples of 4.
+// decays [rows, heads] (modes 1 and 2; or null) receives the product of every row's decays.
 HB_EXPORT int hb_state_scan(int mode, const float* conv, int conv_stride, int k_off, int q_off, int v_off, const float* proj, int proj_stride,
                             int decay_off, int step_off, const float* a_log, const float* dt_bias, const float* skip, float* state,
                             long long slot_stride, int state_off, const int* slots, const int* row_start, float* out, int rows, int heads,
-                            int groups, int n, int n_padded, int e, float q_scale, cudaStream_t stream) {
+                            int groups, int n, int n_padded, int e, float q_scale, float* decays, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (n <= 0 || n > 256 || e <= 0 || heads <= 0 || groups <= 0 || heads % groups || rows > 65535 || heads > 65535) return HB_UNSUPPORTED_SIZE;
     if (n_padded < n || (n_padded & 3) || (state_off & 3) || (slot_stride & 3) || (((uintptr_t)state) & 15)) return HB_BAD_ARGUMENT;
     ScanArgs a{conv + k_off, conv + q_off, conv + v_off, conv_stride, conv_stride, conv_stride, proj, proj_stride, decay_off, step_off, proj, proj_stride, a_log, dt_bias, skip,
-               state, (size_t)slot_stride, state_off, slots, row_start, out, heads, groups, n, n_padded, e, q_scale};
+               state, (size_t)slot_stride, state_off, slots, row_start, out, heads, groups, n, n_padded, e, q_scale, 0, 0, decays};
+    if (decays && mode == MODE_DELTA) return HB_BAD_ARGUMENT;  // its correction is not a product of decays
     if (mode == MODE_DELTA) return launch_scan<MODE_DELTA>(a, rows, stream);
     if (mode == MODE_STATE_SPACE) return launch_scan<MODE_STATE_SPACE>(a, rows, stream);
     if (mode == MODE_RETENTION) return launch_scan<MODE_RETENTION>(a, rows, stream);
@@ -489,6 +515,143 @@ HB_EXPORT int hb_wkv_scan(const float* k, int k_stride, const float* q, int q_st
     ScanArgs a{k, q, v, k_stride, q_stride, v_stride, x, x_stride, x_off, 0, x, x_stride, w0, bonus, nullptr, state, (size_t)slot_stride, state_off, slots, row_start, out,
                heads, heads, n, n_padded, e, 1.f};
     return launch_scan<MODE_WKV>(a, rows, stream);
+}
+
+// ---------------------------------------------------------------- a matrix memory with exponential gates
+// Per head: S <- exp(f + m' - m) S + exp(i - m) k v^T and a vector n that follows the same recurrence with k alone, where i and f are the logarithms of
+// the input and of the forget gate and m = max(f + m', i) a running maximum that starts at 0;   o = S^T q / (max(|n . q|, exp(-m)) + 1e-6).
+// The maximum depends on the gates alone, so it is walked first (matrix_memory_gates: a warp per row and head; the lanes make the gates of
+// 32 tokens side by side, then every lane walks the chain m = max(f + m, i) through them in order, so its bits do not depend on how a row was
+// cut).  The scan (MODE_GIVEN) then knows its decay and step; n is the column of S whose value is always 1.  matrix_memory_norm divides, norms each
+// head by its root mean square, and applies weight and gate.
+namespace {
+__global__ void __launch_bounds__(32) matrix_memory_gates_kernel(const float* __restrict__ x, int x_stride, int i_off, int f_off, const float* __restrict__ i_bias,
+                                                                 const float* __restrict__ f_bias, float cap, float* __restrict__ state, size_t slot_stride,
+                                                                 int m_off, const int* __restrict__ slots, const int* __restrict__ row_start,
+                                                                 float* __restrict__ gates, int heads) {
+    const int head = blockIdx.x, row = blockIdx.y, lane = threadIdx.x;
+    const int t0 = row_start[row], t1 = row_start[row + 1];
+    float* const kept = state + (size_t)slots[row] * slot_stride + m_off + head;
+    const float bi = i_bias[head], bf = f_bias[head];
+    float m = *kept, raw_i = 0.f, raw_f = 0.f;
+    if (t0 + lane < t1) {
+        raw_i = x[(size_t)(t0 + lane) * x_stride + i_off + head];
+        raw_f = x[(size_t)(t0 + lane) * x_stride + f_off + head];
+    }
+    for (int base = t0; base < t1; base += 32) {
+        const float in = cap * tanhf((raw_i + bi) / cap);
+        const float z = cap * tanhf((raw_f + bf) / cap);
+        const float forget = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+        const int next = base + 32 + lane;
+        if (next < t1) {  // in flight while the chain is walked
+            raw_i = x[(size_t)next * x_stride + i_off + head];
+            raw_f = x[(size_t)next * x_stride + f_off + head];
+        }
+        const int count = min(32, t1 - base);
+        float before = m, after = m;
+        if (count == 32) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+                const float fj = __shfl_sync(0xffffffffu, forget, j), ij = __shfl_sync(0xffffffffu, in, j), was = m;
+                m = fmaxf(fj + m, ij);
+                if (lane == j) { before = was; after = m; }
+            }
+        } else {
+            for (int j = 0; j < count; ++j) {
+                const float fj = __shfl_sync(0xffffffffu, forget, j), ij = __shfl_sync(0xffffffffu, in, j), was = m;
+                m = fmaxf(fj + m, ij);
+                if (lane == j) { before = was; after = m; }
+            }
+        }
+        if (lane < count) {
+            float* g = gates + (size_t)(base + lane) * 3 * heads + head;
+            g[0] = expf((forget + before) - after);
+            g[heads] = expf(in - after);
+            g[2 * heads] = expf(-after);
+        }
+    }
+    if (lane == 0) *kept = m;
+}
+
+// A warp per (token, head).
+template <typename TO>
+__global__ void __launch_bounds__(128) matrix_memory_norm_kernel(const float* __restrict__ y, int head_stride, const float* __restrict__ gates,
+                                                                 const float* __restrict__ gate, int gate_stride, int gate_off, const float* __restrict__ weight,
+                                                                 int heads, int e, float eps, TO* __restrict__ out, int out_stride, int by_four) {
+    const int t = blockIdx.x, head = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (head >= heads) return;
+    const float* row = y + ((size_t)t * heads + head) * head_stride;
+    const float* g = gate + (size_t)t * gate_stride + gate_off + (size_t)head * e;
+    const float* w = weight + (size_t)head * e;
+    TO* dst = out + (size_t)t * out_stride + (size_t)head * e;
+    const float below = fmaxf(fabsf(row[e]), gates[(size_t)t * 3 * heads + 2 * heads + head]) + 1e-6f;
+    float sum = 0.f;
+    if (by_four) {
+        for (int j = lane * 4; j < e; j += 128) {
+            float v[4];
+            load4(row + j, v);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) { v[k] /= below; sum = fmaf(v[k], v[k], sum); }
+        }
+    } else {
+        for (int j = lane; j < e; j += 32) { const float v = row[j] / below; sum = fmaf(v, v, sum); }
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(sum) / (float)e + eps);
+    if (by_four) {
+        for (int j = lane * 4; j < e; j += 128) {
+            float v[4], gv[4], wv[4];
+            load4(row + j, v);
+            load4(g + j, gv);
+            load4(w + j, wv);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) v[k] = v[k] / below * inv * wv[k] * sigmoid_of(gv[k]);
+            store4(dst + j, v);
+        }
+    } else {
+        for (int j = lane; j < e; j += 32) dst[j] = from_float<TO>(row[j] / below * inv * w[j] * sigmoid_of(g[j]));
+    }
+}
+}  // namespace
+
+// x [tokens, x_stride]: the gates' pre-activations, head h at i_off + h and f_off + h; log input gate i = cap tanh((x + i_bias) / cap), log forget gate
+// f = log sigmoid(cap tanh((x + f_bias) / cap)).  The running maximum of (slot, head) lies at state + slot * slot_stride + m_off + head.
+// gates [tokens, 3, heads] receives the token's decay exp(f + m' - m), its step exp(i - m) and exp(-m).
+HB_EXPORT int hb_matrix_memory_gates(const float* x, int x_stride, int i_off, int f_off, const float* i_bias, const float* f_bias, float cap, float* state,
+                                     long long slot_stride, int m_off, const int* slots, const int* row_start, float* gates, int rows, int heads, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (heads <= 0 || rows > 65535 || !(cap > 0.f)) return HB_UNSUPPORTED_SIZE;
+    matrix_memory_gates_kernel<<<dim3(heads, rows), 32, 0, stream>>>(x, x_stride, i_off, f_off, i_bias, f_bias, cap, state, (size_t)slot_stride, m_off, slots, row_start,
+                                                                   gates, heads);
+    return launch_status();
+}
+
+// Keys, queries (times q_scale) and values at k_off, q_off and v_off of `x`, decay and step per token from hb_matrix_memory_gates.  The state of (slot, head) is
+// [values + 1, n_padded], its last row the sum of keys; out [tokens, heads, out_e] with out_e > values, entry `values` being n . q.
+HB_EXPORT int hb_matrix_memory_scan(const float* x, int x_stride, int k_off, int q_off, int v_off, const float* gates, float* state, long long slot_stride, int state_off,
+                                    const int* slots, const int* row_start, float* out, int rows, int heads, int n, int n_padded, int values, int out_e, float q_scale,
+                                    float* decays, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (n <= 0 || n > 256 || values <= 0 || heads <= 0 || rows > 65535 || heads > 65535 || out_e <= values) return HB_UNSUPPORTED_SIZE;
+    if (n_padded < n || (n_padded & 3) || (state_off & 3) || (slot_stride & 3) || (((uintptr_t)state) & 15)) return HB_BAD_ARGUMENT;
+    ScanArgs a{x + k_off, x + q_off, x + v_off, x_stride, x_stride, x_stride, gates, 3 * heads, 0, heads, gates, 3 * heads, nullptr, nullptr, nullptr,
+               state, (size_t)slot_stride, state_off, slots, row_start, out, heads, heads, n, n_padded, values + 1, q_scale, values, out_e, decays};
+    return launch_scan<MODE_GIVEN>(a, rows, stream);
+}
+
+// y [tokens, heads, head_stride] as hb_matrix_memory_scan left it, gates as hb_matrix_memory_gates did: each head's y / (max(|n . q|, exp(-m)) + 1e-6) is divided by its root mean square,
+// multiplied by weight [heads * e] and by sigmoid(gate[token, gate_off + head * e + j]).
+HB_EXPORT int hb_matrix_memory_norm(const float* y, int head_stride, const float* gates, const float* gate, int gate_stride, int gate_off, const float* weight,
+                                    int heads, int e, float eps, void* out, int out_is_bf16, int out_stride, int tokens, cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (heads <= 0 || e <= 0 || heads > 4 * 65535 || head_stride <= e) return HB_UNSUPPORTED_SIZE;
+    const int by_four = e % 4 == 0 && head_stride % 4 == 0 && gate_stride % 4 == 0 && gate_off % 4 == 0 && out_stride % 4 == 0 &&
+                        (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)weight) & 15) == 0 && ((uintptr_t)out & (out_is_bf16 ? 7 : 15)) == 0;
+    const dim3 grid(tokens, (heads + 3) / 4);
+    if (out_is_bf16)
+        matrix_memory_norm_kernel<<<grid, 128, 0, stream>>>(y, head_stride, gates, gate, gate_stride, gate_off, weight, heads, e, eps, (__nv_bfloat16*)out, out_stride, by_four);
+    else
+        matrix_memory_norm_kernel<<<grid, 128, 0, stream>>>(y, head_stride, gates, gate, gate_stride, gate_off, weight, heads, e, eps, (float*)out, out_stride, by_four);
+    return launch_status();
 }
 
 // ---------------------------------------------------------------- token shift
@@ -955,10 +1118,10 @@ HB_EXPORT int hb_selective_scan(const float* x, int x_stride, const float* dt, i
 namespace {
 __global__ void join_segments_kernel(float* __restrict__ ends, size_t end_stride, float* __restrict__ state, size_t slot_stride, int state_off,
                                      const int* __restrict__ slots, const int* __restrict__ seg_start, const int* __restrict__ seg_row, int segments,
-                                     const float* __restrict__ decay, int per_head, int entries) {
+                                     const float* __restrict__ decay, int per_head, int entries, const float* __restrict__ seg_decay, int heads) {
     const int entry = blockIdx.x * blockDim.x + threadIdx.x;
     if (entry >= entries) return;
-    const float log_decay = log2f(decay[entry / per_head]);
+    const float log_decay = seg_decay ? 0.f : log2f(decay[entry / per_head]);
     constexpr int AHEAD = 8;  // what the segments add is asked for before the chain through them starts: one trip to memory, not one per segment
     int j = 0;
     while (j < segments) {
@@ -973,7 +1136,7 @@ __global__ void join_segments_kernel(float* __restrict__ ends, size_t end_stride
                 if (j + k < segments && seg_row[j + k] == row) {
                     added[k] = ends[(size_t)(j + k) * end_stride + entry];
                     const int length = seg_start[j + k + 1] - seg_start[j + k];
-                    fade[k] = log_decay == 0.f ? 1.f : exp2f((float)length * log_decay);
+                    fade[k] = seg_decay ? seg_decay[(size_t)(j + k) * heads + entry / per_head] : (log_decay == 0.f ? 1.f : exp2f((float)length * log_decay));
                     count = k + 1;
                 }
             }
@@ -1000,7 +1163,19 @@ HB_EXPORT int hb_join_segments(float* ends, long long end_stride, float* state, 
     if (heads <= 0 || per_head <= 0) return HB_BAD_ARGUMENT;
     const int entries = heads * per_head;
     join_segments_kernel<<<(entries + 255) / 256, 256, 0, stream>>>(ends, (size_t)end_stride, state, (size_t)slot_stride, state_off, slots, seg_start, seg_row,
-                                                                 segments, decay, per_head, entries);
+                                                                 segments, decay, per_head, entries, nullptr, heads);
+    return launch_status();
+}
+
+// The same where a head's decay differs from token to token: seg_decay [segments, heads] holds its product over every segment (the first pass leaves it).
+HB_EXPORT int hb_join_segments_by_decay(float* ends, long long end_stride, float* state, long long slot_stride, int state_off, const int* slots,
+                                        const int* seg_start, const int* seg_row, int segments, const float* seg_decay, int heads, int per_head,
+                                        cudaStream_t stream) {
+    if (segments <= 0) return 0;
+    if (heads <= 0 || per_head <= 0 || !seg_decay) return HB_BAD_ARGUMENT;
+    const int entries = heads * per_head;
+    join_segments_kernel<<<(entries + 255) / 256, 256, 0, stream>>>(ends, (size_t)end_stride, state, (size_t)slot_stride, state_off, slots, seg_start, seg_row,
+                                                                 segments, nullptr, per_head, entries, seg_decay, heads);
     return launch_status();
 }
 

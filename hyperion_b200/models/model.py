@@ -35,7 +35,10 @@ class DecoderModel:
             norms = {name: parts.make(parts.NORMS, norm, self.build) for name, norm in layer.norms.items()}
             if layer.arrangement not in parts.ARRANGEMENTS:
                 raise KeyError(f"no arrangement {layer.arrangement!r} is registered")
-            self.layers.append(parts.ARRANGEMENTS[layer.arrangement](mixer, feed_forward, norms))
+            arranged = parts.ARRANGEMENTS[layer.arrangement](mixer, feed_forward, norms)
+            if layer.connections:
+                arranged.connections = {name: parts.make(parts.CONNECTIONS, connection, self.build) for name, connection in layer.connections.items()}
+            self.layers.append(arranged)
         self.offsets = parts.make(parts.STREAM_OFFSETS, spec.offsets, self.build) if spec.offsets is not None else None
         self.final_norm = parts.make(parts.NORMS, spec.final_norm, self.build)
         self.head = parts.make(parts.HEADS, spec.head, self.build)
@@ -53,6 +56,8 @@ class DecoderModel:
                 yield layer_spec.feed_forward.prefix, layer.feed_forward
             for name, norm_spec in layer_spec.norms.items():
                 yield norm_spec.prefix, layer.norms[name]
+            for name, connection_spec in layer_spec.connections.items():
+                yield connection_spec.prefix, layer.connections[name]
         if self.offsets is not None:
             yield self.spec.offsets.prefix, self.offsets
         yield self.spec.final_norm.prefix, self.final_norm

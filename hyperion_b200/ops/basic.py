@@ -521,12 +521,18 @@ def rotate_heads_(x: torch.Tensor, col0: int, heads: int, head_dim: int, positio
 def heads_store(x: torch.Tensor, q_off: int, k_off: int, v_off: int, q_heads: int, kv_heads: int, head_dim: int, v_dim: int, positions: torch.Tensor, *,
                 q_out: torch.Tensor, maps: int = 1, bias: torch.Tensor | None = None, q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None,
                 eps: float = 0.0, cache: torch.Tensor | None = None, block_table: torch.Tensor | None = None, token_row: torch.Tensor | None = None,
-                page_size: int = 0) -> None:
-    """Float projections ``x`` [tokens, *] of heads that nothing rotates: ``bias`` [columns] float is added, query and key heads pass an optional RMS
+                page_size: int = 0, inv_freq: torch.Tensor | None = None, rot_dims: int = 0, rot_half: bool = False, amplitude: float = 1.0,
+                unit_norm: bool = False, temperature: tuple[float, int] | None = None) -> None:
+    """Float projections ``x`` [tokens, *] of heads: ``bias`` [columns] float is added, query and key heads pass an optional RMS
     norm (one weight [head_dim] for all of them), queries [q_heads, maps, head_dim] go to ``q_out``, keys [kv_heads, maps, head_dim] and values
     [kv_heads, v_dim] to ``cache`` (either arrangement of :func:`paged_strides`, with maps * head_dim as the keys' size).  Without a cache:
-    queries only."""
-    require_cuda(x, positions, q_out, bias, q_norm, k_norm, cache, block_table, token_row)
+    queries only.  ``unit_norm``: query and key heads are divided by sqrt(mean(x^2) + eps) without a weight.  ``inv_freq`` [rot_dims / 2] float: the
+    first ``rot_dims`` entries of query and key heads turn in pairs (``rot_half``: i with i + rot_dims / 2, else 2i with 2i + 1) by position *
+    inv_freq[i], cosine and sine times ``amplitude``.  ``temperature`` (coef, every): queries are multiplied by
+    1 + coef * ln(floor((position + 1) / every) + 1)."""
+    require_cuda(x, positions, q_out, bias, q_norm, k_norm, cache, block_table, token_row, inv_freq)
+    if inv_freq is not None and (inv_freq.dtype != torch.float32 or not inv_freq.is_contiguous() or inv_freq.numel() < rot_dims // 2):
+        raise KernelError("heads_store: a dense float32 frequency per rotated pair")
     if x.dtype != torch.float32 or x.stride(-1) != 1 or q_out.stride(-1) != 1 or q_out.shape[1] < q_heads * maps * head_dim:
         raise KernelError("heads_store: float32 projections and queries with unit inner stride")
     if bias is not None and (bias.dtype != torch.float32 or not bias.is_contiguous() or bias.numel() > x.shape[1]):
@@ -541,12 +547,16 @@ def heads_store(x: torch.Tensor, q_off: int, k_off: int, v_off: int, q_heads: in
         v_cache_off, page_stride, head_stride, token_stride = paged_strides(cache, maps * head_dim, v_dim)
         pages = cache.shape[0]
     v_cache = ctypes.c_void_p(cache.data_ptr() + v_cache_off * cache.element_size()) if cache is not None else ctypes.c_void_p(0)
-    check(library("heads_prepare").hb_heads_store(
-        ptr(x), i32(x.shape[0]), i32(x.stride(0)), ptr(bias), i32(q_off), i32(k_off), i32(v_off), i32(q_heads * maps), i32(kv_heads * maps), i32(kv_heads), i32(maps),
-        i32(head_dim), i32(v_dim), ptr(q_norm), ptr(k_norm), f32(eps), ptr(positions), ptr(q_out), i32(q_out.stride(0)), i32(is_bf16(q_out)), ptr(cache), v_cache,
-        ctypes.c_longlong(page_stride), ctypes.c_longlong(head_stride), i32(token_stride), ptr(block_table),
-        i32(block_table.shape[1] if block_table is not None else 0), ptr(token_row), i32(page_size), i32(pages), ptr(status_word(x.device)), stream_ptr()),
-        "heads_store")
+    common = (ptr(x), i32(x.shape[0]), i32(x.stride(0)), ptr(bias), i32(q_off), i32(k_off), i32(v_off), i32(q_heads * maps), i32(kv_heads * maps), i32(kv_heads),
+              i32(maps), i32(head_dim), i32(v_dim), ptr(q_norm), ptr(k_norm), f32(eps), ptr(positions), ptr(q_out), i32(q_out.stride(0)), i32(is_bf16(q_out)), ptr(cache),
+              v_cache, ctypes.c_longlong(page_stride), ctypes.c_longlong(head_stride), i32(token_stride), ptr(block_table),
+              i32(block_table.shape[1] if block_table is not None else 0), ptr(token_row), i32(page_size), i32(pages))
+    if inv_freq is None and not unit_norm and temperature is None:
+        check(library("heads_prepare").hb_heads_store(*common, ptr(status_word(x.device)), stream_ptr()), "heads_store")
+        return
+    coef, every = temperature if temperature is not None else (0.0, 1)
+    check(library("heads_prepare").hb_heads_turn(*common, ptr(inv_freq), i32(rot_dims if inv_freq is not None else 0), i32(1 if rot_half else 0), f32(amplitude),
+                                                 i32(1 if unit_norm else 0), f32(coef), i32(every), ptr(status_word(x.device)), stream_ptr()), "heads_store")
 
 
 def pair_norms_take(hidden: int) -> bool:
@@ -608,3 +618,69 @@ def soft_cap_(x: torch.Tensor, cap: float) -> torch.Tensor:
         raise KernelError("soft_cap_: a dense float32 tensor")
     check(library("elementwise").hb_soft_cap(ptr(x), f32(cap), ctypes.c_longlong(x.numel()), stream_ptr()), "soft_cap")
     return x
+
+
+def relu_squared(x: torch.Tensor) -> torch.Tensor:
+    """max(x, 0)^2, computed in float, in the element type of ``x``."""
+    require_cuda(x)
+    if not x.is_contiguous():
+        raise KernelError("relu_squared: a dense tensor")
+    out = torch.empty_like(x)
+    check(library("elementwise").hb_relu_squared(ptr(x), ptr(out), i32(is_bf16(x)), ctypes.c_longlong(x.numel()), stream_ptr()), "relu_squared")
+    return out
+
+
+LARGEST_STREAMS = 16  # csrc/hyper_connections.cu
+
+
+def streams_module(streams: int) -> tuple[str, dict]:
+    """The build of ``csrc/hyper_connections.cu`` that takes this number of streams."""
+    return "hyper_connections", {"HB_STREAMS": streams if streams <= 4 else 0}
+
+
+def hyper_connect(h: torch.Tensor, streams: int, read: torch.Tensor | None, weight: torch.Tensor, eps: float, out_dtype: torch.dtype, *, results=(), norms=(None, None),
+                  result_eps: float = 0.0, result_scale: float = 1.0, mix: torch.Tensor | None = None, share: torch.Tensor | None = None,
+                  rows: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+    """One boundary between two sublayers of a model with several residual streams.  ``h`` is [tokens, streams, hidden] float, or [tokens, hidden] while
+    all streams are still equal.  With ``results`` (one or two sublayer results, tensors or products in their split-K pieces without a bias; each
+    divided by its own root mean square and multiplied by its entry of ``norms`` unless that is None; their sum times ``result_scale`` is y):
+    x_t <- sum_s mix[s, t] x_s + share[t] y.  Then u = sum_s read[s] x_s (``read`` None: the plain sum), and u / rms(u) * ``weight`` is returned in
+    ``out_dtype`` together with the streams ([tokens, streams, hidden], written in place where ``h`` had them already; ``h`` itself when nothing was
+    pending).  ``rows`` (int32 indices): only those rows are worked on and the streams stay as they were."""
+    from .gemm import SplitSum
+
+    single = h.dim() == 2
+    tokens, hidden = h.shape[0], h.shape[-1]
+    if h.dtype != torch.float32 or not h.is_contiguous() or (not single and (h.dim() != 3 or h.shape[1] != streams)):
+        raise KernelError("hyper_connect: dense float32 streams [tokens, streams, hidden], or [tokens, hidden] for streams that are all equal")
+    if len(results) > 2 or (len(results) == 0) != (mix is None):
+        raise KernelError("hyper_connect: one or two sublayer results with a mixing matrix, or none without")
+    for t, count in ((mix, streams * streams), (share, streams), (read, streams), (weight, hidden), (norms[0], hidden), (norms[1], hidden)):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != count or not t.is_contiguous()):
+            raise KernelError("hyper_connect: mixing weights and norm weights are dense float32")
+    taken = []
+    for y in results:
+        if isinstance(y, SplitSum) and (y.bias is not None or not y.partials.is_contiguous()):
+            y = y.tensor()
+        if tuple(y.shape) != (tokens, hidden) or (not isinstance(y, SplitSum) and not y.is_contiguous()):
+            raise KernelError("hyper_connect: sublayer results are dense [tokens, hidden]")
+        taken.append(y)
+    dense = {y.dtype for y in taken if not isinstance(y, SplitSum)}
+    if len(dense) > 1 or (dense == {torch.bfloat16} and out_dtype == torch.float32):  # sublayers of unlike precision
+        taken = [y if isinstance(y, SplitSum) else y.float() for y in taken]
+        dense = {torch.float32}
+    pieces = [y.partials.shape[0] if isinstance(y, SplitSum) else 0 for y in taken] + [0, 0]
+    data = [y.partials if isinstance(y, SplitSum) else y for y in taken] + [None, None]
+    require_cuda(h, read, weight, mix, share, rows, *data, *norms)
+    n_rows = rows.numel() if rows is not None else tokens
+    out = torch.empty((n_rows, hidden), dtype=out_dtype, device=h.device)
+    new = None
+    if taken and rows is None:
+        new = torch.empty((tokens, streams, hidden), dtype=torch.float32, device=h.device) if single else h
+    bf16 = dense == {torch.bfloat16} or (not dense and out_dtype == torch.bfloat16)
+    module, defines = streams_module(streams)
+    check(library(module, **defines).hb_hyper_connect(
+        ptr(h), i32(1 if single else 0), ptr(new), i32(streams), ptr(data[0]), i32(pieces[0]), ptr(data[1]), i32(pieces[1]), ctypes.c_longlong(tokens * hidden),
+        i32(1 if bf16 else 0), ptr(norms[0]), ptr(norms[1]), f32(result_eps), f32(result_scale), ptr(mix), ptr(share), ptr(read), ptr(weight), f32(eps), ptr(out),
+        i32(is_bf16(out)), ptr(rows), i32(n_rows), i32(hidden), stream_ptr()), "hyper_connect")
+    return out, (h if new is None else new)

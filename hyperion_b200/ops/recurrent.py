@@ -81,16 +81,66 @@ def silu_columns_(x: torch.Tensor, col0: int, columns: int) -> None:
 def state_scan(mode: int, conv: torch.Tensor, k_off: int, q_off: int, v_off: int, proj: torch.Tensor, decay_off: int, step_off: int,
                a_log: torch.Tensor, dt_bias: torch.Tensor, skip: torch.Tensor | None, state: torch.Tensor, state_off: int, slots: torch.Tensor,
                row_start: torch.Tensor, rows: int, heads: int, groups: int, n: int, n_padded: int, e: int, q_scale: float = 1.0,
-               states_only: bool = False) -> torch.Tensor | None:
+               states_only: bool = False, decays: torch.Tensor | None = None) -> torch.Tensor | None:
     """Walk every row's tokens through the recurrence of ``mode`` from and into its slot of ``state``; returns [tokens, heads * e]
-    (nothing with ``states_only``: the walk then only leaves the rows' states)."""
-    require_cuda(conv, proj, a_log, dt_bias, skip, state, slots, row_start)
+    (nothing with ``states_only``: the walk then only leaves the rows' states).  ``decays`` [rows, heads] float (not for the delta rule) receives the
+    product of every row's decays."""
+    require_cuda(conv, proj, a_log, dt_bias, skip, state, slots, row_start, decays)
     _floats(conv, proj, a_log, dt_bias, skip, state)
     out = None if states_only else torch.empty((conv.shape[0], heads * e), dtype=torch.float32, device=conv.device)
     check(library("recurrent").hb_state_scan(i32(mode), ptr(conv), i32(conv.stride(0)), i32(k_off), i32(q_off), i32(v_off), ptr(proj), i32(proj.stride(0)),
                                              i32(decay_off), i32(step_off), ptr(a_log), ptr(dt_bias), ptr(skip), ptr(state),
                                              ctypes.c_longlong(state.stride(0)), i32(state_off), ptr(slots), ptr(row_start), ptr(out), i32(rows),
-                                             i32(heads), i32(groups), i32(n), i32(n_padded), i32(e), f32(q_scale), stream_ptr()), "state_scan")
+                                             i32(heads), i32(groups), i32(n), i32(n_padded), i32(e), f32(q_scale), ptr(decays), stream_ptr()), "state_scan")
+    return out
+
+
+def matrix_memory_gates(x: torch.Tensor, i_off: int, f_off: int, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, state: torch.Tensor, m_off: int,
+                        slots: torch.Tensor, row_start: torch.Tensor, rows: int, heads: int) -> torch.Tensor:
+    """The gates of a matrix memory: log input gate i = cap tanh((x + i_bias) / cap) and log forget gate f = log sigmoid(cap tanh((x + f_bias) / cap)) from the columns
+    ``i_off ..`` and ``f_off ..`` of ``x``, and the running maximum m = max(f + m', i) of every row, which starts from and ends in its slot of
+    ``state`` at ``m_off``.  Returns [tokens, 3, heads]: the decay exp(f + m' - m), the step exp(i - m), and exp(-m)."""
+    require_cuda(x, i_bias, f_bias, state, slots, row_start)
+    _floats(x, i_bias, f_bias, state)
+    gates = torch.empty((x.shape[0], 3, heads), dtype=torch.float32, device=x.device)
+    check(library("recurrent").hb_matrix_memory_gates(ptr(x), i32(x.stride(0)), i32(i_off), i32(f_off), ptr(i_bias), ptr(f_bias), f32(cap), ptr(state),
+                                                      ctypes.c_longlong(state.stride(0)), i32(m_off), ptr(slots), ptr(row_start), ptr(gates), i32(rows), i32(heads),
+                                                      stream_ptr()), "matrix_memory_gates")
+    return gates
+
+
+def matrix_memory_columns(values: int) -> int:
+    """Columns per head of what :func:`matrix_memory_scan` returns: the values, the normaliser, and as many more as keep rows on 16-byte boundaries."""
+    return -(-(values + 1) // 4) * 4
+
+
+def matrix_memory_scan(x: torch.Tensor, k_off: int, q_off: int, v_off: int, gates: torch.Tensor, state: torch.Tensor, state_off: int, slots: torch.Tensor,
+                       row_start: torch.Tensor, rows: int, heads: int, n: int, n_padded: int, values: int, q_scale: float, states_only: bool = False,
+                       decays: torch.Tensor | None = None) -> torch.Tensor | None:
+    """S <- a S + b k v^T per head with decay a and step b from ``gates`` (:func:`matrix_memory_gates`), and the same for the sum of keys, a further column of S.
+    Keys, queries and values are columns of ``x``; every row's tokens walk from and into its slot of ``state`` ([heads, values + 1, n_padded] floats at
+    ``state_off``).  Returns [tokens, heads, :func:`matrix_memory_columns`]: S^T q and, at entry ``values``, n . q, with q times ``q_scale``."""
+    require_cuda(x, gates, state, slots, row_start, decays)
+    _floats(x, gates, state)
+    columns = matrix_memory_columns(values)
+    out = None if states_only else torch.empty((x.shape[0], heads, columns), dtype=torch.float32, device=x.device)
+    check(library("recurrent").hb_matrix_memory_scan(ptr(x), i32(x.stride(0)), i32(k_off), i32(q_off), i32(v_off), ptr(gates), ptr(state), ctypes.c_longlong(state.stride(0)),
+                                                     i32(state_off), ptr(slots), ptr(row_start), ptr(out), i32(rows), i32(heads), i32(n), i32(n_padded), i32(values), i32(columns),
+                                                     f32(q_scale), ptr(decays), stream_ptr()), "matrix_memory_scan")
+    return out
+
+
+def matrix_memory_norm(y: torch.Tensor, gates: torch.Tensor, gate: torch.Tensor, gate_off: int, weight: torch.Tensor, values: int, eps: float,
+                       out: torch.Tensor) -> torch.Tensor:
+    """What follows :func:`matrix_memory_scan`: every head of ``y`` over max(|n . q|, exp(-m)) + 1e-6, divided by its root mean square, times ``weight``
+    [heads * values] and the sigmoid of the columns ``gate_off ..`` of ``gate``; written to ``out`` [tokens, >= heads * values]."""
+    require_cuda(y, gates, gate, weight, out)
+    _floats(y, gates, gate, weight)
+    tokens, heads, columns = y.shape
+    if weight.numel() != heads * values or out.shape[0] != tokens or out.shape[1] < heads * values or out.stride(1) != 1:
+        raise KernelError("matrix_memory_norm: a weight per column and an output of [tokens, >= heads * values]")
+    check(library("recurrent").hb_matrix_memory_norm(ptr(y), i32(columns), ptr(gates), ptr(gate), i32(gate.stride(0)), i32(gate_off), ptr(weight), i32(heads), i32(values),
+                                                     f32(eps), ptr(out), i32(is_bf16(out)), i32(out.stride(0)), i32(tokens), stream_ptr()), "matrix_memory_norm")
     return out
 
 
@@ -243,6 +293,22 @@ def retention_in_segments(proj: torch.Tensor, k_off: int, q_off: int, v_off: int
     check(library("recurrent").hb_join_segments(ptr(ends), ctypes.c_longlong(ends.stride(0)), ptr(state), ctypes.c_longlong(state.stride(0)), i32(0), ptr(slots),
                                                 ptr(seg_start), ptr(seg_row), i32(segments), ptr(decay), i32(heads), i32(per_head), stream_ptr()), "join_segments")
     return state_scan(MODE_RETENTION, proj, k_off, q_off, v_off, proj, 0, 0, decay, decay, None, ends, 0, own, seg_start, segments, heads, heads, n, n_padded, e)
+
+
+def scan_in_segments(scan, per_head: int, state: torch.Tensor, state_off: int, slots: torch.Tensor, seg_start: torch.Tensor, seg_row: torch.Tensor, segments: int, heads: int):
+    """A scan whose state fades by a number per token and head, S <- a S + (something that does not depend on S), with long rows cut into segments that are walked
+    side by side (see :func:`retention_in_segments`; here a segment's decay is the product its first pass leaves).  ``scan(state, slots, row_start, rows,
+    states_only, decays)`` walks rows whose matrices (``per_head`` floats a head) are the first ``heads * per_head`` floats of a record; the rows' own
+    matrices lie at ``state_off`` of ``state``."""
+    require_cuda(state, slots, seg_start, seg_row)
+    ends = torch.zeros((segments, heads * per_head), dtype=torch.float32, device=state.device)
+    decays = torch.empty((segments, heads), dtype=torch.float32, device=state.device)
+    own = torch.arange(segments, dtype=torch.int32, device=state.device)
+    scan(ends, own, seg_start, segments, True, decays)
+    check(library("recurrent").hb_join_segments_by_decay(ptr(ends), ctypes.c_longlong(ends.stride(0)), ptr(state), ctypes.c_longlong(state.stride(0)), i32(state_off),
+                                                         ptr(slots), ptr(seg_start), ptr(seg_row), i32(segments), ptr(decays), i32(heads), i32(per_head),
+                                                         stream_ptr()), "join_segments")
+    return scan(ends, own, seg_start, segments, False, None)
 
 
 def selective_in_segments(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, b_off: int, c_off: int, a: torch.Tensor, skip: torch.Tensor,

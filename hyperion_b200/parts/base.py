@@ -31,8 +31,9 @@ from .spec import PartSpec
 class WeightSpec:
     shape: tuple[int, ...]
     integer: bool = False  # integer tables are kept as int32, everything else as a float type
-    init: str = "normal"  # how random weights fill it: "normal" = N(0, std), "one_plus_normal" = 1 + N(0, std)
+    init: str = "normal"  # how random weights fill it: "normal" = N(mean, std), "one_plus_normal" = 1 + N(0, std)
     any_extent: tuple[int, ...] = ()  # dimensions whose extent a checkpoint decides (the part reads it off the tensor); ``shape`` is what random weights get
+    mean: float = 0.0  # of "normal" random weights
 
 
 @dataclass(frozen=True)
@@ -175,12 +176,21 @@ class StreamOffsets(Part):
         raise NotImplementedError
 
 
+class Connection(Part):
+    """How one sublayer reads from and writes to several residual streams (``parts/streams.py``)."""
+
+    def read(self, h: torch.Tensor, pending: Any, norm: Norm) -> tuple[torch.Tensor, torch.Tensor]:
+        """Write what is pending to the streams, then (the normalised rows the sublayer reads, the streams)."""
+        raise NotImplementedError
+
+
 class Arrangement:
     """How one layer wires its parts.  ``forward`` gets the residual stream ``h`` and a pending
     ``delta`` not yet added to it (so the add fuses with the next norm) and returns the new pair."""
 
     def __init__(self, mixer: Mixer, feed_forward: FeedForward, norms: Mapping[str, Norm]):
         self.mixer, self.feed_forward, self.norms = mixer, feed_forward, dict(norms)
+        self.connections: dict[str, "Connection"] = {}  # set by the model where the layer names some
 
     def forward(self, h: torch.Tensor, delta: Optional[torch.Tensor], step: Any, cache: Any, own_cache: bool):
         raise NotImplementedError
@@ -193,6 +203,7 @@ POSITIONS: dict[str, Callable[[PartSpec, BuildContext], PositionEncoding]] = {}
 EMBEDDINGS: dict[str, Callable[[PartSpec, BuildContext], Embedding]] = {}
 HEADS: dict[str, Callable[[PartSpec, BuildContext], Head]] = {}
 STREAM_OFFSETS: dict[str, Callable[[PartSpec, BuildContext], StreamOffsets]] = {}
+CONNECTIONS: dict[str, Callable[[PartSpec, BuildContext], Connection]] = {}
 ARRANGEMENTS: dict[str, Callable[..., Arrangement]] = {}
 
 
@@ -209,6 +220,7 @@ def register_position(kind: str, factory) -> None: _register(POSITIONS, kind, fa
 def register_embedding(kind: str, factory) -> None: _register(EMBEDDINGS, kind, factory)
 def register_head(kind: str, factory) -> None: _register(HEADS, kind, factory)
 def register_stream_offsets(kind: str, factory) -> None: _register(STREAM_OFFSETS, kind, factory)
+def register_connection(kind: str, factory) -> None: _register(CONNECTIONS, kind, factory)
 def register_arrangement(kind: str, factory) -> None: _register(ARRANGEMENTS, kind, factory)
 
 

@@ -111,3 +111,26 @@ class SideBySideTwoNormsBlock(Arrangement):
 
 
 register_arrangement("side_by_side_two_norms", SideBySideTwoNormsBlock)
+
+
+class HyperConnectedBlock(Arrangement):
+    """Several residual streams: a sublayer reads one mixture of them through its norm and writes its result to all of them,
+    u = sum_s a[s] x_s;  y = sublayer(norm(u));  x_t <- sum_s B[s, t] x_s + c[t] y,
+    first the mixer, then (when the layer has one) the feed-forward.  Norm names: ``input`` and ``post_mixer``; connection names: ``mixer`` and
+    ``feed_forward`` (``parts/streams.py``).  ``h`` is [tokens, hidden] while the streams are all equal and [tokens, streams, hidden] from the first
+    write on; what a sublayer returned travels on as a :class:`StreamDelta`, and the launch that makes the next sublayer's rows writes it."""
+
+    def forward(self, h, delta, step, cache, own_cache):
+        from .norm import StreamDelta
+
+        connection = self.connections["mixer"]
+        x, h = connection.read(h, delta, self.norms["input"])
+        delta = StreamDelta(self.mixer.forward(x, step, cache, own_cache), connection)
+        if self.feed_forward is not None:
+            connection = self.connections["feed_forward"]
+            x, h = connection.read(h, delta, self.norms["post_mixer"])
+            delta = StreamDelta(self.feed_forward.forward(x, step), connection)
+        return h, delta
+
+
+register_arrangement("hyper_connected", HyperConnectedBlock)

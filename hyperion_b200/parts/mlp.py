@@ -62,10 +62,10 @@ register_feed_forward("swiglu", SwiGLU)
 
 
 class ActivatedMLP(FeedForward):
-    """The feed-forward without a gate: down(act(up(x))), no biases, act = the tanh form of GELU or its exact (erf) form.
-    Parameters: ``hidden_size``, ``intermediate_size``, ``activation`` (``gelu_tanh`` or ``gelu_erf``), ``names`` (``{"up": ..., "down": ...}``)."""
+    """The feed-forward without a gate: down(act(up(x))), no biases, act = the tanh form of GELU, its exact (erf) form or the square of relu.
+    Parameters: ``hidden_size``, ``intermediate_size``, ``activation`` (``gelu_tanh``, ``gelu_erf`` or ``relu_squared``), ``names`` (``{"up": ..., "down": ...}``)."""
 
-    ACTIVATIONS = {"gelu_tanh": "gelu_tanh", "gelu_erf": "gelu_erf"}  # the name of the activation -> the operation of ``ops``
+    ACTIVATIONS = {"gelu_tanh": "gelu_tanh", "gelu_erf": "gelu_erf", "relu_squared": "relu_squared"}  # the name of the activation -> the operation of ``ops``
 
     def __init__(self, spec: PartSpec, build: BuildContext):
         super().__init__(spec, build)

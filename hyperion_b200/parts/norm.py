@@ -88,8 +88,39 @@ class SumOfTwo:
         return first.float() + second.float()
 
 
+@dataclass
+class NormedSum:
+    """What one or two sublayers that read the same rows returned, each still to be divided by its own root mean square and multiplied by its own weight before
+    their sum, times ``scale``, is the sublayer's result.  The launch that adds it to the residual streams (``ops.hyper_connect``) does all of it, and takes
+    a result in its split-K pieces; any other reader calls :meth:`tensor`."""
+
+    results: tuple
+    weights: tuple
+    eps: float
+    scale: float
+
+    def tensor(self) -> torch.Tensor:
+        total = None
+        for y, weight in zip(self.results, self.weights):
+            rows = (y.tensor() if hasattr(y, "tensor") else y).float()
+            normed = ops.add_rmsnorm(rows, None, weight, self.eps, torch.float32)
+            total = normed if total is None else total + normed
+        return total * self.scale
+
+
+@dataclass
+class StreamDelta:
+    """What a sublayer returned, still to be written to the residual streams by its ``connection`` (``parts/streams.py``); the next boundary between two sublayers
+    does it in its own launch, and so does the norm behind the last layer, which reads the sum of the streams."""
+
+    y: object
+    connection: object
+
+
 def with_offset(h: torch.Tensor, delta, row: torch.Tensor):
     """The pending addition ``delta`` (None, a tensor, split-K pieces or a :class:`NormedDelta`) with ``row`` added after it."""
+    if isinstance(delta, StreamDelta):
+        raise ValueError("a model with several residual streams adds no offsets to them")
     if isinstance(delta, NormedDelta):
         if delta.offset is not None:
             row = delta.offset + row
@@ -130,6 +161,12 @@ class RMSNorm(Norm):
         return ops.add_pair_norms(h, first, second, self.weight, other.weight, self.eps, self.dtype)
 
     def forward(self, h, delta, rows=None):
+        if isinstance(delta, StreamDelta):
+            if self.groups > 1:
+                raise ValueError("a norm in groups does not read the sum of several residual streams")
+            return delta.connection.read_sum(h, delta, self, rows)
+        if isinstance(delta, NormedSum):
+            delta = delta.tensor()
         if isinstance(delta, SumOfTwo) and self.groups == 1 and ops.pair_norms_take(h.shape[1]):
             return ops.add_pair_norms(h, delta.first, delta.second, self.weight, None, self.eps, self.dtype, rows)[0]
         if isinstance(delta, WeightedRows):

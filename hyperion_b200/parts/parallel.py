@@ -7,9 +7,12 @@ projection reads, times its scale, into its columns of one buffer, and one more 
 gives the sum: two products for any number of branches.  A branch keeps what it needs between steps like any mixer; the
 combination asks for all of it as a tuple.  Parameters: ``hidden_size``, ``branches``: a tuple of (PartSpec, scale).
 
-A branch is a mixer that also offers: ``in_names`` (its input matrices' tensor names, in the order of its columns),
-``in_width`` and ``core_width`` (columns it takes of the first product and gives to the second), ``out_name``, and
-``core(proj, col0, step, cache, out, scale)``.  Used alone, a branch is an ordinary mixer.
+A branch is a mixer of the kind ``parts/branch.py`` describes.
+
+``parallel_normed_mixers``: one or two branches on the same rows whose results are normalised before they are added:
+y = scale * sum_b branch_b(x) / rms(branch_b(x)) * weight_b, the root mean square over the whole row with ``eps`` inside it.  One input product for all branches,
+an output product each; the results travel on as they are (:class:`NormedSum`), and the launch that adds them to the stream norms and sums them.
+Parameters: ``hidden_size``, ``branches``: a tuple of (PartSpec, name of the norm's weight), ``eps``, ``scale``.
 
 ``biased_attention``: causal grouped-query softmax attention without any rotation; all it knows about positions is a learned
 bias per head and bucket of distance:  score(i, j) = (q_i . k_j) * scale + rel[bucket(i - j), head].  With B buckets and
@@ -41,11 +44,9 @@ from ..ops import attention as fast_attention
 from ..ops import recurrent
 from .attention import GroupedQueryAttention
 from .base import MIXERS, POSITIONS, BuildContext, Mixer, PagedTokens, RequestState, WeightSpec, make, register_mixer
+from .branch import Branch, common_dtype
+from .norm import NormedSum
 from .spec import PartSpec
-
-
-def _common_dtype(tensors) -> torch.dtype:
-    return torch.float32 if any(t.dtype == torch.float32 for t in tensors) else tensors[0].dtype
 
 
 def _round_up(value: int, step: int) -> int:
@@ -57,39 +58,6 @@ def distance_bucket(n: int, buckets: int, far: int) -> int:
     if n < half:
         return n
     return min(buckets - 1, half + int(math.floor(math.log(n / half) / math.log(far / half) * (buckets - half))))
-
-
-class Branch(Mixer):
-    """A mixer that can run beside others on one input (see the module's text)."""
-
-    in_names: tuple[str, ...]
-    out_name: str
-    in_width: int
-    core_width: int
-    hidden: int
-
-    def core(self, proj: torch.Tensor, col0: int, step, cache, out: torch.Tensor, scale: float) -> None:
-        """``proj`` [tokens, *] float: this branch's input projections start at column ``col0``.  Write what the output
-        projection reads, times ``scale``, to ``out`` [tokens, core_width] (a view, activation type)."""
-        raise NotImplementedError
-
-    def load_core(self, tensors: Mapping[str, torch.Tensor]) -> None:
-        """Everything but the input and output matrices."""
-
-    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
-        mats = [tensors[name] for name in self.in_names]
-        dtype = _common_dtype(mats)
-        self.w_in = torch.cat([m.to(dtype) for m in mats], dim=0).contiguous()
-        self.w_o = tensors[self.out_name].contiguous()
-        self.load_core(tensors)
-
-    def forward(self, x, step, cache, own_cache):
-        if cache is None or not own_cache:
-            raise ValueError(f"{type(self).__name__} keeps something per request; the schedule gave it none")
-        proj = ops.linear(x, self.w_in, None, torch.float32)
-        out = torch.empty((x.shape[0], self.core_width), dtype=self.dtype, device=x.device)
-        self.core(proj, 0, step, cache, out, 1.0)
-        return ops.linear(out, self.w_o, None, self.dtype, may_leave_partials=True)  # the result is a residual delta
 
 
 class BiasedAttention(Branch):
@@ -260,7 +228,7 @@ class ParallelMixers(Mixer):
             branch.load_core(own)
             ins += [own[name] for name in branch.in_names]
             outs.append(own[branch.out_name])
-        dtype = _common_dtype(ins + outs)
+        dtype = common_dtype(ins + outs)
         self.w_in = torch.cat([m.to(dtype) for m in ins], dim=0).contiguous()
         self.w_o = torch.cat([m.to(dtype) for m in outs], dim=1).contiguous()
 
@@ -289,6 +257,79 @@ class ParallelMixers(Mixer):
         return ops.linear(out, self.w_o, None, self.dtype, may_leave_partials=True)  # the result is a residual delta
 
 
+class ParallelNormedMixers(Mixer):
+    COLUMN_STEP = 8  # every branch's columns of the input product start on a multiple of this, so that they stay whole 16-byte pieces
+
+    def __init__(self, spec: PartSpec, build: BuildContext):
+        super().__init__(spec, build)
+        p = spec.params
+        self.hidden, self.eps, self.scale = int(p["hidden_size"]), float(p["eps"]), float(p["scale"])
+        self.branches: list[Branch] = []
+        self.prefixes: list[str] = []
+        self.norm_names: list[str] = []
+        self.columns: list[int] = []
+        at = 0
+        for branch_spec, norm_name in p["branches"]:
+            branch = make(MIXERS, branch_spec, build)
+            if not isinstance(branch, Branch):
+                raise ValueError(f"a mixer of kind {branch_spec.kind!r} cannot run beside others (it is no Branch)")
+            if branch.hidden != self.hidden or getattr(branch, "shares_kv", False):
+                raise ValueError("branches read and write rows of the combination's width and keep caches of their own")
+            self.branches.append(branch)
+            self.prefixes.append(branch_spec.prefix)  # relative to the combination's own prefix
+            self.norm_names.append(str(norm_name))
+            self.columns.append(at)
+            at += _round_up(branch.in_width, self.COLUMN_STEP)
+        if not 1 <= len(self.branches) <= 2:
+            raise ValueError(f"{len(self.branches)} mixers side by side: one or two can be normed and added")
+
+    def weights(self) -> dict[str, WeightSpec]:
+        wanted = {prefix + name: spec for prefix, branch in zip(self.prefixes, self.branches) for name, spec in branch.weights().items()}
+        wanted.update({name: WeightSpec((self.hidden,), init="one_plus_normal") for name in self.norm_names})
+        return wanted
+
+    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        ins, self.w_out = [], []
+        for prefix, branch in zip(self.prefixes, self.branches):
+            own = {name: tensors[prefix + name] for name in branch.weights()}
+            branch.load_core(own)
+            ins.append([own[name] for name in branch.in_names])
+            self.w_out.append(own[branch.out_name].contiguous())
+        dtype = common_dtype([m for mats in ins for m in mats])
+        rows = []
+        for branch, mats in zip(self.branches, ins):
+            rows += [m.to(dtype) for m in mats]
+            gap = _round_up(branch.in_width, self.COLUMN_STEP) - branch.in_width
+            if gap:
+                rows.append(torch.zeros((gap, self.hidden), dtype=dtype, device=mats[0].device))
+        self.w_in = torch.cat(rows, dim=0).contiguous()
+        self.norm_weights = [tensors[name].to(torch.float32).contiguous() for name in self.norm_names]
+
+    def cache_request(self):
+        return tuple(branch.cache_request() for branch in self.branches)
+
+    def kernel_modules(self):
+        return [module for branch in self.branches for module in branch.kernel_modules()]
+
+    def step_plans(self):
+        plans = {}
+        for branch in self.branches:
+            plans.update(getattr(branch, "step_plans", lambda: {})())
+        return plans
+
+    def forward(self, x, step, cache, own_cache):
+        if cache is None or not own_cache or len(cache) != len(self.branches):
+            raise ValueError("parallel mixers keep what their branches keep; the schedule gave them something else")
+        proj = ops.linear(x, self.w_in, None, torch.float32)
+        results = []
+        for branch, column, w_out, view in zip(self.branches, self.columns, self.w_out, cache):
+            out = torch.empty((x.shape[0], branch.core_width), dtype=self.dtype, device=x.device)
+            branch.core(proj, column, step, view, out, 1.0)
+            results.append(ops.linear(out, w_out, None, self.dtype, may_leave_partials=True))
+        return NormedSum(tuple(results), tuple(self.norm_weights), self.eps, self.scale)
+
+
+register_mixer("parallel_normed_mixers", ParallelNormedMixers)
 register_mixer("biased_attention", BiasedAttention)
 register_mixer("retention", Retention)
 register_mixer("parallel_mixers", ParallelMixers)

@@ -46,6 +46,14 @@ The decay and the gate come through two small matrices each; their inner sizes a
 Parameters: ``hidden_size``, ``heads``, ``kv_heads``, ``head_dim``, ``value_dim``, ``conv`` (taps), ``eps``, ``decay_rank`` and ``gate_rank`` (what
 random weights get).  Tensors: q, k, v, q.conv, k.conv, v.conv, b, a1, a2, A_log, dt_bias, g1, g2, norm, o.
 
+Matrix memory with exponential gates (``matrix_memory``; the mLSTM of Beck et al., "xLSTM: Extended Long Short-Term Memory"), per head:
+    q = W_q x n^(-1/2), k = W_k x, v = W_v x;   i = cap tanh((W_i x + b_i) / cap);   f = log sigmoid(cap tanh((W_f x + b_f) / cap))
+    m' = max(f + m, i);   S <- exp(f + m - m') S + exp(i - m') k v^T;   n <- exp(f + m - m') n + exp(i - m') k;   o = S^T q / (max(|n . q|, exp(-m')) + 1e-6)
+    y = o / rms(o) per head, times norm (a weight per column), times sigmoid(W_g x), then W_o.
+The running maximum m starts at 0.  The record holds the heads' matrices with n as one more column each, then the heads' m.
+Parameters: ``hidden_size``, ``heads``, ``head_dim``, ``value_dim``, ``gate_cap``, ``eps``.  Tensors: q, k, v, g, i, i.b, f, f.b, norm, o.
+``mamba2`` and ``matrix_memory`` are branches (``parts/branch.py``): they also run beside another mixer on the same input.
+
 Lightning attention (``lightning``): a matrix state per head that fades by a constant of the head, with nothing between the projections and
 the recurrence but an activation:
     q, k, v = silu(W_q x), silu(W_k x), silu(W_v x);  S <- decay_h S + k v^T;  o = S^T q
@@ -61,7 +69,11 @@ import torch
 from .. import ops
 from ..ops import recurrent
 from .base import BuildContext, Mixer, RequestState, WeightSpec, register_mixer
+from .branch import Branch
 from .spec import PartSpec
+
+
+SEGMENT_BLOCKS = 100  # the most blocks of a one-pass scan at which cutting long rows into segments pays
 
 
 def _round_up(value: int, step: int) -> int:
@@ -96,6 +108,15 @@ class _ScanMixer(Mixer):
 
     def _float(self, tensor: torch.Tensor) -> torch.Tensor:
         return tensor.to(torch.float32).contiguous()
+
+    def _walk(self, scan, step, state, slots, per_head: int, columns: int):
+        """``scan`` (as ``recurrent.scan_in_segments`` takes it) over the step's rows, long rows in segments side by side while one pass would leave the GPU mostly
+        idle, as for the package's other recurrences that are linear in their state."""
+        blocks = self.heads * -(-columns // 32)
+        segments = step.host.get("scan_segments", 0) if self.dtype == torch.bfloat16 and blocks <= SEGMENT_BLOCKS else 0
+        if segments:
+            return recurrent.scan_in_segments(scan, per_head, state, 0, slots, step.extra["scan_seg_start"], step.extra["scan_seg_row"], segments, self.heads)
+        return scan(state, slots, step.row_start, step.n_rows)
 
 
 class GatedDeltaRule(_ScanMixer):
@@ -145,8 +166,10 @@ class GatedDeltaRule(_ScanMixer):
         return ops.linear(y, self.w_o, None, self.dtype, may_leave_partials=True)  # the result is a residual delta
 
 
-class StateSpaceMixer(_ScanMixer):
+class StateSpaceMixer(_ScanMixer, Branch):
     mode = recurrent.MODE_STATE_SPACE
+    in_names = ("in",)
+    out_name = "o"
 
     def __init__(self, spec: PartSpec, build: BuildContext):
         super().__init__(spec, build)
@@ -154,13 +177,14 @@ class StateSpaceMixer(_ScanMixer):
         self.hidden, self.heads, self.groups = int(p["hidden_size"]), int(p["heads"]), int(p["groups"])
         self.n, self.e, self.taps, self.eps = int(p["state"]), int(p["value_dim"]), int(p["conv"]), float(p["eps"])
         self.norm_groups = int(p.get("norm_groups", 1))
-        self.inner = self.heads * self.e
+        self.inner = self.core_width = self.heads * self.e
         if self.inner % self.norm_groups:
             raise ValueError(f"{self.norm_groups} norm groups do not divide the inner width {self.inner}")
         self.conv_channels = self.inner + 2 * self.groups * self.n
         # columns of the in-projection: [z | x | B | C | dt]
         self.conv_col0 = self.inner
         self.dt_off = self.inner + self.conv_channels
+        self.in_width = self.dt_off + self.heads
         self._finish_layout()
 
     def weights(self) -> dict[str, WeightSpec]:
@@ -168,25 +192,77 @@ class StateSpaceMixer(_ScanMixer):
                 "conv.b": WeightSpec((self.conv_channels,)), "dt_bias": WeightSpec((self.heads,)), "A_log": WeightSpec((self.heads,)),
                 "D": WeightSpec((self.heads,)), "norm": WeightSpec((self.inner,), init="one_plus_normal"), "o": WeightSpec((self.hidden, self.inner))}
 
-    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
-        self.w_in = tensors["in"].contiguous()
+    def load_core(self, tensors: Mapping[str, torch.Tensor]) -> None:
         self.w_conv, self.b_conv = self._float(tensors["conv"]), self._float(tensors["conv.b"])
         self.a_log, self.dt_bias, self.skip = self._float(tensors["A_log"]), self._float(tensors["dt_bias"]), self._float(tensors["D"])
         self.norm = self._float(tensors["norm"])
-        self.w_o = tensors["o"].contiguous()
 
-    def forward(self, x, step, cache, own_cache):
-        if cache is None or not own_cache:
-            raise ValueError("the state-space mixer keeps a state per request; the schedule gave it none")
-        proj = ops.linear(x, self.w_in, None, torch.float32)
+    def step_plans(self):
+        return recurrent.segment_planner(self.dtype)
+
+    def core(self, proj, col0, step, cache, out, scale):
         state, slots, rows = cache.state, cache.slots, step.n_rows
-        conv = recurrent.causal_conv_silu(proj, self.conv_col0, self.w_conv, self.b_conv, state, self.conv_off, slots, step.token_row, step.row_start)
-        recurrent.conv_state_update(proj, self.conv_col0, self.conv_channels, self.taps, state, self.conv_off, slots, step.row_start, rows)
+        conv_col, dt_off = col0 + self.conv_col0, col0 + self.dt_off
+        conv = recurrent.causal_conv_silu(proj, conv_col, self.w_conv, self.b_conv, state, self.conv_off, slots, step.token_row, step.row_start)
+        recurrent.conv_state_update(proj, conv_col, self.conv_channels, self.taps, state, self.conv_off, slots, step.row_start, rows)
         bn = self.groups * self.n
-        y = recurrent.state_scan(self.mode, conv, self.inner, self.inner + bn, 0, proj, self.dt_off, self.dt_off, self.a_log, self.dt_bias, self.skip,
-                                 state, 0, slots, step.row_start, rows, self.heads, self.groups, self.n, self.n_padded, self.e)
-        y = recurrent.gated_group_norm(y, proj, 0, self.norm, self.inner // self.norm_groups, True, self.eps, self.dtype)
-        return ops.linear(y, self.w_o, None, self.dtype, may_leave_partials=True)  # the result is a residual delta
+
+        def scan(state, slots, row_start, rows, states_only=False, decays=None):
+            return recurrent.state_scan(self.mode, conv, self.inner, self.inner + bn, 0, proj, dt_off, dt_off, self.a_log, self.dt_bias, self.skip, state, 0, slots, row_start,
+                                        rows, self.heads, self.groups, self.n, self.n_padded, self.e, states_only=states_only, decays=decays)
+
+        y = self._walk(scan, step, state, slots, self.e * self.n_padded, self.e)
+        recurrent.gated_group_norm(y, proj, col0, self.norm, self.inner // self.norm_groups, True, self.eps, self.dtype, scale=scale, out=out)
+
+
+class MatrixMemoryMixer(_ScanMixer, Branch):
+    in_names = ("q", "k", "v", "g", "i", "f")
+    out_name = "o"
+
+    def __init__(self, spec: PartSpec, build: BuildContext):
+        super().__init__(spec, build)
+        p = spec.params
+        self.hidden, self.heads = int(p["hidden_size"]), int(p["heads"])
+        self.n, self.e = int(p["head_dim"]), int(p.get("value_dim") or p["head_dim"])
+        self.cap, self.eps = float(p["gate_cap"]), float(p["eps"])
+        if self.n > 256:
+            raise ValueError(f"a state of {self.n} per column is above the scan kernel's limit of 256")
+        if not self.cap > 0:
+            raise ValueError(f"gates capped at {self.cap}")
+        self.qk_width, self.core_width = self.heads * self.n, self.heads * self.e
+        self.in_width = 2 * self.qk_width + 2 * self.core_width + 2 * self.heads
+        self.n_padded = _round_up(self.n, 4)
+        self.per_head = (self.e + 1) * self.n_padded  # the columns of the values, then the sum of keys
+        self.max_off = self.heads * self.per_head
+        self.record = _round_up(self.max_off + self.heads, 4)
+
+    def weights(self) -> dict[str, WeightSpec]:
+        h = self.hidden
+        return {"q": WeightSpec((self.qk_width, h)), "k": WeightSpec((self.qk_width, h)), "v": WeightSpec((self.core_width, h)), "g": WeightSpec((self.core_width, h)),
+                "i": WeightSpec((self.heads, h)), "i.b": WeightSpec((self.heads,)), "f": WeightSpec((self.heads, h)), "f.b": WeightSpec((self.heads,)),
+                "norm": WeightSpec((self.core_width,), init="one_plus_normal"), "o": WeightSpec((h, self.core_width))}
+
+    def load_core(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        self.b_i, self.b_f, self.norm = self._float(tensors["i.b"]), self._float(tensors["f.b"]), self._float(tensors["norm"])
+
+    def step_plans(self):
+        return recurrent.segment_planner(self.dtype)
+
+    def core(self, proj, col0, step, cache, out, scale):
+        if scale != 1.0:
+            raise ValueError("a matrix memory's result takes no factor of its own")
+        state, slots = cache.state, cache.slots
+        k_off, v_off = col0 + self.qk_width, col0 + 2 * self.qk_width
+        g_off = v_off + self.core_width
+        i_off = g_off + self.core_width
+        gates = recurrent.matrix_memory_gates(proj, i_off, i_off + self.heads, self.b_i, self.b_f, self.cap, state, self.max_off, slots, step.row_start, step.n_rows, self.heads)
+
+        def scan(state, slots, row_start, rows, states_only=False, decays=None):
+            return recurrent.matrix_memory_scan(proj, k_off, col0, v_off, gates, state, 0, slots, row_start, rows, self.heads, self.n, self.n_padded, self.e, self.n ** -0.5,
+                                                states_only=states_only, decays=decays)
+
+        y = self._walk(scan, step, state, slots, self.per_head, self.e + 1)
+        recurrent.matrix_memory_norm(y, gates, proj, g_off, self.norm, self.e, self.eps, out)
 
 
 class SelectiveScanMixer(Mixer):
@@ -410,4 +486,5 @@ register_mixer("lightning", LightningAttention)
 register_mixer("delta_rule", GatedDeltaRule)
 register_mixer("mamba1", SelectiveScanMixer)
 register_mixer("mamba2", StateSpaceMixer)
+register_mixer("matrix_memory", MatrixMemoryMixer)
 register_mixer("wkv", WkvMixer)

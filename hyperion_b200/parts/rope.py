@@ -8,6 +8,8 @@ y[i+d/2] = x[i+d/2] c + x[i] s over the whole head (reference.rs:91-109).  Param
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 from .. import ops
@@ -105,3 +107,40 @@ class PartialHalfRotaryEncoding(InterleavedRotaryEncoding):
 
 
 register_position("rope_half_partial", PartialHalfRotaryEncoding)
+
+
+def slowed_frequencies(dims: int, base: float, factor: float, original: float, fast: float, slow: float) -> torch.Tensor:
+    """float64 [dims / 2]: base**(-2i/dims), kept where a pair turns at least ``fast`` times within ``original`` positions, divided by ``factor`` where it turns
+    at most ``slow`` times, and a mixture along a ramp over the pairs in between."""
+
+    def pair_that_turns(times: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * times)) / (2.0 * math.log(base))
+
+    low = max(math.floor(pair_that_turns(fast)), 0)
+    high = min(math.ceil(pair_that_turns(slow)), dims - 1)
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    freq = torch.tensor(base, dtype=torch.float64) ** (-2.0 * i / max(1, dims))
+    ramp = ((i - low) / max(high - low, 0.001)).clamp(0.0, 1.0)
+    return freq / factor * ramp + freq * (1.0 - ramp)
+
+
+class SlowedHalfRotaryEncoding(PartialHalfRotaryEncoding):
+    """The rotation of :class:`PartialHalfRotaryEncoding` stretched to longer texts than the model was first made for (YaRN: Peng et al., "YaRN: Efficient Context
+    Window Extension of Large Language Models"): frequencies as :func:`slowed_frequencies` gives them, cosine and sine both multiplied by
+    ``amplitude`` = 0.1 ln(factor) + 1.  Parameters: ``dims``, ``base``, ``factor``, ``original``, ``fast``, ``slow``."""
+
+    def __init__(self, spec: PartSpec, build: BuildContext):
+        super().__init__(PartSpec(spec.kind, spec.prefix, {"dims": spec.params["dims"], "base": spec.params["base"]}), build)
+        p = spec.params
+        values = tuple(float(p[name]) for name in ("factor", "original", "fast", "slow"))
+        self.factor, self.amplitude = values[0], 0.1 * math.log(values[0]) + 1.0
+        key = ("slowed_frequencies", self.dims, self.base, *values, str(build.device))
+        if key not in build.shared:
+            build.shared[key] = slowed_frequencies(self.dims, self.base, *values).to(torch.float32).to(build.device)
+        self.inv_freq = build.shared[key]
+
+    def apply_(self, x, heads, head_dim, positions):
+        raise ValueError("this rotation also scales what it turns; the part that uses it passes the amplitude to the kernel that stores its heads")
+
+
+register_position("rope_half_slowed", SlowedHalfRotaryEncoding)

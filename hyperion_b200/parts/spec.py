@@ -31,6 +31,7 @@ class LayerSpec:
     mixer: PartSpec
     feed_forward: Optional[PartSpec]  # None: the layer has a mixer only
     norms: Mapping[str, PartSpec]
+    connections: Mapping[str, PartSpec] = field(default_factory=dict)  # how sublayers read from and write to several residual streams
 
 
 @dataclass(frozen=True)

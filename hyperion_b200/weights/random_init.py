@@ -30,7 +30,7 @@ def random_tensor(name: str, wanted: WeightSpec, seed: int, std: float, device: 
     if dtype not in (torch.bfloat16, torch.float32):
         raise ValueError(f"random weights are made as bfloat16 or float32, got {dtype}")
     key = philox_normal.tensor_key(seed, name)
-    mean = 1.0 if wanted.init == "one_plus_normal" else 0.0
+    mean = 1.0 if wanted.init == "one_plus_normal" else wanted.mean
     count = 1
     for extent in wanted.shape:
         count *= int(extent)
