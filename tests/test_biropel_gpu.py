@@ -1,0 +1,925 @@
+"""Biropel on the GPU against the plain implementation (``tests/plain/biropel_plain.py``): every mechanism alone, whole prompts against
+token-by-token decoding, portions down to two tokens, batches of unequal requests against each alone, pages and state slots that are freed
+and taken again, keys just inside and just outside a window, at page borders and far away, the matrix memory's and the state-space mixer's states
+over long texts, long decoding, sizes that differ in every respect between the configurations, layers that read another layer's keys and values through
+windows of their own, one to many residual streams, and greedy generation through ``Engine.generate``.
+
+The configurations and weights are made here.  Weights are drawn so that a fault shows: matrices of N(0, gain^2 / in) make the attention
+peaked, mixing matrices keep the streams apart, gates of the recurrences forget slowly, and where a test is about one key a marker token, whose
+key points where the last query points, makes that key's score stand out.  float32 runs are held to 3e-4 of the largest logit, which no wrong key,
+window, state or lost page survives; bfloat16 runs to 5e-2 of a row's root-mean-square logit.
+"""
+from __future__ import annotations
+
+import json
+import math
+import subprocess
+import sys
+from pathlib import Path
+
+import numpy as np
+import pytest
+import torch
+
+from plain import biropel_plain as plain
+
+pytestmark = pytest.mark.gpu
+ROOT = Path(__file__).resolve().parent.parent
+TOLERANCE = {"float32": 3e-4, "bfloat16": 5e-2}
+
+
+# ------------------------------------------------------------------------------------------ configurations
+def heads(count, kv_heads, dim, vdim, scale, window=None, cap=None, rot=None, scaling=None, temp=None, kv_from=None):
+    m = {"heads": count, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale}
+    if window is not None:
+        m["mask"] = {"size": window}
+    if cap is not None:
+        m["softcap"] = cap
+    if rot is not None:
+        m["rot"] = {"dims": rot[0], "base": rot[1]}
+        if scaling is not None:
+            m["rot"]["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    if temp is not None:
+        m["q_temp"] = {"coef": temp[0], "every": temp[1]}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return m
+
+
+def state_space(count, vdim, state, groups, norm_groups, conv):
+    return {"heads": count, "vdim": vdim, "state": state, "groups": groups, "norm_groups": norm_groups, "conv": conv}
+
+
+def memory(count, dim, vdim, cap):
+    return {"heads": count, "dim": dim, "vdim": vdim, "gate_cap": cap}
+
+
+def layer(kind, mixer, ff=None):
+    return {"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": ff} if ff is not None else None}
+
+
+def attention(m, ff=None):
+    return layer("attention", m, ff)
+
+
+def beside_states(left, right, ff=None):
+    return layer("parallel", {"left": left, "right": right}, ff)
+
+
+def beside_memory(left, right, ff=None):
+    return layer("parallel_2", {"left": left, "right": right}, ff)
+
+
+def document(width, vocab, streams, layers, eps=1e-5):
+    return {"architecture": "Biropel", "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": eps}, "layers": layers}
+
+
+# Two models that differ in every size, in the order of their layers, in eps and in the number of streams; keys and values of unequal size and of shapes that
+# the tensor-core kernels take, windows that are no multiple of a page and none, a layer that reads another's keys through a wider and one that reads
+# them through a narrower window, groups and norm groups that differ, convolutions of two to five taps, layers without a feed-forward.
+CONFIGS = {
+    "A": document(64, 131, 2, [beside_memory(heads(4, 2, 24, 16, 0.4, cap=12.0, temp=(0.7, 20)), memory(3, 20, 12, 4.0), 72),
+                               attention(heads(4, 2, 24, 20, 0.25, window=20, rot=(10, 300.0)), 40),
+                               beside_states(heads(6, 3, 12, 18, 0.3, window=33, cap=8.0, rot=(8, 1e4), scaling=(8.0, 64.0, 8.0, 1.0)), state_space(6, 10, 12, 3, 4, 3)),
+                               attention(heads(6, 2, 24, 20, 0.2, window=45, rot=(10, 300.0), kv_from=1)),
+                               attention(heads(2, 2, 24, 20, 0.3, window=7, rot=(10, 300.0), kv_from=1), 24)], eps=2e-3),
+    "B": document(96, 211, 4, [attention(heads(6, 3, 64, 64, 0.1, window=33, rot=(32, 1e4)), 60),
+                               beside_states(heads(2, 1, 128, 128, 0.08, window=50, cap=30.0, rot=(128, 5e4), scaling=(2.0, 128.0, 16.0, 2.0)), state_space(4, 24, 16, 1, 1, 5), 100),
+                               beside_memory(heads(4, 4, 48, 48, 0.25, cap=20.0, temp=(0.3, 64)), memory(2, 32, 40, 9.0), 50),
+                               attention(heads(3, 3, 64, 64, 0.15, window=80, rot=(32, 1e4), kv_from=0), 28),
+                               beside_states(heads(4, 2, 16, 16, 0.3), state_space(3, 8, 40, 3, 3, 2), 16),
+                               beside_memory(heads(2, 1, 64, 64, 0.2), memory(5, 9, 7, 30.0))], eps=1e-6),
+}
+# One layer each: a mechanism alone as far as the design allows it (a mixer of two halves keeps both).
+STATES, MEMORY = state_space(4, 12, 16, 2, 2, 4), memory(3, 16, 12, 10.0)
+ALONE = {
+    "attention": document(48, 97, 2, [attention(heads(4, 2, 24, 20, 0.3, window=24, rot=(8, 1e3)))]),
+    "attention_48": document(48, 97, 3, [attention(heads(6, 2, 48, 48, 0.2, window=24, rot=(12, 1e3)))]),
+    "attention_64": document(64, 97, 2, [attention(heads(4, 2, 64, 64, 0.15, window=24, rot=(16, 1e3)))]),
+    "attention_128": document(64, 61, 1, [attention(heads(6, 2, 128, 128, 0.1, window=100, rot=(128, 1e4)))]),
+    "shared": document(64, 97, 2, [attention(heads(4, 2, 64, 64, 0.15, window=10, rot=(16, 1e3))), attention(heads(2, 2, 64, 64, 0.1, window=24, rot=(16, 1e3), kv_from=0))]),
+    "stretched": document(48, 97, 2, [beside_states(heads(4, 2, 24, 20, 0.3, window=24, cap=15.0, rot=(8, 1e3), scaling=(4.0, 64.0, 8.0, 1.0)), STATES)]),
+    "stretched_48": document(48, 97, 2, [beside_states(heads(4, 2, 48, 48, 0.25, window=24, cap=15.0, rot=(12, 1e3), scaling=(4.0, 64.0, 8.0, 1.0)), STATES)]),
+    "stretched_64": document(64, 97, 2, [beside_states(heads(4, 2, 64, 64, 0.2, window=24, cap=15.0, rot=(16, 1e3), scaling=(4.0, 64.0, 8.0, 1.0)), STATES)]),
+    "open": document(48, 61, 2, [beside_memory(heads(4, 2, 24, 20, 0.7, cap=25.0, temp=(0.3, 100)), MEMORY)]),
+    "open_64": document(64, 61, 2, [beside_memory(heads(4, 2, 64, 64, 0.25, cap=25.0, temp=(0.3, 100)), MEMORY)]),
+    "memory_wide": document(40, 61, 2, [beside_memory(heads(2, 1, 8, 8, 0.5), memory(2, 130, 33, 15.0))]),
+    "states_wide": document(40, 61, 2, [beside_states(heads(2, 1, 8, 8, 0.5, window=9), state_space(2, 40, 140, 1, 1, 4))]),
+    "feed_forward": document(48, 97, 2, [attention(heads(2, 2, 8, 8, 0.5, window=8, rot=(4, 1e3)), 136)]),
+    "five_streams": document(40, 61, 5, [attention(heads(2, 2, 8, 8, 0.5, window=8, rot=(4, 1e3)), 24), beside_states(heads(2, 1, 8, 8, 0.5, window=9), STATES, 24)]),
+}
+
+
+def make_weights(doc: dict, seed: int, gain: float = 1.5) -> dict[str, torch.Tensor]:
+    """bfloat16 tensors under the design's names: matrices N(0, gain^2 / in), norm weights around 1, biases of the size of what they stand beside, mixing matrices
+    that keep most of a stream and trade some, recurrences that forget over tens of tokens."""
+    from hyperion_b200.models import DecoderModel, get_architecture
+
+    entry = get_architecture("Biropel")
+    model = DecoderModel(entry.build_spec(entry.read_config(doc)), torch.float32, torch.device("meta"))
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, wanted in model.expected_tensors().items():
+        shape = tuple(wanted.shape)
+        last = name.rsplit(".", 1)[-1]
+        connection = ".hc" in name
+        if connection and last == "mix":
+            t = 0.8 * torch.eye(shape[0]) + 0.25 * torch.randn(shape, generator=g)
+        elif connection:
+            t = (0.5 if last == "in" else 1.0) + 0.4 * torch.randn(shape, generator=g)
+        elif last in ("norm", "norm1", "norm2", "out"):
+            t = 1.0 + 0.2 * torch.randn(shape, generator=g)
+        elif last == "A_log":
+            t = torch.log(0.05 + 2.0 * torch.rand(shape, generator=g))
+        elif last == "dt_bias":
+            t = torch.randn(shape, generator=g) - 2.0
+        elif last == "D":
+            t = torch.randn(shape, generator=g)
+        elif last == "conv":
+            t = torch.randn(shape, generator=g) * 0.6
+        elif name.endswith(".f.b"):
+            t = 3.0 + torch.randn(shape, generator=g)
+        elif last == "b":
+            t = 0.5 * torch.randn(shape, generator=g)
+        elif name == "embed":
+            t = torch.randn(shape, generator=g)
+        else:
+            t = torch.randn(shape, generator=g) * (gain / shape[-1] ** 0.5)
+        out[name] = t.to(torch.bfloat16)
+    return out
+
+
+def align_keys_with_queries(doc: dict, weights: dict[str, torch.Tensor]) -> None:
+    """Make one score stand out.  The last token of the vocabulary is the marker, the one before it the query: the marker's embedding is half the query's and half its
+    own direction.  Keys are made by the matrices (and biases) that make the queries (every key head takes its first query head's), and the marker's own direction
+    adds the query's key once more, so a marker's key meets the query with a larger score than even the query's own key does."""
+    query = weights["embed"][-2].float()
+    own = torch.randn(query.shape, generator=torch.Generator().manual_seed(99))
+    own -= query * (own @ query) / (query @ query)
+    weights["embed"][-1] = ((query + own) / 2 ** 0.5).to(torch.bfloat16)
+    lift = torch.outer(query / query.norm(), own / own.norm()) * 1.5
+    for index, entry in enumerate(doc["layers"]):
+        m, p = entry["mixer"], f"l{index}.mix."
+        if entry["type"] != "attention":
+            m, p = m["left"], p + "left."
+        if "kv_from" in m:  # its queries are those that the lender's keys were made for
+            every = doc["layers"][0]["mixer"]["heads"] // m["heads"]
+            weights[p + "q"] = weights["l0.mix.q"].view(-1, m["dim"], query.numel())[::every].reshape(m["heads"] * m["dim"], -1).clone()
+            weights[p + "q.b"] = weights["l0.mix.q.b"].view(-1, m["dim"])[::every].reshape(-1).clone()
+            continue
+        rep = m["heads"] // m["kv_heads"]
+        k = weights[p + "q"].view(m["heads"], m["dim"], -1)[::rep].reshape(m["kv_heads"] * m["dim"], -1).float()
+        weights[p + "k"] = (k + k @ lift).to(torch.bfloat16)
+        if p + "k.b" in weights:
+            weights[p + "k.b"] = weights[p + "q.b"].view(m["heads"], m["dim"])[::rep].reshape(-1).clone()
+
+
+MARKED = ("attention", "attention_48", "attention_64", "shared", "stretched", "stretched_48", "stretched_64", "open", "open_64")
+
+
+@pytest.fixture(scope="module")
+def folders(tmp_path_factory):
+    from hyperion_b200.weights import write_file
+
+    root = tmp_path_factory.mktemp("biropel_models")
+    made = {}
+    for index, (name, doc) in enumerate({**CONFIGS, **ALONE}.items()):
+        folder = root / name
+        folder.mkdir()
+        (folder / "config.json").write_text(json.dumps(doc))
+        weights = make_weights(doc, 23 + index, gain=1.2 if name in CONFIGS else 1.5)
+        if name in MARKED:
+            align_keys_with_queries(doc, weights)
+        write_file(folder / "model.safetensors", weights)
+        made[name] = folder
+    return made
+
+
+_plain_cache: dict = {}
+
+
+def plain_logits(folder: Path, ids) -> np.ndarray:
+    key = (str(folder), tuple(ids))
+    if key not in _plain_cache:
+        config, weights = plain.read_model_folder(folder)
+        _plain_cache[key] = plain.forward(config, weights, list(ids)).numpy()
+    return _plain_cache[key]
+
+
+def ids_for(seed: int, count: int, vocab: int) -> list[int]:
+    return torch.randint(0, vocab, (count,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+def engine_for(folder, dtype, **options):
+    from hyperion_b200.api import Engine
+
+    options.setdefault("page_size", 16)
+    options.setdefault("max_tokens", 1024)
+    options.setdefault("max_requests", 4)
+    return Engine.from_folder(folder, dtype=dtype, **options)
+
+
+def row_errors(got: np.ndarray, want: np.ndarray) -> np.ndarray:
+    got, want = np.atleast_2d(got), np.atleast_2d(want)
+    return np.sqrt(((got - want) ** 2).mean(axis=1)) / np.sqrt((want ** 2).mean(axis=1))
+
+
+def relative_error(got: np.ndarray, want: np.ndarray) -> float:
+    """The largest difference against the largest logit: the sharp measure, which a float32 run meets.  For bfloat16 results the worst row's
+    root-mean-square difference against its root-mean-square logit."""
+    sharp = float(np.abs(got - want).max() / np.abs(want).max())
+    return sharp if sharp <= TOLERANCE["float32"] else float(row_errors(got, want).max())
+
+
+def assert_close(got: np.ndarray, want: np.ndarray, dtype: str, what=None, deep: bool = False) -> None:
+    """``deep`` (a model of several layers in bfloat16): three rows in a hundred may be off, and the middle row stays within half the tolerance (a fault of a kernel or
+    a cache moves every row).  float32 is held to its line without exceptions."""
+    assert np.isfinite(got).all(), what
+    if deep and dtype == "bfloat16":
+        errors = row_errors(got, want)
+        over, middle = float((errors > TOLERANCE[dtype]).mean()), float(np.median(errors))
+        assert over <= 0.03 and middle <= TOLERANCE[dtype] / 2, (what, over, middle)
+        return
+    error = relative_error(got, want)
+    assert error <= TOLERANCE[dtype], (what, error)
+
+
+def run_cut(engine, name, ids, sizes) -> np.ndarray:
+    """One request in portions of the given sizes (cycled), every position's logits."""
+    from hyperion_b200.engine.batch import StepEntry
+
+    rows, at, k = [], 0, 0
+    while at < len(ids):
+        n = min(sizes[k % len(sizes)], len(ids) - at)
+        k += 1
+        rows.append(engine.step([StepEntry(name, ids[at:at + n], list(range(n)))]).cpu().numpy().copy())
+        at += n
+    engine.finish(name)
+    engine.check()
+    return np.concatenate(rows)
+
+
+# ------------------------------------------------------------------------------------------ every mechanism alone
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", sorted(ALONE))
+def test_one_layer_of_each_kind(folders, name, dtype):
+    """A model of one layer (two where one reads the other's keys): the whole prompt at once, again in portions of 5, 2, 1, 9 tokens, and
+    over larger pages."""
+    vocab = ALONE[name]["vocab"]
+    ids = ids_for(3, 75, vocab)
+    want = plain_logits(folders[name], ids)
+    for page_size in (8, 64):
+        engine = engine_for(folders[name], dtype, page_size=page_size)
+        deep = len(ALONE[name]["layers"]) > 1
+        assert_close(run_cut(engine, "w", ids, [len(ids)]), want, dtype, "whole", deep)
+        assert_close(run_cut(engine, "p", ids, [5, 2, 1, 9]), want, dtype, "portions", deep)
+
+
+def test_which_kernels_a_shape_takes(folders):
+    for name, fast in (("attention", False), ("attention_48", True), ("attention_64", True)):
+        for dtype in ("float32", "bfloat16"):
+            assert engine_for(folders[name], dtype).model.layers[0].mixer.fast == (fast and dtype == "bfloat16"), (name, dtype)
+
+
+@pytest.mark.parametrize("streams", [1, 2, 3, 4, 7, 16])
+def test_a_boundary_between_two_sublayers(streams):
+    """Streams that are still one row and streams apart; nothing pending, one result (dense, in pieces), two normed results; rows picked out behind the last layer."""
+    from hyperion_b200 import ops
+    from hyperion_b200.ops.gemm import SplitSum
+
+    for hidden in (8, 37, 130, 516, 1024, 2048, 4096, 5000):
+        if hidden > 600 and streams not in (3, 7):
+            continue
+        g = torch.Generator().manual_seed(hidden + streams)
+        tokens, eps, y_eps = 13, 1e-5, 1e-3
+        w = {"c.in": 0.5 + torch.randn(streams, generator=g), "c.out": torch.randn(streams, generator=g), "c.mix": torch.randn(streams, streams, generator=g)}
+        read = torch.randn(streams, generator=g)
+        weight, n0, n1 = (1 + 0.2 * torch.randn(hidden, generator=g) for _ in range(3))
+        wide = {k: v.double() for k, v in w.items()}
+        for dtype, tolerance in ((torch.float32, 2e-5), (torch.bfloat16, 1e-2)):
+            a, b = (torch.randn(tokens, hidden, generator=g).to(dtype) for _ in range(2))
+            pieces = torch.randn(5, tokens, hidden, generator=g)
+            summed = SplitSum(pieces.cuda(), None, dtype)
+            both = 0.5 * (plain.rms_norm(a.double(), n0.double(), y_eps) + plain.rms_norm(b.double(), n1.double(), y_eps))
+            mixed = 0.5 * (plain.rms_norm(pieces.double().sum(0), n0.double(), y_eps) + plain.rms_norm(b.double(), n1.double(), y_eps))
+            cases = {"nothing": ((), None), "dense": ((a.cuda(),), a.double()), "pieces": ((summed,), pieces.double().sum(0)), "two": ((a.cuda(), b.cuda()), both),
+                     "two, one in pieces": ((summed, b.cuda()), mixed)}
+            for equal in (False, True):
+                start = 3 * torch.randn((tokens, hidden) if equal else (tokens, streams, hidden), generator=g)
+                old = start.double()[:, None].expand(tokens, streams, hidden) if equal else start.double()
+                for name, (results, y) in cases.items():
+                    normed = {"norms": (n0.cuda(), n1.cuda()), "result_eps": y_eps, "result_scale": 0.5} if len(results) == 2 else {}
+                    pending = {"results": results, "mix": w["c.mix"].cuda(), "share": w["c.out"].cuda(), **normed} if results else {}
+                    new = old if y is None else plain.write_streams(old.transpose(0, 1), y, wide, "c.").transpose(0, 1)
+                    h = start.cuda()
+                    x, after = ops.hyper_connect(h, streams, read.cuda(), weight.cuda(), eps, dtype, **pending)
+                    want = plain.rms_norm(torch.einsum("s,tsw->tw", read.double(), new), weight.double(), eps)
+                    what = (hidden, dtype, equal, name)
+                    assert x.dtype == dtype and (x.cpu().double() - want).abs().max() <= tolerance * want.abs().max(), what
+                    if results:
+                        assert after.shape == (tokens, streams, hidden) and (after.cpu().double() - new).abs().max() <= 2e-5 * new.abs().max(), what
+                        assert equal or after.data_ptr() == h.data_ptr()
+                    else:
+                        assert after is h and torch.equal(h.cpu(), start), what
+                    rows = torch.tensor([12, 3, 3], dtype=torch.int32)
+                    h = start.cuda()
+                    x, after = ops.hyper_connect(h, streams, None, weight.cuda(), eps, dtype, rows=rows.cuda(), **pending)
+                    want = plain.rms_norm(new.sum(1), weight.double(), eps)[rows.long()]
+                    assert torch.equal(h.cpu(), start) and (x.cpu().double() - want).abs().max() <= tolerance * want.abs().max(), what
+
+
+def test_relu_squared():
+    from hyperion_b200 import ops
+
+    for shape in ((3, 7), (5, 64), (130, 520)):
+        x = 3 * torch.randn(shape, generator=torch.Generator().manual_seed(1))
+        for dtype, tolerance in ((torch.float32, 1e-6), (torch.bfloat16, 5e-3)):
+            y = x.to(dtype)
+            want = torch.relu(y.double()).pow(2)
+            assert (ops.relu_squared(y.cuda()).cpu().double() - want).abs().max() <= tolerance * want.abs().max()
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_heads_are_normed_turned_and_tempered(dtype):
+    """Queries to a buffer, keys and values to pages in either arrangement; sizes and rotated dimensions that are and are not whole 16-byte pieces; either pairing;
+    columns of a wider product; with and without biases, the unit norm, an amplitude and the temperature; few tokens and many, far positions."""
+    from hyperion_b200 import ops
+
+    g = torch.Generator().manual_seed(7)
+    tolerance = 1e-5 if dtype == torch.float32 else 1e-2
+    for q_heads, kv_heads, d, e, dims, half, unit, bias, temp, amplitude in (
+            (4, 2, 24, 20, 8, True, False, True, None, 1.0), (4, 2, 24, 24, 24, True, True, False, (0.5, 7), 1.3), (3, 1, 7, 5, 6, True, False, True, None, 0.7),
+            (6, 3, 64, 64, 10, True, False, True, None, 1.0), (2, 2, 64, 64, 0, True, True, False, (0.3, 100), 1.0), (1, 1, 200, 40, 144, True, True, True, (1.0, 1), 1.1),
+            (2, 1, 1, 1, 0, True, True, True, (0.2, 3), 1.0), (2, 1, 16, 16, 12, False, False, False, None, 1.2), (5, 5, 96, 96, 48, True, False, True, None, 1.0),
+            (2, 2, 640, 8, 640, True, True, False, None, 1.0)):
+        for tokens, offset in ((3, 5), (530, 0), (4, 60)):
+            page, pages = 8, 80
+            qw, kw, vw, before = q_heads * d, kv_heads * d, kv_heads * e, 4
+            x = torch.randn(tokens, before + qw + kw + vw + 3, generator=g)
+            b = torch.randn(qw + kw + vw, generator=g) if bias else None
+            inv = torch.rand(dims // 2, generator=g) if dims else None
+            cache = torch.zeros((pages, 2, kv_heads, page, e) if d == e else (pages, kv_heads, page, d + e), dtype=dtype).cuda()
+            table = torch.randperm(pages, generator=g).int().view(1, pages)
+            positions = torch.arange(tokens, dtype=torch.int32) + offset
+            q = torch.empty(tokens, qw, dtype=dtype).cuda()
+            ops.heads_store(x.cuda()[:, before:], 0, qw, qw + kw, q_heads, kv_heads, d, e, positions.cuda(), q_out=q, bias=b.cuda() if bias else None, eps=1e-3, cache=cache,
+                            block_table=table.cuda(), token_row=torch.zeros(tokens, dtype=torch.int32).cuda(), page_size=page, inv_freq=inv.cuda() if dims else None, rot_dims=dims,
+                            rot_half=half, amplitude=amplitude, unit_norm=unit, temperature=temp)
+            full = x[:, before : before + qw + kw + vw].double() + (b.double() if bias else 0)
+
+            def turned(z):
+                if unit:
+                    z = plain.unit_rms(z, 1e-3)
+                if not dims:
+                    return z
+                angle = (positions.float()[:, None] * inv[None]).double()
+                c, s = torch.cos(angle)[:, None] * amplitude, torch.sin(angle)[:, None] * amplitude
+                out = z.clone()
+                lo, hi = (slice(0, dims // 2), slice(dims // 2, dims)) if half else (slice(0, dims, 2), slice(1, dims, 2))
+                out[..., lo], out[..., hi] = z[..., lo] * c - z[..., hi] * s, z[..., hi] * c + z[..., lo] * s
+                return out
+
+            want_q, want_k = turned(full[:, :qw].reshape(tokens, q_heads, d)), turned(full[:, qw : qw + kw].reshape(tokens, kv_heads, d))
+            if temp is not None:
+                want_q = want_q * torch.tensor([1 + temp[0] * math.log((int(p) + 1) // temp[1] + 1) for p in positions], dtype=torch.float64)[:, None, None]
+            want_v = full[:, qw + kw :].reshape(tokens, kv_heads, e)
+            what = (q_heads, d, e, dims, half, tokens)
+            assert (q.cpu().double().view(tokens, q_heads, d) - want_q).abs().max() <= tolerance * want_q.abs().max(), what
+            where, slot = table[0, (positions // page).long()].long(), (positions % page).long()
+            host = cache.cpu().double()
+            if d == e:
+                got_k, got_v = host[where, 0, :, slot], host[where, 1, :, slot]
+            else:
+                got_k, got_v = host[where, :, slot][..., :d], host[where, :, slot][..., d:]
+            assert (got_k - want_k).abs().max() <= tolerance * want_k.abs().max(), what
+            assert (got_v - want_v).abs().max() <= tolerance * want_v.abs().max(), what
+
+
+def _memory_case(heads, n, e, counts, seed, cap=5.0):
+    """Random inputs of a matrix memory for rows of the given lengths, its record's layout, and what the plain recurrence gives per row from a zero state."""
+    g = torch.Generator().manual_seed(seed)
+    tokens = sum(counts)
+    x = torch.randn(tokens, 2 * heads * n + heads * e + 2 * heads, generator=g)
+    bias_i, bias_f = torch.randn(heads, generator=g), 3 + torch.randn(heads, generator=g)
+    start = [0]
+    for c in counts:
+        start.append(start[-1] + c)
+    return x, bias_i, bias_f, torch.tensor(start, dtype=torch.int32)
+
+
+def _plain_memory(x, bias_i, bias_f, heads, n, e, cap):
+    """The recurrence for one row in double: (S^T q, n . q, running maximum) per token."""
+    T = x.shape[0]
+    x = x.double()
+    q, k = x[:, : heads * n].reshape(T, heads, n) * n ** -0.5, x[:, heads * n : 2 * heads * n].reshape(T, heads, n)
+    v = x[:, 2 * heads * n : 2 * heads * n + heads * e].reshape(T, heads, e)
+    i = plain.soft_cap(x[:, -2 * heads : -heads] + bias_i.double(), cap)
+    f = torch.nn.functional.logsigmoid(plain.soft_cap(x[:, -heads:] + bias_f.double(), cap))
+    S, s, m = torch.zeros(heads, n, e).double(), torch.zeros(heads, n).double(), torch.zeros(heads).double()
+    rows = []
+    for t in range(T):
+        new = torch.maximum(f[t] + m, i[t])
+        keep, take = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
+        S = keep[:, None, None] * S + take[:, None, None] * k[t][:, :, None] * v[t][:, None]
+        s, m = keep[:, None] * s + take[:, None] * k[t], new
+        rows.append((torch.einsum("hne,hn->he", S, q[t]), (s * q[t]).sum(-1), m))
+    return tuple(torch.stack(z) for z in zip(*rows))
+
+
+@pytest.mark.parametrize("shape", [(3, 16, 12), (1, 1, 1), (2, 33, 31), (4, 64, 32), (2, 130, 65), (1, 256, 40)])
+def test_the_matrix_memory_kernels(shape):
+    """Gates, scan and what follows it, rows of 1 to 131 tokens at once and one row cut in two, against the plain recurrence."""
+    from hyperion_b200.ops import recurrent
+
+    heads, n, e = shape
+    cap, eps, n_padded = 5.0, 1e-5, -(-n // 4) * 4
+    counts = [1, 70, 2, 131, 32]
+    x, bi, bf, start = _memory_case(heads, n, e, counts, 3 + n)
+    per_head = (e + 1) * n_padded
+    m_off = heads * per_head
+    record = -(-(m_off + heads) // 4) * 4
+    state = torch.zeros(7, record).cuda()
+    slots = torch.tensor([4, 0, 6, 2, 1], dtype=torch.int32).cuda()
+    dev, i_off = x.cuda(), 2 * heads * n + heads * e
+    weight, gate = 1 + 0.2 * torch.randn(heads * e), torch.randn(sum(counts), heads * e)
+
+    def run(rows_x, row_start, row_slots, rows):
+        gates = recurrent.matrix_memory_gates(rows_x, i_off, i_off + heads, bi.cuda(), bf.cuda(), cap, state, m_off, row_slots, row_start, rows, heads)
+        return gates, recurrent.matrix_memory_scan(rows_x, heads * n, 0, 2 * heads * n, gates, state, 0, row_slots, row_start, rows, heads, n, n_padded, e, n ** -0.5)
+
+    gates, y = run(dev, start.cuda(), slots, len(counts))
+    out = torch.empty(sum(counts), heads * e).cuda()
+    recurrent.matrix_memory_norm(y, gates, gate.cuda(), 0, weight.cuda(), e, eps, out)
+    for row, count in enumerate(counts):
+        a, b = int(start[row]), int(start[row + 1])
+        raw, normaliser, top = _plain_memory(x[a:b], bi, bf, heads, n, e, cap)
+        assert (gates[a:b, 2].cpu().double() - torch.exp(-top)).abs().max() <= 2e-5 * torch.exp(-top).max()
+        assert (y[a:b, :, :e].cpu().double() - raw).abs().max() <= 2e-5 * max(1.0, float(raw.abs().max()))
+        assert (y[a:b, :, e].cpu().double() - normaliser).abs().max() <= 2e-5 * max(1.0, float(normaliser.abs().max()))
+        o = plain.unit_rms(raw / (torch.maximum(normaliser.abs(), torch.exp(-top)) + 1e-6)[..., None], eps).reshape(count, heads * e)
+        want = o * weight.double() * torch.sigmoid(gate[a:b].double())
+        assert (out[a:b].cpu().double() - want).abs().max() <= 1e-3 * max(1.0, float(want.abs().max()))
+    after = state.clone()
+    # the longest row again, cut after 37 tokens: the same bits, and the same state
+    state.zero_()
+    a = int(start[3])
+    one = torch.tensor([2], dtype=torch.int32).cuda()
+    first = run(dev[a : a + 37], torch.tensor([0, 37], dtype=torch.int32).cuda(), one, 1)
+    second = run(dev[a + 37 : a + 131], torch.tensor([0, 94], dtype=torch.int32).cuda(), one, 1)
+    assert torch.equal(torch.cat([first[0], second[0]]), gates[a : a + 131]) and torch.equal(torch.cat([first[1], second[1]])[..., : e + 1], y[a : a + 131, :, : e + 1])
+    assert torch.equal(state[2], after[2])
+
+
+def test_long_rows_in_segments():
+    """The matrix memory and the state-space scan with long rows cut into segments that are walked side by side: the one-pass results and states to rounding, from
+    states that are not zero, beside rows that are not cut."""
+    from hyperion_b200.ops import recurrent
+
+    heads, n, e, n_padded, cap = 3, 40, 24, 40, 5.0
+    counts = [700, 5, 1100, 300]
+    x, bi, bf, start = _memory_case(heads, n, e, counts, 5)
+    cut = recurrent.plan_segments(counts)
+    seg_start, seg_row = (torch.tensor(v, dtype=torch.int32).cuda() for v in cut)
+    per_head = (e + 1) * n_padded
+    m_off = heads * per_head
+    begin = torch.zeros(5, m_off + 4)
+    begin[:, :m_off] = torch.randn(5, m_off, generator=torch.Generator().manual_seed(1))
+    slots = torch.tensor([3, 0, 4, 1], dtype=torch.int32).cuda()
+    dev, i_off, rows_of = x.cuda(), 2 * heads * n + heads * e, start.cuda()
+
+    def memory_scan(gates):
+        return lambda s, sl, rs, rows, states_only=False, decays=None: recurrent.matrix_memory_scan(dev, heads * n, 0, 2 * heads * n, gates, s, 0, sl, rs, rows, heads, n, n_padded, e,
+                                                                                                   n ** -0.5, states_only=states_only, decays=decays)
+
+    one, many = begin.cuda(), begin.cuda()
+    gates = [recurrent.matrix_memory_gates(dev, i_off, i_off + heads, bi.cuda(), bf.cuda(), cap, s, m_off, slots, rows_of, 4, heads) for s in (one, many)]
+    y = memory_scan(gates[0])(one, slots, rows_of, 4)[..., : e + 1]
+    z = recurrent.scan_in_segments(memory_scan(gates[1]), per_head, many, 0, slots, seg_start, seg_row, len(cut[1]), heads)[..., : e + 1]
+    assert (y - z).abs().max() <= 1e-4 * y.abs().max() and (one - many).abs().max() <= 1e-4 * one.abs().max()
+    a_log, dt_bias, skip = torch.log(torch.tensor([0.05, 0.5, 1.5])).cuda(), torch.tensor([-3.0, -2.0, -1.0]).cuda(), torch.ones(heads).cuda()
+    one, many = begin[:, : heads * e * n_padded].contiguous().cuda(), begin[:, : heads * e * n_padded].contiguous().cuda()
+
+    def state_scan(s, sl, rs, rows, states_only=False, decays=None):
+        return recurrent.state_scan(recurrent.MODE_STATE_SPACE, dev, heads * n, 0, 2 * heads * n, dev, i_off, i_off, a_log, dt_bias, skip, s, 0, sl, rs, rows, heads, heads, n, n_padded, e,
+                                    states_only=states_only, decays=decays)
+
+    y = state_scan(one, slots, rows_of, 4)
+    z = recurrent.scan_in_segments(state_scan, e * n_padded, many, 0, slots, seg_start, seg_row, len(cut[1]), heads)
+    assert (y - z).abs().max() <= 1e-4 * y.abs().max() and (one - many).abs().max() <= 1e-4 * one.abs().max()
+
+
+# ------------------------------------------------------------------------------------------ whole models
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", sorted(CONFIGS))
+def test_prefill_against_token_by_token_and_portions(folders, name, dtype):
+    vocab = CONFIGS[name]["vocab"]
+    ids = ids_for(5, 150, vocab)
+    want = plain_logits(folders[name], ids)
+    engine = engine_for(folders[name], dtype, page_size=8 if name == "A" else 16)
+    results = {"whole": run_cut(engine, "w", ids, [len(ids)]), "single": run_cut(engine, "s", ids, [1]),
+               "pairs": run_cut(engine, "p", ids, [2]), "mixed sizes": run_cut(engine, "m", ids, [7, 2, 16, 3, 33, 1, 1, 64])}
+    for how, got in results.items():
+        assert_close(got, want, dtype, how, deep=True)
+        if dtype == "float32":
+            assert np.array_equal(got, results["whole"]), how  # float32: the same bits however the work is cut
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", sorted(CONFIGS))
+def test_unequal_requests_together_over_pages_and_slots_that_are_used_again(folders, name, dtype):
+    """Six requests of unequal length through a cache of 3 slots and too few pages for all: portions of some beside single tokens of
+    others, a request sitting out now and then; as one ends, the next takes its pages and its slot."""
+    from hyperion_b200.engine.batch import StepEntry
+
+    vocab = CONFIGS[name]["vocab"]
+    lengths = [90, 41, 130, 17, 66, 101]
+    requests = {f"r{i}": ids_for(50 + i, n, vocab) for i, n in enumerate(lengths)}
+    want = {rid: plain_logits(folders[name], ids) for rid, ids in requests.items()}
+    engine = engine_for(folders[name], dtype, page_size=16, max_tokens=3 * 144, max_requests=3)
+    waiting, live, sizes, k, step = list(requests), {}, [5, 2, 19, 3, 8, 2, 30, 4], 0, 0
+    got_rows, want_rows, owners, slots = [], [], {}, {}
+    while waiting or live:
+        while waiting and len(live) < 3:
+            live[waiting.pop(0)] = 0
+        entries = []
+        for j, rid in enumerate(list(live)):
+            ids, at = requests[rid], live[rid]
+            if (step + j) % 5 == 4 and len(live) > 1:
+                continue
+            n = 1 if at >= len(ids) - 10 else min(sizes[k % len(sizes)], len(ids) - 10 - at)
+            k += 1
+            entries.append(StepEntry(rid, ids[at:at + n], list(range(n))))
+        logits = engine.step(entries).cpu().numpy()
+        row = 0
+        for index, entry in enumerate(entries):
+            at = live[entry.request]
+            n = len(entry.tokens)
+            got_rows.append(logits[row:row + n])
+            want_rows.append(want[entry.request][at:at + n])
+            row += n
+            live[entry.request] = at + n
+            slots.setdefault(int(engine.runner.last_context.rows.slots[index]), set()).add(entry.request)
+            for group in range(len(engine.cache.paged)):
+                for page in engine.cache.table(group, entry.request):
+                    if page >= 0:
+                        owners.setdefault((group, page), set()).add(entry.request)
+            if at + n == len(requests[entry.request]):
+                engine.finish(entry.request)
+                del live[entry.request]
+        step += 1
+    engine.check()
+    engine.cache.check()
+    assert_close(np.concatenate(got_rows), np.concatenate(want_rows), dtype, deep=True)
+    for group in range(len(engine.cache.paged)):  # in every group some page served more than one request, and so did some slot
+        assert max(len(users) for (g, _), users in owners.items() if g == group) >= 2
+    assert max(len(users) for users in slots.values()) >= 2
+
+
+def _marked(seed: int, length: int, vocab: int, places) -> list[int]:
+    """Random tokens that end in the query token, with the marker at the given positions and nowhere else."""
+    ids = ids_for(seed, length, vocab - 2)  # the last two tokens of the vocabulary are kept for the marked places
+    ids[-1] = vocab - 2
+    for place in places:
+        ids[place] = vocab - 1
+    return ids
+
+
+def _as_a_prompt_and_decoded(engine, ids, want, dtype, what):
+    """The last row of the whole prompt, and of a tail of 30 tokens decoded one by one behind a portion."""
+    from hyperion_b200.engine.batch import StepEntry
+
+    whole = engine.step([StepEntry("w", ids, [len(ids) - 1])]).cpu().numpy()[0]
+    engine.finish("w")
+    assert relative_error(whole, want[-1]) <= TOLERANCE[dtype], (what, "whole")
+    head = len(ids) - 30
+    engine.step([StepEntry("d", ids[:head], [])])
+    for at in range(head, len(ids)):
+        last = engine.step([StepEntry("d", [ids[at]], [0])]).cpu().numpy()[0].copy()
+        assert relative_error(last, want[at]) <= TOLERANCE[dtype], (what, at)
+    engine.finish("d")
+
+
+def _mixer_with_window(entry):
+    return entry["mixer"] if entry["type"] == "attention" else entry["mixer"]["left"]
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["attention", "attention_48", "attention_64", "shared", "stretched", "stretched_48", "stretched_64"])
+def test_keys_just_inside_and_just_outside_the_window(folders, name, dtype):
+    """A window of 24 positions over pages of 8: a marker whose key scores high against the last query stands 23 places back (the last key the
+    window keeps), 24 places back (the first it does not), one place, one page and two pages back, and 22 and 25; the prompts end at and around
+    multiples of a page.  In ``shared`` the window is the borrowing layer's, wider than the one of the layer that owns the keys."""
+    vocab, window = ALONE[name]["vocab"], 24
+    engine = engine_for(folders[name], dtype, page_size=8)
+    for length in (120, 121, 71):
+        for back in (1, 8, 16, window - 2, window - 1, window, window + 1):
+            ids = _marked(700 + length + back, length, vocab, [length - 1 - back])
+            _as_a_prompt_and_decoded(engine, ids, plain_logits(folders[name], ids), dtype, (length, back))
+    engine.check()
+    # the marked key and the window's edge matter: the plain logits move by more than either tolerance when the key is taken away, and
+    # a window that is one place longer or shorter moves them too
+    seen, unseen = _marked(1, 120, vocab, [119 - (window - 1)]), _marked(1, 120, vocab, [119 - window])
+    without = list(seen)
+    without[119 - (window - 1)] = 0
+    base = plain_logits(folders[name], seen)[-1]
+    assert relative_error(plain_logits(folders[name], without)[-1], base) > TOLERANCE["bfloat16"]
+    config, weights = plain.read_model_folder(folders[name])
+    for ids, size in ((seen, window - 1), (unseen, window + 1)):
+        other = json.loads(json.dumps(config))
+        _mixer_with_window(other["layers"][-1])["mask"]["size"] = size
+        assert relative_error(plain.forward(other, weights, ids).numpy()[-1], plain_logits(folders[name], ids)[-1]) > TOLERANCE["bfloat16"]
+
+
+def test_pages_of_a_window_go_back(folders):
+    """A request of 300 tokens through one layer with a window of 24 over pages of 8, in a pool of eight pages."""
+    from hyperion_b200.engine.batch import StepEntry
+
+    for name in ("attention_48", "stretched_64"):
+        ids = ids_for(17, 300, ALONE[name]["vocab"])
+        want = plain_logits(folders[name], ids)
+        for dtype in ("float32", "bfloat16"):
+            engine = engine_for(folders[name], dtype, page_size=8, max_tokens=64)
+            got = []
+            for at in range(0, 300, 20):
+                got.append(engine.step([StepEntry("r", ids[at:at + 20], list(range(20)))]).cpu().numpy().copy())
+                assert sum(page >= 0 for page in engine.cache.table(0, "r")) <= 4
+            engine.check()
+            assert_close(np.concatenate(got), want, dtype)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["open", "open_64"])
+def test_a_key_far_away_among_hundreds(folders, name, dtype):
+    """No window: the marker stands 1, 7, 8, 9, 64, 300 and 690 places behind the last query among 700 tokens (in bfloat16 the prompt's recurrence runs in segments), as a
+    whole prompt and with the tail decoded; queries have a temperature that steps at every 100 positions."""
+    vocab = ALONE[name]["vocab"]
+    engine = engine_for(folders[name], dtype, page_size=8, max_tokens=1536)
+    for back in (1, 7, 8, 9, 64, 300, 690):
+        ids = _marked(800 + back, 700, vocab, [699 - back])
+        _as_a_prompt_and_decoded(engine, ids, plain_logits(folders[name], ids), dtype, back)
+    engine.check()
+    without = list(ids)
+    without[699 - 690] = 0
+    assert relative_error(plain_logits(folders[name], without)[-1], plain_logits(folders[name], ids)[-1]) > TOLERANCE["bfloat16"]
+
+
+@pytest.mark.parametrize("name", ["open", "states_wide", "memory_wide", "stretched_64"])
+def test_states_over_long_texts(folders, name):
+    """1,300 tokens: one prompt (in bfloat16 the scans run in segments), portions whose sizes straddle the segments' length, and a decoded tail."""
+    ids = ids_for(21, 1300, ALONE[name]["vocab"])
+    want = plain_logits(folders[name], ids)
+    for dtype in ("float32", "bfloat16"):
+        engine = engine_for(folders[name], dtype, max_tokens=2048)
+        whole = run_cut(engine, "w", ids, [1300])
+        assert_close(whole, want, dtype, "whole", deep=True)
+        cut = run_cut(engine, "p", ids, [513, 600, 100] + [1] * 87)
+        assert_close(cut, want, dtype, "portions", deep=True)
+        if dtype == "float32":
+            assert np.array_equal(whole, cut)
+
+
+def test_every_tensor_and_option_matters(folders):
+    """What the runs above are held to moves by many tolerances when a bias, a gate, a state, a cap, a temperature, the stretching or one residual stream is left out."""
+    ids = ids_for(3, 75, 61)
+
+    def moves(name, change):
+        config, weights = plain.read_model_folder(folders[name])
+        change(config, weights)
+        assert relative_error(plain.forward(config, weights, ids).numpy(), plain_logits(folders[name], ids)) > 50 * TOLERANCE["float32"], (name, change)
+
+    def tensor(key, value):
+        return lambda config, weights: weights.__setitem__(key, torch.full_like(weights[key], value))
+
+    def dropped(*path):
+        def change(config, weights):
+            at = config["layers"][0]["mixer"]
+            for step in path[:-1]:
+                at = at[step]
+            del at[path[-1]]
+        return change
+
+    for key in ("l0.mix.q.b", "l0.mix.k.b", "l0.mix.v.b", "l0.mix.g", "l0.hc1.out", "l0.hc1.mix"):
+        moves("attention", tensor(key, 0.0))
+    moves("attention", dropped("rot"))
+    for key in ("l0.hc2.in", "l1.hc1.in", "l1.hc2.in", "l0.hc2.out", "l1.hc1.out"):
+        moves("five_streams", tensor(key, 1.0))
+    for key in ("l0.hc1.mix", "l0.hc2.mix", "l1.hc1.mix"):  # indexed from, to
+        moves("five_streams", lambda c, w: w.__setitem__(key, w[key].T.contiguous()))
+    for key in ("l0.mix.right.conv.b", "l0.mix.right.D", "l0.mix.right.A_log", "l0.mix.right.dt_bias", "l0.mix.left.out", "l0.mix.right.out"):
+        moves("stretched", tensor(key, 3.0))
+    moves("stretched", dropped("left", "softcap"))
+    moves("stretched", dropped("left", "rot", "scaling"))
+    for key in ("l0.mix.right.f.b",  # (an input gate's bias scales a head's whole state, which the head's norm takes out again)
+                "l0.mix.right.g", "l0.mix.right.i", "l0.mix.right.f", "l0.mix.right.norm"):
+        moves("open", tensor(key, 0.0))
+    moves("open", dropped("left", "softcap"))
+    moves("open", lambda c, w: c["layers"][0]["mixer"]["left"]["q_temp"].__setitem__("every", 10))
+    moves("open", lambda c, w: c["layers"][0]["mixer"]["right"].__setitem__("gate_cap", 1.0))
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", sorted(CONFIGS))
+def test_first_tokens_and_long_decoding(folders, name, dtype):
+    from hyperion_b200.engine.batch import StepEntry
+
+    vocab = CONFIGS[name]["vocab"]
+    ids = ids_for(8, 400, vocab)
+    want = plain_logits(folders[name], ids)
+    engine = engine_for(folders[name], dtype, page_size=32, max_tokens=512)
+    rows = []
+    for token in ids:  # position 0 alone, then every other one: a one-token prompt and 399 decoded tokens
+        rows.append(engine.step([StepEntry("r", [token], [0])]).cpu().numpy()[0].copy())
+    engine.finish("r")
+    pair = engine.step([StepEntry("pair", ids[:2], [0, 1])]).cpu().numpy().copy()
+    engine.finish("pair")
+    engine.check()
+    single = np.stack(rows)
+    assert_close(single, want, dtype, deep=True)
+    assert_close(single[:8], want[:8], dtype, "the first tokens")
+    assert_close(pair, want[:2], dtype)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["attention_64", "attention_128", "stretched_64", "open_64"])
+def test_options_in_the_tensor_core_kernels(folders, name, dtype):
+    """450 tokens: as one prompt (tiles whose queries' windows begin in the middle of a key tile), in two portions and a tail decoded token by token (the split-key
+    kernel), and three requests of unequal progress side by side."""
+    from hyperion_b200.engine.batch import StepEntry
+
+    vocab = ALONE[name]["vocab"]
+    ids = ids_for(77, 450, vocab)
+    want = plain_logits(folders[name], ids)
+    engine = engine_for(folders[name], dtype, max_tokens=2048)
+    assert_close(run_cut(engine, "w", ids, [len(ids)]), want, dtype, "whole")
+    got = [engine.step([StepEntry("d", ids[:300], list(range(300)))]).cpu().numpy().copy()]
+    got.append(engine.step([StepEntry("d", ids[300:420], list(range(120)))]).cpu().numpy().copy())
+    for at in range(420, 450):
+        got.append(engine.step([StepEntry("d", [ids[at]], [0])]).cpu().numpy().copy())
+    engine.finish("d")
+    assert_close(np.concatenate(got), want, dtype, "two portions and a decoded tail")
+    engine.step([StepEntry("a", ids[:199], []), StepEntry("b", ids[:30], [])])
+    got = engine.step([StepEntry("a", [ids[199]], [0]), StepEntry("b", ids[30:330], list(range(300))), StepEntry("c", ids[:2], [0, 1])]).cpu().numpy()
+    engine.check()
+    assert_close(got, np.concatenate([want[199:200], want[30:330], want[:2]]), dtype, "side by side")
+
+
+@pytest.mark.parametrize("name", sorted(CONFIGS))
+def test_greedy_generation_through_the_scheduler(folders, name):
+    from hyperion_b200.sampling import SamplingParams
+
+    vocab = CONFIGS[name]["vocab"]
+    prompts = [ids_for(300 + i, n, vocab) for i, n in enumerate([5, 37, 1, 80, 23])]
+    config, weights = plain.read_model_folder(folders[name])
+
+    def greedy(prompt, count):
+        ids = list(prompt)
+        for _ in range(count):
+            ids.append(int(plain.forward(config, weights, ids)[-1].argmax()))
+        return ids[len(prompt):]
+
+    want = [greedy(prompt, 6) for prompt in prompts]
+    engine = engine_for(folders[name], "float32", max_tokens=3 * 128, max_requests=3)
+    got = engine.generate(prompts, SamplingParams(temperature=0.0, max_tokens=6, ignore_eos=True), max_batch_tokens=48, prefill_chunk_busy=16)
+    assert got == want
+    engine = engine_for(folders[name], "bfloat16", max_tokens=3 * 128, max_requests=3)
+    got = engine.generate(prompts, SamplingParams(temperature=0.0, max_tokens=6, ignore_eos=True), max_batch_tokens=48, prefill_chunk_busy=16)
+    assert all(len(tokens) == 6 for tokens in got)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_replay_through_the_command(folders, dtype, tmp_path):
+    """bin/trace_run on a model of this design: two requests side by side, one ends, a third takes its place."""
+    name, vocab = "A", CONFIGS["A"]["vocab"]
+    a, b, c = ids_for(1, 70, vocab), ids_for(2, 33, vocab), ids_for(3, 50, vocab)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:40], "want": [39]}, {"id": "b", "tokens": b[:31], "want": [0, 30]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": a[40:42], "want": [0, 1]}, {"id": "b", "tokens": b[31:32], "want": [0]}], "end": []},
+             {"step": 2, "entries": [{"id": "b", "tokens": b[32:], "want": [0]}], "end": ["b"]},
+             {"step": 3, "entries": [{"id": "c", "tokens": c, "want": [49]}, {"id": "a", "tokens": a[42:], "want": [27]}], "end": ["a", "c"]}]
+    text = "".join(json.dumps(s) + "\n" for s in steps)
+    done = subprocess.run([sys.executable, str(ROOT / "bin" / "trace_run"), "--model", str(folders[name]), "--dtype", dtype, "--out", str(tmp_path),
+                           "--max-tokens", "192"], input=text, capture_output=True, text=True, timeout=900)
+    assert done.returncode == 0, done.stderr[-3000:]
+    assert [line for line in done.stdout.splitlines() if line.startswith("done ")] == [f"done {i}" for i in range(4)]
+    ref = {"a": plain_logits(folders[name], a), "b": plain_logits(folders[name], b), "c": plain_logits(folders[name], c)}
+    read = lambda step: np.fromfile(tmp_path / f"{step}.f32", dtype="<f4").reshape(-1, vocab)
+    expected = {0: [ref["a"][39], ref["b"][0], ref["b"][30]], 1: [ref["a"][40], ref["a"][41], ref["b"][31]], 2: [ref["b"][32]],
+                3: [ref["c"][49], ref["a"][69]]}
+    for step, rows in expected.items():
+        assert_close(read(step), np.stack(rows), dtype, step)
+
+
+def test_the_command_line_writes_a_random_model_and_generates_with_it(tmp_path):
+    """``python -m hyperion_b200 random`` from a config.json of this design, then ``generate`` on the folder it wrote:
+    the tokens are the plain implementation's greedy ones."""
+    config = tmp_path / "config.json"
+    config.write_text(json.dumps(CONFIGS["A"]))
+    folder = tmp_path / "model"
+    run = lambda *args: subprocess.run([sys.executable, "-m", "hyperion_b200", *args], capture_output=True, text=True, timeout=900, cwd=ROOT)
+    done = run("random", "--config", str(config), "--out", str(folder), "--seed", "5", "--std", "0.3")
+    assert done.returncode == 0, done.stderr[-2000:]
+    prompt = ids_for(71, 19, CONFIGS["A"]["vocab"])
+    done = run("generate", "-m", str(folder), "--dtype", "float32", "--prompt-ids", ",".join(map(str, prompt)), "--max-tokens", "5", "--temperature", "0",
+               "--ignore-eos", "--max-batch", "2")
+    assert done.returncode == 0, done.stderr[-2000:]
+    got = json.loads(done.stdout.strip().splitlines()[-1])
+    plain_config, weights = plain.read_model_folder(folder)
+    ids = list(prompt)
+    for _ in range(5):
+        ids.append(int(plain.forward(plain_config, weights, ids)[-1].argmax()))
+    assert got["tokens"] == ids[len(prompt):] and got["finish_reason"] == "length"
+
+
+# ------------------------------------------------------------------------------------------ configurations drawn at random
+def _random_document(seed: int) -> dict:
+    """A model whose every size, option and constant is drawn: streams, widths, heads and groupings, head sizes that the tensor-core kernels take and
+    others, windows, rotations, caps, temperatures, recurrences, layers without a feed-forward, layers that read an earlier layer's keys, in any order."""
+    import random
+
+    r = random.Random(seed)
+    layers: list = []
+    width = r.choice([32, 40, 54, 64, 80, 128])
+
+    def rotated(dim):
+        return (2 * r.randint(1, dim // 2), r.choice([50.0, 1e4, 1e6])) if dim > 1 and r.random() < 0.8 else None
+
+    for _ in range(r.randint(2, 6)):
+        ff = r.choice([8, 20, 36, 100]) if r.random() < 0.75 else None
+        kv = r.choice([1, 2, 3])
+        count, window, dim = kv * r.choice([1, 2, 3]), r.choice([None, r.randint(1, 70), r.randint(1, 70)]), r.choice([4, 8, 12, 16, 24, 32, 48, 64])
+        vdim = r.choice([dim, dim, 12, 20])
+        scale = r.choice([0.1, 0.3, dim ** -0.5])
+        lenders = [i for i, entry in enumerate(layers) if entry["type"] == "attention" and "kv_from" not in entry["mixer"]]
+        kind = r.choice(["attention", "shared", "states", "states", "memory", "memory"])
+        if kind == "shared" and lenders:
+            source = r.choice(lenders)
+            m = layers[source]["mixer"]
+            lent = {**m, "heads": m["kv_heads"] * r.choice([1, 2]), "scale": scale, "kv_from": source}
+            lent.pop("mask", None)
+            if window is not None:
+                lent["mask"] = {"size": window}
+            layers.append(attention(lent, ff))
+        elif kind in ("attention", "shared"):
+            layers.append(attention(heads(count, kv, dim, vdim, scale, window=window, rot=rotated(dim)), ff))
+        elif kind == "states":
+            rot = rotated(dim)
+            scaling = (r.choice([1.5, 4.0, 32.0]), float(r.choice([16, 64, 512])), r.choice([4.0, 32.0]), 1.0) if rot is not None and r.random() < 0.8 else None
+            groups = r.choice([1, 2])
+            inner_heads, e = groups * r.choice([1, 2, 3]), r.choice([4, 7, 16, 33])
+            parts = r.choice([n for n in (1, 2, 3, inner_heads) if inner_heads * e % n == 0])
+            layers.append(beside_states(heads(count, kv, dim, vdim, scale, window=window, cap=r.choice([None, 3.0, 20.0]), rot=rot, scaling=scaling),
+                                        state_space(inner_heads, e, r.choice([3, 8, 16, 70]), groups, parts, r.randint(1, 5)), ff))
+        else:
+            layers.append(beside_memory(heads(count, kv, dim, vdim, scale, cap=r.choice([None, 3.0, 20.0]), temp=r.choice([None, (0.5, 7), (-0.1, 30)])),
+                                        memory(r.randint(1, 4), r.choice([3, 8, 24, 40]), r.choice([4, 9, 32]), r.choice([1.0, 6.0, 15.0])), ff))
+    return document(width, r.randint(40, 300), r.choice([1, 2, 3, 4]), layers, eps=r.choice([1e-6, 1e-5, 1e-3]))
+
+
+@pytest.mark.parametrize("seed", range(10))
+def test_configurations_drawn_at_random(seed, tmp_path):
+    """Ten models drawn at random, in float32 against the plain implementation: a whole prompt, the same in portions, and two requests of
+    unequal progress side by side; in bfloat16 the middle row of the whole prompt and of the portions."""
+    from hyperion_b200.engine.batch import StepEntry
+    from hyperion_b200.weights import write_file
+
+    doc = _random_document(seed)
+    folder = tmp_path / "model"
+    folder.mkdir()
+    (folder / "config.json").write_text(json.dumps(doc))
+    write_file(folder / "model.safetensors", make_weights(doc, 100 + seed, gain=1.2))
+    ids, other = ids_for(seed, 90, doc["vocab"]), ids_for(seed + 50, 37, doc["vocab"])
+    want, want_other = plain_logits(folder, ids), plain_logits(folder, other)
+    engine = engine_for(folder, "float32", page_size=8, max_tokens=512)
+    assert_close(run_cut(engine, "w", ids, [len(ids)]), want, "float32", ("whole", doc))
+    assert_close(run_cut(engine, "p", ids, [3, 1, 2, 17]), want, "float32", ("portions", doc))
+    engine.step([StepEntry("a", ids[:61], []), StepEntry("b", other[:5], [])])
+    got = engine.step([StepEntry("a", [ids[61]], [0]), StepEntry("b", other[5:], list(range(32)))]).cpu().numpy()
+    engine.check()
+    assert_close(got, np.concatenate([want[61:62], want_other[5:]]), "float32", ("side by side", doc))
+    engine = engine_for(folder, "bfloat16", page_size=8, max_tokens=512)
+    for sizes in ([len(ids)], [3, 1, 2, 17]):
+        errors = row_errors(run_cut(engine, "w", ids, sizes), want)
+        assert np.median(errors) <= TOLERANCE["bfloat16"], (float(np.median(errors)), sizes, doc)
+
+
+def test_sizes_of_one(tmp_path):
+    """Every size that can be one is one (streams, heads, key and value sizes, a window of one position, a state of one entry, one tap, an inner size of one), and a
+    model of many heads and streams: whole, in portions and token by token, in both precisions."""
+    from hyperion_b200.weights import write_file
+
+    docs = {
+        "ones": document(8, 17, 1, [attention(heads(1, 1, 2, 1, 1.0, window=1, rot=(2, 10.0)), 1), beside_states(heads(1, 1, 1, 1, 1.0, window=1), state_space(1, 1, 1, 1, 1, 1), 4),
+                                    beside_memory(heads(1, 1, 1, 1, 0.5, temp=(1.0, 1)), memory(1, 1, 1, 1.0)), attention(heads(1, 1, 2, 1, 0.5, window=2, rot=(2, 10.0), kv_from=0))], eps=1e-4),
+        "many": document(24, 50, 6, [beside_states(heads(16, 1, 8, 16, 0.3, window=33, cap=5.0, rot=(2, 100.0)), state_space(24, 3, 5, 12, 8, 6), 8),
+                                     beside_memory(heads(12, 1, 16, 16, 0.25), memory(20, 4, 5, 3.0), 8)]),
+    }
+    for name, doc in docs.items():
+        folder = tmp_path / name
+        folder.mkdir()
+        (folder / "config.json").write_text(json.dumps(doc))
+        write_file(folder / "model.safetensors", make_weights(doc, 7, gain=1.2))
+        ids = ids_for(1, 90, doc["vocab"])
+        want = plain_logits(folder, ids)
+        for dtype in ("float32", "bfloat16"):
+            engine = engine_for(folder, dtype, page_size=8, max_tokens=512)
+            for sizes in ([len(ids)], [3, 1, 2, 17], [1]):
+                assert_close(run_cut(engine, "w", ids, sizes), want, dtype, (name, sizes), deep=True)
