@@ -1192,6 +1192,222 @@ def zurevik_workload(args) -> int:
     return 0
 
 
+BIROPEL_SIZES = {
+    # width; heads, kv heads and head size of every attention; window; matrix memory (heads, key size, value size); state space (heads, value size, state,
+    # groups); feed-forward; residual streams.  Eight layers A P M P A' M P M (A = windowed attention with a gate, A' = the same over the keys and values of the A before it,
+    # P = windowed attention beside the state-space mixer, M = attention over every key beside the matrix memory), every layer with a feed-forward, 32,000 tokens
+    "2k": {"width": 2048, "heads": (16, 4, 128), "window": 1024, "memory": (16, 128, 128), "states": (16, 128, 128, 1), "ff": 8192, "streams": 4},
+    "4k": {"width": 4096, "heads": (32, 8, 128), "window": 2048, "memory": (32, 128, 128), "states": (32, 128, 128, 1), "ff": 14336, "streams": 4},
+}
+
+
+def biropel_document(size: dict, vocab: int = 32000) -> dict:
+    heads, kv_heads, dim = size["heads"]
+    base = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+    windowed = {**base, "mask": {"size": size["window"]}}
+    mlp = {"kind": "dense", "ff": size["ff"]}
+    scaling = {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}
+    m_heads, m_dim, m_vdim = size["memory"]
+    s_heads, s_vdim, state, groups = size["states"]
+
+    def a(kv_from=None):
+        mixer = {**windowed, "rot": {"dims": dim // 2, "base": 1e6}}
+        return {"type": "attention", "mlp": mlp, "mixer": {**mixer, "kv_from": kv_from} if kv_from is not None else mixer}
+
+    p = {"type": "parallel", "mlp": mlp, "mixer": {"left": {**windowed, "softcap": 30.0, "rot": {"dims": dim, "base": 1e6, "scaling": scaling}},
+                                                   "right": {"heads": s_heads, "vdim": s_vdim, "state": state, "groups": groups, "norm_groups": groups, "conv": 4}}}
+    m = {"type": "parallel_2", "mlp": mlp, "mixer": {"left": {**base, "softcap": 50.0, "q_temp": {"coef": 0.1, "every": 1024}},
+                                                     "right": {"heads": m_heads, "dim": m_dim, "vdim": m_vdim, "gate_cap": 15.0}}}
+    return {"architecture": "Biropel", "vocab": vocab, "width": size["width"], "streams": size["streams"], "norm": {"eps": 1e-6}, "layers": [a(), p, m, p, a(0), m, p, m]}
+
+
+def biropel_like_document(size: dict, vocab: int = 32000) -> dict:
+    """The closest model of the package at equal size: Mirovik with attention beside a recurrence and a dense feed-forward in all eight layers."""
+    heads, kv_heads, dim = size["heads"]
+    r_heads, r_dim, r_vdim = size["memory"]
+    mixer = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "bias_max": 256, "buckets": 32},
+             "right": {"heads": r_heads, "dim": r_dim, "vdim": r_vdim, "decay": [1.0 - 2.0 ** (-5 - 5 * h / max(1, r_heads - 1)) for h in range(r_heads)],
+                       "rot": {"dims": r_dim // 2, "base": 1e6}}, "left_scale": 1.0, "right_scale": 1.0}
+    layer = {"type": "parallel", "mixer": mixer, "mlp": {"kind": "dense", "ff": size["ff"]}}
+    return {"architecture": "Mirovik", "vocab": vocab, "width": size["width"], "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "layers": [layer] * 8}
+
+
+def biropel_kernels(size: dict, measured: dict) -> dict:
+    """The design's own kernels alone at this size, a prompt of 2,048 tokens in one row and 8 rows of one decoded token behind 2,048: time, the bytes
+    each must move against the measured copy bandwidth, for attention the bfloat16 operations against the measured product rate, for the scans the float32
+    operations; beside each the like kernel of the closest model (Mirovik)."""
+    import types
+
+    import torch
+
+    from hyperion_b200 import ops
+    from hyperion_b200.ops import attention as fast, recurrent
+
+    dev = torch.device("cuda")
+    hbm, peak = measured["hbm_gbs"] * 1e9, measured["bf16_tflops"] * 1e12
+    out: dict = {}
+    width, page, streams = size["width"], 16, size["streams"]
+
+    def report(name, ms, bytes_moved, bf16_flops=None, fp32_flops=None):
+        entry = {"us": round(ms * 1e3, 2), "bytes": int(bytes_moved), "of_measured_bandwidth": round(bytes_moved / (ms / 1e3) / hbm, 3)}
+        if bf16_flops is not None:
+            entry["of_measured_bf16_rate"] = round(bf16_flops / (ms / 1e3) / peak, 3)
+        if fp32_flops is not None:
+            entry["fp32_tflops"] = round(fp32_flops / (ms / 1e3) / 1e12, 2)
+        out[name] = entry
+
+    heads, kv_heads, dim = size["heads"]
+    window = size["window"]
+    for shape, counts, before in (("prefill_2048", [PROMPT], 0), ("decode_8", [1] * 8, PROMPT)):
+        tokens, rows = sum(counts), len(counts)
+        token_row = torch.tensor([r for r, c in enumerate(counts) for _ in range(c)], dtype=torch.int32, device=dev)
+        row_start = torch.tensor([sum(counts[:r]) for r in range(rows + 1)], dtype=torch.int32, device=dev)
+        slots = torch.arange(rows, dtype=torch.int32, device=dev)
+        positions = torch.cat([torch.arange(c, dtype=torch.int32) + before for c in counts]).to(dev)
+        context = before + max(counts)
+        per_row = -(-context // page)
+        table = torch.arange(rows * per_row, dtype=torch.int32, device=dev).view(rows, per_row)
+        # a boundary between two sublayers: one result, and two normed ones; beside it the one-stream boundary of the closest model
+        h = torch.randn(tokens, streams, width, device=dev)
+        a, b = (torch.randn(tokens, width, device=dev).to(torch.bfloat16) for _ in range(2))
+        weight, mix = torch.ones(width, device=dev), torch.eye(streams, device=dev)
+        share, read = torch.ones(streams, device=dev) * 0.1, torch.ones(streams, device=dev) / streams
+        one = lambda: ops.hyper_connect(h, streams, read, weight, 1e-6, torch.bfloat16, results=(a,), mix=mix, share=share)
+        two = lambda: ops.hyper_connect(h, streams, read, weight, 1e-6, torch.bfloat16, results=(a, b), norms=(weight, weight), result_eps=1e-6, result_scale=0.5, mix=mix, share=share)
+        report(f"hyper_connect/{shape}", timed(one), tokens * width * (8 * streams + 2 + 2))
+        report(f"hyper_connect_two_normed/{shape}", timed(two), tokens * width * (8 * streams + 4 + 2))
+        g = torch.randn(tokens, width, device=dev)
+        report(f"mirovik.norm_add_norm/{shape}", timed(lambda: ops.norm_add_norm(g, a, weight, 1e-6, None, weight, 1e-6, torch.bfloat16)), tokens * width * (4 + 4 + 2 + 2))
+        # heads to their buffers and pages: turned, with biases; unit norm and temperature
+        cols = (heads + 2 * kv_heads) * dim
+        proj = torch.randn(tokens, cols + heads * dim, device=dev)
+        q = torch.empty(tokens, heads * dim, dtype=torch.bfloat16, device=dev)
+        cache = (torch.randn(rows * per_row, 2, kv_heads, page, dim, device=dev) * 0.5).to(torch.bfloat16)
+        bias, inv_freq = torch.randn(cols, device=dev), torch.rand(dim // 2, device=dev)
+        k_off, v_off = heads * dim, (heads + kv_heads) * dim
+        where = {"cache": cache, "block_table": table, "token_row": token_row, "page_size": page}
+        report(f"attention.heads_turned/{shape}", timed(lambda: ops.heads_store(proj, 0, k_off, v_off, heads, kv_heads, dim, dim, positions, q_out=q, bias=bias, inv_freq=inv_freq,
+                                                                             rot_dims=dim, rot_half=True, amplitude=1.1, **where)), tokens * cols * 6)
+        report(f"attention.heads_unit_normed/{shape}", timed(lambda: ops.heads_store(proj, 0, k_off, v_off, heads, kv_heads, dim, dim, positions, q_out=q, unit_norm=True, eps=1e-6,
+                                                                                  temperature=(0.1, 1024), **where)), tokens * cols * 6)
+        norms = torch.ones(heads * dim, device=dev)
+        report(f"mirovik.heads_prepare/{shape}", timed(lambda: ops.heads_prepare_wide(proj, 0, k_off, v_off, heads, kv_heads, dim, dim, positions, q_out=q, q_norm=norms,
+                                                                                   k_norm=norms[: kv_heads * dim].contiguous(), norm_whole=True, eps=1e-6, **where)), tokens * cols * 6)
+        # attention: windowed and over every key, capped; the biased attention of the closest model; the gate
+        fake_rows = [types.SimpleNamespace(count=c, position=before) for c in counts]
+        seen = lambda w: sum(min(p + 1, w) if w else p + 1 for p in positions.tolist())
+        attn = torch.empty(tokens, heads * dim, dtype=torch.bfloat16, device=dev)
+        tile = fast.tile_rows(dim, page)
+        tiles, items = fast.plan(fake_rows, fast.tile_tokens(heads, kv_heads, tile))
+        work = torch.tensor(tiles if len(tiles) else items, dtype=torch.int32, device=dev)
+        table_bias = torch.randn(heads, 257, device=dev)
+        for label, w, extras in (("windowed_attention", window, {}), ("windowed_capped_attention", window, {"softcap": 30.0}), ("capped_attention", 0, {"softcap": 50.0}),
+                                 ("mirovik.biased_attention", 0, {"bias": table_bias})):
+            splits = fast.choose_splits(max(1, len(items)), heads, kv_heads, min(context, w + fast.KEY_TILE) if w else context)
+            if len(tiles):
+                run = lambda: fast.attention_tiles(q, heads, cache, table, token_row, positions, work, len(tiles) // 3, dim ** -0.5, w, attn, tile_size=tile, **extras)
+            else:
+                run = lambda: fast.attention_tokens(q, heads, cache, table, token_row, positions, work, len(items), splits, dim ** -0.5, w, attn, **extras)
+            report(f"{label}/{shape}", timed(run), rows * (min(context, w) if w else context) * 2 * kv_heads * dim * 2 + tokens * heads * dim * 4, bf16_flops=4.0 * seen(w) * heads * dim)
+        report(f"attention.gate/{shape}", timed(lambda: ops.sigmoid_gate_(attn, proj, cols)), tokens * heads * dim * (2 + 2 + 4))
+        # the matrix memory: gates, scan (one pass, and as the engine walks a long row), what follows it; retention of the closest model
+        m_heads, n, e = size["memory"]
+        m_cols = 2 * m_heads * n + 2 * m_heads * e
+        m_proj = torch.randn(tokens, m_cols + 2 * m_heads, device=dev) * 0.5
+        n_padded, per_head = n, (e + 1) * n
+        m_state = torch.zeros(rows, m_heads * per_head + m_heads, device=dev)
+        b_i, b_f = torch.zeros(m_heads, device=dev), torch.full((m_heads,), 4.0, device=dev)
+        make = lambda: recurrent.matrix_memory_gates(m_proj, m_cols, m_cols + m_heads, b_i, b_f, 15.0, m_state, m_heads * per_head, slots, row_start, rows, m_heads)
+        report(f"memory.gates/{shape}", timed(make), tokens * m_heads * 20)
+        gates = make()
+
+        def memory_scan(state, own, starts, count, states_only=False, decays=None):
+            return recurrent.matrix_memory_scan(m_proj, m_heads * n, 0, 2 * m_heads * n, gates, state, 0, own, starts, count, m_heads, n, n_padded, e, n ** -0.5,
+                                                states_only=states_only, decays=decays)
+
+        moved = 4 * (tokens * (2 * m_heads * n + 2 * m_heads * e) + 2 * rows * m_heads * e * n)
+        report(f"memory.scan/{shape}", timed(lambda: memory_scan(m_state, slots, row_start, rows)), moved, fp32_flops=4.0 * tokens * m_heads * n * e)
+        cut = recurrent.plan_segments(counts)
+        if cut is not None:
+            seg_start, seg_row = torch.tensor(cut[0], dtype=torch.int32, device=dev), torch.tensor(cut[1], dtype=torch.int32, device=dev)
+            report(f"memory.scan_in_segments/{shape}", timed(lambda: recurrent.scan_in_segments(memory_scan, per_head, m_state, 0, slots, seg_start, seg_row, len(cut[1]), m_heads)), moved,
+                   fp32_flops=7.0 * tokens * m_heads * n * e)
+        y = memory_scan(m_state, slots, row_start, rows)
+        gated = torch.empty(tokens, m_heads * e, dtype=torch.bfloat16, device=dev)
+        m_norm = torch.ones(m_heads * e, device=dev)
+        report(f"memory.norm/{shape}", timed(lambda: recurrent.matrix_memory_norm(y, gates, m_proj, 2 * m_heads * n + m_heads * e, m_norm, e, 1e-6, gated)), tokens * m_heads * e * 10)
+        decay, r_state = torch.full((m_heads,), 0.99, device=dev), torch.zeros(rows, m_heads * e * n, device=dev)
+        retention = lambda: recurrent.state_scan(recurrent.MODE_RETENTION, m_proj, m_heads * n, 0, 2 * m_heads * n, m_proj, 0, 0, decay, decay, None, r_state, 0, slots, row_start, rows,
+                                                 m_heads, m_heads, n, n, e)
+        report(f"mirovik.retention_scan/{shape}", timed(retention), moved, fp32_flops=4.0 * tokens * m_heads * n * e)
+        if cut is not None:
+            report(f"mirovik.retention_in_segments/{shape}", timed(lambda: recurrent.retention_in_segments(m_proj, m_heads * n, 0, 2 * m_heads * n, decay, r_state, slots, seg_start,
+                                                                                                          seg_row, len(cut[1]), m_heads, n, n, e)), moved, fp32_flops=8.0 * tokens * m_heads * n * e)
+        o = retention()
+        report(f"mirovik.gated_norm/{shape}", timed(lambda: recurrent.gated_group_norm(o, m_proj, 2 * m_heads * n + m_heads * e, None, e, False, 1e-6, torch.bfloat16)), tokens * m_heads * e * 10)
+        # the state-space mixer: convolution, scan, gated norm over groups of the inner width
+        s_heads, s_e, state, groups = size["states"]
+        inner, bn = s_heads * s_e, groups * state
+        channels = inner + 2 * bn
+        s_proj = torch.randn(tokens, inner + channels + s_heads, device=dev) * 0.5
+        w_conv, b_conv = torch.randn(channels, 4, device=dev) * 0.3, torch.zeros(channels, device=dev)
+        c_state = torch.zeros(rows, 3 * channels, device=dev)
+        report(f"states.conv/{shape}", timed(lambda: recurrent.causal_conv_silu(s_proj, inner, w_conv, b_conv, c_state, 0, slots, token_row, row_start)), tokens * channels * 8)
+        report(f"states.conv_keep/{shape}", timed(lambda: recurrent.conv_state_update(s_proj, inner, channels, 4, c_state, 0, slots, row_start, rows)), rows * channels * 3 * 8)
+        conv = recurrent.causal_conv_silu(s_proj, inner, w_conv, b_conv, c_state, 0, slots, token_row, row_start)
+        zeros, ones = torch.zeros(s_heads, device=dev), torch.ones(s_heads, device=dev)
+        s_state = torch.zeros(rows, s_heads * s_e * state, device=dev)
+
+        def state_scan(st, own, starts, count, states_only=False, decays=None):
+            return recurrent.state_scan(recurrent.MODE_STATE_SPACE, conv, inner, inner + bn, 0, s_proj, inner + channels, inner + channels, zeros, zeros, ones, st, 0, own, starts, count,
+                                        s_heads, groups, state, state, s_e, states_only=states_only, decays=decays)
+
+        moved = 4 * (tokens * (2 * bn + 2 * inner) + 2 * rows * inner * state)
+        report(f"states.scan/{shape}", timed(lambda: state_scan(s_state, slots, row_start, rows)), moved, fp32_flops=4.0 * tokens * inner * state)
+        if cut is not None:
+            report(f"states.scan_in_segments/{shape}", timed(lambda: recurrent.scan_in_segments(state_scan, s_e * state, s_state, 0, slots, seg_start, seg_row, len(cut[1]), s_heads)), moved,
+                   fp32_flops=7.0 * tokens * inner * state)
+        y = state_scan(s_state, slots, row_start, rows)
+        s_norm = torch.ones(inner, device=dev)
+        report(f"states.gated_norm/{shape}", timed(lambda: recurrent.gated_group_norm(y, s_proj, 0, s_norm, inner // groups, True, 1e-6, torch.bfloat16)), tokens * inner * 10)
+        # the feed-forward's activation
+        act = torch.randn(tokens, size["ff"], device=dev).to(torch.bfloat16)
+        report(f"relu_squared/{shape}", timed(lambda: ops.relu_squared(act)), act.numel() * 4)
+        report(f"mirovik.gelu_tanh/{shape}", timed(lambda: ops.gelu_tanh(act)), act.numel() * 4)
+    return out
+
+
+def biropel_workload(args) -> int:
+    """Prefill (one prompt of 2,048 tokens in one step) and decode (batch 8 from a context of 2,048) of the Biropel design at two sizes that
+    resemble real layers, beside the closest model of the package, Mirovik with attention beside retention and a dense feed-forward in every layer, at equal width, heads,
+    recurrence, feed-forward and number of layers; random weights."""
+    import torch
+
+    from hyperion_b200.api import Engine
+    from hyperion_b200.config import BiropelConfig, MirovikConfig
+
+    measured, kind = peaks()
+    for name, size in BIROPEL_SIZES.items():
+        if args.size and name != args.size:
+            continue
+        arms = {"biropel": ("Biropel", BiropelConfig.from_dict(biropel_document(size))), "mirovik": ("Mirovik", MirovikConfig.from_dict(biropel_like_document(size)))}
+        line = {"workload": "biropel", "size": name, "dtype": "bf16", "data": "synthetic: random weights and token ids",
+                "layers": "A P M P A' M P M beside eight layers of attention beside retention, all with a dense feed-forward", "peaks": kind}
+        for arm, (architecture, config) in arms.items():
+            engine = Engine.from_random(architecture, config, seed=0, dtype="bfloat16", page_size=16, max_tokens=8 * (PROMPT + 256), max_requests=8)
+            prefill = time_prefill(engine)
+            decode = time_decode(engine, 8, 16, max(3, args.warmup), decode_tokens=max(3, args.warmup) + 160)
+            line[arm] = {"prefill_ms": round(prefill["ms"], 3), "prefill_tokens_per_s": round(PROMPT / prefill["ms"] * 1e3),
+                         "decode_ms_per_step": round(decode["ms_per_step"], 4), "decode_tokens_per_s": round(decode["tok_s"], 1),
+                         "decode_launches_per_step": round(decode["launches"] / decode["steps"], 1)}
+            del engine
+            torch.cuda.empty_cache()
+        if not args.skip_points:
+            line["kernels"] = biropel_kernels(size, measured)
+        print(json.dumps(line), flush=True)
+    return 0
+
+
 def main() -> int:
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
@@ -1204,13 +1420,13 @@ def main() -> int:
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
     parser.add_argument("--skip-points", action="store_true", help="leave out the batch 1 / 64 points, prefill and e2e")
     parser.add_argument("--only", default=None, choices=["prefill"], help="time one part alone (for profiling)")
-    parser.add_argument("--workload", default=None, choices=["mixed-1.5b", "batch-32b", "reference-tables", "nunivik", "mirovik", "kudazen", "tobadra", "zurevik"],
+    parser.add_argument("--workload", default=None, choices=["mixed-1.5b", "batch-32b", "reference-tables", "nunivik", "mirovik", "kudazen", "tobadra", "zurevik", "biropel"],
                         help="one of the other workloads instead: 128 requests with prompts of 16..4096 tokens and 256 decoded tokens "
                              "each through generate() at the 1.5B shape; batch 16 with prompts of 4,096 and 512 decoded tokens at the 32B shape; "
                              "or the reference's own published tables (decode by batch at context 512, prefill by length) at the 0.5B and 7B shapes; "
                              "or the Nunivik design at two layer sizes beside the Qwen2 model of equal size, with its own kernels timed alone; "
                              "or the Mirovik design at two layer sizes beside the Nunivik model of equal size, likewise")
-    parser.add_argument("--size", default=None, choices=["2k", "4k"], help="with --workload nunivik, mirovik, kudazen, tobadra or zurevik: one of its sizes only")
+    parser.add_argument("--size", default=None, choices=["2k", "4k"], help="with --workload nunivik, mirovik, kudazen, tobadra, zurevik or biropel: one of its sizes only")
     args = parser.parse_args()
     if args.impl == "reference":
         return reference_arm()
@@ -1226,6 +1442,8 @@ def main() -> int:
         return tobadra_workload(args)
     if args.workload == "zurevik":
         return zurevik_workload(args)
+    if args.workload == "biropel":
+        return biropel_workload(args)
     if args.workload:
         return other_workload(args.workload)
     if args.gpus != 1 or int(os.environ.get("WORLD_SIZE", "1")) != 1:
