@@ -1321,18 +1321,19 @@ def biropel_kernels(size: dict, measured: dict) -> dict:
         report(f"memory.gates/{shape}", timed(make), tokens * m_heads * 20)
         gates = make()
 
-        def memory_scan(state, own, starts, count, states_only=False, decays=None):
-            return recurrent.matrix_memory_scan(m_proj, m_heads * n, 0, 2 * m_heads * n, gates, state, 0, own, starts, count, m_heads, n, n_padded, e, n ** -0.5,
-                                                states_only=states_only, decays=decays)
+        def memory_scan():
+            return recurrent.matrix_memory_scan(m_proj, m_heads * n, 0, 2 * m_heads * n, gates, m_state, 0, slots, row_start, rows, m_heads, n, n_padded, e, n ** -0.5)
 
         moved = 4 * (tokens * (2 * m_heads * n + 2 * m_heads * e) + 2 * rows * m_heads * e * n)
-        report(f"memory.scan/{shape}", timed(lambda: memory_scan(m_state, slots, row_start, rows)), moved, fp32_flops=4.0 * tokens * m_heads * n * e)
-        cut = recurrent.plan_segments(counts)
-        if cut is not None:
-            seg_start, seg_row = torch.tensor(cut[0], dtype=torch.int32, device=dev), torch.tensor(cut[1], dtype=torch.int32, device=dev)
-            report(f"memory.scan_in_segments/{shape}", timed(lambda: recurrent.scan_in_segments(memory_scan, per_head, m_state, 0, slots, seg_start, seg_row, len(cut[1]), m_heads)), moved,
-                   fp32_flops=7.0 * tokens * m_heads * n * e)
-        y = memory_scan(m_state, slots, row_start, rows)
+        report(f"memory.scan/{shape}", timed(memory_scan), moved, fp32_flops=4.0 * tokens * m_heads * n * e)
+        cut = recurrent.plan_chunks(counts)
+        if cut is not None:  # as the bfloat16 engine walks a long row
+            chunk_start, chunk_row = torch.tensor(cut[0], dtype=torch.int32, device=dev), torch.tensor(cut[1], dtype=torch.int32, device=dev)
+            in_chunks = lambda: recurrent.chunked_scan(recurrent.KIND_GIVEN, m_proj[:, m_heads * n :], m_proj, m_proj[:, 2 * m_heads * n :], gates.view(tokens, 4 * m_heads), 3 * m_heads, m_heads,
+                                                       m_state, 0, slots, chunk_start, chunk_row, len(cut[1]), m_heads, m_heads, n, n_padded, e, sums_keys=True, q_scale=n ** -0.5,
+                                                       columns=recurrent.matrix_memory_columns(e))
+            report(f"memory.scan_in_chunks/{shape}", timed(in_chunks), moved, bf16_flops=2.0 * tokens * m_heads * (3 * n * e + recurrent.CHUNK / 2 * (n + e)))
+        y = memory_scan()
         gated = torch.empty(tokens, m_heads * e, dtype=torch.bfloat16, device=dev)
         m_norm = torch.ones(m_heads * e, device=dev)
         report(f"memory.norm/{shape}", timed(lambda: recurrent.matrix_memory_norm(y, gates, m_proj, 2 * m_heads * n + m_heads * e, m_norm, e, 1e-6, gated)), tokens * m_heads * e * 10)
@@ -1340,9 +1341,11 @@ def biropel_kernels(size: dict, measured: dict) -> dict:
         retention = lambda: recurrent.state_scan(recurrent.MODE_RETENTION, m_proj, m_heads * n, 0, 2 * m_heads * n, m_proj, 0, 0, decay, decay, None, r_state, 0, slots, row_start, rows,
                                                  m_heads, m_heads, n, n, e)
         report(f"mirovik.retention_scan/{shape}", timed(retention), moved, fp32_flops=4.0 * tokens * m_heads * n * e)
-        if cut is not None:
+        segments = recurrent.plan_segments(counts)
+        if segments is not None:
+            seg_start, seg_row = torch.tensor(segments[0], dtype=torch.int32, device=dev), torch.tensor(segments[1], dtype=torch.int32, device=dev)
             report(f"mirovik.retention_in_segments/{shape}", timed(lambda: recurrent.retention_in_segments(m_proj, m_heads * n, 0, 2 * m_heads * n, decay, r_state, slots, seg_start,
-                                                                                                          seg_row, len(cut[1]), m_heads, n, n, e)), moved, fp32_flops=8.0 * tokens * m_heads * n * e)
+                                                                                                          seg_row, len(segments[1]), m_heads, n, n, e)), moved, fp32_flops=8.0 * tokens * m_heads * n * e)
         o = retention()
         report(f"mirovik.gated_norm/{shape}", timed(lambda: recurrent.gated_group_norm(o, m_proj, 2 * m_heads * n + m_heads * e, None, e, False, 1e-6, torch.bfloat16)), tokens * m_heads * e * 10)
         # the state-space mixer: convolution, scan, gated norm over groups of the inner width
@@ -1358,16 +1361,17 @@ def biropel_kernels(size: dict, measured: dict) -> dict:
         zeros, ones = torch.zeros(s_heads, device=dev), torch.ones(s_heads, device=dev)
         s_state = torch.zeros(rows, s_heads * s_e * state, device=dev)
 
-        def state_scan(st, own, starts, count, states_only=False, decays=None):
-            return recurrent.state_scan(recurrent.MODE_STATE_SPACE, conv, inner, inner + bn, 0, s_proj, inner + channels, inner + channels, zeros, zeros, ones, st, 0, own, starts, count,
-                                        s_heads, groups, state, state, s_e, states_only=states_only, decays=decays)
+        def state_scan():
+            return recurrent.state_scan(recurrent.MODE_STATE_SPACE, conv, inner, inner + bn, 0, s_proj, inner + channels, inner + channels, zeros, zeros, ones, s_state, 0, slots, row_start,
+                                        rows, s_heads, groups, state, state, s_e)
 
         moved = 4 * (tokens * (2 * bn + 2 * inner) + 2 * rows * inner * state)
-        report(f"states.scan/{shape}", timed(lambda: state_scan(s_state, slots, row_start, rows)), moved, fp32_flops=4.0 * tokens * inner * state)
+        report(f"states.scan/{shape}", timed(state_scan), moved, fp32_flops=4.0 * tokens * inner * state)
         if cut is not None:
-            report(f"states.scan_in_segments/{shape}", timed(lambda: recurrent.scan_in_segments(state_scan, s_e * state, s_state, 0, slots, seg_start, seg_row, len(cut[1]), s_heads)), moved,
-                   fp32_flops=7.0 * tokens * inner * state)
-        y = state_scan(s_state, slots, row_start, rows)
+            in_chunks = lambda: recurrent.chunked_scan(recurrent.KIND_STATE_SPACE, conv[:, inner:], conv[:, inner + bn :], conv, s_proj, inner + channels, 0, s_state, 0, slots, chunk_start,
+                                                       chunk_row, len(cut[1]), s_heads, groups, state, state, s_e, a_log=zeros, dt_bias=zeros, skip=ones)
+            report(f"states.scan_in_chunks/{shape}", timed(in_chunks), moved, bf16_flops=2.0 * tokens * s_heads * (3 * state * s_e + recurrent.CHUNK / 2 * (state + s_e)))
+        y = state_scan()
         s_norm = torch.ones(inner, device=dev)
         report(f"states.gated_norm/{shape}", timed(lambda: recurrent.gated_group_norm(y, s_proj, 0, s_norm, inner // groups, True, 1e-6, torch.bfloat16)), tokens * inner * 10)
         # the feed-forward's activation

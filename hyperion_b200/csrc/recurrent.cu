@@ -90,7 +90,6 @@ struct ScanArgs {
     float q_scale;
     int values;          // value columns of a head (0: e); a column from there on takes the constant 1
     int out_e;           // columns of a head in `out` (0: e)
-    float* decays;       // [rows, heads] or null: the product of a row's decays per head (what joins segments scanned side by side)
 };
 
 template <int NG, int LPC, int CPT, int MODE>  // NG groups of four entries per lane, LPC lanes per column (n <= NG * 4 * LPC), CPT columns per thread
@@ -141,7 +140,6 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
         bonus[r] = (WKV && index < a.n) ? a.dt_bias[(size_t)head * a.n + index] : 0.f;
     }
     const float skip = MODE == MODE_STATE_SPACE ? a.skip[head] : 0.f;
-    float faded = 1.f;
 
     float pk[PER_WARP][NPR], pq[PER_WARP][NPR], pv[PER_WARP][VR], pdecay[PER_WARP], pstep[PER_WARP], pw[PER_WARP][VEC ? NPR : 1];
     auto prefetch = [&](int first) {
@@ -315,16 +313,6 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
                         for (int i = 0; i < 4; ++i) s[c][r][i] *= decay;
                     u[c] = step * cv[c];
                 }
-                faded *= decay;
-                if (!a.out) {  // only the states are wanted: the query meets nothing
-#pragma unroll
-                    for (int c = 0; c < CPT; ++c)
-#pragma unroll
-                        for (int r = 0; r < NG; ++r)
-#pragma unroll
-                            for (int i = 0; i < 4; ++i) s[c][r][i] = fmaf(ck[r][i], u[c], s[c][r][i]);
-                    continue;
-                }
             }
 #pragma unroll
             for (int c = 0; c < CPT; ++c) {
@@ -350,7 +338,6 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanArgs
         publish(buffer ^ 1);
         __syncthreads();
     }
-    if (a.decays && blockIdx.x == 0 && threadIdx.x == 0) a.decays[(size_t)row * a.heads + head] = faded;
 #pragma unroll
     for (int c = 0; c < CPT; ++c) {
         const int col = col0 + cw + GROUPS * c;
@@ -472,17 +459,15 @@ HB_EXPORT int hb_conv_state_update(const float* x, int x_stride, int col0, int c
 // mode 0: gated delta rule (keys and queries made unit vectors, q times q_scale; decay = exp(-exp(a_log) softplus(proj[decay_off] + dt_bias)),
 // step = sigmoid(proj[step_off])).  mode 1: state space (step = softplus(proj[decay_off] + dt_bias), decay = exp(-exp(a_log) step), skip = D).
 // The state of (slot, head) is S^T [e, n_padded] at state + slot * slot_stride + state_off; n_padded, state_off and slot_stride are multiples of 4.
-// decays [rows, heads] (modes 1 and 2; or null) receives the product of every row's decays.
 HB_EXPORT int hb_state_scan(int mode, const float* conv, int conv_stride, int k_off, int q_off, int v_off, const float* proj, int proj_stride,
                             int decay_off, int step_off, const float* a_log, const float* dt_bias, const float* skip, float* state,
                             long long slot_stride, int state_off, const int* slots, const int* row_start, float* out, int rows, int heads,
-                            int groups, int n, int n_padded, int e, float q_scale, float* decays, cudaStream_t stream) {
+                            int groups, int n, int n_padded, int e, float q_scale, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (n <= 0 || n > 256 || e <= 0 || heads <= 0 || groups <= 0 || heads % groups || rows > 65535 || heads > 65535) return HB_UNSUPPORTED_SIZE;
     if (n_padded < n || (n_padded & 3) || (state_off & 3) || (slot_stride & 3) || (((uintptr_t)state) & 15)) return HB_BAD_ARGUMENT;
     ScanArgs a{conv + k_off, conv + q_off, conv + v_off, conv_stride, conv_stride, conv_stride, proj, proj_stride, decay_off, step_off, proj, proj_stride, a_log, dt_bias, skip,
-               state, (size_t)slot_stride, state_off, slots, row_start, out, heads, groups, n, n_padded, e, q_scale, 0, 0, decays};
-    if (decays && mode == MODE_DELTA) return HB_BAD_ARGUMENT;  // its correction is not a product of decays
+               state, (size_t)slot_stride, state_off, slots, row_start, out, heads, groups, n, n_padded, e, q_scale};
     if (mode == MODE_DELTA) return launch_scan<MODE_DELTA>(a, rows, stream);
     if (mode == MODE_STATE_SPACE) return launch_scan<MODE_STATE_SPACE>(a, rows, stream);
     if (mode == MODE_RETENTION) return launch_scan<MODE_RETENTION>(a, rows, stream);
@@ -520,57 +505,80 @@ HB_EXPORT int hb_wkv_scan(const float* k, int k_stride, const float* q, int q_st
 // ---------------------------------------------------------------- a matrix memory with exponential gates
 // Per head: S <- exp(f + m' - m) S + exp(i - m) k v^T and a vector n that follows the same recurrence with k alone, where i and f are the logarithms of
 // the input and of the forget gate and m = max(f + m', i) a running maximum that starts at 0;   o = S^T q / (max(|n . q|, exp(-m)) + 1e-6).
-// The maximum depends on the gates alone, so it is walked first (matrix_memory_gates: a warp per row and head; the lanes make the gates of
-// 32 tokens side by side, then every lane walks the chain m = max(f + m, i) through them in order, so its bits do not depend on how a row was
-// cut).  The scan (MODE_GIVEN) then knows its decay and step; n is the column of S whose value is always 1.  matrix_memory_norm divides, norms each
+// The maximum depends on the gates alone, so it is walked first (matrix_memory_gates: a block per row and head; one thread walks the chain
+// m = max(f + m, i) through a run of 128 tokens in order, so its bits do not depend on how a row was cut, while the others make the next run's gates
+// and the last run's results).  The scan (MODE_GIVEN) then knows its decay and step; n is the column of S whose value is always 1.  matrix_memory_norm divides, norms each
 // head by its root mean square, and applies weight and gate.
 namespace {
-__global__ void __launch_bounds__(32) matrix_memory_gates_kernel(const float* __restrict__ x, int x_stride, int i_off, int f_off, const float* __restrict__ i_bias,
-                                                                 const float* __restrict__ f_bias, float cap, float* __restrict__ state, size_t slot_stride,
-                                                                 int m_off, const int* __restrict__ slots, const int* __restrict__ row_start,
-                                                                 float* __restrict__ gates, int heads) {
-    const int head = blockIdx.x, row = blockIdx.y, lane = threadIdx.x;
-    const int t0 = row_start[row], t1 = row_start[row + 1];
+constexpr int GATE_TOKENS = 128;
+
+__global__ void __launch_bounds__(32 + GATE_TOKENS) matrix_memory_gates_kernel(const float* __restrict__ x, int x_stride, int i_off, int f_off,
+                                                                               const float* __restrict__ i_bias, const float* __restrict__ f_bias, float cap,
+                                                                               float* __restrict__ state, size_t slot_stride, int m_off, const int* __restrict__ slots,
+                                                                               const int* __restrict__ row_start, float* __restrict__ gates, int heads) {
+    __shared__ __align__(16) float in[2][GATE_TOKENS], forget[2][GATE_TOKENS];
+    __shared__ float top[2][GATE_TOKENS + 1];  // the maximum before the run of tokens, then after each of them
+    const int head = blockIdx.x, row = blockIdx.y, mine = (int)threadIdx.x - 32;
+    const int t0 = row_start[row], count = row_start[row + 1] - t0, runs = (count + GATE_TOKENS - 1) / GATE_TOKENS;
     float* const kept = state + (size_t)slots[row] * slot_stride + m_off + head;
     const float bi = i_bias[head], bf = f_bias[head];
-    float m = *kept, raw_i = 0.f, raw_f = 0.f;
-    if (t0 + lane < t1) {
-        raw_i = x[(size_t)(t0 + lane) * x_stride + i_off + head];
-        raw_f = x[(size_t)(t0 + lane) * x_stride + f_off + head];
+    float m = *kept, raw_i = 0.f, raw_f = 0.f, i0 = 0.f, f0 = 0.f, i1 = 0.f, f1 = 0.f;  // this thread's gates of the last two runs
+    if (mine >= 0 && mine < count) {
+        raw_i = x[(size_t)(t0 + mine) * x_stride + i_off + head];
+        raw_f = x[(size_t)(t0 + mine) * x_stride + f_off + head];
     }
-    for (int base = t0; base < t1; base += 32) {
-        const float in = cap * tanhf((raw_i + bi) / cap);
-        const float z = cap * tanhf((raw_f + bf) / cap);
-        const float forget = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
-        const int next = base + 32 + lane;
-        if (next < t1) {  // in flight while the chain is walked
-            raw_i = x[(size_t)next * x_stride + i_off + head];
-            raw_f = x[(size_t)next * x_stride + f_off + head];
-        }
-        const int count = min(32, t1 - base);
-        float before = m, after = m;
-        if (count == 32) {
+    for (int run = 0; run < runs + 2; ++run) {  // at once: the gates of `run`, the chain through the run before, the results of the one before that
+        if (mine >= 0) {
+            const int done = (run - 2) * GATE_TOKENS + mine;
+            if (run >= 2 && done < count) {
+                const float before = top[run & 1][mine], after = top[run & 1][mine + 1], fade = (f0 + before) - after;
+                float* g = gates + (size_t)(t0 + done) * 4 * heads + head;
+                g[0] = expf(fade);
+                g[heads] = expf(i0 - after);
+                g[2 * heads] = expf(-after);
+                g[3 * heads] = fade;
+            }
+            i0 = i1; f0 = f1;
+            if (run < runs) {
+                const float z = cap * tanhf((raw_f + bf) / cap);
+                i1 = cap * tanhf((raw_i + bi) / cap);
+                f1 = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+                in[run & 1][mine] = i1;
+                forget[run & 1][mine] = f1;
+                const int next = (run + 1) * GATE_TOKENS + mine;
+                if (next < count) {
+                    raw_i = x[(size_t)(t0 + next) * x_stride + i_off + head];
+                    raw_f = x[(size_t)(t0 + next) * x_stride + f_off + head];
+                }
+            }
+        } else if (threadIdx.x == 0 && run >= 1 && run <= runs) {
+            const int which = (run - 1) & 1, live = min(GATE_TOKENS, count - (run - 1) * GATE_TOKENS);
+            top[which][0] = m;
+            int j = 0;
+            for (; j + 16 <= live; j += 16) {
+                float f[16], i[16];
 #pragma unroll
-            for (int j = 0; j < 32; ++j) {
-                const float fj = __shfl_sync(0xffffffffu, forget, j), ij = __shfl_sync(0xffffffffu, in, j), was = m;
-                m = fmaxf(fj + m, ij);
-                if (lane == j) { before = was; after = m; }
+                for (int k = 0; k < 16; k += 4) {
+                    float part[4];
+                    load4(&forget[which][j + k], part);
+                    f[k] = part[0]; f[k + 1] = part[1]; f[k + 2] = part[2]; f[k + 3] = part[3];
+                    load4(&in[which][j + k], part);
+                    i[k] = part[0]; i[k + 1] = part[1]; i[k + 2] = part[2]; i[k + 3] = part[3];
+                }
+#pragma unroll
+                for (int k = 0; k < 16; ++k) {
+                    m = fmaxf(f[k] + m, i[k]);
+                    top[which][j + k + 1] = m;
+                }
             }
-        } else {
-            for (int j = 0; j < count; ++j) {
-                const float fj = __shfl_sync(0xffffffffu, forget, j), ij = __shfl_sync(0xffffffffu, in, j), was = m;
-                m = fmaxf(fj + m, ij);
-                if (lane == j) { before = was; after = m; }
+            for (; j < live; ++j) {
+                m = fmaxf(forget[which][j] + m, in[which][j]);
+                top[which][j + 1] = m;
             }
         }
-        if (lane < count) {
-            float* g = gates + (size_t)(base + lane) * 3 * heads + head;
-            g[0] = expf((forget + before) - after);
-            g[heads] = expf(in - after);
-            g[2 * heads] = expf(-after);
-        }
+        __syncthreads();
     }
-    if (lane == 0) *kept = m;
+    if (threadIdx.x == 0) *kept = m;
 }
 
 // A warp per (token, head).
@@ -584,7 +592,7 @@ __global__ void __launch_bounds__(128) matrix_memory_norm_kernel(const float* __
     const float* g = gate + (size_t)t * gate_stride + gate_off + (size_t)head * e;
     const float* w = weight + (size_t)head * e;
     TO* dst = out + (size_t)t * out_stride + (size_t)head * e;
-    const float below = fmaxf(fabsf(row[e]), gates[(size_t)t * 3 * heads + 2 * heads + head]) + 1e-6f;
+    const float below = fmaxf(fabsf(row[e]), gates[(size_t)t * 4 * heads + 2 * heads + head]) + 1e-6f;
     float sum = 0.f;
     if (by_four) {
         for (int j = lane * 4; j < e; j += 128) {
@@ -615,12 +623,12 @@ __global__ void __launch_bounds__(128) matrix_memory_norm_kernel(const float* __
 
 // x [tokens, x_stride]: the gates' pre-activations, head h at i_off + h and f_off + h; log input gate i = cap tanh((x + i_bias) / cap), log forget gate
 // f = log sigmoid(cap tanh((x + f_bias) / cap)).  The running maximum of (slot, head) lies at state + slot * slot_stride + m_off + head.
-// gates [tokens, 3, heads] receives the token's decay exp(f + m' - m), its step exp(i - m) and exp(-m).
+// gates [tokens, 4, heads] receives the token's decay exp(f + m' - m), its step exp(i - m), exp(-m) and the decay's logarithm.
 HB_EXPORT int hb_matrix_memory_gates(const float* x, int x_stride, int i_off, int f_off, const float* i_bias, const float* f_bias, float cap, float* state,
                                      long long slot_stride, int m_off, const int* slots, const int* row_start, float* gates, int rows, int heads, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (heads <= 0 || rows > 65535 || !(cap > 0.f)) return HB_UNSUPPORTED_SIZE;
-    matrix_memory_gates_kernel<<<dim3(heads, rows), 32, 0, stream>>>(x, x_stride, i_off, f_off, i_bias, f_bias, cap, state, (size_t)slot_stride, m_off, slots, row_start,
+    matrix_memory_gates_kernel<<<dim3(heads, rows), 32 + GATE_TOKENS, 0, stream>>>(x, x_stride, i_off, f_off, i_bias, f_bias, cap, state, (size_t)slot_stride, m_off, slots, row_start,
                                                                    gates, heads);
     return launch_status();
 }
@@ -629,12 +637,12 @@ HB_EXPORT int hb_matrix_memory_gates(const float* x, int x_stride, int i_off, in
 // [values + 1, n_padded], its last row the sum of keys; out [tokens, heads, out_e] with out_e > values, entry `values` being n . q.
 HB_EXPORT int hb_matrix_memory_scan(const float* x, int x_stride, int k_off, int q_off, int v_off, const float* gates, float* state, long long slot_stride, int state_off,
                                     const int* slots, const int* row_start, float* out, int rows, int heads, int n, int n_padded, int values, int out_e, float q_scale,
-                                    float* decays, cudaStream_t stream) {
+                                    cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (n <= 0 || n > 256 || values <= 0 || heads <= 0 || rows > 65535 || heads > 65535 || out_e <= values) return HB_UNSUPPORTED_SIZE;
     if (n_padded < n || (n_padded & 3) || (state_off & 3) || (slot_stride & 3) || (((uintptr_t)state) & 15)) return HB_BAD_ARGUMENT;
-    ScanArgs a{x + k_off, x + q_off, x + v_off, x_stride, x_stride, x_stride, gates, 3 * heads, 0, heads, gates, 3 * heads, nullptr, nullptr, nullptr,
-               state, (size_t)slot_stride, state_off, slots, row_start, out, heads, heads, n, n_padded, values + 1, q_scale, values, out_e, decays};
+    ScanArgs a{x + k_off, x + q_off, x + v_off, x_stride, x_stride, x_stride, gates, 4 * heads, 0, heads, gates, 4 * heads, nullptr, nullptr, nullptr,
+               state, (size_t)slot_stride, state_off, slots, row_start, out, heads, heads, n, n_padded, values + 1, q_scale, values, out_e};
     return launch_scan<MODE_GIVEN>(a, rows, stream);
 }
 
@@ -1118,10 +1126,10 @@ HB_EXPORT int hb_selective_scan(const float* x, int x_stride, const float* dt, i
 namespace {
 __global__ void join_segments_kernel(float* __restrict__ ends, size_t end_stride, float* __restrict__ state, size_t slot_stride, int state_off,
                                      const int* __restrict__ slots, const int* __restrict__ seg_start, const int* __restrict__ seg_row, int segments,
-                                     const float* __restrict__ decay, int per_head, int entries, const float* __restrict__ seg_decay, int heads) {
+                                     const float* __restrict__ decay, int per_head, int entries) {
     const int entry = blockIdx.x * blockDim.x + threadIdx.x;
     if (entry >= entries) return;
-    const float log_decay = seg_decay ? 0.f : log2f(decay[entry / per_head]);
+    const float log_decay = log2f(decay[entry / per_head]);
     constexpr int AHEAD = 8;  // what the segments add is asked for before the chain through them starts: one trip to memory, not one per segment
     int j = 0;
     while (j < segments) {
@@ -1136,7 +1144,7 @@ __global__ void join_segments_kernel(float* __restrict__ ends, size_t end_stride
                 if (j + k < segments && seg_row[j + k] == row) {
                     added[k] = ends[(size_t)(j + k) * end_stride + entry];
                     const int length = seg_start[j + k + 1] - seg_start[j + k];
-                    fade[k] = seg_decay ? seg_decay[(size_t)(j + k) * heads + entry / per_head] : (log_decay == 0.f ? 1.f : exp2f((float)length * log_decay));
+                    fade[k] = log_decay == 0.f ? 1.f : exp2f((float)length * log_decay);
                     count = k + 1;
                 }
             }
@@ -1163,22 +1171,9 @@ HB_EXPORT int hb_join_segments(float* ends, long long end_stride, float* state, 
     if (heads <= 0 || per_head <= 0) return HB_BAD_ARGUMENT;
     const int entries = heads * per_head;
     join_segments_kernel<<<(entries + 255) / 256, 256, 0, stream>>>(ends, (size_t)end_stride, state, (size_t)slot_stride, state_off, slots, seg_start, seg_row,
-                                                                 segments, decay, per_head, entries, nullptr, heads);
+                                                                 segments, decay, per_head, entries);
     return launch_status();
 }
-
-// The same where a head's decay differs from token to token: seg_decay [segments, heads] holds its product over every segment (the first pass leaves it).
-HB_EXPORT int hb_join_segments_by_decay(float* ends, long long end_stride, float* state, long long slot_stride, int state_off, const int* slots,
-                                        const int* seg_start, const int* seg_row, int segments, const float* seg_decay, int heads, int per_head,
-                                        cudaStream_t stream) {
-    if (segments <= 0) return 0;
-    if (heads <= 0 || per_head <= 0 || !seg_decay) return HB_BAD_ARGUMENT;
-    const int entries = heads * per_head;
-    join_segments_kernel<<<(entries + 255) / 256, 256, 0, stream>>>(ends, (size_t)end_stride, state, (size_t)slot_stride, state_off, slots, seg_start, seg_row,
-                                                                 segments, nullptr, per_head, entries, seg_decay, heads);
-    return launch_status();
-}
-
 
 // The same joining for the selective scan, whose decay differs per channel and state entry: over a segment it is exp(A[c, i] * the sum
 // of the channel's steps), which the first pass leaves in dt_sums [segments, inner].

@@ -81,17 +81,16 @@ def silu_columns_(x: torch.Tensor, col0: int, columns: int) -> None:
 def state_scan(mode: int, conv: torch.Tensor, k_off: int, q_off: int, v_off: int, proj: torch.Tensor, decay_off: int, step_off: int,
                a_log: torch.Tensor, dt_bias: torch.Tensor, skip: torch.Tensor | None, state: torch.Tensor, state_off: int, slots: torch.Tensor,
                row_start: torch.Tensor, rows: int, heads: int, groups: int, n: int, n_padded: int, e: int, q_scale: float = 1.0,
-               states_only: bool = False, decays: torch.Tensor | None = None) -> torch.Tensor | None:
+               states_only: bool = False) -> torch.Tensor | None:
     """Walk every row's tokens through the recurrence of ``mode`` from and into its slot of ``state``; returns [tokens, heads * e]
-    (nothing with ``states_only``: the walk then only leaves the rows' states).  ``decays`` [rows, heads] float (not for the delta rule) receives the
-    product of every row's decays."""
-    require_cuda(conv, proj, a_log, dt_bias, skip, state, slots, row_start, decays)
+    (nothing with ``states_only``: the walk then only leaves the rows' states)."""
+    require_cuda(conv, proj, a_log, dt_bias, skip, state, slots, row_start)
     _floats(conv, proj, a_log, dt_bias, skip, state)
     out = None if states_only else torch.empty((conv.shape[0], heads * e), dtype=torch.float32, device=conv.device)
     check(library("recurrent").hb_state_scan(i32(mode), ptr(conv), i32(conv.stride(0)), i32(k_off), i32(q_off), i32(v_off), ptr(proj), i32(proj.stride(0)),
                                              i32(decay_off), i32(step_off), ptr(a_log), ptr(dt_bias), ptr(skip), ptr(state),
                                              ctypes.c_longlong(state.stride(0)), i32(state_off), ptr(slots), ptr(row_start), ptr(out), i32(rows),
-                                             i32(heads), i32(groups), i32(n), i32(n_padded), i32(e), f32(q_scale), ptr(decays), stream_ptr()), "state_scan")
+                                             i32(heads), i32(groups), i32(n), i32(n_padded), i32(e), f32(q_scale), stream_ptr()), "state_scan")
     return out
 
 
@@ -99,10 +98,10 @@ def matrix_memory_gates(x: torch.Tensor, i_off: int, f_off: int, i_bias: torch.T
                         slots: torch.Tensor, row_start: torch.Tensor, rows: int, heads: int) -> torch.Tensor:
     """The gates of a matrix memory: log input gate i = cap tanh((x + i_bias) / cap) and log forget gate f = log sigmoid(cap tanh((x + f_bias) / cap)) from the columns
     ``i_off ..`` and ``f_off ..`` of ``x``, and the running maximum m = max(f + m', i) of every row, which starts from and ends in its slot of
-    ``state`` at ``m_off``.  Returns [tokens, 3, heads]: the decay exp(f + m' - m), the step exp(i - m), and exp(-m)."""
+    ``state`` at ``m_off``.  Returns [tokens, 4, heads]: the decay exp(f + m' - m), the step exp(i - m), exp(-m), and the decay's logarithm."""
     require_cuda(x, i_bias, f_bias, state, slots, row_start)
     _floats(x, i_bias, f_bias, state)
-    gates = torch.empty((x.shape[0], 3, heads), dtype=torch.float32, device=x.device)
+    gates = torch.empty((x.shape[0], 4, heads), dtype=torch.float32, device=x.device)
     check(library("recurrent").hb_matrix_memory_gates(ptr(x), i32(x.stride(0)), i32(i_off), i32(f_off), ptr(i_bias), ptr(f_bias), f32(cap), ptr(state),
                                                       ctypes.c_longlong(state.stride(0)), i32(m_off), ptr(slots), ptr(row_start), ptr(gates), i32(rows), i32(heads),
                                                       stream_ptr()), "matrix_memory_gates")
@@ -115,18 +114,17 @@ def matrix_memory_columns(values: int) -> int:
 
 
 def matrix_memory_scan(x: torch.Tensor, k_off: int, q_off: int, v_off: int, gates: torch.Tensor, state: torch.Tensor, state_off: int, slots: torch.Tensor,
-                       row_start: torch.Tensor, rows: int, heads: int, n: int, n_padded: int, values: int, q_scale: float, states_only: bool = False,
-                       decays: torch.Tensor | None = None) -> torch.Tensor | None:
+                       row_start: torch.Tensor, rows: int, heads: int, n: int, n_padded: int, values: int, q_scale: float) -> torch.Tensor:
     """S <- a S + b k v^T per head with decay a and step b from ``gates`` (:func:`matrix_memory_gates`), and the same for the sum of keys, a further column of S.
     Keys, queries and values are columns of ``x``; every row's tokens walk from and into its slot of ``state`` ([heads, values + 1, n_padded] floats at
     ``state_off``).  Returns [tokens, heads, :func:`matrix_memory_columns`]: S^T q and, at entry ``values``, n . q, with q times ``q_scale``."""
-    require_cuda(x, gates, state, slots, row_start, decays)
+    require_cuda(x, gates, state, slots, row_start)
     _floats(x, gates, state)
     columns = matrix_memory_columns(values)
-    out = None if states_only else torch.empty((x.shape[0], heads, columns), dtype=torch.float32, device=x.device)
+    out = torch.empty((x.shape[0], heads, columns), dtype=torch.float32, device=x.device)
     check(library("recurrent").hb_matrix_memory_scan(ptr(x), i32(x.stride(0)), i32(k_off), i32(q_off), i32(v_off), ptr(gates), ptr(state), ctypes.c_longlong(state.stride(0)),
                                                      i32(state_off), ptr(slots), ptr(row_start), ptr(out), i32(rows), i32(heads), i32(n), i32(n_padded), i32(values), i32(columns),
-                                                     f32(q_scale), ptr(decays), stream_ptr()), "matrix_memory_scan")
+                                                     f32(q_scale), stream_ptr()), "matrix_memory_scan")
     return out
 
 
@@ -295,20 +293,72 @@ def retention_in_segments(proj: torch.Tensor, k_off: int, q_off: int, v_off: int
     return state_scan(MODE_RETENTION, proj, k_off, q_off, v_off, proj, 0, 0, decay, decay, None, ends, 0, own, seg_start, segments, heads, heads, n, n_padded, e)
 
 
-def scan_in_segments(scan, per_head: int, state: torch.Tensor, state_off: int, slots: torch.Tensor, seg_start: torch.Tensor, seg_row: torch.Tensor, segments: int, heads: int):
-    """A scan whose state fades by a number per token and head, S <- a S + (something that does not depend on S), with long rows cut into segments that are walked
-    side by side (see :func:`retention_in_segments`; here a segment's decay is the product its first pass leaves).  ``scan(state, slots, row_start, rows,
-    states_only, decays)`` walks rows whose matrices (``per_head`` floats a head) are the first ``heads * per_head`` floats of a record; the rows' own
-    matrices lie at ``state_off`` of ``state``."""
-    require_cuda(state, slots, seg_start, seg_row)
-    ends = torch.zeros((segments, heads * per_head), dtype=torch.float32, device=state.device)
-    decays = torch.empty((segments, heads), dtype=torch.float32, device=state.device)
-    own = torch.arange(segments, dtype=torch.int32, device=state.device)
-    scan(ends, own, seg_start, segments, True, decays)
-    check(library("recurrent").hb_join_segments_by_decay(ptr(ends), ctypes.c_longlong(ends.stride(0)), ptr(state), ctypes.c_longlong(state.stride(0)), i32(state_off),
-                                                         ptr(slots), ptr(seg_start), ptr(seg_row), i32(segments), ptr(decays), i32(heads), i32(per_head),
-                                                         stream_ptr()), "join_segments")
-    return scan(ends, own, seg_start, segments, False, None)
+CHUNK = 64  # csrc/chunked_scan.cu
+CHUNKED_FROM = 128  # tokens of a step's longest row from which its recurrences are walked in chunks
+KIND_STATE_SPACE, KIND_GIVEN = 0, 1
+
+
+def plan_chunks(counts) -> tuple[list[int], list[int]] | None:
+    """Every row cut into chunks of ``CHUNK`` tokens, the last one shorter: (first token of every chunk plus the end, the row of every chunk), or None when no row is
+    long enough for the chunked form to pay."""
+    if max(counts) < CHUNKED_FROM:
+        return None
+    starts, rows, at = [], [], 0
+    for row, count in enumerate(counts):
+        for first in range(0, int(count), CHUNK):
+            starts.append(at + first)
+            rows.append(row)
+        at += int(count)
+    return starts + [at], rows
+
+
+def chunk_planner(dtype: torch.dtype) -> dict:
+    """The step planner of mixers that walk long rows in chunks on the tensor cores (:func:`chunked_scan`): in bfloat16, a step with a long row gets ``scan_chunk_start``
+    and ``scan_chunk_row`` among its arrays and their number in ``step.host["scan_chunks"]`` (0 otherwise)."""
+    if dtype != torch.bfloat16:
+        return {}
+
+    def plan(rows, packer, host):
+        if "scan_chunks" in host:
+            return
+        counts = rows.counts if hasattr(rows, "counts") else [row.count for row in rows]
+        cut = plan_chunks([int(c) for c in counts])
+        host["scan_chunks"] = 0 if cut is None else len(cut[1])
+        if cut is not None:
+            packer.add("scan_chunk_start", cut[0])
+            packer.add("scan_chunk_row", cut[1])
+
+    return {("scan_chunks", CHUNK): plan}
+
+
+def chunked_scan(kind: int, k: torch.Tensor, q: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, decay_off: int, step_off: int, state: torch.Tensor, state_off: int,
+                 slots: torch.Tensor, chunk_start: torch.Tensor, chunk_row: torch.Tensor, chunks: int, heads: int, groups: int, n: int, n_padded: int, e: int, *,
+                 a_log: torch.Tensor | None = None, dt_bias: torch.Tensor | None = None, skip: torch.Tensor | None = None, sums_keys: bool = False,
+                 q_scale: float = 1.0, columns: int | None = None) -> torch.Tensor:
+    """A recurrence whose state fades by one number per token and head, S <- a S + b k v^T, o = S^T q, over the chunks of a step (:func:`plan_chunks`) on the tensor cores.
+    ``k``, ``q`` (group g at g * n, the query times ``q_scale``) and ``v`` (head h at h * e) are float views [tokens, *].  ``KIND_STATE_SPACE``: the
+    step is softplus(``gate``[decay_off + h] + dt_bias), a = exp(-exp(a_log) step), D = ``skip``; ``KIND_GIVEN``: ln a and b are the columns ``decay_off + h`` and
+    ``step_off + h`` of ``gate``.  The rows' states ([heads, e, n_padded], with ``sums_keys`` one more row for the sum of keys) lie at ``state_off`` of ``state``.  Returns
+    [tokens, heads, ``columns``] (``e`` unless stated; with ``sums_keys`` entry e of a head is n . q).  Differs from the one-pass scan by bfloat16 roundings of
+    keys, queries, values and weighted scores."""
+    require_cuda(k, q, v, gate, state, slots, chunk_start, chunk_row, a_log, dt_bias, skip)
+    _floats(k, q, v, gate, state, a_log, dt_bias, skip)
+    rows = e + (1 if sums_keys else 0)
+    columns = columns or rows
+    per_head = rows * n_padded
+    n16 = -(-n // 16) * 16
+    ends = torch.empty((chunks, heads * per_head), dtype=torch.float32, device=k.device)
+    begins = torch.empty((chunks, heads * rows * 2 * n16), dtype=torch.bfloat16, device=k.device)
+    decays = torch.empty((chunks, heads), dtype=torch.float32, device=k.device)
+    out = torch.empty((k.shape[0], heads, columns), dtype=torch.float32, device=k.device)
+    check(library("chunked_scan").hb_chunked_scan(
+        i32(kind), ptr(k), i32(k.stride(0)), ptr(q), i32(q.stride(0)), ptr(v), i32(v.stride(0)), ptr(gate), i32(gate.stride(0)), i32(decay_off), i32(step_off), ptr(a_log), ptr(dt_bias),
+        ptr(skip), ptr(ends), ptr(decays), ptr(begins), ptr(state), ctypes.c_longlong(state.stride(0)), i32(state_off), ptr(slots), ptr(chunk_start), ptr(chunk_row), i32(chunks),
+        ptr(out), i32(columns), i32(heads), i32(groups), i32(n), i32(n_padded), i32(e), i32(1 if sums_keys else 0), f32(q_scale), stream_ptr()), "chunked_scan")
+    from . import native
+
+    native.LAUNCHES[0] += 2  # three kernels: the chunks' sums, the chain through them, the outputs
+    return out
 
 
 def selective_in_segments(x: torch.Tensor, dt: torch.Tensor, bc: torch.Tensor, b_off: int, c_off: int, a: torch.Tensor, skip: torch.Tensor,

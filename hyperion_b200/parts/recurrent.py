@@ -52,7 +52,8 @@ Matrix memory with exponential gates (``matrix_memory``; the mLSTM of Beck et al
     y = o / rms(o) per head, times norm (a weight per column), times sigmoid(W_g x), then W_o.
 The running maximum m starts at 0.  The record holds the heads' matrices with n as one more column each, then the heads' m.
 Parameters: ``hidden_size``, ``heads``, ``head_dim``, ``value_dim``, ``gate_cap``, ``eps``.  Tensors: q, k, v, g, i, i.b, f, f.b, norm, o.
-``mamba2`` and ``matrix_memory`` are branches (``parts/branch.py``): they also run beside another mixer on the same input.
+``mamba2`` and ``matrix_memory`` are branches (``parts/branch.py``): they also run beside another mixer on the same input.  Both walk a bfloat16 step with a long row
+in chunks on the tensor cores (``csrc/chunked_scan.cu``: the state, its decays and steps stay float).
 
 Lightning attention (``lightning``): a matrix state per head that fades by a constant of the head, with nothing between the projections and
 the recurrence but an activation:
@@ -73,11 +74,12 @@ from .branch import Branch
 from .spec import PartSpec
 
 
-SEGMENT_BLOCKS = 100  # the most blocks of a one-pass scan at which cutting long rows into segments pays
-
-
 def _round_up(value: int, step: int) -> int:
     return -(-value // step) * step
+
+
+def _chunked_module(dtype: torch.dtype) -> list[tuple[str, dict]]:
+    return [("chunked_scan", {})] if dtype == torch.bfloat16 else []
 
 
 class _ScanMixer(Mixer):
@@ -108,15 +110,6 @@ class _ScanMixer(Mixer):
 
     def _float(self, tensor: torch.Tensor) -> torch.Tensor:
         return tensor.to(torch.float32).contiguous()
-
-    def _walk(self, scan, step, state, slots, per_head: int, columns: int):
-        """``scan`` (as ``recurrent.scan_in_segments`` takes it) over the step's rows, long rows in segments side by side while one pass would leave the GPU mostly
-        idle, as for the package's other recurrences that are linear in their state."""
-        blocks = self.heads * -(-columns // 32)
-        segments = step.host.get("scan_segments", 0) if self.dtype == torch.bfloat16 and blocks <= SEGMENT_BLOCKS else 0
-        if segments:
-            return recurrent.scan_in_segments(scan, per_head, state, 0, slots, step.extra["scan_seg_start"], step.extra["scan_seg_row"], segments, self.heads)
-        return scan(state, slots, step.row_start, step.n_rows)
 
 
 class GatedDeltaRule(_ScanMixer):
@@ -197,8 +190,11 @@ class StateSpaceMixer(_ScanMixer, Branch):
         self.a_log, self.dt_bias, self.skip = self._float(tensors["A_log"]), self._float(tensors["dt_bias"]), self._float(tensors["D"])
         self.norm = self._float(tensors["norm"])
 
+    def kernel_modules(self):
+        return super().kernel_modules() + _chunked_module(self.dtype)
+
     def step_plans(self):
-        return recurrent.segment_planner(self.dtype)
+        return recurrent.chunk_planner(self.dtype)
 
     def core(self, proj, col0, step, cache, out, scale):
         state, slots, rows = cache.state, cache.slots, step.n_rows
@@ -206,12 +202,14 @@ class StateSpaceMixer(_ScanMixer, Branch):
         conv = recurrent.causal_conv_silu(proj, conv_col, self.w_conv, self.b_conv, state, self.conv_off, slots, step.token_row, step.row_start)
         recurrent.conv_state_update(proj, conv_col, self.conv_channels, self.taps, state, self.conv_off, slots, step.row_start, rows)
         bn = self.groups * self.n
-
-        def scan(state, slots, row_start, rows, states_only=False, decays=None):
-            return recurrent.state_scan(self.mode, conv, self.inner, self.inner + bn, 0, proj, dt_off, dt_off, self.a_log, self.dt_bias, self.skip, state, 0, slots, row_start,
-                                        rows, self.heads, self.groups, self.n, self.n_padded, self.e, states_only=states_only, decays=decays)
-
-        y = self._walk(scan, step, state, slots, self.e * self.n_padded, self.e)
+        chunks = step.host.get("scan_chunks", 0)
+        if chunks:  # long rows in bfloat16: the tensor cores walk the step in chunks
+            y = recurrent.chunked_scan(recurrent.KIND_STATE_SPACE, conv[:, self.inner :], conv[:, self.inner + bn :], conv, proj, dt_off, 0, state, 0, slots,
+                                       step.extra["scan_chunk_start"], step.extra["scan_chunk_row"], chunks, self.heads, self.groups, self.n, self.n_padded, self.e,
+                                       a_log=self.a_log, dt_bias=self.dt_bias, skip=self.skip).view(proj.shape[0], self.inner)
+        else:
+            y = recurrent.state_scan(self.mode, conv, self.inner, self.inner + bn, 0, proj, dt_off, dt_off, self.a_log, self.dt_bias, self.skip, state, 0, slots, step.row_start,
+                                     rows, self.heads, self.groups, self.n, self.n_padded, self.e)
         recurrent.gated_group_norm(y, proj, col0, self.norm, self.inner // self.norm_groups, True, self.eps, self.dtype, scale=scale, out=out)
 
 
@@ -245,8 +243,11 @@ class MatrixMemoryMixer(_ScanMixer, Branch):
     def load_core(self, tensors: Mapping[str, torch.Tensor]) -> None:
         self.b_i, self.b_f, self.norm = self._float(tensors["i.b"]), self._float(tensors["f.b"]), self._float(tensors["norm"])
 
+    def kernel_modules(self):
+        return super().kernel_modules() + _chunked_module(self.dtype)
+
     def step_plans(self):
-        return recurrent.segment_planner(self.dtype)
+        return recurrent.chunk_planner(self.dtype)
 
     def core(self, proj, col0, step, cache, out, scale):
         if scale != 1.0:
@@ -256,12 +257,14 @@ class MatrixMemoryMixer(_ScanMixer, Branch):
         g_off = v_off + self.core_width
         i_off = g_off + self.core_width
         gates = recurrent.matrix_memory_gates(proj, i_off, i_off + self.heads, self.b_i, self.b_f, self.cap, state, self.max_off, slots, step.row_start, step.n_rows, self.heads)
-
-        def scan(state, slots, row_start, rows, states_only=False, decays=None):
-            return recurrent.matrix_memory_scan(proj, k_off, col0, v_off, gates, state, 0, slots, row_start, rows, self.heads, self.n, self.n_padded, self.e, self.n ** -0.5,
-                                                states_only=states_only, decays=decays)
-
-        y = self._walk(scan, step, state, slots, self.per_head, self.e + 1)
+        chunks = step.host.get("scan_chunks", 0)
+        if chunks:  # long rows in bfloat16: the tensor cores walk the step in chunks
+            flat = gates.view(proj.shape[0], 4 * self.heads)
+            y = recurrent.chunked_scan(recurrent.KIND_GIVEN, proj[:, k_off:], proj[:, col0:], proj[:, v_off:], flat, 3 * self.heads, self.heads, state, 0, slots,
+                                       step.extra["scan_chunk_start"], step.extra["scan_chunk_row"], chunks, self.heads, self.heads, self.n, self.n_padded, self.e,
+                                       sums_keys=True, q_scale=self.n ** -0.5, columns=recurrent.matrix_memory_columns(self.e))
+        else:
+            y = recurrent.matrix_memory_scan(proj, k_off, col0, v_off, gates, state, 0, slots, step.row_start, step.n_rows, self.heads, self.n, self.n_padded, self.e, self.n ** -0.5)
         recurrent.matrix_memory_norm(y, gates, proj, g_off, self.norm, self.e, self.eps, out)
 
 

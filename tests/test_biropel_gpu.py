@@ -470,42 +470,52 @@ def test_the_matrix_memory_kernels(shape):
     assert torch.equal(state[2], after[2])
 
 
-def test_long_rows_in_segments():
-    """The matrix memory and the state-space scan with long rows cut into segments that are walked side by side: the one-pass results and states to rounding, from
-    states that are not zero, beside rows that are not cut."""
+@pytest.mark.parametrize("shape", [(3, 40, 24), (2, 128, 128), (4, 7, 5), (1, 250, 65), (6, 64, 100)])
+def test_scans_in_chunks(shape):
+    """The matrix memory and the state-space scan in chunks on the tensor cores against the one-pass scan: rows of 1 to 700 tokens, from states that are not zero, keys
+    shared by several heads, decays from nearly 1 to nearly 0, columns of a wider matrix."""
     from hyperion_b200.ops import recurrent
 
-    heads, n, e, n_padded, cap = 3, 40, 24, 40, 5.0
-    counts = [700, 5, 1100, 300]
+    heads, n, e = shape
+    n_padded, cap = -(-n // 4) * 4, 5.0
+    counts = [300, 1, 64, 700, 63, 129]
     x, bi, bf, start = _memory_case(heads, n, e, counts, 5)
-    cut = recurrent.plan_segments(counts)
-    seg_start, seg_row = (torch.tensor(v, dtype=torch.int32).cuda() for v in cut)
+    bf[0] = 9.0  # this head hardly forgets
+    cut = recurrent.plan_chunks(counts)
+    assert sum(counts) == cut[0][-1] and max(b - a for a, b in zip(cut[0], cut[0][1:])) == 64 and cut[1] == [0] * 5 + [1, 2] + [3] * 11 + [4] + [5] * 3
+    assert recurrent.plan_chunks([5, 100, 127]) is None
+    chunk_start, chunk_row = (torch.tensor(v, dtype=torch.int32).cuda() for v in cut)
     per_head = (e + 1) * n_padded
     m_off = heads * per_head
-    begin = torch.zeros(5, m_off + 4)
-    begin[:, :m_off] = torch.randn(5, m_off, generator=torch.Generator().manual_seed(1))
-    slots = torch.tensor([3, 0, 4, 1], dtype=torch.int32).cuda()
+    record = -(-(m_off + heads) // 4) * 4
+    begin = torch.zeros(8, record)
+    begin[:, :m_off] = torch.randn(8, m_off, generator=torch.Generator().manual_seed(1))
+    begin[:, :m_off].view(8, heads, e + 1, n_padded)[..., n:] = 0
+    slots = torch.tensor([3, 0, 4, 1, 7, 6], dtype=torch.int32).cuda()
     dev, i_off, rows_of = x.cuda(), 2 * heads * n + heads * e, start.cuda()
 
-    def memory_scan(gates):
-        return lambda s, sl, rs, rows, states_only=False, decays=None: recurrent.matrix_memory_scan(dev, heads * n, 0, 2 * heads * n, gates, s, 0, sl, rs, rows, heads, n, n_padded, e,
-                                                                                                   n ** -0.5, states_only=states_only, decays=decays)
+    def compare(y, z, one, many):
+        scale = y.abs().mean(dim=0, keepdim=True) + y.abs().mean()
+        assert ((y - z).abs() / scale).max() <= 0.1 and ((y - z) / scale).pow(2).mean().sqrt() <= 1e-2
+        assert (one - many).abs().max() <= 2e-2 * one.abs().max() and ((one - many).pow(2).mean() / one.pow(2).mean()).sqrt() <= 5e-3
 
     one, many = begin.cuda(), begin.cuda()
-    gates = [recurrent.matrix_memory_gates(dev, i_off, i_off + heads, bi.cuda(), bf.cuda(), cap, s, m_off, slots, rows_of, 4, heads) for s in (one, many)]
-    y = memory_scan(gates[0])(one, slots, rows_of, 4)[..., : e + 1]
-    z = recurrent.scan_in_segments(memory_scan(gates[1]), per_head, many, 0, slots, seg_start, seg_row, len(cut[1]), heads)[..., : e + 1]
-    assert (y - z).abs().max() <= 1e-4 * y.abs().max() and (one - many).abs().max() <= 1e-4 * one.abs().max()
-    a_log, dt_bias, skip = torch.log(torch.tensor([0.05, 0.5, 1.5])).cuda(), torch.tensor([-3.0, -2.0, -1.0]).cuda(), torch.ones(heads).cuda()
-    one, many = begin[:, : heads * e * n_padded].contiguous().cuda(), begin[:, : heads * e * n_padded].contiguous().cuda()
-
-    def state_scan(s, sl, rs, rows, states_only=False, decays=None):
-        return recurrent.state_scan(recurrent.MODE_STATE_SPACE, dev, heads * n, 0, 2 * heads * n, dev, i_off, i_off, a_log, dt_bias, skip, s, 0, sl, rs, rows, heads, heads, n, n_padded, e,
-                                    states_only=states_only, decays=decays)
-
-    y = state_scan(one, slots, rows_of, 4)
-    z = recurrent.scan_in_segments(state_scan, e * n_padded, many, 0, slots, seg_start, seg_row, len(cut[1]), heads)
-    assert (y - z).abs().max() <= 1e-4 * y.abs().max() and (one - many).abs().max() <= 1e-4 * one.abs().max()
+    gates = [recurrent.matrix_memory_gates(dev, i_off, i_off + heads, bi.cuda(), bf.cuda(), cap, s, m_off, slots, rows_of, len(counts), heads) for s in (one, many)]
+    y = recurrent.matrix_memory_scan(dev, heads * n, 0, 2 * heads * n, gates[0], one, 0, slots, rows_of, len(counts), heads, n, n_padded, e, n ** -0.5)
+    z = recurrent.chunked_scan(recurrent.KIND_GIVEN, dev[:, heads * n :], dev, dev[:, 2 * heads * n :], gates[1].view(len(x), 4 * heads), 3 * heads, heads, many, 0, slots, chunk_start,
+                               chunk_row, len(cut[1]), heads, heads, n, n_padded, e, sums_keys=True, q_scale=n ** -0.5, columns=y.shape[2])
+    compare(y[..., : e + 1], z[..., : e + 1], one, many)
+    groups = 2 if heads % 2 == 0 else 1
+    a_log, dt_bias = torch.linspace(-4, 1, heads).cuda(), torch.linspace(-5, 3, heads).cuda()
+    skip = torch.randn(heads, generator=torch.Generator().manual_seed(2)).cuda()
+    one, many = (begin[:, : heads * e * n_padded].contiguous().cuda() for _ in range(2))
+    for s in (one, many):
+        s.view(8, heads, e, n_padded)[..., n:] = 0
+    y = recurrent.state_scan(recurrent.MODE_STATE_SPACE, dev, heads * n, 0, 2 * heads * n, dev, i_off, i_off, a_log, dt_bias, skip, one, 0, slots, rows_of, len(counts), heads, groups, n,
+                             n_padded, e)
+    z = recurrent.chunked_scan(recurrent.KIND_STATE_SPACE, dev[:, heads * n :], dev, dev[:, 2 * heads * n :], dev, i_off, 0, many, 0, slots, chunk_start, chunk_row, len(cut[1]), heads,
+                               groups, n, n_padded, e, a_log=a_log, dt_bias=dt_bias, skip=skip)
+    compare(y.view(z.shape), z, one, many)
 
 
 # ------------------------------------------------------------------------------------------ whole models
@@ -650,7 +660,7 @@ def test_pages_of_a_window_go_back(folders):
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("name", ["open", "open_64"])
 def test_a_key_far_away_among_hundreds(folders, name, dtype):
-    """No window: the marker stands 1, 7, 8, 9, 64, 300 and 690 places behind the last query among 700 tokens (in bfloat16 the prompt's recurrence runs in segments), as a
+    """No window: the marker stands 1, 7, 8, 9, 64, 300 and 690 places behind the last query among 700 tokens (in bfloat16 the prompt's recurrence runs in chunks), as a
     whole prompt and with the tail decoded; queries have a temperature that steps at every 100 positions."""
     vocab = ALONE[name]["vocab"]
     engine = engine_for(folders[name], dtype, page_size=8, max_tokens=1536)
@@ -665,7 +675,7 @@ def test_a_key_far_away_among_hundreds(folders, name, dtype):
 
 @pytest.mark.parametrize("name", ["open", "states_wide", "memory_wide", "stretched_64"])
 def test_states_over_long_texts(folders, name):
-    """1,300 tokens: one prompt (in bfloat16 the scans run in segments), portions whose sizes straddle the segments' length, and a decoded tail."""
+    """1,300 tokens: one prompt (in bfloat16 the scans run in chunks), portions that end inside a chunk or hold none, and a decoded tail."""
     ids = ids_for(21, 1300, ALONE[name]["vocab"])
     want = plain_logits(folders[name], ids)
     for dtype in ("float32", "bfloat16"):
