@@ -37,11 +37,12 @@ struct ChunkArgs {
     int sums;            // 1: the state has a row for the sum of keys
     float q_scale;
     int by_four;         // columns and strides allow 16-byte loads
+    int by_two;          // outputs may be stored in pairs
 };
 
 __device__ __forceinline__ float softplus_of(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
-// L[j] (the running sum of ln a) and the step of every token of the chunk (threads 0 .. 63 of the block); past the end: L stays, step 0.
+// L[j] (the running sum of log2 a) and the step of every token of the chunk (threads 0 .. 63 of the block); past the end: L stays, step 0.
 template <int KIND>
 __device__ __forceinline__ void chunk_gates(const ChunkArgs& a, int first, int count, int head, float* L, float* step, float* warp_total) {
     const int j = threadIdx.x, lane = j & 31;
@@ -67,7 +68,7 @@ __device__ __forceinline__ void chunk_gates(const ChunkArgs& a, int first, int c
     }
     __syncthreads();
     if (j < CHUNK) {
-        L[j] = j >= 32 ? sum + *warp_total : sum;
+        L[j] = (j >= 32 ? sum + *warp_total : sum) * 1.4426950408889634f;
         step[j] = b;
     }
     __syncthreads();
@@ -86,14 +87,26 @@ struct Tile {
     int live, columns, quads;  // quads: pieces per row
     bool by_four;
 
+    // a walk over the tile's pieces in steps of THREADS without a division per piece
     template <int THREADS>
-    __device__ __forceinline__ void fetch(int base, float (&x)[AHEAD][4]) const {
+    struct Walk {
+        int r, quad, rows, rest, quads;
+        __device__ __forceinline__ Walk(int first, int quads_) : r(first / quads_), quad(first % quads_), rows(THREADS / quads_), rest(THREADS % quads_), quads(quads_) {}
+        __device__ __forceinline__ void next() {
+            r += rows;
+            quad += rest;
+            if (quad >= quads) { quad -= quads; ++r; }
+        }
+    };
+
+    template <int THREADS>
+    __device__ __forceinline__ void fetch(Walk<THREADS> at, float (&x)[AHEAD][4]) const {
 #pragma unroll
-        for (int u = 0; u < AHEAD; ++u) {
-            const int item = base + u * THREADS, r = item / quads, c = (item - r * quads) * 4;
+        for (int u = 0; u < AHEAD; ++u, at.next()) {
             x[u][0] = x[u][1] = x[u][2] = x[u][3] = 0.f;
-            if (r < live) {
-                const float* p = src + (size_t)r * stride + c;
+            const int c = at.quad * 4;
+            if (at.r < live) {
+                const float* p = src + (size_t)at.r * stride + c;
                 if (by_four && c + 4 <= columns) {
                     load4(p, x[u]);
                 } else {
@@ -105,16 +118,15 @@ struct Tile {
     }
 
     template <int THREADS>
-    __device__ __forceinline__ void place(int base, const float (&x)[AHEAD][4], __nv_bfloat16* dst, int ld, const float* row_factor, float factor) const {
+    __device__ __forceinline__ void place(Walk<THREADS> at, const float (&x)[AHEAD][4], __nv_bfloat16* dst, int ld, const float* row_factor, float factor) const {
 #pragma unroll
-        for (int u = 0; u < AHEAD; ++u) {
-            const int item = base + u * THREADS, r = item / quads, c = (item - r * quads) * 4;
-            if (r >= CHUNK) continue;
-            const float f = row_factor ? row_factor[r] * factor : factor;
+        for (int u = 0; u < AHEAD; ++u, at.next()) {
+            if (at.r >= CHUNK) continue;
+            const float f = row_factor ? row_factor[at.r] * factor : factor;
             uint2 packed;
             packed.x = pack(x[u][0] * f, x[u][1] * f);
             packed.y = pack(x[u][2] * f, x[u][3] * f);
-            *reinterpret_cast<uint2*>(dst + (size_t)r * ld + c) = packed;
+            *reinterpret_cast<uint2*>(dst + at.r * ld + at.quad * 4) = packed;
         }
     }
 };
@@ -137,7 +149,7 @@ template <int KIND, int NMAX, int ETILE>
 __global__ void __launch_bounds__(2 * ETILE) chunk_states_kernel(const ChunkArgs a) {
     constexpr int THREADS = 2 * ETILE;
     extern __shared__ __align__(16) unsigned char memory[];
-    __shared__ float L[CHUNK], step[CHUNK], warp_total;
+    __shared__ __align__(16) float L[CHUNK], step[CHUNK], warp_total;
     const int chunk = blockIdx.x, head = blockIdx.y, e0 = blockIdx.z * ETILE;
     const int first = a.start[chunk], count = a.start[chunk + 1] - first;
     const int n16 = (a.n + 15) & ~15, k_ld = n16 + 8;
@@ -149,20 +161,22 @@ __global__ void __launch_bounds__(2 * ETILE) chunk_states_kernel(const ChunkArgs
 
     const Tile keys{a.k + (size_t)first * a.k_stride + (size_t)group * a.n, (size_t)a.k_stride, count, a.n, n16 / 4, a.by_four != 0};
     const Tile values{a.v + (size_t)first * a.v_stride + (size_t)head * a.e + e0, (size_t)a.v_stride, count, min(ETILE, a.e - e0), ETILE / 4, a.by_four != 0};
+    const Tile::Walk<THREADS> key_walk(threadIdx.x, keys.quads), value_walk(threadIdx.x, ETILE / 4);
     float x[AHEAD][4], y[AHEAD][4];
-    keys.fetch<THREADS>(threadIdx.x, x);
-    values.fetch<THREADS>(threadIdx.x, y);  // AHEAD pieces per thread are the whole tile
+    keys.fetch(key_walk, x);
+    values.fetch(value_walk, y);  // AHEAD pieces per thread are the whole tile
     chunk_gates<KIND>(a, first, count, head, L, step, &warp_total);
     const float last = L[CHUNK - 1];
-    if (threadIdx.x < CHUNK) step[threadIdx.x] *= expf(last - L[threadIdx.x]);  // the weight of a token in the chunk's sum
-    if (threadIdx.x == 0 && blockIdx.z == 0) a.decays[(size_t)chunk * a.heads + head] = expf(last);
-    keys.place<THREADS>(threadIdx.x, x, ks, k_ld, nullptr, 1.f);
+    if (threadIdx.x < CHUNK) step[threadIdx.x] *= exp2f(last - L[threadIdx.x]);  // the weight of a token in the chunk's sum
+    if (threadIdx.x == 0 && blockIdx.z == 0) a.decays[(size_t)chunk * a.heads + head] = exp2f(last);
+    keys.place(key_walk, x, ks, k_ld, nullptr, 1.f);
     for (int base = threadIdx.x + AHEAD * THREADS; base < CHUNK * keys.quads; base += AHEAD * THREADS) {
-        keys.fetch<THREADS>(base, x);
-        keys.place<THREADS>(base, x, ks, k_ld, nullptr, 1.f);
+        const Tile::Walk<THREADS> walk(base, keys.quads);
+        keys.fetch(walk, x);
+        keys.place(walk, x, ks, k_ld, nullptr, 1.f);
     }
     __syncthreads();  // the weights are there
-    values.place<THREADS>(threadIdx.x, y, vs, v_ld, step, 1.f);
+    values.place(value_walk, y, vs, v_ld, step, 1.f);
     __syncthreads();
 
     float acc[NMAX / 8][4];
@@ -252,85 +266,102 @@ __device__ __forceinline__ void copy_ahead(uint32_t to, const void* from, bool l
 }
 
 // The outputs of a chunk from its start state: grid (chunks, heads, tiles of value columns); warp w owns tokens 16 (w % 4) .. + 15 and 64 of the tile's columns.
+// First the queries meet the start state; then keys and values take the state's place in shared memory, which lets two blocks share an SM.
 template <int KIND, int ETILE>
-__global__ void __launch_bounds__(2 * ETILE) chunk_outputs_kernel(const ChunkArgs a) {
+__global__ void __launch_bounds__(2 * ETILE, 256 / ETILE) chunk_outputs_kernel(const ChunkArgs a) {
     constexpr int THREADS = 2 * ETILE, COLUMNS = 64;
     extern __shared__ __align__(16) unsigned char memory[];
-    __shared__ float L[CHUNK], step[CHUNK], warp_total;
+    __shared__ __align__(16) float L[CHUNK], step[CHUNK], warp_total;
     const int chunk = blockIdx.x, head = blockIdx.y, e0 = blockIdx.z * ETILE;
     const int first = a.start[chunk], count = a.start[chunk + 1] - first;
     const int n16 = (a.n + 15) & ~15, ld = n16 + 8;
     constexpr int v_ld = ETILE + 8;
     __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(memory);
-    __nv_bfloat16* ks = qs + CHUNK * ld;
-    __nv_bfloat16* s_hi = ks + CHUNK * ld;
+    __nv_bfloat16* s_hi = qs + CHUNK * ld;
     __nv_bfloat16* s_lo = s_hi + ETILE * ld;
-    __nv_bfloat16* vs = s_lo + ETILE * ld;
+    __nv_bfloat16* ks = s_hi;  // CHUNK <= ETILE rows
+    __nv_bfloat16* vs = ks + CHUNK * ld;
     const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) & 3, column0 = (threadIdx.x >> 7) * COLUMNS;
     const int group = head / (a.heads / a.groups);
     const __nv_bfloat16* begin = a.begins + ((size_t)chunk * a.heads + head) * (a.e + a.sums) * 2 * n16;
 
-    for (int item = threadIdx.x; item < ETILE * (n16 / 4); item += THREADS) {  // both halves of a state row lie side by side: n16 / 8 pieces each
-        const int r = item / (n16 / 4), piece = item - r * (n16 / 4), half = piece >= n16 / 8, c = (piece - half * (n16 / 8)) * 8;
-        const bool live = e0 + r < a.e;
-        copy_ahead(shared_address((half ? s_lo : s_hi) + r * ld + c), begin + (size_t)(live ? e0 + r : 0) * 2 * n16 + half * n16 + c, live);
+    {
+        const int pieces = n16 / 4;  // both halves of a state row lie side by side: n16 / 8 pieces of 16 bytes each
+        Tile::Walk<THREADS> at(threadIdx.x, pieces);
+        for (; at.r < ETILE; at.next()) {
+            const int half = at.quad >= pieces / 2, c = (at.quad - half * (pieces / 2)) * 8;
+            const bool live = e0 + at.r < a.e;
+            copy_ahead(shared_address((half ? s_lo : s_hi) + at.r * ld + c), begin + (size_t)(live ? e0 + at.r : 0) * 2 * n16 + at.quad * 8, live);
+        }
     }
     asm volatile("cp.async.commit_group;");
     const Tile queries{a.q + (size_t)first * a.q_stride + (size_t)group * a.n, (size_t)a.q_stride, count, a.n, n16 / 4, a.by_four != 0};
     const Tile keys{a.k + (size_t)first * a.k_stride + (size_t)group * a.n, (size_t)a.k_stride, count, a.n, n16 / 4, a.by_four != 0};
     const Tile values{a.v + (size_t)first * a.v_stride + (size_t)head * a.e + e0, (size_t)a.v_stride, count, min(ETILE, a.e - e0), ETILE / 4, a.by_four != 0};
-    {
-        float x[AHEAD][4], y[AHEAD][4], z[AHEAD][4];
-        queries.fetch<THREADS>(threadIdx.x, x);
-        keys.fetch<THREADS>(threadIdx.x, y);
-        values.fetch<THREADS>(threadIdx.x, z);  // AHEAD pieces per thread are the whole tile
-        chunk_gates<KIND>(a, first, count, head, L, step, &warp_total);
-        queries.place<THREADS>(threadIdx.x, x, qs, ld, nullptr, a.q_scale);
-        keys.place<THREADS>(threadIdx.x, y, ks, ld, nullptr, 1.f);
-        values.place<THREADS>(threadIdx.x, z, vs, v_ld, nullptr, 1.f);
-        for (int base = threadIdx.x + AHEAD * THREADS; base < CHUNK * keys.quads; base += AHEAD * THREADS) {
-            queries.fetch<THREADS>(base, x);
-            keys.fetch<THREADS>(base, y);
-            queries.place<THREADS>(base, x, qs, ld, nullptr, a.q_scale);
-            keys.place<THREADS>(base, y, ks, ld, nullptr, 1.f);
-        }
+    const Tile::Walk<THREADS> walk(threadIdx.x, n16 / 4), value_walk(threadIdx.x, ETILE / 4);
+    float x[AHEAD][4], y[AHEAD][4];
+    queries.fetch(walk, x);
+    chunk_gates<KIND>(a, first, count, head, L, step, &warp_total);
+    queries.place(walk, x, qs, ld, nullptr, a.q_scale);
+    for (int base = threadIdx.x + AHEAD * THREADS; base < CHUNK * queries.quads; base += AHEAD * THREADS) {
+        const Tile::Walk<THREADS> more(base, queries.quads);
+        queries.fetch(more, x);
+        queries.place(more, x, qs, ld, nullptr, a.q_scale);
     }
     asm volatile("cp.async.wait_all;");
     __syncthreads();
 
     const int row0 = warp * 16, g = lane >> 2, t2 = (lane & 3) * 2;
-    if (row0 < count) {
-        float acc[COLUMNS / 8][4], score[CHUNK / 8][4];
+    const bool active = row0 < count;
+    float acc[COLUMNS / 8][4];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-            score[i][0] = score[i][1] = score[i][2] = score[i][3] = 0.f;
-        }
+    for (int i = 0; i < COLUMNS / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    const int spot = ((lane >> 4) * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8;  // this lane's row of the four matrices of a step, rows n-major
+    if (active) {
         for (int c = 0; c < n16; c += 16) {
             uint32_t qa[4];
             load_matrices(qa, shared_address(qs + (row0 + (lane & 15)) * ld + c + (lane >> 4) * 8));
-            const int at = ((lane >> 4) * 8 + (lane & 7)) * ld + c + ((lane >> 3) & 1) * 8;
 #pragma unroll
             for (int i = 0; i < COLUMNS / 16; ++i) {
                 uint32_t b[4];
-                load_matrices(b, shared_address(s_hi + (column0 + i * 16) * ld + at));
+                load_matrices(b, shared_address(s_hi + (column0 + i * 16) * ld + spot + c));
                 multiply(acc[2 * i], qa, b[0], b[1]);
                 multiply(acc[2 * i + 1], qa, b[2], b[3]);
-                load_matrices(b, shared_address(s_lo + (column0 + i * 16) * ld + at));
+                load_matrices(b, shared_address(s_lo + (column0 + i * 16) * ld + spot + c));
                 multiply(acc[2 * i], qa, b[0], b[1]);
                 multiply(acc[2 * i + 1], qa, b[2], b[3]);
             }
+        }
+    }
+    keys.fetch(walk, x);
+    values.fetch(value_walk, y);  // AHEAD pieces per thread are the whole tile
+    __syncthreads();  // the state has been read
+    keys.place(walk, x, ks, ld, nullptr, 1.f);
+    for (int base = threadIdx.x + AHEAD * THREADS; base < CHUNK * keys.quads; base += AHEAD * THREADS) {
+        const Tile::Walk<THREADS> more(base, keys.quads);
+        keys.fetch(more, x);
+        keys.place(more, x, ks, ld, nullptr, 1.f);
+    }
+    values.place(value_walk, y, vs, v_ld, nullptr, 1.f);
+    __syncthreads();
+    if (active) {
+        float score[CHUNK / 8][4];
+#pragma unroll
+        for (int i = 0; i < CHUNK / 8; ++i) score[i][0] = score[i][1] = score[i][2] = score[i][3] = 0.f;
+        for (int c = 0; c < n16; c += 16) {
+            uint32_t qa[4];
+            load_matrices(qa, shared_address(qs + (row0 + (lane & 15)) * ld + c + (lane >> 4) * 8));
 #pragma unroll
             for (int i = 0; i < CHUNK / 16; ++i) {
                 if (i > warp) continue;  // keys behind every query of this warp
                 uint32_t b[4];
-                load_matrices(b, shared_address(ks + i * 16 * ld + at));
+                load_matrices(b, shared_address(ks + i * 16 * ld + spot + c));
                 multiply(score[2 * i], qa, b[0], b[1]);
                 multiply(score[2 * i + 1], qa, b[2], b[3]);
             }
         }
         const float top = L[row0 + g], bottom = L[row0 + g + 8];
-        const float fade_top = expf(top), fade_bottom = expf(bottom);
+        const float fade_top = exp2f(top), fade_bottom = exp2f(bottom);
 #pragma unroll
         for (int i = 0; i < COLUMNS / 8; ++i) {
             acc[i][0] *= fade_top; acc[i][1] *= fade_top;
@@ -339,13 +370,16 @@ __global__ void __launch_bounds__(2 * ETILE) chunk_outputs_kernel(const ChunkArg
         float sum_top = 0.f, sum_bottom = 0.f;
 #pragma unroll
         for (int i = 0; i < CHUNK / 8; ++i) {
+            if (i > 2 * warp + 1) continue;
+            const float2 ahead = *reinterpret_cast<const float2*>(&L[i * 8 + t2]), weight = *reinterpret_cast<const float2*>(&step[i * 8 + t2]);
 #pragma unroll
-            for (int x = 0; x < 2; ++x) {
-                const int j = i * 8 + t2 + x;
-                score[i][x] = j <= row0 + g ? score[i][x] * (expf(top - L[j]) * step[j]) : 0.f;
-                score[i][2 + x] = j <= row0 + g + 8 ? score[i][2 + x] * (expf(bottom - L[j]) * step[j]) : 0.f;
-                sum_top += score[i][x];
-                sum_bottom += score[i][2 + x];
+            for (int z = 0; z < 2; ++z) {
+                const int j = i * 8 + t2 + z;
+                const float l = z ? ahead.y : ahead.x, b = z ? weight.y : weight.x;
+                score[i][z] = j <= row0 + g ? score[i][z] * (exp2f(top - l) * b) : 0.f;
+                score[i][2 + z] = j <= row0 + g + 8 ? score[i][2 + z] * (exp2f(bottom - l) * b) : 0.f;
+                sum_top += score[i][z];
+                sum_bottom += score[i][2 + z];
             }
         }
 #pragma unroll
@@ -366,14 +400,26 @@ __global__ void __launch_bounds__(2 * ETILE) chunk_outputs_kernel(const ChunkArg
         for (int half = 0; half < 2; ++half) {
             const int i = row0 + g + half * 8;
             if (i >= count) continue;
-            float* dst = a.out + ((size_t)(first + i) * a.heads + head) * a.out_e + e0 + column0;
-            const float* own = a.v + (size_t)(first + i) * a.v_stride + (size_t)head * a.e + e0 + column0;
+            float* dst = a.out + ((size_t)(first + i) * a.heads + head) * a.out_e + e0 + column0 + t2;
+            const float* own = a.v + (size_t)(first + i) * a.v_stride + (size_t)head * a.e + e0 + column0 + t2;
+            const int live = a.e - e0 - column0 - t2;  // entries from this lane's first one to the head's end
+            float mine[COLUMNS / 8][2];
+            if (KIND == KIND_STATE_SPACE) {
+#pragma unroll
+                for (int c = 0; c < COLUMNS / 8; ++c) {
+#pragma unroll
+                    for (int z = 0; z < 2; ++z) mine[c][z] = c * 8 + z < live ? skip * own[c * 8 + z] : 0.f;
+                }
+            }
 #pragma unroll
             for (int c = 0; c < COLUMNS / 8; ++c) {
-#pragma unroll
-                for (int x = 0; x < 2; ++x) {
-                    const int column = c * 8 + t2 + x;
-                    if (e0 + column0 + column < a.e) dst[column] = KIND == KIND_STATE_SPACE ? fmaf(skip, own[column], acc[c][2 * half + x]) : acc[c][2 * half + x];
+                float2 o = make_float2(acc[c][2 * half], acc[c][2 * half + 1]);
+                if (KIND == KIND_STATE_SPACE) { o.x += mine[c][0]; o.y += mine[c][1]; }
+                if (a.by_two && c * 8 + 1 < live) {
+                    *reinterpret_cast<float2*>(dst + c * 8) = o;
+                } else {
+                    if (c * 8 < live) dst[c * 8] = o.x;
+                    if (c * 8 + 1 < live) dst[c * 8 + 1] = o.y;
                 }
             }
         }
@@ -425,7 +471,7 @@ int launch_states(const ChunkArgs& a, int chunks, cudaStream_t stream) {
 
 template <int KIND, int ETILE>
 int launch_outputs(const ChunkArgs& a, int chunks, cudaStream_t stream) {
-    const int n16 = (a.n + 15) & ~15, bytes = (2 * CHUNK + 2 * ETILE) * (n16 + 8) * 2 + CHUNK * (ETILE + 8) * 2;
+    const int n16 = (a.n + 15) & ~15, state = 2 * ETILE * (n16 + 8) * 2, tiles = CHUNK * (n16 + 8) * 2 + CHUNK * (ETILE + 8) * 2, bytes = CHUNK * (n16 + 8) * 2 + (state > tiles ? state : tiles);
     const int status = allow_shared(chunk_outputs_kernel<KIND, ETILE>, bytes);
     if (status) return status;
     chunk_outputs_kernel<KIND, ETILE><<<dim3(chunks, a.heads, (a.e + ETILE - 1) / ETILE), 2 * ETILE, bytes, stream>>>(a);
@@ -464,7 +510,7 @@ HB_EXPORT int hb_chunked_scan(int kind, const float* k, int k_stride, const floa
     if (kind == KIND_STATE_SPACE && (!a_log || !dt_bias || !skip || sums)) return HB_BAD_ARGUMENT;
     const int by_four = ((k_stride | q_stride | v_stride | n | e) & 3) == 0 && (((uintptr_t)k | (uintptr_t)q | (uintptr_t)v) & 15) == 0;
     const ChunkArgs a{k, q, v, k_stride, q_stride, v_stride, gate, gate_stride, decay_off, step_off, a_log, dt_bias, skip, ends, (size_t)heads * (e + sums) * n_padded, decays,
-                      (__nv_bfloat16*)begins, start, out, out_e, heads, groups, n, n_padded, e, sums, q_scale, by_four};
+                      (__nv_bfloat16*)begins, start, out, out_e, heads, groups, n, n_padded, e, sums, q_scale, by_four, out_e % 2 == 0 && ((uintptr_t)out & 7) == 0};
     if (kind == KIND_STATE_SPACE) return launch_chunks<KIND_STATE_SPACE>(a, chunks, state, slot_stride, state_off, slots, chunk_row, stream);
     if (kind == KIND_GIVEN) return launch_chunks<KIND_GIVEN>(a, chunks, state, slot_stride, state_off, slots, chunk_row, stream);
     return HB_BAD_ARGUMENT;

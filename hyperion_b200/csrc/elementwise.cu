@@ -853,12 +853,34 @@ __global__ void sigmoid_gate_kernel(T* __restrict__ x, int x_stride, const float
     }
 }
 
+// Four columns per access, for rows of whole pieces.
+template <typename T>
+__global__ void sigmoid_gate4_kernel(T* __restrict__ x, int x_stride, const float* __restrict__ gate, int gate_stride, int gate_off, float scale, int width) {
+    const int t = blockIdx.y, c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (c >= width) return;
+    float g[4], v[4];
+    load4(gate + (size_t)t * gate_stride + gate_off + c, g);
+    load4(x + (size_t)t * x_stride + c, v);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] *= scale / (1.f + expf(-g[e]));
+    store4(x + (size_t)t * x_stride + c, v);
+}
+
 HB_EXPORT int hb_sigmoid_gate(void* x, int is_bf16, int x_stride, const float* gate, int gate_stride, int gate_off, float scale, int tokens, int width,
                               cudaStream_t stream) {
     if (tokens <= 0 || width <= 0) return 0;
     for (int first = 0; first < tokens; first += 65535) {
         const int count = tokens - first < 65535 ? tokens - first : 65535;
         const dim3 grid((width + 255) / 256 < 8 ? (width + 255) / 256 : 8, count);
+        if (((width | x_stride | gate_stride | gate_off) & 3) == 0 && ((uintptr_t)gate & 15) == 0 && ((uintptr_t)x & (is_bf16 ? 7 : 15)) == 0) {
+            const dim3 fours((width / 4 + 255) / 256, count);
+            if (is_bf16)
+                sigmoid_gate4_kernel<<<fours, 256, 0, stream>>>((__nv_bfloat16*)x + (size_t)first * x_stride, x_stride, gate + (size_t)first * gate_stride, gate_stride, gate_off,
+                                                                scale, width);
+            else
+                sigmoid_gate4_kernel<<<fours, 256, 0, stream>>>((float*)x + (size_t)first * x_stride, x_stride, gate + (size_t)first * gate_stride, gate_stride, gate_off, scale, width);
+            continue;
+        }
         if (is_bf16)
             sigmoid_gate_kernel<<<grid, 256, 0, stream>>>((__nv_bfloat16*)x + (size_t)first * x_stride, x_stride, gate + (size_t)first * gate_stride, gate_stride,
                                                           gate_off, scale, width);

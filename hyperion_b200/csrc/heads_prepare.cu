@@ -567,17 +567,6 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
                                                                     const int* __restrict__ token_row, int page_size, int pages, int* status, const TurnArgs turn) {
     __shared__ float2 turned[TURN ? TURN_PAIRS : 1];  // (cosine, sine) of every pair at this token's position
     let_next_kernel_start();
-    if constexpr (TURN) {  // positions come with the step's one copy from the host, not from a kernel
-        if (turn.inv_freq) {
-            const float at = (float)positions[blockIdx.x];
-            for (int i = threadIdx.x; i < turn.rot_dims / 2; i += STORE_THREADS) {
-                float sine, cosine;
-                sincosf(at * turn.inv_freq[i], &sine, &cosine);
-                turned[i] = make_float2(cosine * turn.amplitude, sine * turn.amplitude);
-            }
-            __syncthreads();
-        }
-    }
     wait_for_previous_kernels();
     const int t = blockIdx.x, runs = (v_dim + head_dim - 1) / head_dim, groups = STORE_THREADS / lanes, lane = threadIdx.x & (lanes - 1);
     const int first_item = blockIdx.y * groups * JOBS + threadIdx.x / lanes;
@@ -626,6 +615,17 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
             const HeadJob<TO> job = job_of(first_item + u * groups);
             const int i = lane * VEC;
             if (i < job.dim) fetch_entries<VEC>(row + job.col + i, bias ? bias + job.col + i : nullptr, kept[u]);
+        }
+    }
+    if constexpr (TURN) {  // while the heads are on their way
+        if (turn.inv_freq) {
+            const float at = (float)positions[t];
+            for (int i = threadIdx.x; i < turn.rot_dims / 2; i += STORE_THREADS) {
+                float sine, cosine;
+                sincosf(at * turn.inv_freq[i], &sine, &cosine);
+                turned[i] = make_float2(cosine * turn.amplitude, sine * turn.amplitude);
+            }
+            __syncthreads();
         }
     }
 #pragma unroll

@@ -67,21 +67,23 @@ __device__ __forceinline__ void take_result(const HyperArgs& a, int which, size_
 
 // SMAX: the streams, or (HB_STREAMS 0) the most of them.
 template <typename TD, typename TO, int VEC, int CHUNKS, int SMAX>
-__global__ void __launch_bounds__(512) hyper_connect_kernel(const HyperArgs a) {
+__global__ void __launch_bounds__(512, CHUNKS == 1 && SMAX <= 4 ? 2 : 1) hyper_connect_kernel(const HyperArgs a) {
     constexpr bool EXACT = HB_STREAMS > 0, AHEAD = EXACT && CHUNKS * SMAX * VEC <= 48;  // few streams: all of a row's are asked for before the sums of squares
     __shared__ float scratch[32];
     const int r = blockIdx.x, step = blockDim.x * VEC, hidden = a.hidden;
     const int streams = EXACT ? SMAX : a.streams;
-    float mix[EXACT ? SMAX : 1][EXACT ? SMAX : 1], share[EXACT ? SMAX : 1], read[EXACT ? SMAX : 1];
+    __shared__ __align__(16) float mix[EXACT ? SMAX : 1][EXACT ? SMAX : 1], share[EXACT ? SMAX : 1], read[EXACT ? SMAX : 1];  // mix[t][s]: from s to t
     let_next_kernel_start();
     if constexpr (EXACT) {  // no kernel writes weights: these loads overlap the kernel before
-#pragma unroll
-        for (int s = 0; s < SMAX; ++s) {
-            read[s] = a.read ? a.read[s] : 1.f;
-            share[s] = a.mix ? a.share[s] : 0.f;
-#pragma unroll
-            for (int t = 0; t < SMAX; ++t) mix[s][t] = a.mix ? a.mix[s * SMAX + t] : (s == t ? 1.f : 0.f);
+        if (threadIdx.x < SMAX * SMAX) {
+            const int t = threadIdx.x / SMAX, s = threadIdx.x % SMAX;
+            mix[t][s] = a.mix ? a.mix[s * SMAX + t] : (s == t ? 1.f : 0.f);
         }
+        if (threadIdx.x < SMAX) {
+            read[threadIdx.x] = a.read ? a.read[threadIdx.x] : 1.f;
+            share[threadIdx.x] = a.mix ? a.share[threadIdx.x] : 0.f;
+        }
+        __syncthreads();
     }
     wait_for_previous_kernels();
     const int row = a.rows ? a.rows[r] : r;
@@ -176,7 +178,7 @@ __global__ void __launch_bounds__(512) hyper_connect_kernel(const HyperArgs a) {
 #pragma unroll
                 for (int s = 0; s < SMAX; ++s) {
                     if (s >= streams) continue;
-                    const float m = EXACT ? mix[EXACT ? s : 0][EXACT ? t : 0] : a.mix[s * streams + t];
+                    const float m = EXACT ? mix[EXACT ? t : 0][EXACT ? s : 0] : a.mix[s * streams + t];
 #pragma unroll
                     for (int e = 0; e < VEC; ++e) now[e] = fmaf(m, x[s][e], now[e]);
                 }

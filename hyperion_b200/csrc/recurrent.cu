@@ -53,6 +53,67 @@ __global__ void causal_conv_silu_kernel(const float* __restrict__ x, int x_strid
     out[(size_t)t * channels + c] = silu_f(acc);
 }
 
+// The same for channels and strides that are whole 16-byte pieces: a thread takes four neighbouring channels through RUN consecutive tokens of the batch
+// and keeps the last TAPS - 1 inputs in registers; the sums are the scalar kernel's, term by term.
+template <int TAPS, int RUN>
+__global__ void causal_conv_silu4_kernel(const float* __restrict__ x, int x_stride, int col0, int channels, const float* __restrict__ weight, const float* __restrict__ bias,
+                                         const float* __restrict__ state, size_t slot_stride, int state_off, const int* __restrict__ slots,
+                                         const int* __restrict__ token_row, const int* __restrict__ row_start, float* __restrict__ out, int first_token, int tokens) {
+    const int t0 = first_token + blockIdx.y * RUN, c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (c >= channels) return;
+    float now[RUN][4];
+#pragma unroll
+    for (int u = 0; u < RUN; ++u)
+        if (t0 + u < tokens) load4(x + (size_t)(t0 + u) * x_stride + col0 + c, now[u]);
+    float w[4 * TAPS], b[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) {
+        float piece[4];
+        load4(weight + (size_t)c * TAPS + 4 * k, piece);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) w[4 * k + e] = piece[e];
+    }
+    if (bias) load4(bias + c, b);
+    float past[TAPS > 1 ? TAPS - 1 : 1][4];  // oldest first
+    int r = -1, start = 0;
+#pragma unroll
+    for (int u = 0; u < RUN; ++u) {
+        const int t = t0 + u;
+        if (t >= tokens) break;
+        const int row = token_row[t];
+        if (row != r) {  // the first token of this thread's run, or of another request: its earlier inputs from the batch or from the request's state
+            r = row;
+            start = row_start[r];
+            const int i = t - start;
+            const float* kept = state + (size_t)slots[r] * slot_stride + state_off;
+#pragma unroll
+            for (int k = 0; k < TAPS - 1; ++k) {
+                const int j = TAPS - 1 - k;  // this many tokens back
+                if (i - j >= 0) load4(x + (size_t)(t - j) * x_stride + col0 + c, past[k]);
+                else load4(kept + (size_t)(TAPS - 1 + i - j) * channels + c, past[k]);
+            }
+        }
+        float result[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            float acc = b[e];
+#pragma unroll
+            for (int k = 0; k < TAPS - 1; ++k) acc = fmaf(w[e * TAPS + k], past[k][e], acc);
+            acc = fmaf(w[e * TAPS + TAPS - 1], now[u][e], acc);
+            result[e] = silu_f(acc);
+        }
+        store4(out + (size_t)t * channels + c, result);
+#pragma unroll
+        for (int k = 0; k + 1 < TAPS - 1; ++k)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) past[k][e] = past[k + 1][e];
+        if (TAPS > 1) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) past[TAPS > 1 ? TAPS - 2 : 0][e] = now[u][e];
+        }
+    }
+}
+
 // The request's last taps - 1 inputs after this step's tokens (runs after the convolution has read the old ones).
 __global__ void conv_state_update_kernel(const float* __restrict__ x, int x_stride, int col0, int channels, int taps, float* __restrict__ state,
                                          size_t slot_stride, int state_off, const int* __restrict__ slots, const int* __restrict__ row_start,
@@ -404,6 +465,53 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, int y_strid
     }
 }
 
+// The same for groups of whole 16-byte pieces, up to 2,048 pieces: a thread keeps its columns in registers between the sum and the result.
+template <typename TO, int CHUNKS>
+__global__ void __launch_bounds__(512) gated_group_norm4_kernel(const float* __restrict__ y, int y_stride, const float* __restrict__ gate, int gate_stride, int gate_off,
+                                                                const float* __restrict__ weight, int weight_len, int group, int gate_first, float eps, float scale,
+                                                                TO* __restrict__ out, int out_stride, int sigmoid_gate) {
+    __shared__ float scratch[32];
+    const int t = blockIdx.x, first = blockIdx.y * group;
+    const float* yrow = y + (size_t)t * y_stride + first;
+    const float* grow = gate + (size_t)t * gate_stride + gate_off + first;
+    float v[CHUNKS][4], g[CHUNKS][4];
+#pragma unroll
+    for (int c = 0; c < CHUNKS; ++c) {
+        const int j = (c * blockDim.x + threadIdx.x) * 4;
+        if (j < group) {
+            load4(yrow + j, v[c]);
+            load4(grow + j, g[c]);
+        }
+    }
+    float sum = 0.f;
+#pragma unroll
+    for (int c = 0; c < CHUNKS; ++c) {
+        const int j = (c * blockDim.x + threadIdx.x) * 4;
+        if (j >= group) continue;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            g[c][e] = gate_f(g[c][e], sigmoid_gate);
+            if (gate_first) v[c][e] *= g[c][e];
+            sum = fmaf(v[c][e], v[c][e], sum);
+        }
+    }
+    const float inv = 1.0f / sqrtf(block_sum(sum, scratch) / (float)group + eps);
+#pragma unroll
+    for (int c = 0; c < CHUNKS; ++c) {
+        const int j = (c * blockDim.x + threadIdx.x) * 4;
+        if (j >= group) continue;
+        float w[4] = {1.f, 1.f, 1.f, 1.f}, o[4];
+        if (weight) load4(weight + (first + j) % weight_len, w);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            o[e] = v[c][e] * inv * w[e];
+            if (!gate_first) o[e] *= g[c][e];
+            o[e] *= scale;
+        }
+        store4(out + (size_t)t * out_stride + first + j, o);
+    }
+}
+
 // The same for groups of up to 1,024 columns: a warp per (token, group), four of them in a block; the lanes' partial sums
 // meet in a butterfly of fixed shape.
 template <typename TO>
@@ -438,7 +546,24 @@ HB_EXPORT int hb_causal_conv_silu(const float* x, int x_stride, int col0, int ch
                                   const int* row_start, float* out, int tokens, cudaStream_t stream) {
     if (tokens <= 0 || channels <= 0) return 0;
     if (taps < 1) return HB_BAD_ARGUMENT;
+    const bool by_four = taps <= 5 && ((x_stride | col0 | channels | state_off) & 3) == 0 && (slot_stride & 3) == 0 &&
+                         (((uintptr_t)x | (uintptr_t)weight | (uintptr_t)bias | (uintptr_t)state | (uintptr_t)out) & 15) == 0;
     for (int first = 0; first < tokens; first += 65535) {  // the grid's second dimension holds 65,535 tokens
+        if (by_four) {
+            const int end = tokens - first < 65535 ? tokens : first + 65535, across = (channels / 4 + 127) / 128;
+#define HB_CONV4(T, RUN)                                                                                                                                        \
+    causal_conv_silu4_kernel<T, RUN><<<dim3(across, (end - first + RUN - 1) / RUN), 128, 0, stream>>>(x, x_stride, col0, channels, weight, bias, state,          \
+                                                                                                     (size_t)slot_stride, state_off, slots, token_row, row_start, \
+                                                                                                     out, first, end)
+#define HB_CONV4_TAPS(T)                                     \
+    case T:                                                  \
+        if (tokens >= 128) HB_CONV4(T, 8); else HB_CONV4(T, 1); \
+        break
+            switch (taps) { HB_CONV4_TAPS(1); HB_CONV4_TAPS(2); HB_CONV4_TAPS(3); HB_CONV4_TAPS(4); HB_CONV4_TAPS(5); }
+#undef HB_CONV4_TAPS
+#undef HB_CONV4
+            continue;
+        }
         const int count = tokens - first < 65535 ? tokens - first : 65535;
         causal_conv_silu_kernel<<<dim3((channels + 255) / 256, count), 256, 0, stream>>>(x, x_stride, col0, channels, weight, bias, taps, state, (size_t)slot_stride,
                                                                                         state_off, slots, token_row, row_start, out, first);
@@ -787,6 +912,19 @@ HB_EXPORT int hb_gated_group_norm(const float* y, int y_stride, const float* gat
         else
             gated_group_norm_warp_kernel<<<warps, 128, 0, stream>>>(y, y_stride, gate, gate_stride, gate_off, weight, weight_len, group, groups, gate_first,
                                                                     eps, scale, (float*)out, out_stride, sigmoid_gate);
+        return launch_status();
+    }
+    const bool by_four = group % 4 == 0 && group <= 8192 && weight_len % 4 == (weight ? 0 : 1) && ((y_stride | gate_stride | gate_off | out_stride) & 3) == 0 &&
+                         (((uintptr_t)y | (uintptr_t)gate | (uintptr_t)weight) & 15) == 0 && ((uintptr_t)out & (out_is_bf16 ? 7 : 15)) == 0;
+    if (by_four) {
+        const dim3 each(tokens, groups);
+        const int pieces = group / 4, lanes = pieces <= 512 ? ((pieces + 31) / 32) * 32 : 512;  // from the group's size alone
+#define HB_GROUP4(TO, CHUNKS)                                                                                                                                      \
+    gated_group_norm4_kernel<TO, CHUNKS><<<each, lanes, 0, stream>>>(y, y_stride, gate, gate_stride, gate_off, weight, weight_len, group, gate_first, eps, scale, \
+                                                                     (TO*)out, out_stride, sigmoid_gate)
+        if (pieces <= 512) { if (out_is_bf16) HB_GROUP4(__nv_bfloat16, 1); else HB_GROUP4(float, 1); }
+        else { if (out_is_bf16) HB_GROUP4(__nv_bfloat16, 4); else HB_GROUP4(float, 4); }
+#undef HB_GROUP4
         return launch_status();
     }
     const int threads = group >= 4096 ? 1024 : (group >= 2048 ? 512 : 256);  // a wide group (one norm over all heads): fewer trips per thread
