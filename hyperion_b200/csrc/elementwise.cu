@@ -1301,6 +1301,34 @@ __global__ void relu_squared_bf16x8_kernel(const uint4* __restrict__ x, uint4* _
     }
 }
 
+// The same of a product still in its split-K pieces ([splits, count] floats, added up in split order): what would add them up applies the activation at once.
+template <typename T>
+__global__ void relu_squared_of_pieces_kernel(const float* __restrict__ pieces, int splits, size_t count, T* __restrict__ out) {
+    let_next_kernel_start();
+    wait_for_previous_kernels();
+    for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4; i < count; i += (size_t)gridDim.x * blockDim.x * 4) {
+        float sum[4] = {0.f, 0.f, 0.f, 0.f}, piece[4];
+#pragma unroll 8
+        for (int k = 0; k < splits; ++k) {
+            load4(pieces + (size_t)k * count + i, piece);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sum[e] += piece[e];
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sum[e] = activated(sum[e], HB_ACT_RELU_SQUARED);
+        store4(out + i, sum);
+    }
+}
+
+HB_EXPORT int hb_relu_squared_of_pieces(const float* pieces, int splits, long long count, void* out, int out_is_bf16, cudaStream_t stream) {
+    if (count <= 0) return 0;
+    if (splits < 1 || count % 4 || (((uintptr_t)pieces | (uintptr_t)out) & 15)) return HB_UNSUPPORTED_SIZE;
+    const long long wanted = (count / 4 + 127) / 128;
+    const dim3 blocks((unsigned)(wanted < 16384 ? wanted : 16384));
+    if (out_is_bf16) return launch_after_previous(relu_squared_of_pieces_kernel<__nv_bfloat16>, blocks, dim3(128), 0, stream, pieces, splits, (size_t)count, (__nv_bfloat16*)out);
+    return launch_after_previous(relu_squared_of_pieces_kernel<float>, blocks, dim3(128), 0, stream, pieces, splits, (size_t)count, (float*)out);
+}
+
 HB_EXPORT int hb_relu_squared(const void* x, void* out, int is_bf16, long long count, cudaStream_t stream) {
     if (count <= 0) return 0;
     const bool eights = is_bf16 && count % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0;

@@ -620,8 +620,18 @@ def soft_cap_(x: torch.Tensor, cap: float) -> torch.Tensor:
     return x
 
 
-def relu_squared(x: torch.Tensor) -> torch.Tensor:
-    """max(x, 0)^2, computed in float, in the element type of ``x``."""
+def relu_squared(x) -> torch.Tensor:
+    """max(x, 0)^2, computed in float, in the element type of ``x``: a tensor, or a product still in its split-K pieces (``ops.gemm.SplitSum``), which this adds up."""
+    from .gemm import SplitSum
+
+    if isinstance(x, SplitSum):
+        splits, m, n = x.partials.shape
+        if x.bias is None and x.partials.is_contiguous() and (m * n) % 4 == 0:
+            require_cuda(x.partials)
+            out = torch.empty((m, n), dtype=x.dtype, device=x.partials.device)
+            check(library("elementwise").hb_relu_squared_of_pieces(ptr(x.partials), i32(splits), ctypes.c_longlong(m * n), ptr(out), i32(is_bf16(out)), stream_ptr()), "relu_squared")
+            return out
+        x = x.tensor()
     require_cuda(x)
     if not x.is_contiguous():
         raise KernelError("relu_squared: a dense tensor")

@@ -87,7 +87,8 @@ class ActivatedMLP(FeedForward):
         return [("elementwise", {}), ("sgemm_f32", {}) if self.dtype == torch.float32 else ("gemm_tcgen05", {})]
 
     def forward(self, x, step):
-        act = getattr(ops, self.ACTIVATIONS[self.activation])(ops.linear(x, self.w_up, None, self.dtype))
+        up = ops.linear(x, self.w_up, None, self.dtype, may_leave_partials=self.activation == "relu_squared")  # that operation adds split-K pieces up itself
+        act = getattr(ops, self.ACTIVATIONS[self.activation])(up)
         return ops.linear(act, self.w_down, None, self.dtype, may_leave_partials=True)  # the result is a residual delta
 
 

@@ -41,7 +41,7 @@ import torch
 
 from .. import ops
 from ..ops import attention as fast_attention
-from ..ops import recurrent
+from ..ops import native, recurrent
 from .attention import GroupedQueryAttention
 from .base import MIXERS, POSITIONS, BuildContext, Mixer, PagedTokens, RequestState, WeightSpec, make, register_mixer
 from .branch import Branch, common_dtype
@@ -258,12 +258,14 @@ class ParallelMixers(Mixer):
 
 
 class ParallelNormedMixers(Mixer):
+    BESIDE_TOKENS = 64  # steps of at most this many tokens run their branches side by side
     COLUMN_STEP = 8  # every branch's columns of the input product start on a multiple of this, so that they stay whole 16-byte pieces
 
     def __init__(self, spec: PartSpec, build: BuildContext):
         super().__init__(spec, build)
         p = spec.params
         self.hidden, self.eps, self.scale = int(p["hidden_size"]), float(p["eps"]), float(p["scale"])
+        self.shared = build.shared
         self.branches: list[Branch] = []
         self.prefixes: list[str] = []
         self.norm_names: list[str] = []
@@ -321,12 +323,31 @@ class ParallelNormedMixers(Mixer):
         if cache is None or not own_cache or len(cache) != len(self.branches):
             raise ValueError("parallel mixers keep what their branches keep; the schedule gave them something else")
         proj = ops.linear(x, self.w_in, None, torch.float32)
-        results = []
-        for branch, column, w_out, view in zip(self.branches, self.columns, self.w_out, cache):
-            out = torch.empty((x.shape[0], branch.core_width), dtype=self.dtype, device=x.device)
-            branch.core(proj, column, step, view, out, 1.0)
-            results.append(ops.linear(out, w_out, None, self.dtype, may_leave_partials=True))
+        # A step of few tokens is a chain of small kernels that leave most of the GPU idle: there the second branch runs on a stream of its own, from the input product
+        # to its own output product, beside the first.  Results do not depend on it.
+        beside = self._side_stream() if len(self.branches) == 2 and x.shape[0] <= self.BESIDE_TOKENS else None
+        if beside is None:
+            results = [self._branch(index, x, proj, step, view) for index, view in enumerate(cache)]
+        else:
+            here = torch.cuda.current_stream()
+            beside.wait_stream(here)
+            with torch.cuda.stream(beside), native.stream_bound():
+                second = self._branch(1, x, proj, step, cache[1])
+            results = [self._branch(0, x, proj, step, cache[0]), second]
+            here.wait_stream(beside)
         return NormedSum(tuple(results), tuple(self.norm_weights), self.eps, self.scale)
+
+    def _branch(self, index: int, x, proj, step, view):
+        branch = self.branches[index]
+        out = torch.empty((x.shape[0], branch.core_width), dtype=self.dtype, device=x.device)
+        branch.core(proj, self.columns[index], step, view, out, 1.0)
+        return ops.linear(out, self.w_out[index], None, self.dtype, may_leave_partials=True)
+
+    def _side_stream(self) -> torch.cuda.Stream:
+        key = ("side_stream", str(self.device))
+        if key not in self.shared:
+            self.shared[key] = torch.cuda.Stream(device=self.device)
+        return self.shared[key]
 
 
 register_mixer("parallel_normed_mixers", ParallelNormedMixers)
