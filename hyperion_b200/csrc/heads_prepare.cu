@@ -574,17 +574,6 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
     const float* row = x + (size_t)t * stride;
     TO* key_at = nullptr;
     TO* value_at = nullptr;
-    if (stored && first_item + (JOBS - 1) * groups >= q_heads) {  // some head of this group goes to the token's page
-        const int pos = positions[t], block = pos / page_size;
-        const int page = (pos >= 0 && block < table_width) ? block_table[(size_t)token_row[t] * table_width + block] : -1;
-        if (page >= 0 && page < pages) {
-            const size_t at = (size_t)page * page_stride + (size_t)(pos - block * page_size) * token_stride;
-            key_at = k_cache + at;
-            value_at = v_cache + at;
-        } else {
-            atomicOr(status, HB_STATUS_BAD_PAGE);
-        }
-    }
     auto job_of = [&](int item) {
         HeadJob<TO> job{q_off, head_dim, nullptr, nullptr, 0};
         if (item < q_heads) {
@@ -597,9 +586,9 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
                 job.col = k_off + which * head_dim;
                 job.weight = k_norm;
                 job.kind = 1;
-                if (key_at) job.dst = key_at + (size_t)(which / maps) * head_stride + (size_t)(which % maps) * head_dim;
+                if (key_at) job.dst = maps == 1 ? key_at + (size_t)which * head_stride : key_at + (size_t)(which / maps) * head_stride + (size_t)(which % maps) * head_dim;
             } else {
-                const int head = (which - k_heads) / runs, first = ((which - k_heads) % runs) * head_dim;
+                const int head = runs == 1 ? which - k_heads : (which - k_heads) / runs, first = runs == 1 ? 0 : ((which - k_heads) % runs) * head_dim;
                 job.col = v_off + head * v_dim + first;
                 job.kind = 2;
                 job.dim = min(head_dim, v_dim - first);
@@ -615,6 +604,17 @@ __global__ void __launch_bounds__(STORE_THREADS) heads_store_kernel(const float*
             const HeadJob<TO> job = job_of(first_item + u * groups);
             const int i = lane * VEC;
             if (i < job.dim) fetch_entries<VEC>(row + job.col + i, bias ? bias + job.col + i : nullptr, kept[u]);
+        }
+    }
+    if (stored && first_item + (JOBS - 1) * groups >= q_heads) {  // some head of this group goes to the token's page; the heads are on their way
+        const int pos = positions[t], block = pos / page_size;
+        const int page = (pos >= 0 && block < table_width) ? block_table[(size_t)token_row[t] * table_width + block] : -1;
+        if (page >= 0 && page < pages) {
+            const size_t at = (size_t)page * page_stride + (size_t)(pos - block * page_size) * token_stride;
+            key_at = k_cache + at;
+            value_at = v_cache + at;
+        } else {
+            atomicOr(status, HB_STATUS_BAD_PAGE);
         }
     }
     if constexpr (TURN) {  // while the heads are on their way

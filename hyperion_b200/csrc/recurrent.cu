@@ -717,32 +717,42 @@ __global__ void __launch_bounds__(128) matrix_memory_norm_kernel(const float* __
     const float* g = gate + (size_t)t * gate_stride + gate_off + (size_t)head * e;
     const float* w = weight + (size_t)head * e;
     TO* dst = out + (size_t)t * out_stride + (size_t)head * e;
-    const float below = fmaxf(fabsf(row[e]), gates[(size_t)t * 4 * heads + 2 * heads + head]) + 1e-6f;
-    float sum = 0.f;
-    if (by_four) {
-        for (int j = lane * 4; j < e; j += 128) {
-            float v[4];
-            load4(row + j, v);
+    if (by_four && e <= 512) {  // the head stays in registers
+        float v[4][4], gv[4][4];
 #pragma unroll
-            for (int k = 0; k < 4; ++k) { v[k] /= below; sum = fmaf(v[k], v[k], sum); }
+        for (int c = 0; c < 4; ++c) {
+            const int j = (c * 32 + lane) * 4;
+            if (j < e) {
+                load4(row + j, v[c]);
+                load4(g + j, gv[c]);
+            }
         }
-    } else {
-        for (int j = lane; j < e; j += 32) { const float v = row[j] / below; sum = fmaf(v, v, sum); }
-    }
-    const float inv = 1.0f / sqrtf(warp_sum(sum) / (float)e + eps);
-    if (by_four) {
-        for (int j = lane * 4; j < e; j += 128) {
-            float v[4], gv[4], wv[4];
-            load4(row + j, v);
-            load4(g + j, gv);
+        const float over = 1.0f / (fmaxf(fabsf(row[e]), gates[(size_t)t * 4 * heads + 2 * heads + head]) + 1e-6f);
+        float sum = 0.f;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            if ((c * 32 + lane) * 4 >= e) continue;
+#pragma unroll
+            for (int k = 0; k < 4; ++k) { v[c][k] *= over; sum = fmaf(v[c][k], v[c][k], sum); }
+        }
+        const float inv = 1.0f / sqrtf(warp_sum(sum) / (float)e + eps);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            const int j = (c * 32 + lane) * 4;
+            if (j >= e) continue;
+            float wv[4];
             load4(w + j, wv);
 #pragma unroll
-            for (int k = 0; k < 4; ++k) v[k] = v[k] / below * inv * wv[k] * sigmoid_of(gv[k]);
-            store4(dst + j, v);
+            for (int k = 0; k < 4; ++k) v[c][k] = v[c][k] * inv * wv[k] * sigmoid_of(gv[c][k]);
+            store4(dst + j, v[c]);
         }
-    } else {
-        for (int j = lane; j < e; j += 32) dst[j] = from_float<TO>(row[j] / below * inv * w[j] * sigmoid_of(g[j]));
+        return;
     }
+    const float below = fmaxf(fabsf(row[e]), gates[(size_t)t * 4 * heads + 2 * heads + head]) + 1e-6f;
+    float sum = 0.f;
+    for (int j = lane; j < e; j += 32) { const float v = row[j] / below; sum = fmaf(v, v, sum); }
+    const float inv = 1.0f / sqrtf(warp_sum(sum) / (float)e + eps);
+    for (int j = lane; j < e; j += 32) dst[j] = from_float<TO>(row[j] / below * inv * w[j] * sigmoid_of(g[j]));
 }
 }  // namespace
 

@@ -96,6 +96,7 @@ class ModelRunner:
         arrays = packer.finish()
         if packer.generation != self._packer_generation:  # the device buffer moved: captured graphs point at the old one
             self.graphs.clear()
+            self._graph_pool = None  # a pool that no graph uses any more is gone
             self._packer_generation = packer.generation
         extra = {k: v for k, v in arrays.items() if k not in ("token_ids", "positions", "token_row", "row_start", "slots", "want")
                  and not k.startswith("table")}

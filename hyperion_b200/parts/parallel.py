@@ -258,7 +258,6 @@ class ParallelMixers(Mixer):
 
 
 class ParallelNormedMixers(Mixer):
-    BESIDE_TOKENS = 64  # steps of at most this many tokens run their branches side by side
     COLUMN_STEP = 8  # every branch's columns of the input product start on a multiple of this, so that they stay whole 16-byte pieces
 
     def __init__(self, spec: PartSpec, build: BuildContext):
@@ -323,9 +322,9 @@ class ParallelNormedMixers(Mixer):
         if cache is None or not own_cache or len(cache) != len(self.branches):
             raise ValueError("parallel mixers keep what their branches keep; the schedule gave them something else")
         proj = ops.linear(x, self.w_in, None, torch.float32)
-        # A step of few tokens is a chain of small kernels that leave most of the GPU idle: there the second branch runs on a stream of its own, from the input product
-        # to its own output product, beside the first.  Results do not depend on it.
-        beside = self._side_stream() if len(self.branches) == 2 and x.shape[0] <= self.BESIDE_TOKENS else None
+        # The second branch runs on a stream of its own, from the input product to its own output product, beside the first: a decode step is a chain of small kernels
+        # that leave most of the GPU idle (7 % of a step at batch 8), and a prompt's recurrence has phases that do.  Results do not depend on it.
+        beside = self._side_stream() if len(self.branches) == 2 else None
         if beside is None:
             results = [self._branch(index, x, proj, step, view) for index, view in enumerate(cache)]
         else:
