@@ -1378,6 +1378,10 @@ def biropel_kernels(size: dict, measured: dict) -> dict:
         act = torch.randn(tokens, size["ff"], device=dev).to(torch.bfloat16)
         report(f"relu_squared/{shape}", timed(lambda: ops.relu_squared(act)), act.numel() * 4)
         report(f"mirovik.gelu_tanh/{shape}", timed(lambda: ops.gelu_tanh(act)), act.numel() * 4)
+        w_up = (torch.randn(size["ff"], width, device=dev) * 0.02).to(torch.bfloat16)
+        moved, flops = w_up.numel() * 2 + tokens * (width + size["ff"]) * 2, 2.0 * tokens * width * size["ff"]
+        report(f"up_product_with_relu_squared/{shape}", timed(lambda: ops.relu_squared_linear(a, w_up)), moved, bf16_flops=flops)
+        report(f"mirovik.up_product_then_gelu/{shape}", timed(lambda: ops.gelu_tanh(ops.linear(a, w_up, None, torch.bfloat16))), moved, bf16_flops=flops)
     return out
 
 

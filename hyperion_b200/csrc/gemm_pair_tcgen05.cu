@@ -141,6 +141,10 @@ __device__ __forceinline__ void store_row(const GemmParams& p, unsigned lane_add
                 v[j] = g / (1.0f + expf(-g)) * uu;
             }
         }
+        if constexpr (EPI == EPI_RELU_SQUARED) {  // applied to the product's float result
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = activated(v[j], HB_ACT_RELU_SQUARED);
+        }
         if (r >= p.m) continue;
         if constexpr (EPI == EPI_F32) {
             float* dst = reinterpret_cast<float*>(p.c) + (size_t)r * p.ldc + out_col;
@@ -351,15 +355,15 @@ int resident_pairs() {
 
 // C = A W^T (+ bias) on pairs of SMs.  a [m, k] (row stride lda), w [n, k] (row stride ldw), bfloat16, k-contiguous.
 //   epilogue 0: c bfloat16 [m, n]; 1: c float [m, n]; 2: SwiGLU, c bfloat16 [m, n / 2] where every 256 rows of w
-//   are 128 gate rows followed by their 128 up rows (n a multiple of 256).
+//   are 128 gate rows followed by their 128 up rows (n a multiple of 256); 4: c = max(., 0)^2 of the product, bfloat16 [m, n], no bias.
 HB_EXPORT int hb_gemm_pair_bf16(const void* a, int lda, const void* w, int ldw, void* c, int ldc, const float* bias_f, const void* bias_h,
                                 int m, int n, int k, int epilogue, int* status, cudaStream_t stream) {
     if (m <= 0 || n <= 0) return 0;
     if (k <= 0) return HB_BAD_ARGUMENT;
     if (epilogue == EPI_SWIGLU && n % 256) return HB_UNSUPPORTED_SIZE;
-    if (epilogue != EPI_BF16 && epilogue != EPI_F32 && epilogue != EPI_SWIGLU) return HB_BAD_ARGUMENT;
+    if (epilogue != EPI_BF16 && epilogue != EPI_F32 && epilogue != EPI_SWIGLU && (epilogue != EPI_RELU_SQUARED || bias_f || bias_h)) return HB_BAD_ARGUMENT;
     GemmParams p{c, bias_f, (const bf16*)bias_h, nullptr, m, n, k, ldc, (k + BK - 1) / BK, status};
-    const int resident = epilogue == EPI_BF16 ? resident_pairs<EPI_BF16>() : (epilogue == EPI_F32 ? resident_pairs<EPI_F32>() : resident_pairs<EPI_SWIGLU>());
+    const int resident = epilogue == EPI_BF16 ? resident_pairs<EPI_BF16>() : (epilogue == EPI_F32 ? resident_pairs<EPI_F32>() : (epilogue == EPI_SWIGLU ? resident_pairs<EPI_SWIGLU>() : resident_pairs<EPI_RELU_SQUARED>()));
     const int bn = epilogue == EPI_SWIGLU ? 256 : choose_pair_width(m, n, resident);
     CUtensorMap map_x, map_w;
     if (int code = make_map(&map_x, a, m, k, lda, BM)) return code;
@@ -369,5 +373,6 @@ HB_EXPORT int hb_gemm_pair_bf16(const void* a, int lda, const void* w, int ldw, 
     const int pairs = min(tiles_m * tiles_n, resident);
     if (epilogue == EPI_BF16) return launch_pairs<EPI_BF16>(map_x, map_w, p, tiles_m, tiles_n, bn, pairs, stream);
     if (epilogue == EPI_F32) return launch_pairs<EPI_F32>(map_x, map_w, p, tiles_m, tiles_n, bn, pairs, stream);
+    if (epilogue == EPI_RELU_SQUARED) return launch_pairs<EPI_RELU_SQUARED>(map_x, map_w, p, tiles_m, tiles_n, bn, pairs, stream);
     return launch_pairs<EPI_SWIGLU>(map_x, map_w, p, tiles_m, tiles_n, bn, pairs, stream);
 }

@@ -11,7 +11,7 @@ constexpr int BM = 128, BK = 64, UMMA_K = 16;
 constexpr int THREADS = 192;
 constexpr unsigned WAIT_LIMIT = 1u << 24;
 
-enum Epilogue : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_PARTIAL = 3 };
+enum Epilogue : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_PARTIAL = 3, EPI_RELU_SQUARED = 4 };
 
 struct GemmParams {
     void* c;              // output

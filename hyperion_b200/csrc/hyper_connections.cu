@@ -67,8 +67,8 @@ __device__ __forceinline__ void take_result(const HyperArgs& a, int which, size_
 
 // SMAX: the streams, or (HB_STREAMS 0) the most of them.
 template <typename TD, typename TO, int VEC, int CHUNKS, int SMAX>
-__global__ void __launch_bounds__(512, CHUNKS == 1 && SMAX <= 4 ? 2 : 1) hyper_connect_kernel(const HyperArgs a) {
-    constexpr bool EXACT = HB_STREAMS > 0, AHEAD = EXACT && CHUNKS * SMAX * VEC <= 48;  // few streams: all of a row's are asked for before the sums of squares
+__global__ void __launch_bounds__(512, CHUNKS <= 2 && SMAX <= 4 ? 2 : 1) hyper_connect_kernel(const HyperArgs a) {
+    constexpr bool EXACT = HB_STREAMS > 0, AHEAD = EXACT && CHUNKS == 1;  // a row's streams are asked for before the sums of squares (more of them cost a block of occupancy)
     __shared__ float scratch[32];
     const int r = blockIdx.x, step = blockDim.x * VEC, hidden = a.hidden;
     const int streams = EXACT ? SMAX : a.streams;

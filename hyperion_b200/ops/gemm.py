@@ -16,7 +16,7 @@ import torch
 from .basic import status_word
 from .native import KernelError, check, i32, library, ptr, require_cuda, sm_count, stream_ptr
 
-EPI_BF16, EPI_F32, EPI_SWIGLU = 0, 1, 2
+EPI_BF16, EPI_F32, EPI_SWIGLU, EPI_RELU_SQUARED = 0, 1, 2, 4
 SWIGLU_BLOCK = 128  # the fused epilogue wants 128 gate rows followed by their 128 up rows, repeated
 PAIR_MIN_ROWS = 128  # more rows than this: the pair kernel's 256-row tiles (when this package's kernels take a prompt-sized product at all)
 

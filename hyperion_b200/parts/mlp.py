@@ -65,7 +65,8 @@ class ActivatedMLP(FeedForward):
     """The feed-forward without a gate: down(act(up(x))), no biases, act = the tanh form of GELU, its exact (erf) form or the square of relu.
     Parameters: ``hidden_size``, ``intermediate_size``, ``activation`` (``gelu_tanh``, ``gelu_erf`` or ``relu_squared``), ``names`` (``{"up": ..., "down": ...}``)."""
 
-    ACTIVATIONS = {"gelu_tanh": "gelu_tanh", "gelu_erf": "gelu_erf", "relu_squared": "relu_squared"}  # the name of the activation -> the operation of ``ops``
+    # the name of the activation -> the operation of ``ops`` (the square of relu: product and activation together)
+    ACTIVATIONS = {"gelu_tanh": "gelu_tanh", "gelu_erf": "gelu_erf", "relu_squared": "relu_squared_linear"}
 
     def __init__(self, spec: PartSpec, build: BuildContext):
         super().__init__(spec, build)
@@ -84,11 +85,16 @@ class ActivatedMLP(FeedForward):
         self.w_up, self.w_down = tensors[self.up_name].contiguous(), tensors[self.down_name].contiguous()
 
     def kernel_modules(self):
-        return [("elementwise", {}), ("sgemm_f32", {}) if self.dtype == torch.float32 else ("gemm_tcgen05", {})]
+        if self.dtype == torch.float32:
+            return [("elementwise", {}), ("sgemm_f32", {})]
+        return [("elementwise", {}), ("gemm_tcgen05", {})] + ([("gemm_pair_tcgen05", {})] if self.activation == "relu_squared" else [])
 
     def forward(self, x, step):
-        up = ops.linear(x, self.w_up, None, self.dtype, may_leave_partials=self.activation == "relu_squared")  # that operation adds split-K pieces up itself
-        act = getattr(ops, self.ACTIVATIONS[self.activation])(up)
+        operation = getattr(ops, self.ACTIVATIONS[self.activation])
+        if self.activation == "relu_squared":
+            act = operation(x, self.w_up, self.dtype)
+        else:
+            act = operation(ops.linear(x, self.w_up, None, self.dtype))
         return ops.linear(act, self.w_down, None, self.dtype, may_leave_partials=True)  # the result is a residual delta
 
 

@@ -337,6 +337,14 @@ def test_relu_squared():
             y = x.to(dtype)
             want = torch.relu(y.double()).pow(2)
             assert (ops.relu_squared(y.cuda()).cpu().double() - want).abs().max() <= tolerance * want.abs().max()
+    # behind a product: few rows (pieces that the activation adds up), rows for the library's product, and enough for the product's own epilogue
+    g = torch.Generator().manual_seed(2)
+    for m, n, k in ((8, 520, 2048), (40, 96, 64), (700, 264, 192), (2048, 264, 192), (2240, 1032, 512)):
+        x, w = torch.randn(m, k, generator=g).to(torch.bfloat16), (torch.randn(n, k, generator=g) / k ** 0.5).to(torch.bfloat16)
+        want = torch.relu((x.float() @ w.float().T).double()).pow(2)
+        got = ops.relu_squared_linear(x.cuda(), w.cuda()).cpu().double()
+        assert got.shape == (m, n) and (got - want).abs().max() <= 1e-2 * want.abs().max(), (m, n, k)
+        assert (ops.relu_squared_linear(x.float().cuda(), w.float().cuda()).cpu().double() - want).abs().max() <= 1e-5 * want.abs().max()
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
