@@ -4,9 +4,9 @@
 //     o_i = exp(L_i) S0^T q_i + sum_(j <= i) exp(L_i - L_j) b_j (q_i . k_j) v_j,
 //     S_end = exp(L_end) S0 + sum_j exp(L_end - L_j) b_j k_j v_j^T,
 // so chunks need one another only through S0: chunk_states makes every chunk's own sum (the second line without S0) and its decay exp(L_end),
-// chunk_join walks the short chain per state entry, and chunk_outputs makes the outputs.  Keys, queries, values and the weighted scores are bfloat16
-// operands of mma.sync with float sums; logarithms, decays, steps, the weights on the scores and the state are float, the state entering its
-// product as a bfloat16 and a bfloat16 remainder (16 bits of it; chunk_join leaves it so).
+// chunk_join walks the short chain per state entry, and chunk_outputs makes the outputs.  Products run as mma.sync with float sums.  Keys, queries and
+// values, which are projections, are rounded to bfloat16; everything else is float: logarithms, decays, steps and the state, and where one of them is an operand
+// of a product (weighted scores, weighted values, the state) it enters as a bfloat16 and a bfloat16 remainder, 16 bits of it, in two products.
 // A matrix memory also sums its keys, n <- a n + b k: the state's row behind the values; n . q is the plain sum of a row's weighted scores
 // plus exp(L_i) n0 . q_i.  The one-token-after-another form of the same recurrences (recurrent.cu) serves decoded tokens and the float32 mode.
 // A block takes ETILE value columns of one head and chunk (64, or 128 where a head has them) with two threads per column.
@@ -79,8 +79,15 @@ __device__ __forceinline__ uint32_t pack(float lo, float hi) {
     return *reinterpret_cast<const uint32_t*>(&both);
 }
 
+// Two floats as bfloat16 and what that rounding left of them.
+__device__ __forceinline__ void pack_pair(float a, float b, uint32_t& rounded, uint32_t& rest) {
+    const __nv_bfloat162 both = __floats2bfloat162_rn(a, b);
+    rounded = *reinterpret_cast<const uint32_t*>(&both);
+    rest = pack(a - __low2float(both), b - __high2float(both));
+}
+
 // A tile of CHUNK rows of floats on its way to shared memory as bfloat16: row r at src + r * stride; rows from `live` on and columns from `columns` on are zeros.
-// fetch() asks for AHEAD pieces of four columns from piece `base` on; place() rounds them into rows of `ld` columns, row r times row_factor[r] (null: 1) and `factor`.
+// fetch() asks for AHEAD pieces of four columns from piece `base` on; place() rounds them, times `factor`, into rows of `ld` columns.
 struct Tile {
     const float* src;
     size_t stride;
@@ -118,15 +125,29 @@ struct Tile {
     }
 
     template <int THREADS>
-    __device__ __forceinline__ void place(Walk<THREADS> at, const float (&x)[AHEAD][4], __nv_bfloat16* dst, int ld, const float* row_factor, float factor) const {
+    __device__ __forceinline__ void place(Walk<THREADS> at, const float (&x)[AHEAD][4], __nv_bfloat16* dst, int ld, float factor) const {
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u, at.next()) {
             if (at.r >= CHUNK) continue;
-            const float f = row_factor ? row_factor[at.r] * factor : factor;
             uint2 packed;
-            packed.x = pack(x[u][0] * f, x[u][1] * f);
-            packed.y = pack(x[u][2] * f, x[u][3] * f);
+            packed.x = pack(x[u][0] * factor, x[u][1] * factor);
+            packed.y = pack(x[u][2] * factor, x[u][3] * factor);
             *reinterpret_cast<uint2*>(dst + at.r * ld + at.quad * 4) = packed;
+        }
+    }
+
+    // rows times a float each: the rounded value and the remainder
+    template <int THREADS>
+    __device__ __forceinline__ void place_weighted(Walk<THREADS> at, const float (&x)[AHEAD][4], __nv_bfloat16* hi, __nv_bfloat16* lo, int ld, const float* row_factor) const {
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u, at.next()) {
+            if (at.r >= CHUNK) continue;
+            const float f = row_factor[at.r];
+            uint2 rounded, rest;
+            pack_pair(x[u][0] * f, x[u][1] * f, rounded.x, rest.x);
+            pack_pair(x[u][2] * f, x[u][3] * f, rounded.y, rest.y);
+            *reinterpret_cast<uint2*>(hi + at.r * ld + at.quad * 4) = rounded;
+            *reinterpret_cast<uint2*>(lo + at.r * ld + at.quad * 4) = rest;
         }
     }
 };
@@ -156,6 +177,7 @@ __global__ void __launch_bounds__(2 * ETILE) chunk_states_kernel(const ChunkArgs
     constexpr int v_ld = ETILE + 8;
     __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(memory);
     __nv_bfloat16* vs = ks + CHUNK * k_ld;
+    __nv_bfloat16* vs_rest = vs + CHUNK * v_ld;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int group = head / (a.heads / a.groups);
 
@@ -169,14 +191,14 @@ __global__ void __launch_bounds__(2 * ETILE) chunk_states_kernel(const ChunkArgs
     const float last = L[CHUNK - 1];
     if (threadIdx.x < CHUNK) step[threadIdx.x] *= exp2f(last - L[threadIdx.x]);  // the weight of a token in the chunk's sum
     if (threadIdx.x == 0 && blockIdx.z == 0) a.decays[(size_t)chunk * a.heads + head] = exp2f(last);
-    keys.place(key_walk, x, ks, k_ld, nullptr, 1.f);
+    keys.place(key_walk, x, ks, k_ld, 1.f);
     for (int base = threadIdx.x + AHEAD * THREADS; base < CHUNK * keys.quads; base += AHEAD * THREADS) {
         const Tile::Walk<THREADS> walk(base, keys.quads);
         keys.fetch(walk, x);
-        keys.place(walk, x, ks, k_ld, nullptr, 1.f);
+        keys.place(walk, x, ks, k_ld, 1.f);
     }
     __syncthreads();  // the weights are there
-    values.place(value_walk, y, vs, v_ld, step, 1.f);
+    values.place_weighted(value_walk, y, vs, vs_rest, v_ld, step);
     __syncthreads();
 
     float acc[NMAX / 8][4];
@@ -184,8 +206,10 @@ __global__ void __launch_bounds__(2 * ETILE) chunk_states_kernel(const ChunkArgs
     for (int i = 0; i < NMAX / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
     for (int t = 0; t < CHUNK / 16; ++t) {
-        uint32_t va[4];  // rows: value columns; inner: tokens
-        load_matrices_turned(va, shared_address(vs + (t * 16 + (lane >> 4) * 8 + (lane & 7)) * v_ld + warp * 16 + ((lane >> 3) & 1) * 8));
+        uint32_t va[4], rest[4];  // rows: value columns; inner: tokens
+        const int spot = (t * 16 + (lane >> 4) * 8 + (lane & 7)) * v_ld + warp * 16 + ((lane >> 3) & 1) * 8;
+        load_matrices_turned(va, shared_address(vs + spot));
+        load_matrices_turned(rest, shared_address(vs_rest + spot));
 #pragma unroll
         for (int c = 0; c < NMAX / 16; ++c) {
             if (c * 16 >= n16) continue;
@@ -193,6 +217,8 @@ __global__ void __launch_bounds__(2 * ETILE) chunk_states_kernel(const ChunkArgs
             load_matrices_turned(kb, shared_address(ks + (t * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * k_ld + c * 16 + (lane >> 4) * 8));
             multiply(acc[2 * c], va, kb[0], kb[1]);
             multiply(acc[2 * c + 1], va, kb[2], kb[3]);
+            multiply(acc[2 * c], rest, kb[0], kb[1]);
+            multiply(acc[2 * c + 1], rest, kb[2], kb[3]);
         }
     }
     float* dst = a.ends + (size_t)chunk * a.end_stride + (size_t)head * (a.e + a.sums) * a.n_padded;
@@ -302,11 +328,11 @@ __global__ void __launch_bounds__(2 * ETILE, 256 / ETILE) chunk_outputs_kernel(c
     float x[AHEAD][4], y[AHEAD][4];
     queries.fetch(walk, x);
     chunk_gates<KIND>(a, first, count, head, L, step, &warp_total);
-    queries.place(walk, x, qs, ld, nullptr, a.q_scale);
+    queries.place(walk, x, qs, ld, a.q_scale);
     for (int base = threadIdx.x + AHEAD * THREADS; base < CHUNK * queries.quads; base += AHEAD * THREADS) {
         const Tile::Walk<THREADS> more(base, queries.quads);
         queries.fetch(more, x);
-        queries.place(more, x, qs, ld, nullptr, a.q_scale);
+        queries.place(more, x, qs, ld, a.q_scale);
     }
     asm volatile("cp.async.wait_all;");
     __syncthreads();
@@ -336,13 +362,13 @@ __global__ void __launch_bounds__(2 * ETILE, 256 / ETILE) chunk_outputs_kernel(c
     keys.fetch(walk, x);
     values.fetch(value_walk, y);  // AHEAD pieces per thread are the whole tile
     __syncthreads();  // the state has been read
-    keys.place(walk, x, ks, ld, nullptr, 1.f);
+    keys.place(walk, x, ks, ld, 1.f);
     for (int base = threadIdx.x + AHEAD * THREADS; base < CHUNK * keys.quads; base += AHEAD * THREADS) {
         const Tile::Walk<THREADS> more(base, keys.quads);
         keys.fetch(more, x);
-        keys.place(more, x, ks, ld, nullptr, 1.f);
+        keys.place(more, x, ks, ld, 1.f);
     }
-    values.place(value_walk, y, vs, v_ld, nullptr, 1.f);
+    values.place(value_walk, y, vs, v_ld, 1.f);
     __syncthreads();
     if (active) {
         float score[CHUNK / 8][4];
@@ -385,14 +411,19 @@ __global__ void __launch_bounds__(2 * ETILE, 256 / ETILE) chunk_outputs_kernel(c
 #pragma unroll
         for (int i = 0; i < CHUNK / 16; ++i) {
             if (i > warp) continue;
-            const uint32_t pa[4] = {pack(score[2 * i][0], score[2 * i][1]), pack(score[2 * i][2], score[2 * i][3]), pack(score[2 * i + 1][0], score[2 * i + 1][1]),
-                                    pack(score[2 * i + 1][2], score[2 * i + 1][3])};
+            uint32_t pa[4], rest[4];
+            pack_pair(score[2 * i][0], score[2 * i][1], pa[0], rest[0]);
+            pack_pair(score[2 * i][2], score[2 * i][3], pa[1], rest[1]);
+            pack_pair(score[2 * i + 1][0], score[2 * i + 1][1], pa[2], rest[2]);
+            pack_pair(score[2 * i + 1][2], score[2 * i + 1][3], pa[3], rest[3]);
 #pragma unroll
             for (int c = 0; c < COLUMNS / 16; ++c) {
                 uint32_t b[4];
                 load_matrices_turned(b, shared_address(vs + (i * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * v_ld + column0 + c * 16 + (lane >> 4) * 8));
                 multiply(acc[2 * c], pa, b[0], b[1]);
                 multiply(acc[2 * c + 1], pa, b[2], b[3]);
+                multiply(acc[2 * c], rest, b[0], b[1]);
+                multiply(acc[2 * c + 1], rest, b[2], b[3]);
             }
         }
         const float skip = KIND == KIND_STATE_SPACE ? a.skip[head] : 0.f;
@@ -454,7 +485,7 @@ int allow_shared(Kernel kernel, int bytes) {
 
 template <int KIND, int ETILE>
 int launch_states(const ChunkArgs& a, int chunks, cudaStream_t stream) {
-    const int n16 = (a.n + 15) & ~15, bytes = CHUNK * (n16 + 8) * 2 + CHUNK * (ETILE + 8) * 2;
+    const int n16 = (a.n + 15) & ~15, bytes = CHUNK * (n16 + 8) * 2 + 2 * CHUNK * (ETILE + 8) * 2;
     const dim3 grid(chunks, a.heads, (a.e + ETILE - 1) / ETILE);
 #define HB_CHUNK_STATES(NMAX)                                                                        \
     do {                                                                                             \

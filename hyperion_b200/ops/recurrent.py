@@ -340,7 +340,7 @@ def chunked_scan(kind: int, k: torch.Tensor, q: torch.Tensor, v: torch.Tensor, g
     step is softplus(``gate``[decay_off + h] + dt_bias), a = exp(-exp(a_log) step), D = ``skip``; ``KIND_GIVEN``: ln a and b are the columns ``decay_off + h`` and
     ``step_off + h`` of ``gate``.  The rows' states ([heads, e, n_padded], with ``sums_keys`` one more row for the sum of keys) lie at ``state_off`` of ``state``.  Returns
     [tokens, heads, ``columns``] (``e`` unless stated; with ``sums_keys`` entry e of a head is n . q).  Differs from the one-pass scan by bfloat16 roundings of
-    keys, queries, values and weighted scores."""
+    keys, queries and values."""
     require_cuda(k, q, v, gate, state, slots, chunk_start, chunk_row, a_log, dt_bias, skip)
     _floats(k, q, v, gate, state, a_log, dt_bias, skip)
     rows = e + (1 if sums_keys else 0)

@@ -478,10 +478,12 @@ def test_the_matrix_memory_kernels(shape):
     assert torch.equal(state[2], after[2])
 
 
+@pytest.mark.parametrize("rounded", [False, True])
 @pytest.mark.parametrize("shape", [(3, 40, 24), (2, 128, 128), (4, 7, 5), (1, 250, 65), (6, 64, 100)])
-def test_scans_in_chunks(shape):
+def test_scans_in_chunks(shape, rounded):
     """The matrix memory and the state-space scan in chunks on the tensor cores against the one-pass scan: rows of 1 to 700 tokens, from states that are not zero, keys
-    shared by several heads, decays from nearly 1 to nearly 0, columns of a wider matrix."""
+    shared by several heads, decays from nearly 1 to nearly 0, columns of a wider matrix.  ``rounded``: keys, queries and values are bfloat16 values to begin with, and
+    then the two agree as two float computations do."""
     from hyperion_b200.ops import recurrent
 
     heads, n, e = shape
@@ -489,6 +491,11 @@ def test_scans_in_chunks(shape):
     counts = [300, 1, 64, 700, 63, 129]
     x, bi, bf, start = _memory_case(heads, n, e, counts, 5)
     bf[0] = 9.0  # this head hardly forgets
+    q_scale = n ** -0.5
+    if rounded:
+        x[:, : heads * n] *= q_scale
+        q_scale = 1.0
+        x[:, : 2 * heads * n + heads * e] = x[:, : 2 * heads * n + heads * e].to(torch.bfloat16).float()
     cut = recurrent.plan_chunks(counts)
     assert sum(counts) == cut[0][-1] and max(b - a for a, b in zip(cut[0], cut[0][1:])) == 64 and cut[1] == [0] * 5 + [1, 2] + [3] * 11 + [4] + [5] * 3
     assert recurrent.plan_chunks([5, 100, 127]) is None
@@ -504,14 +511,17 @@ def test_scans_in_chunks(shape):
 
     def compare(y, z, one, many):
         scale = y.abs().mean(dim=0, keepdim=True) + y.abs().mean()
+        if rounded:
+            assert ((y - z).abs() / scale).max() <= 2e-4 and (one - many).abs().max() <= 5e-5 * one.abs().max()
+            return
         assert ((y - z).abs() / scale).max() <= 0.1 and ((y - z) / scale).pow(2).mean().sqrt() <= 1e-2
         assert (one - many).abs().max() <= 2e-2 * one.abs().max() and ((one - many).pow(2).mean() / one.pow(2).mean()).sqrt() <= 5e-3
 
     one, many = begin.cuda(), begin.cuda()
     gates = [recurrent.matrix_memory_gates(dev, i_off, i_off + heads, bi.cuda(), bf.cuda(), cap, s, m_off, slots, rows_of, len(counts), heads) for s in (one, many)]
-    y = recurrent.matrix_memory_scan(dev, heads * n, 0, 2 * heads * n, gates[0], one, 0, slots, rows_of, len(counts), heads, n, n_padded, e, n ** -0.5)
+    y = recurrent.matrix_memory_scan(dev, heads * n, 0, 2 * heads * n, gates[0], one, 0, slots, rows_of, len(counts), heads, n, n_padded, e, q_scale)
     z = recurrent.chunked_scan(recurrent.KIND_GIVEN, dev[:, heads * n :], dev, dev[:, 2 * heads * n :], gates[1].view(len(x), 4 * heads), 3 * heads, heads, many, 0, slots, chunk_start,
-                               chunk_row, len(cut[1]), heads, heads, n, n_padded, e, sums_keys=True, q_scale=n ** -0.5, columns=y.shape[2])
+                               chunk_row, len(cut[1]), heads, heads, n, n_padded, e, sums_keys=True, q_scale=q_scale, columns=y.shape[2])
     compare(y[..., : e + 1], z[..., : e + 1], one, many)
     groups = 2 if heads % 2 == 0 else 1
     a_log, dt_bias = torch.linspace(-4, 1, heads).cuda(), torch.linspace(-5, 3, heads).cuda()
